@@ -440,6 +440,98 @@ int b200_classify_causal_mask(const void* mask, int64_t batch, int64_t tokens,
 int b200_argmax(const void* logits, int64_t* ids, int64_t rows, int64_t vocab,
                 int64_t row_stride, int dtype, void* stream);
 
+/* ---- Hybrid layers -------------------------------------------------------------------
+ * Operators of decoder layers whose mixers are recurrences with a matrix state (retention, the
+ * gated delta rule with a decay per key channel) or attention over cached latents, with an RMS norm
+ * before and after every sublayer and an fp32 residual stream. No counterpart in the reference.
+ *
+ * The rows of a step are the tokens of `sequences` sequences side by side: sequence s owns rows
+ * starts[s] .. starts[s + 1] - 1 (int32 [sequences + 1]), its first row stands at position bases[s]
+ * and its state lives in slot slots[s]; slot -1 is an idle row: it computes zeros and keeps nothing.
+ * token_sequence[row] (int32 [rows]) is the sequence of a row. A portion that starts at position 0
+ * starts from an empty state whatever the slot held before. dtype is B200_F32 or B200_BF16 (weights,
+ * projections, cached latents); state, decays, gates, norms and the residual are fp32.
+ *
+ *   b200_residual_norm   x += norm(y) * (weight_offset + post_weight); h = norm(x) * (weight_offset +
+ *                        next_weight). x fp32 [rows, width]; y of the model dtype, or fp32 split-K
+ *                        partials [splits, rows, y_row_stride] when splits > 0; y NULL: h only;
+ *                        next_weight NULL: no h. Columns of h from width to h_row_stride are zeroed.
+ *   b200_latent_norm     RMS norms (plain weights) of the query latent (columns 0 .. q_rank - 1 of
+ *                        input) and the kv latent (from kv_column); the latter goes to the cache row of
+ *                        the token's position, and to dense [rows, cache_row] when given. kv_weight
+ *                        NULL: the query latent only. Padding columns of the results are zeroed.
+ *   b200_gated_head_norm out = norm over vdim of input (fp32 [rows, heads, vdim]) * weight (or 1) *
+ *                        silu(gate) or sigmoid(gate)
+ *   b200_retention_prep  q and k (rotated on the first rot_dims dimensions of each head, pair
+ *                        (i, i + rot_dims / 2); k times k_scale) and v as fp32 operands
+ *   b200_delta_prep      q, k (short convolution, silu, unit norm; q times q_scale), v (convolution,
+ *                        silu), beta and log g as fp32 operands
+ *   b200_conv_tail       keeps the last `taps` inputs of every sequence for the next portion
+ *   b200_recurrence_scan token by token recurrence on prepared operands. beta NULL: retention, decay
+ *                        is [heads]; otherwise the delta rule, decay is log g [rows, heads, dim]. State
+ *                        [slots, heads, dim, state_row] is read, and written behind the last token.
+ *   b200_head_linear     y[m, h, :] = w[h] x[m, h, :], w [heads, n, k]
+ *   b200_latent_attention  q, out [rows, heads, rank_row] in the latent space, cache [slots, capacity,
+ *                        rank_row]; a row sees the positions up to its own; with sink (model dtype
+ *                        [heads]) the softmax denominator of head h also holds exp(sink[h])
+ *   b200_sequence_positions  positions[r] = lengths[slots[r]] (0 for an idle row)
+ *   b200_advance_slots   lengths[slots[r]] += starts[r + 1] - starts[r], clamped with a status bit */
+#define B200_GATE_SILU 0
+#define B200_GATE_SIGMOID 1
+typedef struct b200_delta_inputs {
+  const void* input;  /* [rows, row_stride]: projections of h; *_column: where an operand starts */
+  const void* gates;  /* [rows, gate_row_stride]: decay projections from decay_column on */
+  const void* q_conv; /* [kv_heads * dim, taps], last column: the current token */
+  const void* k_conv;
+  const void* v_conv; /* [heads * vdim, taps] */
+  const void* a_log;  /* [heads] */
+  const void* dt_bias; /* [heads * dim] */
+  void* ring;         /* [slots, taps, 2 kv_heads dim + heads vdim]: inputs by position % taps */
+  const int32_t* token_sequence;
+  const int32_t* starts;
+  const int32_t* slots;
+  const int32_t* bases;
+  int64_t heads, kv_heads, dim, vdim, taps;
+  int64_t q_column, k_column, v_column, beta_column, decay_column;
+  int64_t row_stride, gate_row_stride;
+  double q_scale;
+} b200_delta_inputs;
+int b200_residual_norm(void* x, const void* y, const void* post_weight, const void* next_weight, void* h,
+                       int64_t rows, int64_t width, int64_t splits, int64_t y_row_stride,
+                       int64_t h_row_stride, double epsilon, double weight_offset, int dtype, void* stream);
+int b200_latent_norm(const void* input, const void* q_weight, const void* kv_weight, void* q_out,
+                     void* cache, void* dense, const int32_t* token_sequence, const int32_t* starts,
+                     const int32_t* slots, const int32_t* bases, int64_t rows, int64_t q_rank,
+                     int64_t kv_rank, int64_t kv_column, int64_t cache_row, int64_t input_row_stride,
+                     int64_t q_row_stride, int64_t capacity, double epsilon, int dtype, int32_t* status,
+                     void* stream);
+int b200_gated_head_norm(const void* input, const void* weight, const void* gate, void* output, int64_t rows,
+                         int64_t heads, int64_t vdim, int64_t gate_row_stride, int64_t output_row_stride,
+                         int gate_kind, double epsilon, int dtype, void* stream);
+int b200_retention_prep(const void* input, const int32_t* token_sequence, const int32_t* starts,
+                        const int32_t* slots, const int32_t* bases, float* q, float* k, float* v,
+                        int64_t rows, int64_t heads, int64_t dim, int64_t vdim, int64_t q_column,
+                        int64_t k_column, int64_t v_column, int64_t row_stride, int64_t rot_dims,
+                        double rot_base, double k_scale, int dtype, void* stream);
+int b200_delta_prep(const b200_delta_inputs* inputs, float* q, float* k, float* v, float* beta,
+                    float* log_decay, int64_t rows, int dtype, void* stream);
+int b200_conv_tail(const b200_delta_inputs* inputs, int64_t sequences, int dtype, void* stream);
+int b200_recurrence_scan(const float* q, const float* k, const float* v, const float* beta, const float* decay,
+                         float* state, float* output, const int32_t* token_sequence, const int32_t* starts,
+                         const int32_t* slots, const int32_t* bases, int64_t sequences, int64_t heads,
+                         int64_t kv_heads, int64_t dim, int64_t vdim, int64_t state_row, void* stream);
+int b200_head_linear(const void* x, const void* w, void* y, int64_t m, int64_t heads, int64_t k, int64_t n,
+                     int64_t x_row_stride, int64_t x_head_stride, int64_t y_row_stride,
+                     int64_t y_head_stride, int dtype, void* stream);
+int b200_latent_attention(const void* q, const void* cache, const void* sink, void* out,
+                          const int32_t* token_sequence, const int32_t* starts, const int32_t* slots,
+                          const int32_t* bases, int64_t rows, int64_t heads, int64_t rank_row,
+                          int64_t capacity, double scale, int dtype, void* stream);
+int b200_sequence_positions(const int64_t* lengths, const int32_t* slots, int32_t* positions, int64_t rows,
+                            void* stream);
+int b200_advance_slots(int64_t* lengths, const int32_t* slots, const int32_t* starts, int64_t rows,
+                       int64_t capacity, int32_t* status, void* stream);
+
 #ifdef __cplusplus
 }
 #endif

@@ -41,8 +41,25 @@ class B200LibraryError(RuntimeError):
 
 _I64P = POINTER(c_int64)
 
+GATE_SILU, GATE_SIGMOID = 0, 1
+
+
+class DeltaInputs(ctypes.Structure):
+    """b200_delta_inputs of include/b200_serve.h."""
+
+    _fields_ = [(name, c_void_p) for name in
+                ("input", "gates", "q_conv", "k_conv", "v_conv", "a_log", "dt_bias", "ring",
+                 "token_sequence", "starts", "slots", "bases")] + \
+               [(name, c_int64) for name in
+                ("heads", "kv_heads", "dim", "vdim", "taps", "q_column", "k_column", "v_column",
+                 "beta_column", "decay_column", "row_stride", "gate_row_stride")] + \
+               [("q_scale", c_double)]
+
+
+_DELTA = POINTER(DeltaInputs)
+
 # What b200_abi_version() of a matching library returns (bumped with every signature change).
-ABI_VERSION = 104
+ABI_VERSION = 105
 
 # name -> (restype, argtypes); mirrors include/b200_serve.h one to one
 SIGNATURES = {
@@ -114,6 +131,17 @@ SIGNATURES = {
     "b200_advance_lengths": (c_int, [c_void_p, c_int64, c_int64, c_int64, c_int64, c_void_p,
                                      c_void_p]),
     "b200_argmax": (c_int, [c_void_p, c_void_p, c_int64, c_int64, c_int64, c_int, c_void_p]),
+    "b200_residual_norm": (c_int, [c_void_p] * 5 + [c_int64] * 5 + [c_double, c_double, c_int, c_void_p]),
+    "b200_latent_norm": (c_int, [c_void_p] * 10 + [c_int64] * 8 + [c_double, c_int, c_void_p, c_void_p]),
+    "b200_gated_head_norm": (c_int, [c_void_p] * 4 + [c_int64] * 5 + [c_int, c_double, c_int, c_void_p]),
+    "b200_retention_prep": (c_int, [c_void_p] * 8 + [c_int64] * 9 + [c_double, c_double, c_int, c_void_p]),
+    "b200_delta_prep": (c_int, [_DELTA] + [c_void_p] * 5 + [c_int64, c_int, c_void_p]),
+    "b200_conv_tail": (c_int, [_DELTA, c_int64, c_int, c_void_p]),
+    "b200_recurrence_scan": (c_int, [c_void_p] * 11 + [c_int64] * 6 + [c_void_p]),
+    "b200_head_linear": (c_int, [c_void_p] * 3 + [c_int64] * 8 + [c_int, c_void_p]),
+    "b200_latent_attention": (c_int, [c_void_p] * 8 + [c_int64] * 4 + [c_double, c_int, c_void_p]),
+    "b200_sequence_positions": (c_int, [c_void_p] * 3 + [c_int64, c_void_p]),
+    "b200_advance_slots": (c_int, [c_void_p] * 3 + [c_int64, c_int64, c_void_p, c_void_p]),
 }
 
 _library: ctypes.CDLL | None = None

@@ -11,6 +11,7 @@ from __future__ import annotations
 
 import concurrent.futures
 import os
+import re
 import shutil
 import subprocess
 import sys
@@ -41,6 +42,21 @@ def sources() -> list[Path]:
     return sorted(CSRC.glob("*.cu"))
 
 
+def _includes(source: Path) -> list[Path]:
+    """The project headers a source includes, directly or through one another."""
+
+    found: list[Path] = []
+    pending = [source]
+    while pending:
+        for name in re.findall(r'^\s*#include\s+"([^"]+)"', pending.pop().read_text(), re.M):
+            for folder in (CSRC, INCLUDE):
+                header = folder / name
+                if header.exists() and header not in found:
+                    found.append(header)
+                    pending.append(header)
+    return found
+
+
 def _stale(target: Path, inputs: list[Path]) -> bool:
     if not target.exists():
         return True
@@ -60,13 +76,12 @@ def _compile(nvcc: str, source: Path, obj: Path) -> None:
 def build(force: bool = False, verbose: bool = False) -> Path:
     nvcc = _nvcc()
     BUILD_DIR.mkdir(parents=True, exist_ok=True)
-    headers = sorted(CSRC.glob("*.cuh")) + sorted(INCLUDE.glob("*.h"))
     jobs = []
     objects = []
     for source in sources():
         obj = BUILD_DIR / (source.stem + ".o")
         objects.append(obj)
-        if force or _stale(obj, [source, *headers]):
+        if force or _stale(obj, [source, *_includes(source)]):
             jobs.append((source, obj))
     if jobs:
         if verbose:

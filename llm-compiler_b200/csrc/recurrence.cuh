@@ -1,0 +1,84 @@
+// Operands of the recurrent mixers as every kernel of theirs computes them (scan, decode step, chunked
+// prefill): rotation, short causal convolution, decays and step sizes, all in fp32.
+#pragma once
+
+#include "hybrid.cuh"
+
+namespace b200 {
+
+constexpr float kUnitEpsilon = 1e-6f;  // inside the root of a unit norm
+
+// cos / sin of position * base^(-2 i / dims). The product and its reduction to one turn are done in
+// double, so that a far position costs no accuracy; the functions then see at most half a turn.
+__device__ __forceinline__ void rotation_of(int64_t position, int i, int dims, double log2_base, float& c,
+                                            float& s) {
+  const double turns = static_cast<double>(position) * exp2(-2.0 * i / dims * log2_base) * 0.15915494309189535;
+  sincospif(2.0f * static_cast<float>(turns - rint(turns)), &s, &c);
+}
+
+struct DeltaInputs {
+  const void* input;   // T [rows, row_stride]: the projections of h
+  const void* gates;   // T [rows, gate_row_stride]: decay columns [heads * dim] from decay_column
+  const void *q_conv, *k_conv, *v_conv;  // T [channels, taps], last column: the current token
+  const void* a_log;   // T [heads]
+  const void* dt_bias; // T [heads * dim]
+  void* ring;          // T [slots, taps, 2 kv_heads dim + heads vdim]: inputs by position % taps
+  SequenceBatch batch;
+  int heads, kv_heads, dim, vdim, taps;
+  int q_column, k_column, v_column, beta_column, decay_column;
+  int64_t row_stride, gate_row_stride;
+  float q_scale;
+};
+
+inline bool delta_inputs_from(const b200_delta_inputs* in, DeltaInputs* out) {
+  if (in == nullptr || !in->input || !in->gates || !in->q_conv || !in->k_conv || !in->v_conv || !in->a_log ||
+      !in->dt_bias || !in->ring || !in->token_sequence || !in->starts || !in->slots || !in->bases ||
+      in->heads <= 0 || in->kv_heads <= 0 || in->heads % in->kv_heads != 0 || in->dim <= 0 || in->vdim <= 0 ||
+      in->taps <= 0)
+    return false;
+  *out = DeltaInputs{in->input, in->gates, in->q_conv, in->k_conv, in->v_conv, in->a_log, in->dt_bias, in->ring,
+                     {in->token_sequence, in->starts, in->slots, in->bases},
+                     static_cast<int>(in->heads), static_cast<int>(in->kv_heads), static_cast<int>(in->dim),
+                     static_cast<int>(in->vdim), static_cast<int>(in->taps), static_cast<int>(in->q_column),
+                     static_cast<int>(in->k_column), static_cast<int>(in->v_column),
+                     static_cast<int>(in->beta_column), static_cast<int>(in->decay_column), in->row_stride,
+                     in->gate_row_stride, static_cast<float>(in->q_scale)};
+  return true;
+}
+
+// Output of the short convolution of operand `which` (0 q, 1 k, 2 v), channel `channel`, for the token
+// at `row` (the local-th of its portion, at `position`). Inputs of earlier portions come from the ring;
+// before the start there are zeros.
+template <typename T>
+__device__ __forceinline__ float short_conv(const DeltaInputs& p, int which, int channel, int64_t row,
+                                            int64_t local, int64_t position, int slot) {
+  const T* taps = static_cast<const T*>(which == 0 ? p.q_conv : which == 1 ? p.k_conv : p.v_conv) +
+                  static_cast<int64_t>(channel) * p.taps;
+  const T* in = static_cast<const T*>(p.input) + row * p.row_stride +
+                (which == 0 ? p.q_column : which == 1 ? p.k_column : p.v_column) + channel;
+  const int qk = p.kv_heads * p.dim;
+  const int channels = 2 * qk + p.heads * p.vdim;
+  const T* ring = static_cast<const T*>(p.ring) + static_cast<int64_t>(slot) * p.taps * channels + which * qk + channel;
+  float sum = 0.0f;
+  for (int back = 0; back < p.taps && back <= position; ++back) {
+    const float value = back <= local ? Elem<T>::load(in - back * p.row_stride)
+                                      : Elem<T>::load(ring + ((position - back) % p.taps) * channels);
+    sum = fmaf(Elem<T>::load(taps + p.taps - 1 - back), value, sum);
+  }
+  return sum;
+}
+
+template <typename T>
+__device__ __forceinline__ float delta_beta(const DeltaInputs& p, int64_t row, int head) {
+  return sigmoid_f32(Elem<T>::load(static_cast<const T*>(p.input) + row * p.row_stride + p.beta_column + head));
+}
+
+// log g of one key channel
+template <typename T>
+__device__ __forceinline__ float delta_log_decay(const DeltaInputs& p, int64_t row, int head, int c) {
+  const float step = Elem<T>::load(static_cast<const T*>(p.gates) + row * p.gate_row_stride + p.decay_column + head * p.dim + c) +
+                     Elem<T>::load(static_cast<const T*>(p.dt_bias) + head * p.dim + c);
+  return -expf(Elem<T>::load(static_cast<const T*>(p.a_log) + head)) * softplus_f32(step);
+}
+
+}  // namespace b200

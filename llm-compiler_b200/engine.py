@@ -33,7 +33,118 @@ from .kv_state import ExecutionError, PagedKVCacheState, PreallocatedKVCacheStat
 from .qwen2 import Qwen2Config, inverse_frequency
 
 
-class Qwen2Engine:
+class ServingEngine:
+    """What the serving engines share: the buffers of a decode step with fixed addresses, its capture
+    in CUDA graphs, the step a serving loop calls and greedy generation. A subclass provides
+    `prefill(input_ids)` (which leaves the next tokens in `next_ids` and `input_ids`),
+    `_decode_step()` (one step from `input_ids`: sets `logits`, fills `next_ids`, advances the
+    state), `_warm_up()` (a step that leaves no trace) and `state` with `check()`."""
+
+    def _init_step(self, batch: int, device: torch.device) -> None:
+        self.batch = batch
+        self.device = device
+        self.input_ids = torch.zeros(batch, dtype=torch.int64, device=device)
+        self.next_ids = torch.zeros(batch, dtype=torch.int64, device=device)
+        self.logits: Optional[torch.Tensor] = None
+        self._graph: Optional[torch.cuda.CUDAGraph] = None
+        self._step_graph: Optional[torch.cuda.CUDAGraph] = None  # the same step between its two host copies
+        self._host_ids = torch.zeros(batch, dtype=torch.int64).pin_memory()
+        self._host_tokens = torch.zeros(batch, dtype=torch.int64).pin_memory()
+        self.kernels_per_step = 0
+
+    def _reserve_blocks(self) -> None:
+        """Host-side storage a step needs, ahead of its launch."""
+
+    def _count_step(self) -> None:
+        """Host-side bookkeeping behind a step."""
+
+    def _warm_up(self) -> None:
+        raise NotImplementedError
+
+    def _decode_step(self) -> None:
+        raise NotImplementedError
+
+    def prefill(self, input_ids: torch.Tensor) -> torch.Tensor:
+        raise NotImplementedError
+
+    def capture(self) -> None:
+        """Captures one decode step in a CUDA graph. A warm-up step runs first so that every
+        workspace exists."""
+
+        self._reserve_blocks()
+        stream = torch.cuda.Stream(device=self.device)
+        stream.wait_stream(torch.cuda.current_stream(self.device))
+        with torch.cuda.stream(stream):
+            self._warm_up()
+        torch.cuda.current_stream(self.device).wait_stream(stream)
+        torch.cuda.synchronize(self.device)
+        graph = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(graph):
+            self._decode_step()
+        self._graph = graph
+        self._graph_logits = self.logits  # each graph writes the logits into a buffer of its own
+        # step(): the copy of the ids from pinned host memory, the step and the copy of the tokens
+        # back as one graph launch instead of three submissions
+        step_graph = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(step_graph):
+            self.input_ids.copy_(self._host_ids, non_blocking=True)
+            self._decode_step()
+            self._host_tokens.copy_(self.next_ids, non_blocking=True)
+        self._step_graph = step_graph
+        self._step_logits = self.logits
+        self.logits = self._graph_logits
+        kernels.runtime(self.device).status.zero_()
+
+    def decode_step(self, *, feed_back: bool = True) -> torch.Tensor:
+        """One decode step for the whole batch on device-resident inputs. Returns the device
+        tensor of greedy tokens; with feed_back they become the next step's input ids."""
+
+        self._reserve_blocks()
+        if self._graph is not None:
+            self._graph.replay()
+            self.logits = self._graph_logits
+        else:
+            self._decode_step()
+        self._count_step()
+        if feed_back:
+            self.input_ids.copy_(self.next_ids, non_blocking=True)
+        return self.next_ids
+
+    def step(self, host_ids: torch.Tensor) -> torch.Tensor:
+        """The call a serving loop makes: host token ids in, host greedy tokens out. Copies
+        the ids from pinned host memory, runs one decode step, copies the tokens back and
+        waits for them."""
+
+        self._host_ids.copy_(host_ids)
+        if self._step_graph is not None:
+            self._reserve_blocks()
+            self._step_graph.replay()
+            self.logits = self._step_logits
+            self._count_step()
+        else:
+            self.input_ids.copy_(self._host_ids, non_blocking=True)
+            self.decode_step(feed_back=False)
+            self._host_tokens.copy_(self.next_ids, non_blocking=True)
+        torch.cuda.current_stream(self.device).synchronize()
+        return self._host_tokens
+
+    def generate(self, prompt_ids: torch.Tensor, steps: int, *, use_graph: bool = True) -> torch.Tensor:
+        """Greedy generation: prefill then `steps` decode steps. Returns B x (steps + 1) token
+        ids (the token sampled from the prompt first)."""
+
+        self.prefill(prompt_ids)
+        history = torch.empty((steps + 1, self.batch), dtype=torch.int64, device=self.device)
+        history[0].copy_(self.next_ids)
+        if use_graph and self._graph is None and steps > 0:
+            self.capture()
+        for index in range(steps):
+            self.decode_step()
+            history[index + 1].copy_(self.next_ids)
+        self.state.check()
+        return history.transpose(0, 1).contiguous()
+
+
+class Qwen2Engine(ServingEngine):
     def __init__(self, config: Qwen2Config, weights: Dict[str, torch.Tensor], *, batch: int,
                  capacity: int, numerical_mode: str = "fast",
                  device: Optional[torch.device] = None, kv_layout: str = "contiguous",
@@ -48,10 +159,9 @@ class Qwen2Engine:
         if kv_layout not in ("contiguous", "paged"):
             raise ValueError(f"unknown KV layout {kv_layout!r}")
         self.config = config
-        self.batch = batch
+        self._init_step(batch, device or torch.device("cuda", torch.cuda.current_device()))
         self.capacity = capacity
         self.mode = numerical_mode
-        self.device = device or torch.device("cuda", torch.cuda.current_device())
         self.dtype = weights["embed_tokens.weight"].dtype
         self.scale = config.head_dim ** -0.5
         # the five-launch decode layer (RMSNorm folded into q|k|v and gate|up, cluster split-K
@@ -93,13 +203,6 @@ class Qwen2Engine:
         arena = self.state._length_arena
         self.positions = arena[layers]
         self.attention_lengths = arena[layers + 1]
-        self.input_ids = torch.zeros(batch, dtype=torch.int64, device=self.device)
-        self.next_ids = torch.zeros(batch, dtype=torch.int64, device=self.device)
-        self.logits: Optional[torch.Tensor] = None
-        self._graph: Optional[torch.cuda.CUDAGraph] = None
-        self._step_graph: Optional[torch.cuda.CUDAGraph] = None  # the same step between its two host copies
-        self._host_ids = torch.zeros(batch, dtype=torch.int64).pin_memory()
-        self._host_tokens = torch.zeros(batch, dtype=torch.int64).pin_memory()
         self.max_length_hint = 0  # host-known upper bound of the context (0 = capacity)
         # programmatic dependent launch of the chain (B200_PROGRAMMATIC_LAUNCH=0 turns it off)
         self.programmatic_launch = os.environ.get("B200_PROGRAMMATIC_LAUNCH", "1") != "0"
@@ -107,7 +210,6 @@ class Qwen2Engine:
         # keeps them a launch of their own)
         self.fused_qkv_attention = os.environ.get("B200_FUSED_QKV_ATTENTION", "1") != "0"
         self.split_tokens = 0
-        self.kernels_per_step = 0
         # longest-first service order of decode attention (ragged batches with more
         # (sequence, KV head) pairs than the GPU holds at once): one buffer, rewritten in place
         # by load_context, so that a captured step keeps reading the current order
@@ -262,6 +364,16 @@ class Qwen2Engine:
             self._block_slack -= 1
 
     # ------------------------------------------------------------------- decode ----
+    def _warm_up(self) -> None:
+        """A step whose lengths and ids are put back (the KV row it wrote lies beyond the valid
+        length and is overwritten by the real step)."""
+
+        saved_lengths = self.state._length_arena.clone()
+        saved_ids = self.input_ids.clone()
+        self._decode_step()
+        self.state._length_arena.copy_(saved_lengths)
+        self.input_ids.copy_(saved_ids)
+
     @property
     def chained(self) -> bool:
         """Whether a decode step runs the launch chain (fast bf16, up to 128 sequences)."""
@@ -451,84 +563,3 @@ class Qwen2Engine:
         decision = resolve_dispatch_plan(plan, context_bound)
         self.split_tokens = split_tokens_of(decision.variant)
         return decision
-
-    def capture(self) -> None:
-        """Captures one decode step in a CUDA graph. A warm-up step runs first so that every
-        workspace exists; lengths, positions and ids are restored afterwards (the KV row the
-        warm-up wrote lies beyond the valid length and is overwritten by the real step)."""
-
-        self._reserve_blocks()
-        saved_lengths = self.state._length_arena.clone()
-        saved_ids = self.input_ids.clone()
-        stream = torch.cuda.Stream(device=self.device)
-        stream.wait_stream(torch.cuda.current_stream(self.device))
-        with torch.cuda.stream(stream):
-            self._decode_step()
-            self.state._length_arena.copy_(saved_lengths)
-            self.input_ids.copy_(saved_ids)
-        torch.cuda.current_stream(self.device).wait_stream(stream)
-        torch.cuda.synchronize(self.device)
-        graph = torch.cuda.CUDAGraph()
-        with torch.cuda.graph(graph):
-            self._decode_step()
-        self._graph = graph
-        self._graph_logits = self.logits  # each graph writes the logits into a buffer of its own
-        # step(): the copy of the ids from pinned host memory, the step and the copy of the tokens
-        # back as one graph launch instead of three submissions
-        step_graph = torch.cuda.CUDAGraph()
-        with torch.cuda.graph(step_graph):
-            self.input_ids.copy_(self._host_ids, non_blocking=True)
-            self._decode_step()
-            self._host_tokens.copy_(self.next_ids, non_blocking=True)
-        self._step_graph = step_graph
-        self._step_logits = self.logits
-        self.logits = self._graph_logits
-        kernels.runtime(self.device).status.zero_()
-
-    def decode_step(self, *, feed_back: bool = True) -> torch.Tensor:
-        """One decode step for the whole batch on device-resident inputs. Returns the device
-        tensor of greedy tokens; with feed_back they become the next step's input ids."""
-
-        self._reserve_blocks()
-        if self._graph is not None:
-            self._graph.replay()
-            self.logits = self._graph_logits
-        else:
-            self._decode_step()
-        self._count_step()
-        if feed_back:
-            self.input_ids.copy_(self.next_ids, non_blocking=True)
-        return self.next_ids
-
-    def step(self, host_ids: torch.Tensor) -> torch.Tensor:
-        """The call a serving loop makes: host token ids in, host greedy tokens out. Copies
-        the ids from pinned host memory, runs one decode step, copies the tokens back and
-        waits for them."""
-
-        self._host_ids.copy_(host_ids)
-        if self._step_graph is not None:
-            self._reserve_blocks()
-            self._step_graph.replay()
-            self.logits = self._step_logits
-            self._count_step()
-        else:
-            self.input_ids.copy_(self._host_ids, non_blocking=True)
-            self.decode_step(feed_back=False)
-            self._host_tokens.copy_(self.next_ids, non_blocking=True)
-        torch.cuda.current_stream(self.device).synchronize()
-        return self._host_tokens
-
-    def generate(self, prompt_ids: torch.Tensor, steps: int, *, use_graph: bool = True) -> torch.Tensor:
-        """Greedy generation: prefill then `steps` decode steps. Returns B x (steps + 1) token
-        ids (the token sampled from the prompt first)."""
-
-        self.prefill(prompt_ids)
-        history = torch.empty((steps + 1, self.batch), dtype=torch.int64, device=self.device)
-        history[0].copy_(self.next_ids)
-        if use_graph and self._graph is None and steps > 0:
-            self.capture()
-        for index in range(steps):
-            self.decode_step()
-            history[index + 1].copy_(self.next_ids)
-        self.state.check()
-        return history.transpose(0, 1).contiguous()

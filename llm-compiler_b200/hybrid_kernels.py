@@ -1,0 +1,292 @@
+"""Python wrappers over the C ABI for the hybrid layers' operators (include/b200_serve.h, "Hybrid
+layers"): recurrent mixers, latent attention and the fp32 residual stream. Same rules as kernels.py:
+preconditions raise before anything is launched, launches go to torch's current stream and never
+synchronise, and there is no fallback to PyTorch."""
+
+from __future__ import annotations
+
+from ctypes import byref
+from dataclasses import dataclass
+from typing import List, Optional, Tuple
+
+import torch
+
+from . import _lib
+from .kernels import _check, _code, _count, _ptr, _require_cuda, _stream, runtime
+
+GATES = {"silu": _lib.GATE_SILU, "sigmoid": _lib.GATE_SIGMOID}
+
+
+def pad8(extent: int) -> int:
+    """Row strides and GEMM extents of 16-bit operands are multiples of 8 elements (16 bytes)."""
+
+    return (extent + 7) // 8 * 8
+
+
+@dataclass
+class SequenceBatch:
+    """The rows of a step as sequences: `rows` tokens of `sequences` sequences, and the four device
+    vectors of the header's description. `counts` / `bases_host` are the host's copy of the portion
+    lengths and first positions (None inside a captured decode step, where every count is 1)."""
+
+    rows: int
+    sequences: int
+    token_sequence: torch.Tensor
+    starts: torch.Tensor
+    slots: torch.Tensor
+    bases: torch.Tensor
+    counts: Optional[List[int]] = None
+    bases_host: Optional[List[int]] = None
+    slots_host: Optional[List[int]] = None
+
+    @property
+    def decode(self) -> bool:
+        return self.counts is None or max(self.counts) == 1
+
+    def pointers(self) -> Tuple[int, int, int, int]:
+        return (self.token_sequence.data_ptr(), self.starts.data_ptr(), self.slots.data_ptr(),
+                self.bases.data_ptr())
+
+
+def _require_rows(tensor: torch.Tensor, what: str) -> None:
+    if tensor.ndim != 2 or tensor.stride(1) != 1:
+        raise ValueError(f"{what} must be a matrix with contiguous rows")
+
+
+def residual_norm(x: torch.Tensor, y: Optional[torch.Tensor], post_weight: Optional[torch.Tensor],
+                  next_weight: Optional[torch.Tensor], *, epsilon: float, weight_offset: float,
+                  dtype: torch.dtype) -> Optional[torch.Tensor]:
+    """x += norm(y) * (weight_offset + post_weight) in place on the fp32 residual x [rows, width], then
+    h = norm(x) * (weight_offset + next_weight), returned in `dtype` with rows padded to 8 elements.
+    y: [rows, >= width] in `dtype`, or fp32 split-K partials [splits, rows, >= width]; None: h only."""
+
+    device = _require_cuda(x, y, post_weight, next_weight)
+    if x.ndim != 2 or x.dtype != torch.float32 or not x.is_contiguous():
+        raise ValueError("the residual is a contiguous fp32 matrix")
+    rows, width = x.shape
+    splits = y_stride = 0
+    if y is not None:
+        if y.ndim == 3:
+            if y.dtype != torch.float32 or not y.is_contiguous() or y.shape[1] != rows:
+                raise ValueError("partial sums must be a contiguous fp32 [splits, rows, columns] tensor")
+            splits, y_stride = y.shape[0], y.shape[2]
+        else:
+            _require_rows(y, "the sublayer's result")
+            if y.dtype != dtype or y.shape[0] != rows:
+                raise ValueError("the sublayer's result does not match the residual")
+            y_stride = y.stride(0)
+        if y.shape[-1] < width or post_weight is None or post_weight.shape != (width,) or \
+                post_weight.dtype != dtype:
+            raise ValueError("the norm behind a sublayer needs a weight and a result of the residual's width")
+    h = None
+    if next_weight is not None:
+        if next_weight.shape != (width,) or next_weight.dtype != dtype:
+            raise ValueError("the norm weight must be a vector of the residual's width")
+        h = torch.empty((rows, pad8(width)), dtype=dtype, device=device)
+    rt = runtime(device)
+    code = _lib.load().b200_residual_norm(
+        x.data_ptr(), _ptr(y), _ptr(post_weight), _ptr(next_weight), _ptr(h), rows, width, splits, y_stride,
+        pad8(width), float(epsilon), float(weight_offset), _code(dtype), _stream())
+    _check(code, "b200_residual_norm")
+    _count(rt)
+    return h
+
+
+def latent_norm(projected: torch.Tensor, q_weight: torch.Tensor, kv_weight: Optional[torch.Tensor],
+                cache: Optional[torch.Tensor], batch: SequenceBatch, *, kv_column: int, epsilon: float,
+                dense: bool = False) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
+    """RMS norms of the query latent (column 0 of `projected`) and, with kv_weight, of the kv latent
+    (from kv_column), which is stored in the cache [slots, capacity, row] at the tokens' positions.
+    Returns the query latent (rows padded to 8 elements) and, with dense, the kv latents [rows, row]."""
+
+    device = _require_cuda(projected, q_weight, kv_weight, cache)
+    _require_rows(projected, "the projection")
+    q_rank = q_weight.shape[0]
+    rows = projected.shape[0]
+    if projected.dtype != q_weight.dtype or (kv_weight is not None and (
+            cache is None or cache.dtype != projected.dtype or not cache.is_contiguous())):
+        raise ValueError("projection, weights and cache must share one dtype")
+    q_out = torch.empty((rows, pad8(q_rank)), dtype=projected.dtype, device=device)
+    kv_rank = kv_weight.shape[0] if kv_weight is not None else 0
+    row = cache.shape[2] if kv_weight is not None else 0
+    dense_out = torch.empty((rows, row), dtype=projected.dtype, device=device) \
+        if dense and kv_weight is not None else None
+    rt = runtime(device)
+    code = _lib.load().b200_latent_norm(
+        projected.data_ptr(), q_weight.data_ptr(), _ptr(kv_weight), q_out.data_ptr(),
+        _ptr(cache) if kv_weight is not None else None, _ptr(dense_out), *batch.pointers(), rows, q_rank, kv_rank,
+        kv_column, row, projected.stride(0), q_out.stride(0), cache.shape[1] if kv_weight is not None else 0,
+        float(epsilon), _code(projected.dtype), rt.status.data_ptr(), _stream())
+    _check(code, "b200_latent_norm")
+    _count(rt)
+    return q_out, dense_out
+
+
+def gated_head_norm(read_out: torch.Tensor, weight: Optional[torch.Tensor], gate: torch.Tensor, *, kind: str,
+                    epsilon: float) -> torch.Tensor:
+    """Per-head RMS norm of a read-out (fp32 [rows, heads, vdim]) times `weight` and silu or sigmoid of
+    `gate` [rows, >= heads * vdim]; rows of the result are padded to 8 elements."""
+
+    device = _require_cuda(read_out, weight, gate)
+    rows, heads, vdim = read_out.shape
+    _require_rows(gate, "the gate")
+    if read_out.dtype != torch.float32 or not read_out.is_contiguous() or gate.shape[0] != rows:
+        raise ValueError("the read-out must be contiguous fp32 and match the gate")
+    output = torch.empty((rows, pad8(heads * vdim)), dtype=gate.dtype, device=device)
+    rt = runtime(device)
+    code = _lib.load().b200_gated_head_norm(
+        read_out.data_ptr(), _ptr(weight), gate.data_ptr(), output.data_ptr(), rows, heads, vdim, gate.stride(0),
+        output.stride(0), GATES[kind], float(epsilon), _code(gate.dtype), _stream())
+    _check(code, "b200_gated_head_norm")
+    _count(rt)
+    return output
+
+
+def retention_prep(projected: torch.Tensor, batch: SequenceBatch, *, heads: int, dim: int, vdim: int,
+                   columns: Tuple[int, int, int], rot_dims: int, rot_base: float, k_scale: float):
+    """fp32 operands q, k [rows, heads, dim] (rotated, k scaled) and v [rows, heads, vdim] of a
+    retention layer from the columns (q, k, v) of its projection."""
+
+    device = _require_cuda(projected)
+    _require_rows(projected, "the projection")
+    rows = projected.shape[0]
+    q = torch.empty((rows, heads, dim), dtype=torch.float32, device=device)
+    k = torch.empty_like(q)
+    v = torch.empty((rows, heads, vdim), dtype=torch.float32, device=device)
+    rt = runtime(device)
+    code = _lib.load().b200_retention_prep(
+        projected.data_ptr(), *batch.pointers(), q.data_ptr(), k.data_ptr(), v.data_ptr(), rows, heads, dim, vdim,
+        *columns, projected.stride(0), rot_dims, float(rot_base), float(k_scale), _code(projected.dtype),
+        _stream())
+    _check(code, "b200_retention_prep")
+    _count(rt)
+    return q, k, v
+
+
+def delta_inputs(projected: torch.Tensor, gates: torch.Tensor, conv: Tuple[torch.Tensor, torch.Tensor, torch.Tensor],
+                 a_log: torch.Tensor, dt_bias: torch.Tensor, ring: torch.Tensor, batch: SequenceBatch, *,
+                 heads: int, kv_heads: int, dim: int, vdim: int, columns: Tuple[int, int, int, int],
+                 decay_column: int, q_scale: float) -> "_lib.DeltaInputs":
+    """The argument block of the gated delta rule's kernels: projections (columns of q, k, v and beta),
+    decay projections, convolution taps, and the ring of earlier inputs [slots, taps, channels]."""
+
+    _require_cuda(projected, gates, *conv, a_log, dt_bias, ring)
+    _require_rows(projected, "the projection")
+    _require_rows(gates, "the gate projection")
+    taps = conv[0].shape[1]
+    if ring.shape[1:] != (taps, 2 * kv_heads * dim + heads * vdim) or not ring.is_contiguous():
+        raise ValueError("the ring must hold `taps` inputs of every channel")
+    if len({t.dtype for t in (projected, gates, *conv, a_log, dt_bias, ring)}) != 1:
+        raise ValueError("projections, weights and ring must share one dtype")
+    return _lib.DeltaInputs(
+        projected.data_ptr(), gates.data_ptr(), conv[0].data_ptr(), conv[1].data_ptr(), conv[2].data_ptr(),
+        a_log.data_ptr(), dt_bias.data_ptr(), ring.data_ptr(), *batch.pointers(), heads, kv_heads, dim, vdim, taps,
+        *columns, decay_column, projected.stride(0), gates.stride(0), float(q_scale))
+
+
+def delta_prep(inputs: "_lib.DeltaInputs", rows: int, dtype: torch.dtype, device: torch.device):
+    """fp32 operands of the gated delta rule: q, k [rows, kv_heads, dim], v [rows, heads, vdim],
+    beta [rows, heads] and log g [rows, heads, dim]."""
+
+    q = torch.empty((rows, inputs.kv_heads, inputs.dim), dtype=torch.float32, device=device)
+    k = torch.empty_like(q)
+    v = torch.empty((rows, inputs.heads, inputs.vdim), dtype=torch.float32, device=device)
+    beta = torch.empty((rows, inputs.heads), dtype=torch.float32, device=device)
+    decay = torch.empty((rows, inputs.heads, inputs.dim), dtype=torch.float32, device=device)
+    rt = runtime(device)
+    code = _lib.load().b200_delta_prep(byref(inputs), q.data_ptr(), k.data_ptr(), v.data_ptr(), beta.data_ptr(),
+                                       decay.data_ptr(), rows, _code(dtype), _stream())
+    _check(code, "b200_delta_prep")
+    _count(rt)
+    return q, k, v, beta, decay
+
+
+def conv_tail(inputs: "_lib.DeltaInputs", sequences: int, dtype: torch.dtype, device: torch.device) -> None:
+    """Keeps every sequence's last inputs for the short convolution of its next portion."""
+
+    rt = runtime(device)
+    _check(_lib.load().b200_conv_tail(byref(inputs), sequences, _code(dtype), _stream()), "b200_conv_tail")
+    _count(rt)
+
+
+def recurrence_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta: Optional[torch.Tensor],
+                    decay: torch.Tensor, state: torch.Tensor, batch: SequenceBatch) -> torch.Tensor:
+    """Token by token recurrence over prepared fp32 operands; state [slots, heads, dim, row] is updated
+    in place. beta None: retention with `decay` [heads]; else the delta rule, `decay` is log g
+    [rows, heads, dim]. Returns the read-out [rows, heads, vdim]."""
+
+    device = _require_cuda(q, k, v, beta, decay, state)
+    rows, kv_heads, dim = q.shape
+    heads, vdim = v.shape[1], v.shape[2]
+    if state.dtype != torch.float32 or state.ndim != 4 or not state.is_contiguous() or \
+            state.shape[1] != heads or state.shape[2] != dim or state.shape[3] < vdim:
+        raise ValueError("the state must be contiguous fp32 [slots, heads, dim, >= vdim]")
+    output = torch.empty((rows, heads, vdim), dtype=torch.float32, device=device)
+    rt = runtime(device)
+    code = _lib.load().b200_recurrence_scan(
+        q.data_ptr(), k.data_ptr(), v.data_ptr(), _ptr(beta), decay.data_ptr(), state.data_ptr(), output.data_ptr(),
+        *batch.pointers(), batch.sequences, heads, kv_heads, dim, vdim, state.shape[3], _stream())
+    _check(code, "b200_recurrence_scan")
+    _count(rt)
+    return output
+
+
+def head_linear(x: torch.Tensor, weight: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """y[m, h, :] = weight[h] x[m, h, :]: x [rows, heads, k] (last dimension contiguous), weight
+    [heads, n, k]. `out` may be a [rows, heads, n] view of a wider matrix."""
+
+    device = _require_cuda(x, weight, out)
+    rows, heads, k = x.shape
+    if weight.ndim != 3 or weight.shape[0] != heads or weight.shape[2] != k or not weight.is_contiguous() or \
+            weight.dtype != x.dtype or x.stride(2) != 1:
+        raise ValueError("head_linear needs x [rows, heads, k] and a contiguous weight [heads, n, k]")
+    n = weight.shape[1]
+    if out is None:
+        out = torch.empty((rows, heads, n), dtype=x.dtype, device=device)
+    rt = runtime(device)
+    code = _lib.load().b200_head_linear(x.data_ptr(), weight.data_ptr(), out.data_ptr(), rows, heads, k, n,
+                                        x.stride(0), x.stride(1), out.stride(0), out.stride(1), _code(x.dtype),
+                                        _stream())
+    _check(code, "b200_head_linear")
+    _count(rt)
+    return out
+
+
+def latent_attention(q: torch.Tensor, cache: torch.Tensor, sink: Optional[torch.Tensor], batch: SequenceBatch, *,
+                     scale: float) -> torch.Tensor:
+    """Attention of queries in the latent space [rows, heads, row] over the cached latents [slots,
+    capacity, row] of their sequences; returns the weighted latents [rows, heads, row]."""
+
+    device = _require_cuda(q, cache, sink)
+    rows, heads, row = q.shape
+    if not q.is_contiguous() or not cache.is_contiguous() or cache.shape[2] != row or cache.dtype != q.dtype:
+        raise ValueError("queries and cached latents must be contiguous and of one row size and dtype")
+    output = torch.empty_like(q)
+    rt = runtime(device)
+    code = _lib.load().b200_latent_attention(
+        q.data_ptr(), cache.data_ptr(), _ptr(sink), output.data_ptr(), *batch.pointers(), rows, heads, row,
+        cache.shape[1], float(scale), _code(q.dtype), _stream())
+    _check(code, "b200_latent_attention")
+    _count(rt)
+    return output
+
+
+def sequence_positions(lengths: torch.Tensor, slots: torch.Tensor, positions: torch.Tensor) -> None:
+    """positions[r] = lengths[slots[r]], 0 for an idle row."""
+
+    device = _require_cuda(lengths, slots, positions)
+    rt = runtime(device)
+    _check(_lib.load().b200_sequence_positions(lengths.data_ptr(), slots.data_ptr(), positions.data_ptr(),
+                                               slots.shape[0], _stream()), "b200_sequence_positions")
+    _count(rt)
+
+
+def advance_slots(lengths: torch.Tensor, batch: SequenceBatch, capacity: int) -> None:
+    """lengths[slot] += the step's tokens of that slot, clamped at `capacity` with a status bit."""
+
+    device = _require_cuda(lengths)
+    rt = runtime(device)
+    _check(_lib.load().b200_advance_slots(lengths.data_ptr(), batch.slots.data_ptr(), batch.starts.data_ptr(),
+                                          batch.sequences, capacity, rt.status.data_ptr(), _stream()),
+           "b200_advance_slots")
+    _count(rt)

@@ -876,9 +876,15 @@ def b200_linear(tensor: torch.Tensor, weight: torch.Tensor,
     if epilogue not in _EPILOGUES:
         raise ValueError(f"unknown epilogue {epilogue!r}")
     weight = _dense(weight)
-    source = _dense(tensor) if tensor.ndim <= 4 else tensor
-    if not source.is_contiguous():
-        raise ValueError("inputs of rank > 4 must be contiguous")
+    row_stride = k
+    if tensor.ndim == 2 and tensor.stride(1) == 1 and tensor.stride(0) >= k and (
+            tensor.dtype != torch.bfloat16 or
+            (tensor.stride(0) % 8 == 0 and tensor.data_ptr() % 16 == 0)):
+        source, row_stride = tensor, tensor.stride(0)  # a column slice of a wider matrix
+    else:
+        source = _dense(tensor) if tensor.ndim <= 4 else tensor
+        if not source.is_contiguous():
+            raise ValueError("inputs of rank > 4 must be contiguous")
     m = source.numel() // k
     out_features = n // 2 if epilogue == "swiglu" else n
     output = torch.empty((*tensor.shape[:-1], out_features), dtype=tensor.dtype, device=device)
@@ -896,8 +902,8 @@ def b200_linear(tensor: torch.Tensor, weight: torch.Tensor,
     need = int(library.b200_linear_workspace_bytes(m, k, n, code_dtype, _EPILOGUES[epilogue]))
     workspace = rt.workspace("linear", need)
     code = library.b200_linear(source.data_ptr(), weight.data_ptr(), _ptr(bias), _ptr(residual),
-                               output.data_ptr(), m, k, n, k, code_dtype, _EPILOGUES[epilogue],
-                               _ptr(workspace), need, rt.status.data_ptr(), _stream())
+                               output.data_ptr(), m, k, n, row_stride, code_dtype,
+                               _EPILOGUES[epilogue], _ptr(workspace), need, rt.status.data_ptr(), _stream())
     _check(code, "b200_linear")
     _count(rt)
     return output

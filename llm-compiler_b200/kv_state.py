@@ -16,6 +16,7 @@ by CUDA-graph replay over fixed addresses:
 
 from __future__ import annotations
 
+import bisect
 from dataclasses import dataclass
 from typing import Callable, Optional, Sequence, Tuple
 
@@ -351,3 +352,68 @@ class PagedKVCacheState(PreallocatedKVCacheState):
         run = runner or kernels.b200_paged_decode_attention
         return run(query, pool_key, pool_value, self.block_table, lengths, attention_mask, scale=scale,
                    **options)
+
+
+class SlotState:
+    """State of sequences that come and go: `slots` places, each holding one sequence's part of every
+    layer's state tensors (`layers[i][name]`, the slot is the first dimension), an int64 length per
+    slot, and a free list. What a layer keeps is the layer's own business (cached rows of a fixed
+    capacity, a recurrent matrix state, the last inputs of a convolution): `specs[i]` maps a name to
+    (shape of one slot, dtype). A slot that is given back is not cleared; a sequence that starts at
+    position 0 reads nothing of what the slot held before (the kernels' contract)."""
+
+    def __init__(self, specs: Sequence[dict], *, slots: int, capacity: int,
+                 device: torch.device | str) -> None:
+        if slots <= 0 or capacity <= 0:
+            raise ExecutionError("state needs a positive slot count and capacity")
+        self.slots, self.capacity = slots, capacity
+        self.layers = [{name: torch.zeros((slots, *shape), dtype=dtype, device=device)
+                        for name, (shape, dtype) in spec.items()} for spec in specs]
+        self.lengths = torch.zeros(slots, dtype=torch.int64, device=device)
+        self.host_lengths = [0] * slots
+        self._free = list(range(slots))  # lowest first
+        self._device = torch.device(device)
+
+    def acquire(self) -> int:
+        if not self._free:
+            raise ExecutionError("every state slot is in use")
+        slot = self._free.pop(0)
+        self._reset(slot)
+        return slot
+
+    def release(self, slot: int) -> None:
+        if not 0 <= slot < self.slots or slot in self._free:
+            raise ExecutionError(f"slot {slot} is not in use")
+        bisect.insort(self._free, slot)
+        self._reset(slot)
+
+    def reset_all(self) -> None:
+        """Every slot in use by one sequence each, all empty: the fixed batch of an engine's own
+        prefill."""
+
+        self._free = []
+        self.host_lengths = [0] * self.slots
+        self.lengths.zero_()
+
+    def _reset(self, slot: int) -> None:
+        self.host_lengths[slot] = 0
+        self.lengths[slot] = 0
+
+    def require(self, slot: int, tokens: int) -> None:
+        if self.host_lengths[slot] + tokens > self.capacity:
+            raise ExecutionError(f"{self.host_lengths[slot]} + {tokens} tokens exceed the slot capacity "
+                                 f"{self.capacity}")
+
+    def slots_in_use(self) -> int:
+        return self.slots - len(self._free)
+
+    def bytes(self) -> int:
+        return sum(t.numel() * t.element_size() for layer in self.layers for t in layer.values())
+
+    def check(self) -> None:
+        """Step-boundary host check of the device status word; raises ExecutionError."""
+
+        try:
+            kernels.runtime(self._device).check_status()
+        except kernels.KernelStatusError as error:
+            raise ExecutionError(str(error)) from error

@@ -1,0 +1,209 @@
+"""Sequence mixers of hybrid decoder layers on the sm_100a kernels: retention, latent attention and the
+gated delta rule with a decay per key channel. Each takes its sizes and constants from a spec, packs its
+weights once, says what state a sequence keeps, and maps normed rows h to the sublayer's result for any
+mix of portions and decoded tokens.
+
+Packing: all projections of h are one stacked matrix; every operand starts at a multiple of 8 columns,
+and extents are padded with zero rows / columns to multiples of 8, so that the 16-bit GEMMs take any size.
+"""
+
+from __future__ import annotations
+
+from typing import Dict, List, Optional, Sequence, Tuple
+
+import torch
+
+from . import hybrid_kernels as hk
+from . import kernels
+from .hybrid_kernels import SequenceBatch, pad8
+
+PARTIAL_ROWS = 128  # rows up to which a projection in front of a residual leaves split-K partials
+
+
+def pad_matrix(weight: torch.Tensor, rows: int, columns: int) -> torch.Tensor:
+    """`weight` in the top left corner of a zero matrix."""
+
+    if tuple(weight.shape) == (rows, columns):
+        return weight.contiguous()
+    padded = torch.zeros((rows, columns), dtype=weight.dtype, device=weight.device)
+    padded[:weight.shape[0], :weight.shape[1]].copy_(weight)
+    return padded
+
+
+def stack_projections(weights: Sequence[torch.Tensor], columns: int) -> Tuple[torch.Tensor, List[int]]:
+    """One [sum of padded rows, columns] matrix and the first output column of every part."""
+
+    offsets, total = [], 0
+    for weight in weights:
+        offsets.append(total)
+        total += pad8(weight.shape[0])
+    stacked = torch.zeros((total, columns), dtype=weights[0].dtype, device=weights[0].device)
+    for offset, weight in zip(offsets, weights):
+        stacked[offset:offset + weight.shape[0], :weight.shape[1]].copy_(weight)
+    return stacked, offsets
+
+
+def block_diagonal(parts: Sequence[Tuple[torch.Tensor, int]], columns: int) -> Tuple[torch.Tensor, List[int]]:
+    """Projections of neighbouring column ranges of one matrix as one GEMM: parts are (weight, first
+    input column); returns the matrix and the first output column of every part."""
+
+    stacked, offsets = stack_projections([torch.zeros((w.shape[0], 1), dtype=w.dtype, device=w.device)
+                                          for w, _ in parts], columns)
+    for offset, (weight, first) in zip(offsets, parts):
+        stacked[offset:offset + weight.shape[0], first:first + weight.shape[1]].copy_(weight)
+    return stacked, offsets
+
+
+def pad_heads(weight: torch.Tensor, heads: int, size: int) -> torch.Tensor:
+    """[heads * d, k] -> [heads * size, k] with zero rows behind every head's d."""
+
+    d = weight.shape[0] // heads
+    if d == size:
+        return weight
+    padded = torch.zeros((heads, size, weight.shape[1]), dtype=weight.dtype, device=weight.device)
+    padded[:, :d].copy_(weight.view(heads, d, -1))
+    return padded.view(heads * size, -1)
+
+
+def project_out(rows: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
+    """A projection whose consumer is residual_norm: fp32 split-K partials at decode sizes (the
+    consumer adds them), else the rounded result."""
+
+    if rows.dtype == torch.bfloat16 and rows.shape[0] <= PARTIAL_ROWS:
+        return kernels.b200_linear_partial(rows, weight)
+    return kernels.b200_linear(rows, weight)
+
+
+class Mixer:
+    """One layer's mixer. `state_spec` is what a slot keeps; `shared_state` names the layer whose state
+    this one reads instead of keeping its own."""
+
+    shared_state: Optional[int] = None
+
+    def state_spec(self, capacity: int) -> Dict[str, tuple]:
+        return {}
+
+    def __call__(self, h: torch.Tensor, batch: SequenceBatch, state: Dict[str, torch.Tensor]) -> torch.Tensor:
+        raise NotImplementedError
+
+
+class Retention(Mixer):
+    """q, k, v and a silu gate; S <- decay_h S + k v^T, o = S^T q, read-out normed per head."""
+
+    def __init__(self, weights: Dict[str, torch.Tensor], *, width: int, heads: int, dim: int, vdim: int,
+                 decay: Sequence[float], rot_dims: int, rot_base: float, epsilon: float) -> None:
+        self.heads, self.dim, self.vdim = heads, dim, vdim
+        self.rot_dims, self.rot_base, self.epsilon = rot_dims, rot_base, epsilon
+        self.w_in, (q, k, v, self.gate_column) = stack_projections(
+            [weights[name] for name in ("q", "k", "v", "g")], pad8(width))
+        self.columns = (q, k, v)
+        self.w_out = pad_matrix(weights["o"], pad8(width), pad8(heads * vdim))
+        self.decay = torch.tensor(list(decay), dtype=torch.float32, device=self.w_in.device)
+        self.k_scale = dim ** -0.5
+
+    def state_spec(self, capacity):
+        return {"state": ((self.heads, self.dim, (self.vdim + 3) // 4 * 4), torch.float32)}
+
+    def __call__(self, h, batch, state):
+        projected = kernels.b200_linear(h, self.w_in)
+        q, k, v = hk.retention_prep(projected, batch, heads=self.heads, dim=self.dim, vdim=self.vdim,
+                                    columns=self.columns, rot_dims=self.rot_dims, rot_base=self.rot_base,
+                                    k_scale=self.k_scale)
+        read_out = hk.recurrence_scan(q, k, v, None, self.decay, state["state"], batch)
+        mixed = hk.gated_head_norm(read_out, None, projected[:, self.gate_column:], kind="silu",
+                                   epsilon=self.epsilon)
+        return project_out(mixed, self.w_out)
+
+
+class ChannelDelta(Mixer):
+    """Gated delta rule: short convolutions on q, k, v, unit q and k, one decay per head and key
+    channel, a sigmoid gate on the normed read-out."""
+
+    def __init__(self, weights: Dict[str, torch.Tensor], *, width: int, heads: int, kv_heads: int, dim: int,
+                 vdim: int, epsilon: float) -> None:
+        self.heads, self.kv_heads, self.dim, self.vdim, self.epsilon = heads, kv_heads, dim, vdim, epsilon
+        self.w_in, offsets = stack_projections(
+            [weights[name] for name in ("q", "k", "v", "b", "a1", "g1")], pad8(width))
+        self.columns = tuple(offsets[:4])
+        self.low_column = offsets[4]  # a1 and g1 side by side: the input of the two up projections
+        low = self.w_in.shape[0] - self.low_column
+        self.w_gates, (self.decay_column, self.gate_column) = block_diagonal(
+            [(weights["a2"], 0), (weights["g2"], offsets[5] - offsets[4])], low)
+        self.w_out = pad_matrix(weights["o"], pad8(width), pad8(heads * vdim))
+        self.conv = tuple(weights[name].contiguous() for name in ("q.conv", "k.conv", "v.conv"))
+        self.a_log, self.dt_bias, self.norm = weights["A_log"], weights["dt_bias"], weights["norm"]
+        self.taps = self.conv[0].shape[1]
+        self.q_scale = dim ** -0.5
+
+    def state_spec(self, capacity):
+        return {"state": ((self.heads, self.dim, (self.vdim + 3) // 4 * 4), torch.float32),
+                "ring": ((self.taps, 2 * self.kv_heads * self.dim + self.heads * self.vdim), self.w_in.dtype)}
+
+    def __call__(self, h, batch, state):
+        projected = kernels.b200_linear(h, self.w_in)
+        gates = kernels.b200_linear(projected[:, self.low_column:], self.w_gates)
+        inputs = hk.delta_inputs(projected, gates, self.conv, self.a_log, self.dt_bias, state["ring"], batch,
+                                 heads=self.heads, kv_heads=self.kv_heads, dim=self.dim, vdim=self.vdim,
+                                 columns=self.columns, decay_column=self.decay_column, q_scale=self.q_scale)
+        q, k, v, beta, log_decay = hk.delta_prep(inputs, h.shape[0], h.dtype, h.device)
+        read_out = hk.recurrence_scan(q, k, v, beta, log_decay, state["state"], batch)
+        hk.conv_tail(inputs, batch.sequences, h.dtype, h.device)
+        mixed = hk.gated_head_norm(read_out, self.norm, gates[:, self.gate_column:], kind="sigmoid",
+                                   epsilon=self.epsilon)
+        return project_out(mixed, self.w_out)
+
+
+class LatentAttention(Mixer):
+    """Attention without positions over one cached latent per token; `kv_from` reads the latents that
+    an earlier layer keeps."""
+
+    def __init__(self, weights: Dict[str, torch.Tensor], *, width: int, heads: int, dim: int, vdim: int,
+                 q_rank: int, kv_rank: int, scale: float, epsilon: float, kv_from: Optional[int] = None) -> None:
+        self.heads, self.dim, self.vdim, self.scale, self.epsilon = heads, dim, vdim, scale, epsilon
+        self.q_rank, self.kv_rank, self.shared_state = q_rank, kv_rank, kv_from
+        self.rank_row = (kv_rank + 15) // 16 * 16
+        down = [weights["dq"]] + ([weights["dkv"]] if kv_from is None else [])
+        self.w_down, offsets = stack_projections(down, pad8(width))
+        self.kv_column = offsets[-1]
+        self.q_norm = weights["dq.norm"]
+        self.kv_norm = weights["dkv.norm"] if kv_from is None else None
+        self.sink = weights["sink"].contiguous()
+        self.q_size, self.v_size = pad8(dim), pad8(vdim)
+        self.w_q = pad_matrix(pad_heads(weights["uq"], heads, self.q_size), heads * self.q_size, pad8(q_rank))
+        key = pad_heads(pad_matrix(weights["uk"], heads * dim, self.rank_row), heads, self.q_size)
+        value = pad_heads(pad_matrix(weights["uv"], heads * vdim, self.rank_row), heads, self.v_size)
+        self.w_into = key.view(heads, self.q_size, self.rank_row).transpose(1, 2).contiguous()
+        self.w_from = value.view(heads, self.v_size, self.rank_row).contiguous()
+        out = pad_heads(weights["o"].t().contiguous(), heads, self.v_size).t()
+        self.w_out = pad_matrix(out, pad8(width), heads * self.v_size)
+        self.w_out = self.w_out.contiguous()
+
+    def state_spec(self, capacity):
+        if self.shared_state is not None:
+            return {}
+        return {"latent": ((capacity, self.rank_row), self.w_down.dtype)}
+
+    def __call__(self, h, batch, state):
+        down = kernels.b200_linear(h, self.w_down)
+        cache = state["latent"]
+        query_latent, _ = hk.latent_norm(down, self.q_norm, self.kv_norm, cache, batch, kv_column=self.kv_column,
+                                         epsilon=self.epsilon)
+        rows = h.shape[0]
+        q = kernels.b200_linear(query_latent, self.w_q).view(rows, self.heads, self.q_size)
+        absorbed = hk.head_linear(q, self.w_into)
+        weighted = hk.latent_attention(absorbed, cache, self.sink, batch, scale=self.scale)
+        values = hk.head_linear(weighted, self.w_from)
+        return project_out(values.view(rows, self.heads * self.v_size), self.w_out)
+
+
+class GatedMlp:
+    """down(silu(gate h) * (up h)): the gate and up rows interleaved for the GEMM's SwiGLU epilogue."""
+
+    def __init__(self, weights: Dict[str, torch.Tensor], *, width: int) -> None:
+        ff = pad8(weights["gate"].shape[0])
+        self.w_in = kernels.interleave_gate_up(pad_matrix(weights["gate"], ff, pad8(width)),
+                                               pad_matrix(weights["up"], ff, pad8(width)))
+        self.w_out = pad_matrix(weights["down"], pad8(width), ff)
+
+    def __call__(self, h: torch.Tensor) -> torch.Tensor:
+        return project_out(kernels.b200_linear(h, self.w_in, epilogue="swiglu"), self.w_out)

@@ -142,3 +142,34 @@ def make_prompt_ids(config: Qwen2Config, batch: int, tokens: int, *, seed: int =
     generator = torch.Generator(device="cpu").manual_seed(seed)
     return torch.randint(0, config.vocab_size, (batch, tokens), generator=generator,
                          dtype=torch.int64)
+
+
+def config_from_dict(data: dict) -> Qwen2Config:
+    """Qwen2Config of a checkpoint's config.json."""
+
+    return Qwen2Config(
+        hidden_size=data["hidden_size"], intermediate_size=data["intermediate_size"],
+        num_layers=data["num_hidden_layers"], num_heads=data["num_attention_heads"],
+        num_kv_heads=data.get("num_key_value_heads", data["num_attention_heads"]),
+        rms_norm_eps=data.get("rms_norm_eps", 1e-6), rope_theta=float(data.get("rope_theta", 10000.0)),
+        max_position_embeddings=data.get("max_position_embeddings", 32768), vocab_size=data["vocab_size"],
+        tie_word_embeddings=data.get("tie_word_embeddings", False), head_dim_override=data.get("head_dim", 0))
+
+
+def weights_from_checkpoint(config: Qwen2Config, stored: Dict[str, torch.Tensor]) -> Dict[str, torch.Tensor]:
+    """Checkpoint names (model.embed_tokens.weight, model.layers.0. ..., model.norm.weight) to the names
+    of parameter_shapes; names that are already those pass unchanged."""
+
+    weights: Dict[str, torch.Tensor] = {}
+    for name, tensor in stored.items():
+        if name.startswith("model."):
+            name = name[len("model."):]
+            if name.startswith(("layers.", "norm.")):
+                name = "decoder." + name
+        weights[name] = tensor
+    if config.tie_word_embeddings:
+        weights["lm_head.weight"] = weights["embed_tokens.weight"]
+    for name, shape in parameter_shapes(config):
+        if name not in weights or tuple(weights[name].shape) != shape:
+            raise ValueError(f"tensor {name} of shape {shape} is missing")
+    return weights
