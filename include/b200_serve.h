@@ -470,10 +470,18 @@ int b200_argmax(const void* logits, int64_t* ids, int64_t rows, int64_t vocab,
  *   b200_recurrence_scan token by token recurrence on prepared operands. beta NULL: retention, decay
  *                        is [heads]; otherwise the delta rule, decay is log g [rows, heads, dim]. State
  *                        [slots, heads, dim, state_row] is read, and written behind the last token.
+ *   b200_retention_step, b200_delta_step  a decode step (one row per sequence) in one launch: operands,
+ *                        state update, read-out, norm and gate; the convolution inputs are kept too. With
+ *                        B200_LAUNCH_STABLE_KV_PREFIX the state is read before the dependency wait (no
+ *                        kernel since the last serialised launch writes it). B200_ERR_UNSUPPORTED for
+ *                        states beyond 128 KB per head.
  *   b200_head_linear     y[m, h, :] = w[h] x[m, h, :], w [heads, n, k]
  *   b200_latent_attention  q, out [rows, heads, rank_row] in the latent space, cache [slots, capacity,
  *                        rank_row]; a row sees the positions up to its own; with sink (model dtype
- *                        [heads]) the softmax denominator of head h also holds exp(sink[h])
+ *                        [heads]) the softmax denominator of head h also holds exp(sink[h]). longest:
+ *                        most rows of one sequence; context: an upper bound of the keys (they choose the
+ *                        row tile and the split count; every sequence's keys are then shared out among the
+ *                        splits on the device)
  *   b200_sequence_positions  positions[r] = lengths[slots[r]] (0 for an idle row)
  *   b200_advance_slots   lengths[slots[r]] += starts[r + 1] - starts[r], clamped with a status bit */
 #define B200_GATE_SILU 0
@@ -496,6 +504,25 @@ typedef struct b200_delta_inputs {
   int64_t row_stride, gate_row_stride;
   double q_scale;
 } b200_delta_inputs;
+typedef struct b200_retention_inputs {
+  const void* input;  /* [rows, row_stride]: projections of h */
+  const float* decay; /* [heads] (may be NULL for b200_retention_prep) */
+  const int32_t* token_sequence;
+  const int32_t* starts;
+  const int32_t* slots;
+  const int32_t* bases;
+  int64_t heads, dim, vdim, q_column, k_column, v_column, row_stride, rot_dims;
+  double rot_base, k_scale;
+} b200_retention_inputs;
+typedef struct b200_step_output {
+  float* state;        /* [slots, heads, dim, state_row], state_row a multiple of 4 */
+  const void* gate;    /* [rows, gate_row_stride], head-major */
+  const void* weight;  /* [vdim] or NULL */
+  void* output;        /* [rows, output_row_stride], zeros behind heads * vdim */
+  int64_t state_row, gate_row_stride, output_row_stride;
+  int64_t gate_kind;
+  double epsilon;
+} b200_step_output;
 int b200_residual_norm(void* x, const void* y, const void* post_weight, const void* next_weight, void* h,
                        int64_t rows, int64_t width, int64_t splits, int64_t y_row_stride,
                        int64_t h_row_stride, double epsilon, double weight_offset, int dtype, void* stream);
@@ -508,11 +535,12 @@ int b200_latent_norm(const void* input, const void* q_weight, const void* kv_wei
 int b200_gated_head_norm(const void* input, const void* weight, const void* gate, void* output, int64_t rows,
                          int64_t heads, int64_t vdim, int64_t gate_row_stride, int64_t output_row_stride,
                          int gate_kind, double epsilon, int dtype, void* stream);
-int b200_retention_prep(const void* input, const int32_t* token_sequence, const int32_t* starts,
-                        const int32_t* slots, const int32_t* bases, float* q, float* k, float* v,
-                        int64_t rows, int64_t heads, int64_t dim, int64_t vdim, int64_t q_column,
-                        int64_t k_column, int64_t v_column, int64_t row_stride, int64_t rot_dims,
-                        double rot_base, double k_scale, int dtype, void* stream);
+int b200_retention_prep(const b200_retention_inputs* inputs, float* q, float* k, float* v, int64_t rows,
+                        int dtype, void* stream);
+int b200_retention_step(const b200_retention_inputs* inputs, const b200_step_output* output,
+                        int64_t sequences, int dtype, void* stream);
+int b200_delta_step(const b200_delta_inputs* inputs, const b200_step_output* output, int64_t sequences,
+                    int dtype, void* stream);
 int b200_delta_prep(const b200_delta_inputs* inputs, float* q, float* k, float* v, float* beta,
                     float* log_decay, int64_t rows, int dtype, void* stream);
 int b200_conv_tail(const b200_delta_inputs* inputs, int64_t sequences, int dtype, void* stream);
@@ -523,10 +551,13 @@ int b200_recurrence_scan(const float* q, const float* k, const float* v, const f
 int b200_head_linear(const void* x, const void* w, void* y, int64_t m, int64_t heads, int64_t k, int64_t n,
                      int64_t x_row_stride, int64_t x_head_stride, int64_t y_row_stride,
                      int64_t y_head_stride, int dtype, void* stream);
+int64_t b200_latent_attention_workspace_bytes(int64_t rows, int64_t sequences, int64_t longest,
+                                              int64_t heads, int64_t rank_row, int64_t context, int dtype);
 int b200_latent_attention(const void* q, const void* cache, const void* sink, void* out,
                           const int32_t* token_sequence, const int32_t* starts, const int32_t* slots,
-                          const int32_t* bases, int64_t rows, int64_t heads, int64_t rank_row,
-                          int64_t capacity, double scale, int dtype, void* stream);
+                          const int32_t* bases, int64_t rows, int64_t sequences, int64_t longest,
+                          int64_t heads, int64_t rank_row, int64_t capacity, int64_t context, double scale,
+                          int dtype, void* workspace, int64_t workspace_bytes, void* stream);
 int b200_sequence_positions(const int64_t* lengths, const int32_t* slots, int32_t* positions, int64_t rows,
                             void* stream);
 int b200_advance_slots(int64_t* lengths, const int32_t* slots, const int32_t* starts, int64_t rows,

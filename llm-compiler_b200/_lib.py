@@ -56,7 +56,26 @@ class DeltaInputs(ctypes.Structure):
                [("q_scale", c_double)]
 
 
-_DELTA = POINTER(DeltaInputs)
+class RetentionInputs(ctypes.Structure):
+    """b200_retention_inputs of include/b200_serve.h."""
+
+    _fields_ = [(name, c_void_p) for name in
+                ("input", "decay", "token_sequence", "starts", "slots", "bases")] + \
+               [(name, c_int64) for name in
+                ("heads", "dim", "vdim", "q_column", "k_column", "v_column", "row_stride", "rot_dims")] + \
+               [("rot_base", c_double), ("k_scale", c_double)]
+
+
+class StepOutput(ctypes.Structure):
+    """b200_step_output of include/b200_serve.h."""
+
+    _fields_ = [(name, c_void_p) for name in ("state", "gate", "weight", "output")] + \
+               [(name, c_int64) for name in
+                ("state_row", "gate_row_stride", "output_row_stride", "gate_kind")] + \
+               [("epsilon", c_double)]
+
+
+_DELTA, _RETENTION, _STEP = POINTER(DeltaInputs), POINTER(RetentionInputs), POINTER(StepOutput)
 
 # What b200_abi_version() of a matching library returns (bumped with every signature change).
 ABI_VERSION = 105
@@ -134,12 +153,15 @@ SIGNATURES = {
     "b200_residual_norm": (c_int, [c_void_p] * 5 + [c_int64] * 5 + [c_double, c_double, c_int, c_void_p]),
     "b200_latent_norm": (c_int, [c_void_p] * 10 + [c_int64] * 8 + [c_double, c_int, c_void_p, c_void_p]),
     "b200_gated_head_norm": (c_int, [c_void_p] * 4 + [c_int64] * 5 + [c_int, c_double, c_int, c_void_p]),
-    "b200_retention_prep": (c_int, [c_void_p] * 8 + [c_int64] * 9 + [c_double, c_double, c_int, c_void_p]),
+    "b200_retention_prep": (c_int, [_RETENTION] + [c_void_p] * 3 + [c_int64, c_int, c_void_p]),
+    "b200_retention_step": (c_int, [_RETENTION, _STEP, c_int64, c_int, c_void_p]),
+    "b200_delta_step": (c_int, [_DELTA, _STEP, c_int64, c_int, c_void_p]),
     "b200_delta_prep": (c_int, [_DELTA] + [c_void_p] * 5 + [c_int64, c_int, c_void_p]),
     "b200_conv_tail": (c_int, [_DELTA, c_int64, c_int, c_void_p]),
     "b200_recurrence_scan": (c_int, [c_void_p] * 11 + [c_int64] * 6 + [c_void_p]),
     "b200_head_linear": (c_int, [c_void_p] * 3 + [c_int64] * 8 + [c_int, c_void_p]),
-    "b200_latent_attention": (c_int, [c_void_p] * 8 + [c_int64] * 4 + [c_double, c_int, c_void_p]),
+    "b200_latent_attention_workspace_bytes": (c_int64, [c_int64] * 6 + [c_int]),
+    "b200_latent_attention": (c_int, [c_void_p] * 8 + [c_int64] * 7 + [c_double, c_int, c_void_p, c_int64, c_void_p]),
     "b200_sequence_positions": (c_int, [c_void_p] * 3 + [c_int64, c_void_p]),
     "b200_advance_slots": (c_int, [c_void_p] * 3 + [c_int64, c_int64, c_void_p, c_void_p]),
 }

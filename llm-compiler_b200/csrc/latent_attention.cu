@@ -3,8 +3,9 @@
 // cached rows themselves, and the weighted sum of the rows is carried out of it (W_uv) behind the
 // attention. The softmax denominator may hold a learned term per head (a sink) beside the keys.
 //
-// This file: the per-head projections in and out of the latent space, and attention for any rank up to
-// 1024 on the CUDA cores (fp32 models, and shapes the tensor-core kernel does not take).
+// This file: the per-head projections in and out of the latent space, attention on warp-level tensor
+// cores with the keys split over CTAs (bf16, rank up to 512), and attention for any rank up to 1024 on
+// the CUDA cores (fp32 models, and shapes the tensor-core kernel does not take).
 #include "common.cuh"
 #include "hybrid.cuh"
 
@@ -59,6 +60,379 @@ __global__ void __launch_bounds__(256) head_linear_kernel(const HeadLinearParams
       const int m = m_base + ty * 4 + i, n = n_base + tx * 4 + j;
       if (m < p.m && n < p.n) Elem<T>::store(y + static_cast<int64_t>(m) * p.y_row_stride + n, acc[i][j]);
     }
+}
+
+// bf16: 16 or 64 rows x 64 columns of one head per CTA, four warps, a ring of 64-wide k-blocks.
+// BM 16: the warps split the columns; BM 64: the rows.
+template <int BM>
+__global__ void __launch_bounds__(128) head_linear_bf16_kernel(const HeadLinearParams p) {
+  constexpr int kStages = 3, BN = 64, BK = 64;
+  constexpr int kTilesN = BM == 16 ? 2 : 8;  // n8 tiles of a warp
+  constexpr uint32_t kABytes = BM * 128, kStageBytes = kABytes + BN * 128;
+  extern __shared__ __align__(128) unsigned char ring[];
+  grid_launch_dependents();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int m_base = blockIdx.y * BM, n_base = blockIdx.x * BN;
+  const __nv_bfloat16* x = static_cast<const __nv_bfloat16*>(p.x) + blockIdx.z * p.x_head_stride;
+  const __nv_bfloat16* w = static_cast<const __nv_bfloat16*>(p.w) + static_cast<int64_t>(blockIdx.z) * p.n * p.k;
+  const uint32_t base = smem_u32(ring);
+  const int blocks = (p.k + BK - 1) / BK;
+  auto load = [&](int block) {
+    const uint32_t stage = base + (block % kStages) * kStageBytes;
+    for (int item = threadIdx.x; item < (BM + BN) * 8; item += 128) {
+      const int r = item >> 3, chunk = item & 7, kk = block * BK + chunk * 8;
+      const bool is_a = r < BM;
+      const int row = is_a ? m_base + r : n_base + r - BM;
+      const bool inside = row < (is_a ? p.m : p.n) && kk < p.k;
+      const __nv_bfloat16* src = is_a ? x + (inside ? static_cast<int64_t>(row) * p.x_row_stride + kk : 0)
+                                      : w + (inside ? static_cast<int64_t>(row) * p.k + kk : 0);
+      const uint32_t dst = stage + (is_a ? r * 128 : kABytes + (r - BM) * 128);
+      cp_async16_zfill(dst + swizzle128(is_a ? r : r - BM, chunk) * 16, src, inside ? 16 : 0);
+    }
+  };
+  grid_dependency_wait_cta();
+#pragma unroll
+  for (int b = 0; b < kStages - 1; ++b) {
+    if (b < blocks) load(b);
+    cp_async_commit();
+  }
+  float acc[kTilesN][4] = {};
+  for (int b = 0; b < blocks; ++b) {
+    cp_async_wait<kStages - 2>();
+    __syncthreads();
+    if (b + kStages - 1 < blocks) load(b + kStages - 1);
+    cp_async_commit();
+    const uint32_t a_tile = base + (b % kStages) * kStageBytes, b_tile = a_tile + kABytes;
+    const int a_row = (BM == 16 ? 0 : warp * 16) + (lane & 15);
+#pragma unroll
+    for (int ks = 0; ks < 4; ++ks) {
+      uint32_t a[4];
+      ldmatrix_x4(a, a_tile + a_row * 128 + swizzle128(a_row, ks * 2 + (lane >> 4)) * 16);
+#pragma unroll
+      for (int pair = 0; pair < kTilesN / 2; ++pair) {
+        uint32_t bf[4];  // two n8 tiles x k16
+        const int n = (BM == 16 ? warp * 16 : 0) + pair * 16 + ((lane >> 4) << 3) + (lane & 7);
+        ldmatrix_x4(bf, b_tile + n * 128 + swizzle128(n, ks * 2 + ((lane >> 3) & 1)) * 16);
+        mma_bf16_16816(acc[pair * 2], a, bf[0], bf[1]);
+        mma_bf16_16816(acc[pair * 2 + 1], a, bf[2], bf[3]);
+      }
+    }
+  }
+  __nv_bfloat16* y = static_cast<__nv_bfloat16*>(p.y) + blockIdx.z * p.y_head_stride;
+#pragma unroll
+  for (int t = 0; t < kTilesN; ++t) {
+    const int n = n_base + (BM == 16 ? warp * 16 : 0) + t * 8 + (lane & 3) * 2;
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int m = m_base + (BM == 16 ? 0 : warp * 16) + (lane >> 2) + half * 8;
+      if (m >= p.m || n >= p.n) continue;  // n is even and p.n a multiple of 8
+      *reinterpret_cast<uint32_t*>(y + static_cast<int64_t>(m) * p.y_row_stride + n) =
+          pack_bf16x2(acc[t][half * 2], acc[t][half * 2 + 1]);
+    }
+  }
+}
+
+// ---- attention on the tensor cores ---------------------------------------------------------
+// Rows of a sequence are its (token, head) pairs. A CTA takes 16 MT rows and one split of the keys, 32
+// keys a step: S = Q C^T (four groups of 8 keys x two halves of the rank per warp), softmax in fp32
+// through shared memory, O += P C with a warp on every eighth of the rank. C, the keys and the values in
+// one, is fetched once per step for both products. The probabilities enter the product as the sum of
+// two bf16 numbers, so that they keep 16 bits of mantissa. Splits leave fp32 partial results and
+// (max, sum) pairs; the combining kernel adds the sink to the denominator, once.
+constexpr int kLatentKeys = 32, kLatentStages = 3, kLatentThreads = 256;
+
+struct LatentSplitParams {
+  const __nv_bfloat16* q;      // [rows, heads, rank]
+  const __nv_bfloat16* cache;  // [slots, capacity, rank]
+  float* partial;              // [rows * heads, splits, rank]
+  float2* partial_stats;       // [rows * heads, splits]: max (log2 domain), sum
+  SequenceBatch batch;
+  int heads, rank, splits, pitch;  // pitch: bytes of a row in shared memory
+  int64_t capacity;
+  float scale_log2;
+};
+
+// The keys of split `split`: equal shares of at least 128 keys, in whole steps.
+__device__ __forceinline__ void split_range(int64_t keys, int splits, int split, int64_t& begin, int64_t& end) {
+  int64_t share = (keys + splits - 1) / splits;
+  if (share < 128) share = 128;
+  share = (share + kLatentKeys - 1) / kLatentKeys * kLatentKeys;
+  begin = share * split;
+  end = begin + share < keys ? begin + share : keys;
+}
+
+template <int MT, int NT>
+__global__ void __launch_bounds__(kLatentThreads) latent_attention_split_kernel(const LatentSplitParams p) {
+  constexpr int M = 16 * MT;
+  constexpr int kSPitch = kLatentKeys + 4;           // floats
+  constexpr int kPPitch = kLatentKeys * 2 + 16;      // bytes
+  extern __shared__ __align__(128) unsigned char smem[];
+  __shared__ float row_factor[M];
+  __shared__ float row_max[M], row_sum[M];
+  grid_launch_dependents();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int split = blockIdx.x, sequence = blockIdx.z, row0 = blockIdx.y * M;
+  grid_dependency_wait_cta();
+  const int slot = p.batch.slots[sequence];
+  const int first = p.batch.starts[sequence];
+  const int rows = (p.batch.starts[sequence + 1] - first) * p.heads;
+  if (slot < 0 || row0 >= rows) return;
+  const int64_t base = p.batch.bases[sequence];
+  const int last_row = min(row0 + M, rows) - 1;
+  int64_t keys = base + last_row / p.heads + 1;
+  if (keys > p.capacity) keys = p.capacity;
+  int64_t begin, end;
+  split_range(keys, p.splits, split, begin, end);
+  const int64_t unit0 = static_cast<int64_t>(first) * p.heads + row0;  // row of q and of the partials
+  if (begin >= end) {
+    for (int r = threadIdx.x; r <= last_row - row0; r += kLatentThreads)
+      p.partial_stats[(unit0 + r) * p.splits + split] = make_float2(-INFINITY, 0.0f);
+    return;
+  }
+  const uint32_t q_tile = smem_u32(smem);
+  const uint32_t c_tiles = q_tile + M * p.pitch;
+  float* scores = reinterpret_cast<float*>(smem + M * p.pitch + kLatentStages * kLatentKeys * p.pitch);  // [2][M][kSPitch]
+  unsigned char* probabilities = reinterpret_cast<unsigned char*>(scores + 2 * M * kSPitch);  // [2][M][kPPitch]: high, low
+  const int chunks = p.rank / 8;
+  for (int item = threadIdx.x; item < M * chunks; item += kLatentThreads) {
+    const int r = item / chunks, c = item % chunks;
+    const bool inside = row0 + r <= last_row;
+    cp_async16_zfill(q_tile + r * p.pitch + c * 16, p.q + (inside ? (unit0 + r) * p.rank + c * 8 : 0), inside ? 16 : 0);
+  }
+  const __nv_bfloat16* cache = p.cache + static_cast<int64_t>(slot) * p.capacity * p.rank;
+  const int steps = static_cast<int>((end - begin + kLatentKeys - 1) / kLatentKeys);
+  auto load = [&](int step) {
+    const uint32_t tile = c_tiles + (step % kLatentStages) * kLatentKeys * p.pitch;
+    const int64_t key0 = begin + static_cast<int64_t>(step) * kLatentKeys;
+    for (int item = threadIdx.x; item < kLatentKeys * chunks; item += kLatentThreads) {
+      const int r = item / chunks, c = item % chunks;
+      const bool inside = key0 + r < end;
+      cp_async16_zfill(tile + r * p.pitch + c * 16, cache + (inside ? (key0 + r) * p.rank + c * 8 : 0), inside ? 16 : 0);
+    }
+  };
+#pragma unroll
+  for (int s = 0; s < kLatentStages - 1; ++s) {
+    if (s < steps) load(s);
+    cp_async_commit();  // (the first group holds Q as well)
+  }
+  for (int r = threadIdx.x; r < M; r += kLatentThreads) {
+    row_max[r] = -INFINITY;
+    row_sum[r] = 0.0f;
+  }
+  float acc[MT][NT][4] = {};
+  const int k_steps = p.rank / 16;
+  const int k_begin = (warp >> 2) ? (k_steps + 1) / 2 : 0, k_end = (warp >> 2) ? k_steps : (k_steps + 1) / 2;
+  for (int step = 0; step < steps; ++step) {
+    cp_async_wait<kLatentStages - 2>();
+    __syncthreads();  // the tile has landed; everyone is done with the one that is refilled now
+    if (step + kLatentStages - 1 < steps) load(step + kLatentStages - 1);
+    cp_async_commit();
+    const uint32_t tile = c_tiles + (step % kLatentStages) * kLatentKeys * p.pitch;
+    // ---- scores: this warp's 8 keys, its half of the rank ----
+    {
+      float s[MT][4] = {};
+      const int key = (warp & 3) * 8 + (lane & 7);
+      for (int ks = k_begin; ks < k_end; ++ks) {
+        uint32_t b[2];
+        asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];\n"
+                     : "=r"(b[0]), "=r"(b[1])
+                     : "r"(tile + key * p.pitch + ks * 32 + ((lane >> 3) & 1) * 16));
+#pragma unroll
+        for (int mt = 0; mt < MT; ++mt) {
+          uint32_t a[4];
+          ldmatrix_x4(a, q_tile + (mt * 16 + (lane & 15)) * p.pitch + ks * 32 + (lane >> 4) * 16);
+          mma_bf16_16816(s[mt], a, b[0], b[1]);
+        }
+      }
+      float* out = scores + (warp >> 2) * M * kSPitch + (warp & 3) * 8 + (lane & 3) * 2;
+#pragma unroll
+      for (int mt = 0; mt < MT; ++mt) {
+        *reinterpret_cast<float2*>(out + (mt * 16 + (lane >> 2)) * kSPitch) = make_float2(s[mt][0], s[mt][1]);
+        *reinterpret_cast<float2*>(out + (mt * 16 + (lane >> 2) + 8) * kSPitch) = make_float2(s[mt][2], s[mt][3]);
+      }
+    }
+    __syncthreads();
+    // ---- softmax: 8 lanes a row, 4 keys each ----
+    for (int r = threadIdx.x >> 3; r < M; r += kLatentThreads / 8) {
+      const int c = (threadIdx.x & 7) * 4;
+      const float4 s0 = *reinterpret_cast<const float4*>(scores + r * kSPitch + c);
+      const float4 s1 = *reinterpret_cast<const float4*>(scores + (M + r) * kSPitch + c);
+      float v[4] = {s0.x + s1.x, s0.y + s1.y, s0.z + s1.z, s0.w + s1.w};
+      const int64_t key0 = begin + static_cast<int64_t>(step) * kLatentKeys + c;
+      const int64_t limit = min(base + (row0 + r) / p.heads + 1, end);
+      float top = row_max[r];
+      const float before = top;
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        v[i] = key0 + i < limit ? v[i] * p.scale_log2 : -INFINITY;
+        top = fmaxf(top, v[i]);
+      }
+#pragma unroll
+      for (int o = 4; o > 0; o >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
+      const float reference = top == -INFINITY ? 0.0f : top;  // (no visible key so far: all weights are 0)
+      float sum = 0.0f;
+      uint32_t high[2], low[2];
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const float p0 = exp2f(v[2 * i] - reference), p1 = exp2f(v[2 * i + 1] - reference);
+        sum += p0 + p1;
+        high[i] = pack_bf16x2(p0, p1);
+        low[i] = pack_bf16x2(p0 - bf16_lo(high[i]), p1 - bf16_hi(high[i]));
+      }
+#pragma unroll
+      for (int o = 4; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+      *reinterpret_cast<uint2*>(probabilities + r * kPPitch + c * 2) = make_uint2(high[0], high[1]);
+      *reinterpret_cast<uint2*>(probabilities + (M + r) * kPPitch + c * 2) = make_uint2(low[0], low[1]);
+      if ((threadIdx.x & 7) == 0) {
+        const float factor = exp2f(before - reference);  // (0 on the first visible key)
+        row_factor[r] = factor;
+        row_sum[r] = row_sum[r] * factor + sum;
+        row_max[r] = top;
+      }
+    }
+    __syncthreads();
+    // ---- O += P C on this warp's columns ----
+    const uint32_t p_tile = smem_u32(probabilities);
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt) {
+      const float f0 = row_factor[mt * 16 + (lane >> 2)], f1 = row_factor[mt * 16 + (lane >> 2) + 8];
+#pragma unroll
+      for (int t = 0; t < NT; ++t) {
+        acc[mt][t][0] *= f0; acc[mt][t][1] *= f0;
+        acc[mt][t][2] *= f1; acc[mt][t][3] *= f1;
+      }
+    }
+#pragma unroll
+    for (int ks = 0; ks < kLatentKeys / 16; ++ks) {
+      uint32_t hi[MT][4], lo[MT][4];
+#pragma unroll
+      for (int mt = 0; mt < MT; ++mt) {
+        const uint32_t address = p_tile + (mt * 16 + (lane & 15)) * kPPitch + ks * 32 + (lane >> 4) * 16;
+        ldmatrix_x4(hi[mt], address);
+        ldmatrix_x4(lo[mt], address + M * kPPitch);
+      }
+#pragma unroll
+      for (int t = 0; t < NT; ++t) {
+        const int n_tile = warp * NT + t;
+        if (n_tile * 8 < p.rank) {
+          uint32_t b[2];
+          asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];\n"
+                       : "=r"(b[0]), "=r"(b[1])
+                       : "r"(tile + (ks * 16 + (lane & 15)) * p.pitch + n_tile * 16));
+#pragma unroll
+          for (int mt = 0; mt < MT; ++mt) {
+            mma_bf16_16816(acc[mt][t], hi[mt], b[0], b[1]);
+            mma_bf16_16816(acc[mt][t], lo[mt], b[0], b[1]);
+          }
+        }
+      }
+    }
+  }
+  cp_async_wait<0>();
+#pragma unroll
+  for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int r = mt * 16 + (lane >> 2) + half * 8;
+      if (row0 + r > last_row) continue;
+      float* out = p.partial + ((unit0 + r) * p.splits + split) * p.rank + (lane & 3) * 2;
+#pragma unroll
+      for (int t = 0; t < NT; ++t) {
+        const int n = (warp * NT + t) * 8;
+        if (n < p.rank)
+          *reinterpret_cast<float2*>(out + n) = make_float2(acc[mt][t][half * 2], acc[mt][t][half * 2 + 1]);
+      }
+    }
+  for (int r = threadIdx.x; r <= last_row - row0; r += kLatentThreads)  // (written before the last barrier but one)
+    p.partial_stats[(unit0 + r) * p.splits + split] = make_float2(row_max[r], row_sum[r]);
+}
+
+// out = sum of the splits' results over (sum of their sums + exp(sink)): one CTA per (row, head)
+__global__ void __launch_bounds__(128) latent_combine_kernel(const float* partial, const float2* stats,
+                                                             const __nv_bfloat16* sink, __nv_bfloat16* out,
+                                                             const SequenceBatch batch, int heads, int rank,
+                                                             int splits) {
+  grid_launch_dependents();
+  grid_dependency_wait_cta();
+  const int64_t unit = static_cast<int64_t>(blockIdx.x) * heads + blockIdx.y;
+  __nv_bfloat16* dst = out + unit * rank;
+  if (batch.slots[batch.token_sequence[blockIdx.x]] < 0) {
+    for (int c = threadIdx.x; c < rank; c += blockDim.x) dst[c] = __float2bfloat16_rn(0.0f);
+    return;
+  }
+  const float own = sink != nullptr ? __bfloat162float(sink[blockIdx.y]) * 1.4426950408889634f : -INFINITY;
+  float top = own;
+  for (int s = 0; s < splits; ++s) top = fmaxf(top, stats[unit * splits + s].x);
+  float total = exp2f(own - top);
+  for (int s = 0; s < splits; ++s) {
+    const float2 st = stats[unit * splits + s];
+    total += st.y * exp2f(st.x - top);
+  }
+  const float inverse = 1.0f / total;
+  for (int c = threadIdx.x * 2; c < rank; c += blockDim.x * 2) {
+    float a = 0.0f, b = 0.0f;
+    for (int s = 0; s < splits; ++s) {
+      const float2 st = stats[unit * splits + s];
+      if (st.y == 0.0f) continue;  // a split without keys left no result
+      const float f = exp2f(st.x - top);
+      const float2 v = *reinterpret_cast<const float2*>(partial + (unit * splits + s) * rank + c);
+      a = fmaf(v.x, f, a);
+      b = fmaf(v.y, f, b);
+    }
+    *reinterpret_cast<uint32_t*>(dst + c) = pack_bf16x2(a * inverse, b * inverse);
+  }
+}
+
+struct LatentPlan {
+  int mt, nt, row_blocks, splits, pitch, smem;
+};
+
+// Row tile and split count: about two CTAs a SM (one for the 64-row tile), in whole waves.
+LatentPlan plan_latent(int64_t sequences, int64_t longest, int64_t heads, int64_t rank, int64_t context) {
+  LatentPlan plan{};
+  if (rank % 16 != 0 || rank > 512) return plan;
+  const int64_t rows = longest * heads;
+  plan.mt = rows <= 16 ? 1 : rows <= 32 ? 2 : 4;
+  const int64_t tiles = (rank / 8 + 7) / 8;
+  plan.nt = tiles <= 1 ? 1 : tiles <= 2 ? 2 : tiles <= 4 ? 4 : 8;
+  const int m = 16 * plan.mt;
+  plan.pitch = static_cast<int>(rank * 2 + 16);
+  plan.smem = (m + kLatentStages * kLatentKeys) * plan.pitch + 2 * m * (kLatentKeys + 4) * 4 + 2 * m * (kLatentKeys * 2 + 16);
+  plan.row_blocks = static_cast<int>(ceil_div(rows, m));
+  const int per_sm = plan.smem <= 112 * 1024 && plan.mt <= 2 ? 2 : 1;
+  const int64_t slots = static_cast<int64_t>(kNumSMs) * per_sm, units = sequences * plan.row_blocks;
+  const int64_t most = ceil_div(context, 128);
+  double best = -1.0;
+  plan.splits = 1;
+  for (int64_t s = 1; s <= 64 && s <= most; ++s) {
+    const int64_t ctas = units * s;
+    const double fill = static_cast<double>(ctas) / (ceil_div(ctas, slots) * slots) - 0.01 * s;
+    if (fill > best) {
+      best = fill;
+      plan.splits = static_cast<int>(s);
+    }
+  }
+  return plan;
+}
+
+template <int MT, int NT>
+int launch_split(const LatentSplitParams& p, const LatentPlan& plan, int64_t sequences, cudaStream_t stream) {
+  auto kernel = latent_attention_split_kernel<MT, NT>;
+  if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, plan.smem) != cudaSuccess)
+    return B200_ERR_LAUNCH;
+  const dim3 grid(static_cast<unsigned>(plan.splits), static_cast<unsigned>(plan.row_blocks),
+                  static_cast<unsigned>(sequences));
+  return launch_chained(kernel, grid, dim3(kLatentThreads), plan.smem, stream, p) == cudaSuccess ? B200_OK
+                                                                                                : B200_ERR_LAUNCH;
+}
+template <int MT>
+int launch_split_nt(const LatentSplitParams& p, const LatentPlan& plan, int64_t sequences, cudaStream_t stream) {
+  switch (plan.nt) {
+    case 1: return launch_split<MT, 1>(p, plan, sequences, stream);
+    case 2: return launch_split<MT, 2>(p, plan, sequences, stream);
+    case 4: return launch_split<MT, 4>(p, plan, sequences, stream);
+    default: return launch_split<MT, 8>(p, plan, sequences, stream);
+  }
 }
 
 // ---- attention on the CUDA cores -----------------------------------------------------------
@@ -189,23 +563,70 @@ extern "C" int b200_head_linear(const void* x, const void* w, void* y, int64_t m
   HeadLinearParams p{x, w, y, static_cast<int>(m), static_cast<int>(k), static_cast<int>(n), x_row_stride,
                      x_head_stride, y_row_stride, y_head_stride};
   cudaStream_t s = static_cast<cudaStream_t>(stream);
+  // 16-byte rows and chunks: the tensor-core kernel
+  if (dtype == B200_BF16 && k % 8 == 0 && n % 8 == 0 && x_row_stride % 8 == 0 && x_head_stride % 8 == 0 &&
+      y_row_stride % 2 == 0 && y_head_stride % 2 == 0 && aligned16(x) && aligned16(w) && aligned16(y)) {
+    const int bm = m <= 16 ? 16 : 64;
+    const dim3 tiles(static_cast<unsigned>(ceil_div(n, 64)), static_cast<unsigned>(ceil_div(m, bm)),
+                     static_cast<unsigned>(heads));
+    const int smem = 3 * (bm + 64) * 128;
+    auto kernel = bm == 16 ? head_linear_bf16_kernel<16> : head_linear_bf16_kernel<64>;
+    if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess)
+      return B200_ERR_LAUNCH;
+    return launch_chained(kernel, tiles, dim3(128), smem, s, p) == cudaSuccess ? launch_status() : B200_ERR_LAUNCH;
+  }
   if (dtype == B200_F32) head_linear_kernel<float><<<grid, 256, 0, s>>>(p);
   else head_linear_kernel<__nv_bfloat16><<<grid, 256, 0, s>>>(p);
   return launch_status();
 }
 
+extern "C" int64_t b200_latent_attention_workspace_bytes(int64_t rows, int64_t sequences, int64_t longest,
+                                                         int64_t heads, int64_t rank_row, int64_t context,
+                                                         int dtype) {
+  if (dtype != B200_BF16 || rows <= 0 || sequences <= 0 || longest <= 0 || heads <= 0 || rank_row <= 0 || context <= 0)
+    return 0;
+  const LatentPlan plan = plan_latent(sequences, longest, heads, rank_row, context);
+  return plan.mt == 0 ? 0 : rows * heads * plan.splits * (rank_row + 2) * 4;
+}
+
 extern "C" int b200_latent_attention(const void* q, const void* cache, const void* sink, void* out,
                                      const int32_t* token_sequence, const int32_t* starts, const int32_t* slots,
-                                     const int32_t* bases, int64_t rows, int64_t heads, int64_t rank_row,
-                                     int64_t capacity, double scale, int dtype, void* stream) {
-  if (!q || !cache || !out || !token_sequence || !starts || !slots || !bases || rows < 0 || heads <= 0 ||
-      rank_row <= 0 || capacity <= 0)
+                                     const int32_t* bases, int64_t rows, int64_t sequences, int64_t longest,
+                                     int64_t heads, int64_t rank_row, int64_t capacity, int64_t context,
+                                     double scale, int dtype, void* workspace, int64_t workspace_bytes,
+                                     void* stream) {
+  if (!q || !cache || !out || !token_sequence || !starts || !slots || !bases || rows < 0 || sequences <= 0 ||
+      longest <= 0 || heads <= 0 || rank_row <= 0 || capacity <= 0 || context <= 0)
     return B200_ERR_BAD_ARGUMENT;
   if (dtype != B200_F32 && dtype != B200_BF16) return B200_ERR_UNSUPPORTED;
   if (rows == 0) return B200_OK;
-  if (rows > INT32_MAX || heads > 65535) return B200_ERR_TOO_LARGE;
+  if (rows > INT32_MAX || heads > 65535 || sequences > 65535) return B200_ERR_TOO_LARGE;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (dtype == B200_BF16) {
+    const LatentPlan plan = plan_latent(sequences, longest, heads, rank_row, context);
+    if (plan.mt != 0 && plan.row_blocks <= 65535) {
+      const int64_t need = rows * heads * plan.splits * (rank_row + 2) * 4;
+      if (!workspace || workspace_bytes < need) return B200_ERR_WORKSPACE;
+      if (!aligned16(q) || !aligned16(cache) || !aligned16(workspace)) return B200_ERR_ALIGNMENT;
+      float* partial = static_cast<float*>(workspace);
+      float2* stats = reinterpret_cast<float2*>(partial + rows * heads * plan.splits * rank_row);
+      LatentSplitParams p{static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(cache), partial, stats,
+                          {token_sequence, starts, slots, bases}, static_cast<int>(heads), static_cast<int>(rank_row),
+                          plan.splits, plan.pitch, capacity, static_cast<float>(scale * 1.4426950408889634)};
+      const int code = plan.mt == 1 ? launch_split_nt<1>(p, plan, sequences, s)
+                       : plan.mt == 2 ? launch_split_nt<2>(p, plan, sequences, s)
+                                      : launch_split_nt<4>(p, plan, sequences, s);
+      if (code != B200_OK) return code;
+      const dim3 grid(static_cast<unsigned>(rows), static_cast<unsigned>(heads));
+      const SequenceBatch batch{token_sequence, starts, slots, bases};
+      return launch_chained(latent_combine_kernel, grid, dim3(128), 0, s, static_cast<const float*>(partial),
+                            static_cast<const float2*>(stats), static_cast<const __nv_bfloat16*>(sink),
+                            static_cast<__nv_bfloat16*>(out), batch, static_cast<int>(heads),
+                            static_cast<int>(rank_row), plan.splits) == cudaSuccess
+                 ? launch_status() : B200_ERR_LAUNCH;
+    }
+  }
   LatentAttentionParams p{q, cache, sink, out, {token_sequence, starts, slots, bases}, static_cast<int>(heads),
                           static_cast<int>(rank_row), capacity, static_cast<float>(scale)};
-  cudaStream_t s = static_cast<cudaStream_t>(stream);
   return dtype == B200_F32 ? launch_generic<float>(p, rows, s) : launch_generic<__nv_bfloat16>(p, rows, s);
 }

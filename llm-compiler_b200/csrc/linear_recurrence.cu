@@ -13,18 +13,9 @@ namespace b200 {
 namespace {
 
 // ---- operand preparation ------------------------------------------------------------------
-struct RetentionPrepParams {
-  const void* input;  // T [rows, row_stride]
-  SequenceBatch batch;
-  float *q, *k, *v;   // [rows, heads, dim], [rows, heads, dim], [rows, heads, vdim]
-  int rows, heads, dim, vdim, q_column, k_column, v_column, rot_dims;
-  int64_t row_stride;
-  double log2_base;   // log2 of the rotation base
-  float k_scale;
-};
-
 template <typename T>
-__global__ void __launch_bounds__(256) retention_prep_kernel(const RetentionPrepParams p) {
+__global__ void __launch_bounds__(256) retention_prep_kernel(const RetentionInputs p, float* q,
+                                                             float* k, float* v) {
   extern __shared__ float rotation[];  // cos, sin of this row's position [rot_dims / 2] each
   const int64_t row = blockIdx.x;
   const int half = p.rot_dims / 2;
@@ -44,11 +35,11 @@ __global__ void __launch_bounds__(256) retention_prep_kernel(const RetentionPrep
       value = value * rotation[within] - Elem<T>::load(src + half) * rotation[half + within];
     else if (within < p.rot_dims)
       value = value * rotation[within - half] + Elem<T>::load(src - half) * rotation[within];
-    if (is_k) p.k[row * qk + channel] = value * p.k_scale;
-    else p.q[row * qk + channel] = value;
+    if (is_k) k[row * qk + channel] = value * p.k_scale;
+    else q[row * qk + channel] = value;
   }
   for (int c = threadIdx.x; c < p.heads * p.vdim; c += blockDim.x)
-    p.v[row * p.heads * p.vdim + c] = Elem<T>::load(in + p.v_column + c);
+    v[row * p.heads * p.vdim + c] = Elem<T>::load(in + p.v_column + c);
 }
 
 // One warp per unit of a row: a q head, a k head, a v head, or a head's step size and decays.
@@ -238,25 +229,17 @@ int dispatch_scan(const ScanParams& p, int64_t sequences, cudaStream_t stream) {
 
 using namespace b200;
 
-extern "C" int b200_retention_prep(const void* input, const int32_t* token_sequence, const int32_t* starts,
-                                   const int32_t* slots, const int32_t* bases, float* q, float* k, float* v,
-                                   int64_t rows, int64_t heads, int64_t dim, int64_t vdim, int64_t q_column,
-                                   int64_t k_column, int64_t v_column, int64_t row_stride, int64_t rot_dims,
-                                   double rot_base, double k_scale, int dtype, void* stream) {
-  if (!input || !token_sequence || !starts || !slots || !bases || !q || !k || !v || rows < 0 || heads <= 0 ||
-      dim <= 0 || vdim <= 0 || rot_dims < 0 || rot_dims > dim || rot_dims % 2 != 0 || !(rot_base > 0.0))
-    return B200_ERR_BAD_ARGUMENT;
+extern "C" int b200_retention_prep(const b200_retention_inputs* inputs, float* q, float* k, float* v,
+                                   int64_t rows, int dtype, void* stream) {
+  RetentionInputs p;
+  if (!retention_inputs_from(inputs, &p) || !q || !k || !v || rows < 0) return B200_ERR_BAD_ARGUMENT;
   if (dtype != B200_F32 && dtype != B200_BF16) return B200_ERR_UNSUPPORTED;
   if (rows == 0) return B200_OK;
-  if (rows > INT32_MAX || rot_dims > 8192) return B200_ERR_TOO_LARGE;
-  RetentionPrepParams p{input, {token_sequence, starts, slots, bases}, q, k, v, static_cast<int>(rows),
-                        static_cast<int>(heads), static_cast<int>(dim), static_cast<int>(vdim),
-                        static_cast<int>(q_column), static_cast<int>(k_column), static_cast<int>(v_column),
-                        static_cast<int>(rot_dims), row_stride, log2(rot_base), static_cast<float>(k_scale)};
-  const size_t smem = (rot_dims + 1) * sizeof(float);
+  if (rows > INT32_MAX) return B200_ERR_TOO_LARGE;
+  const size_t smem = (p.rot_dims + 1) * sizeof(float);
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (dtype == B200_F32) retention_prep_kernel<float><<<static_cast<unsigned>(rows), 256, smem, s>>>(p);
-  else retention_prep_kernel<__nv_bfloat16><<<static_cast<unsigned>(rows), 256, smem, s>>>(p);
+  if (dtype == B200_F32) retention_prep_kernel<float><<<static_cast<unsigned>(rows), 256, smem, s>>>(p, q, k, v);
+  else retention_prep_kernel<__nv_bfloat16><<<static_cast<unsigned>(rows), 256, smem, s>>>(p, q, k, v);
   return launch_status();
 }
 

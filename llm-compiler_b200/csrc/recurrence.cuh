@@ -17,6 +17,7 @@ __device__ __forceinline__ void rotation_of(int64_t position, int i, int dims, d
 }
 
 struct DeltaInputs {
+  static constexpr bool kDelta = true;
   const void* input;   // T [rows, row_stride]: the projections of h
   const void* gates;   // T [rows, gate_row_stride]: decay columns [heads * dim] from decay_column
   const void *q_conv, *k_conv, *v_conv;  // T [channels, taps], last column: the current token
@@ -80,5 +81,99 @@ __device__ __forceinline__ float delta_log_decay(const DeltaInputs& p, int64_t r
                      Elem<T>::load(static_cast<const T*>(p.dt_bias) + head * p.dim + c);
   return -expf(Elem<T>::load(static_cast<const T*>(p.a_log) + head)) * softplus_f32(step);
 }
+
+struct RetentionInputs {
+  static constexpr bool kDelta = false;
+  const void* input;  // T [rows, row_stride]
+  const float* decay; // [heads]
+  SequenceBatch batch;
+  int heads, dim, vdim, q_column, k_column, v_column, rot_dims;
+  int64_t row_stride;
+  double log2_base;   // log2 of the rotation base
+  float k_scale;
+};
+
+inline bool retention_inputs_from(const b200_retention_inputs* in, RetentionInputs* out) {
+  if (in == nullptr || !in->input || !in->token_sequence || !in->starts || !in->slots || !in->bases ||
+      in->heads <= 0 || in->dim <= 0 || in->vdim <= 0 || in->rot_dims < 0 || in->rot_dims > in->dim ||
+      in->rot_dims % 2 != 0 || in->rot_dims > 8192 || !(in->rot_base > 0.0))
+    return false;
+  *out = RetentionInputs{in->input, in->decay, {in->token_sequence, in->starts, in->slots, in->bases},
+                         static_cast<int>(in->heads), static_cast<int>(in->dim), static_cast<int>(in->vdim),
+                         static_cast<int>(in->q_column), static_cast<int>(in->k_column),
+                         static_cast<int>(in->v_column), static_cast<int>(in->rot_dims), in->row_stride,
+                         log2(in->rot_base), static_cast<float>(in->k_scale)};
+  return true;
+}
+
+// ---- operands of a single decoded token: q, k (before a unit norm) and the decay of one key channel ----
+template <typename T>
+__device__ __forceinline__ void step_operands(const DeltaInputs& p, int head, int c, int64_t row, int64_t position,
+                                              int slot, float& q, float& k, float& g) {
+  const int channel = head / (p.heads / p.kv_heads) * p.dim + c;
+  q = silu_of(short_conv<T>(p, 0, channel, row, 0, position, slot));
+  k = silu_of(short_conv<T>(p, 1, channel, row, 0, position, slot));
+  g = expf(delta_log_decay<T>(p, row, head, c));
+}
+template <typename T>
+__device__ __forceinline__ void step_operands(const RetentionInputs& p, int head, int c, int64_t row,
+                                              int64_t position, int, float& q, float& k, float& g) {
+  const T* in = static_cast<const T*>(p.input) + row * p.row_stride + head * p.dim + c;
+  const T *qp = in + p.q_column, *kp = in + p.k_column;
+  q = Elem<T>::load(qp);
+  k = Elem<T>::load(kp);
+  const int half = p.rot_dims / 2;
+  if (c < p.rot_dims) {
+    const int i = c < half ? c : c - half;
+    const int other = c < half ? half : -half;
+    float cosine, sine;
+    rotation_of(position, i, p.rot_dims, p.log2_base, cosine, sine);
+    if (c < half) sine = -sine;
+    q = q * cosine + Elem<T>::load(qp + other) * sine;
+    k = k * cosine + Elem<T>::load(kp + other) * sine;
+  }
+  k *= p.k_scale;
+  g = p.decay[head];
+}
+template <typename T>
+__device__ __forceinline__ float step_value(const DeltaInputs& p, int head, int c, int64_t row, int64_t position,
+                                            int slot) {
+  return silu_of(short_conv<T>(p, 2, head * p.vdim + c, row, 0, position, slot));
+}
+template <typename T>
+__device__ __forceinline__ float step_value(const RetentionInputs& p, int head, int c, int64_t row, int64_t, int) {
+  return Elem<T>::load(static_cast<const T*>(p.input) + row * p.row_stride + p.v_column + head * p.vdim + c);
+}
+template <typename T>
+__device__ __forceinline__ float step_beta(const DeltaInputs& p, int64_t row, int head) {
+  return delta_beta<T>(p, row, head);
+}
+template <typename T>
+__device__ __forceinline__ float step_beta(const RetentionInputs&, int64_t, int) { return 1.0f; }
+__device__ __forceinline__ float step_q_scale(const DeltaInputs& p) { return p.q_scale; }
+__device__ __forceinline__ float step_q_scale(const RetentionInputs&) { return 1.0f; }
+
+// This token's convolution inputs into the ring entry of its position, which no CTA of the step reads
+// (the entries read are those of the taps - 1 positions before it).
+template <typename T, int THREADS>
+__device__ __forceinline__ void keep_step_inputs(const DeltaInputs& p, int head, int64_t row, int64_t position,
+                                                 int slot) {
+  if (p.taps <= 1) return;
+  const int shared = p.heads / p.kv_heads, qk = p.kv_heads * p.dim;
+  const int channels = 2 * qk + p.heads * p.vdim;
+  T* ring = static_cast<T*>(p.ring) + (static_cast<int64_t>(slot) * p.taps + position % p.taps) * channels;
+  const T* in = static_cast<const T*>(p.input) + row * p.row_stride;
+  if (head % shared == 0) {
+    const int first = head / shared * p.dim;
+    for (int c = threadIdx.x; c < p.dim; c += THREADS) {
+      ring[first + c] = in[p.q_column + first + c];
+      ring[qk + first + c] = in[p.k_column + first + c];
+    }
+  }
+  for (int c = threadIdx.x; c < p.vdim; c += THREADS)
+    ring[2 * qk + head * p.vdim + c] = in[p.v_column + head * p.vdim + c];
+}
+template <typename T, int THREADS>
+__device__ __forceinline__ void keep_step_inputs(const RetentionInputs&, int, int64_t, int64_t, int) {}
 
 }  // namespace b200

@@ -43,6 +43,13 @@ class SequenceBatch:
     def decode(self) -> bool:
         return self.counts is None or max(self.counts) == 1
 
+    def context_bound(self, capacity: int) -> int:
+        """Upper bound of the positions any row of this step sees."""
+
+        if self.counts is None:
+            return capacity
+        return min(capacity, max(base + count for base, count in zip(self.bases_host, self.counts)))
+
     def pointers(self) -> Tuple[int, int, int, int]:
         return (self.token_sequence.data_ptr(), self.starts.data_ptr(), self.slots.data_ptr(),
                 self.bases.data_ptr())
@@ -142,25 +149,57 @@ def gated_head_norm(read_out: torch.Tensor, weight: Optional[torch.Tensor], gate
     return output
 
 
-def retention_prep(projected: torch.Tensor, batch: SequenceBatch, *, heads: int, dim: int, vdim: int,
-                   columns: Tuple[int, int, int], rot_dims: int, rot_base: float, k_scale: float):
-    """fp32 operands q, k [rows, heads, dim] (rotated, k scaled) and v [rows, heads, vdim] of a
-    retention layer from the columns (q, k, v) of its projection."""
+def retention_inputs(projected: torch.Tensor, decay: torch.Tensor, batch: SequenceBatch, *, heads: int, dim: int,
+                     vdim: int, columns: Tuple[int, int, int], rot_dims: int, rot_base: float,
+                     k_scale: float) -> "_lib.RetentionInputs":
+    """The argument block of the retention kernels: the columns (q, k, v) of the projections, the
+    rotation and the decay of every head."""
 
-    device = _require_cuda(projected)
+    _require_cuda(projected, decay)
     _require_rows(projected, "the projection")
-    rows = projected.shape[0]
-    q = torch.empty((rows, heads, dim), dtype=torch.float32, device=device)
+    if decay.dtype != torch.float32 or decay.shape != (heads,):
+        raise ValueError("retention needs one fp32 decay per head")
+    inputs = _lib.RetentionInputs(projected.data_ptr(), decay.data_ptr(), *batch.pointers(), heads, dim, vdim,
+                                  *columns, projected.stride(0), rot_dims, float(rot_base), float(k_scale))
+    inputs.tensors = (projected, decay, batch)  # alive as long as the block that points into them
+    return inputs
+
+
+def retention_prep(inputs: "_lib.RetentionInputs", rows: int, dtype: torch.dtype, device: torch.device):
+    """fp32 operands q, k [rows, heads, dim] (rotated, k scaled) and v [rows, heads, vdim]."""
+
+    q = torch.empty((rows, inputs.heads, inputs.dim), dtype=torch.float32, device=device)
     k = torch.empty_like(q)
-    v = torch.empty((rows, heads, vdim), dtype=torch.float32, device=device)
+    v = torch.empty((rows, inputs.heads, inputs.vdim), dtype=torch.float32, device=device)
     rt = runtime(device)
-    code = _lib.load().b200_retention_prep(
-        projected.data_ptr(), *batch.pointers(), q.data_ptr(), k.data_ptr(), v.data_ptr(), rows, heads, dim, vdim,
-        *columns, projected.stride(0), rot_dims, float(rot_base), float(k_scale), _code(projected.dtype),
-        _stream())
-    _check(code, "b200_retention_prep")
+    _check(_lib.load().b200_retention_prep(byref(inputs), q.data_ptr(), k.data_ptr(), v.data_ptr(), rows,
+                                           _code(dtype), _stream()), "b200_retention_prep")
     _count(rt)
     return q, k, v
+
+
+def recurrence_step(inputs, state: torch.Tensor, gate: torch.Tensor, weight: Optional[torch.Tensor],
+                    sequences: int, *, kind: str, epsilon: float) -> Optional[torch.Tensor]:
+    """Decode step of a recurrent mixer in one launch (inputs: retention_inputs or delta_inputs): state
+    update, read-out, per-head norm and gate. Returns [sequences, heads * vdim padded to 8], or None
+    where the state of a head is too large for the fused kernel."""
+
+    device = _require_cuda(state, gate, weight)
+    _require_rows(gate, "the gate")
+    if state.dtype != torch.float32 or state.ndim != 4 or not state.is_contiguous() or \
+            state.shape[1] != inputs.heads or state.shape[2] != inputs.dim or state.shape[3] < inputs.vdim:
+        raise ValueError("the state must be contiguous fp32 [slots, heads, dim, >= vdim]")
+    output = torch.empty((sequences, pad8(inputs.heads * inputs.vdim)), dtype=gate.dtype, device=device)
+    block = _lib.StepOutput(state.data_ptr(), gate.data_ptr(), _ptr(weight), output.data_ptr(), state.shape[3],
+                            gate.stride(0), output.stride(0), GATES[kind], float(epsilon))
+    rt = runtime(device)
+    call = _lib.load().b200_delta_step if isinstance(inputs, _lib.DeltaInputs) else _lib.load().b200_retention_step
+    code = call(byref(inputs), byref(block), sequences, _code(gate.dtype), _stream())
+    if code == _lib.ERR_UNSUPPORTED:
+        return None
+    _check(code, "recurrence step")
+    _count(rt)
+    return output
 
 
 def delta_inputs(projected: torch.Tensor, gates: torch.Tensor, conv: Tuple[torch.Tensor, torch.Tensor, torch.Tensor],
@@ -178,10 +217,12 @@ def delta_inputs(projected: torch.Tensor, gates: torch.Tensor, conv: Tuple[torch
         raise ValueError("the ring must hold `taps` inputs of every channel")
     if len({t.dtype for t in (projected, gates, *conv, a_log, dt_bias, ring)}) != 1:
         raise ValueError("projections, weights and ring must share one dtype")
-    return _lib.DeltaInputs(
+    inputs = _lib.DeltaInputs(
         projected.data_ptr(), gates.data_ptr(), conv[0].data_ptr(), conv[1].data_ptr(), conv[2].data_ptr(),
         a_log.data_ptr(), dt_bias.data_ptr(), ring.data_ptr(), *batch.pointers(), heads, kv_heads, dim, vdim, taps,
         *columns, decay_column, projected.stride(0), gates.stride(0), float(q_scale))
+    inputs.tensors = (projected, gates, conv, a_log, dt_bias, ring, batch)
+    return inputs
 
 
 def delta_prep(inputs: "_lib.DeltaInputs", rows: int, dtype: torch.dtype, device: torch.device):
@@ -263,11 +304,17 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, sink: Optional[torch.
         raise ValueError("queries and cached latents must be contiguous and of one row size and dtype")
     output = torch.empty_like(q)
     rt = runtime(device)
-    code = _lib.load().b200_latent_attention(
-        q.data_ptr(), cache.data_ptr(), _ptr(sink), output.data_ptr(), *batch.pointers(), rows, heads, row,
-        cache.shape[1], float(scale), _code(q.dtype), _stream())
+    library = _lib.load()
+    longest = 1 if batch.counts is None else max(batch.counts)
+    context = batch.context_bound(cache.shape[1])
+    need = int(library.b200_latent_attention_workspace_bytes(rows, batch.sequences, longest, heads, row, context,
+                                                            _code(q.dtype)))
+    workspace = rt.workspace("latent_attention", need)
+    code = library.b200_latent_attention(
+        q.data_ptr(), cache.data_ptr(), _ptr(sink), output.data_ptr(), *batch.pointers(), rows, batch.sequences,
+        longest, heads, row, cache.shape[1], context, float(scale), _code(q.dtype), _ptr(workspace), need, _stream())
     _check(code, "b200_latent_attention")
-    _count(rt)
+    _count(rt, 2 if need else 1)
     return output
 
 

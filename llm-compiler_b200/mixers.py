@@ -106,12 +106,18 @@ class Retention(Mixer):
 
     def __call__(self, h, batch, state):
         projected = kernels.b200_linear(h, self.w_in)
-        q, k, v = hk.retention_prep(projected, batch, heads=self.heads, dim=self.dim, vdim=self.vdim,
-                                    columns=self.columns, rot_dims=self.rot_dims, rot_base=self.rot_base,
-                                    k_scale=self.k_scale)
-        read_out = hk.recurrence_scan(q, k, v, None, self.decay, state["state"], batch)
-        mixed = hk.gated_head_norm(read_out, None, projected[:, self.gate_column:], kind="silu",
-                                   epsilon=self.epsilon)
+        inputs = hk.retention_inputs(projected, self.decay, batch, heads=self.heads, dim=self.dim, vdim=self.vdim,
+                                     columns=self.columns, rot_dims=self.rot_dims, rot_base=self.rot_base,
+                                     k_scale=self.k_scale)
+        gate = projected[:, self.gate_column:]
+        mixed = None
+        if batch.decode:
+            mixed = hk.recurrence_step(inputs, state["state"], gate, None, batch.sequences, kind="silu",
+                                       epsilon=self.epsilon)
+        if mixed is None:
+            q, k, v = hk.retention_prep(inputs, h.shape[0], h.dtype, h.device)
+            read_out = hk.recurrence_scan(q, k, v, None, self.decay, state["state"], batch)
+            mixed = hk.gated_head_norm(read_out, None, gate, kind="silu", epsilon=self.epsilon)
         return project_out(mixed, self.w_out)
 
 
@@ -145,11 +151,16 @@ class ChannelDelta(Mixer):
         inputs = hk.delta_inputs(projected, gates, self.conv, self.a_log, self.dt_bias, state["ring"], batch,
                                  heads=self.heads, kv_heads=self.kv_heads, dim=self.dim, vdim=self.vdim,
                                  columns=self.columns, decay_column=self.decay_column, q_scale=self.q_scale)
-        q, k, v, beta, log_decay = hk.delta_prep(inputs, h.shape[0], h.dtype, h.device)
-        read_out = hk.recurrence_scan(q, k, v, beta, log_decay, state["state"], batch)
-        hk.conv_tail(inputs, batch.sequences, h.dtype, h.device)
-        mixed = hk.gated_head_norm(read_out, self.norm, gates[:, self.gate_column:], kind="sigmoid",
-                                   epsilon=self.epsilon)
+        gate = gates[:, self.gate_column:]
+        mixed = None
+        if batch.decode:
+            mixed = hk.recurrence_step(inputs, state["state"], gate, self.norm, batch.sequences, kind="sigmoid",
+                                       epsilon=self.epsilon)
+        if mixed is None:
+            q, k, v, beta, log_decay = hk.delta_prep(inputs, h.shape[0], h.dtype, h.device)
+            read_out = hk.recurrence_scan(q, k, v, beta, log_decay, state["state"], batch)
+            hk.conv_tail(inputs, batch.sequences, h.dtype, h.device)
+            mixed = hk.gated_head_norm(read_out, self.norm, gate, kind="sigmoid", epsilon=self.epsilon)
         return project_out(mixed, self.w_out)
 
 
