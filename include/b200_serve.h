@@ -470,6 +470,9 @@ int b200_argmax(const void* logits, int64_t* ids, int64_t rows, int64_t vocab,
  *   b200_recurrence_scan token by token recurrence on prepared operands. beta NULL: retention, decay
  *                        is [heads]; otherwise the delta rule, decay is log g [rows, heads, dim]. State
  *                        [slots, heads, dim, state_row] is read, and written behind the last token.
+ *   b200_recurrence_chunked  the same results in chunks of 64 tokens on the tensor cores (operands split
+ *                        into two bf16 numbers each); chunk_starts (int32 [sequences + 1]): the first chunk
+ *                        of every sequence, `chunks` in all. dim up to 128, vdim up to 1024.
  *   b200_retention_step, b200_delta_step  a decode step (one row per sequence) in one launch: operands,
  *                        state update, read-out, norm and gate; the convolution inputs are kept too. With
  *                        B200_LAUNCH_STABLE_KV_PREFIX the state is read before the dependency wait (no
@@ -548,6 +551,14 @@ int b200_recurrence_scan(const float* q, const float* k, const float* v, const f
                          float* state, float* output, const int32_t* token_sequence, const int32_t* starts,
                          const int32_t* slots, const int32_t* bases, int64_t sequences, int64_t heads,
                          int64_t kv_heads, int64_t dim, int64_t vdim, int64_t state_row, void* stream);
+int64_t b200_recurrence_chunked_workspace_bytes(int64_t chunks, int64_t heads, int64_t dim, int64_t vdim,
+                                                int delta);
+int b200_recurrence_chunked(const float* q, const float* k, const float* v, const float* beta,
+                            const float* decay, float* state, float* output, const int32_t* token_sequence,
+                            const int32_t* starts, const int32_t* slots, const int32_t* bases,
+                            const int32_t* chunk_starts, int64_t chunks, int64_t sequences, int64_t heads,
+                            int64_t kv_heads, int64_t dim, int64_t vdim, int64_t state_row, void* workspace,
+                            int64_t workspace_bytes, void* stream);
 int b200_head_linear(const void* x, const void* w, void* y, int64_t m, int64_t heads, int64_t k, int64_t n,
                      int64_t x_row_stride, int64_t x_head_stride, int64_t y_row_stride,
                      int64_t y_head_stride, int dtype, void* stream);

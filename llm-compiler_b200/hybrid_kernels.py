@@ -14,6 +14,8 @@ import torch
 from . import _lib
 from .kernels import _check, _code, _count, _ptr, _require_cuda, _stream, runtime
 
+CHUNK = 64  # tokens of a chunk of recurrence_chunked
+CHUNKED_FROM = 24  # longest portion of a step from which the chunked form is the faster one
 GATES = {"silu": _lib.GATE_SILU, "sigmoid": _lib.GATE_SIGMOID}
 
 
@@ -38,10 +40,21 @@ class SequenceBatch:
     counts: Optional[List[int]] = None
     bases_host: Optional[List[int]] = None
     slots_host: Optional[List[int]] = None
+    _chunks: Optional[Tuple[torch.Tensor, int]] = None
 
     @property
     def decode(self) -> bool:
         return self.counts is None or max(self.counts) == 1
+
+    def chunk_table(self) -> Tuple[torch.Tensor, int]:
+        """First chunk of every sequence (int32 [sequences + 1]) and the number of chunks."""
+
+        if self._chunks is None:
+            table = [0]
+            for count in self.counts:
+                table.append(table[-1] + -(-count // CHUNK))
+            self._chunks = (torch.tensor(table, dtype=torch.int32).to(self.starts.device), table[-1])
+        return self._chunks
 
     def context_bound(self, capacity: int) -> int:
         """Upper bound of the positions any row of this step sees."""
@@ -270,6 +283,42 @@ def recurrence_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta: Opt
     _check(code, "b200_recurrence_scan")
     _count(rt)
     return output
+
+
+def recurrence_chunked(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta: Optional[torch.Tensor],
+                       decay: torch.Tensor, state: torch.Tensor, batch: SequenceBatch) -> Optional[torch.Tensor]:
+    """recurrence_scan in chunks of 64 tokens on the tensor cores; None where the sizes do not fit."""
+
+    device = _require_cuda(q, k, v, beta, decay, state)
+    rows, kv_heads, dim = q.shape
+    heads, vdim = v.shape[1], v.shape[2]
+    if state.dtype != torch.float32 or state.ndim != 4 or not state.is_contiguous() or \
+            state.shape[1] != heads or state.shape[2] != dim or state.shape[3] < vdim:
+        raise ValueError("the state must be contiguous fp32 [slots, heads, dim, >= vdim]")
+    library = _lib.load()
+    starts, chunks = batch.chunk_table()
+    need = int(library.b200_recurrence_chunked_workspace_bytes(chunks, heads, dim, vdim, int(beta is not None)))
+    if need == 0:
+        return None
+    output = torch.empty((rows, heads, vdim), dtype=torch.float32, device=device)
+    rt = runtime(device)
+    workspace = rt.workspace("recurrence_chunked", need)
+    code = library.b200_recurrence_chunked(
+        q.data_ptr(), k.data_ptr(), v.data_ptr(), _ptr(beta), decay.data_ptr(), state.data_ptr(), output.data_ptr(),
+        *batch.pointers(), starts.data_ptr(), chunks, batch.sequences, heads, kv_heads, dim, vdim, state.shape[3],
+        _ptr(workspace), need, _stream())
+    _check(code, "b200_recurrence_chunked")
+    _count(rt, 2)
+    return output
+
+
+def recurrence(q, k, v, beta, decay, state, batch: SequenceBatch, dtype: torch.dtype) -> torch.Tensor:
+    """The recurrence over a step's portions: chunked for prompts of 16-bit models, else token by token."""
+
+    output = None
+    if dtype == torch.bfloat16 and batch.counts is not None and max(batch.counts) >= CHUNKED_FROM:
+        output = recurrence_chunked(q, k, v, beta, decay, state, batch)
+    return recurrence_scan(q, k, v, beta, decay, state, batch) if output is None else output
 
 
 def head_linear(x: torch.Tensor, weight: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:

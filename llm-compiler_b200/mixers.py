@@ -116,7 +116,7 @@ class Retention(Mixer):
                                        epsilon=self.epsilon)
         if mixed is None:
             q, k, v = hk.retention_prep(inputs, h.shape[0], h.dtype, h.device)
-            read_out = hk.recurrence_scan(q, k, v, None, self.decay, state["state"], batch)
+            read_out = hk.recurrence(q, k, v, None, self.decay, state["state"], batch, h.dtype)
             mixed = hk.gated_head_norm(read_out, None, gate, kind="silu", epsilon=self.epsilon)
         return project_out(mixed, self.w_out)
 
@@ -158,7 +158,7 @@ class ChannelDelta(Mixer):
                                        epsilon=self.epsilon)
         if mixed is None:
             q, k, v, beta, log_decay = hk.delta_prep(inputs, h.shape[0], h.dtype, h.device)
-            read_out = hk.recurrence_scan(q, k, v, beta, log_decay, state["state"], batch)
+            read_out = hk.recurrence(q, k, v, beta, log_decay, state["state"], batch, h.dtype)
             hk.conv_tail(inputs, batch.sequences, h.dtype, h.device)
             mixed = hk.gated_head_norm(read_out, self.norm, gate, kind="sigmoid", epsilon=self.epsilon)
         return project_out(mixed, self.w_out)

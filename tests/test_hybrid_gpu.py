@@ -211,6 +211,35 @@ def test_delta_write_is_read_by_its_own_token_and_erased_by_the_next():
         close(run_mixer(mixer, h, cuts), want, torch.float32)
 
 
+@pytest.mark.parametrize("kind", ["retention", "delta"])
+@pytest.mark.parametrize("dim,vdim", [(64, 64), (40, 24), (128, 128), (100, 50)])
+def test_chunked_recurrence_equals_the_scan(kind, dim, vdim):
+    """The tensor-core form against the token-by-token fp32 scan on the same operands: split operands keep
+    far more than bf16 would. Several sequences of one step, one of them continued, strong and weak decays."""
+    heads, kv_heads = 4, 4 if kind == "retention" else 2
+    counts, bases = [1, 63, 64, 65, 200], [0, 5, 0, 64, 17]
+    batch = batch_of([(4 - i, bases[i], counts[i]) for i in range(5)])
+    g = torch.Generator(device="cuda").manual_seed(dim)
+    rand = lambda *shape: torch.randn(*shape, generator=g, device="cuda")
+    unit = lambda x: x / x.norm(dim=-1, keepdim=True)
+    q, k = unit(rand(batch.rows, kv_heads, dim)), unit(rand(batch.rows, kv_heads, dim))
+    v = rand(batch.rows, heads, vdim)
+    if kind == "retention":
+        beta, decay = None, torch.tensor([0.05, 0.9, 0.999, 1.0], device="cuda")
+    else:
+        beta = torch.sigmoid(rand(batch.rows, heads))
+        decay = -torch.exp(3 * rand(batch.rows, heads, dim) - 3)
+        decay[::7, 1] = -200.0  # a token that forgets everything
+    start = rand(5, heads, dim, (vdim + 3) // 4 * 4)
+    start[..., vdim:] = 0
+    states = [start.clone(), start.clone()]
+    want = hk.recurrence_scan(q, k, v, beta, decay, states[0], batch)
+    got = hk.recurrence_chunked(q, k, v, beta, decay, states[1], batch)
+    assert bool(torch.isfinite(got).all())
+    for a, b in ((got, want), (states[1], states[0])):
+        assert float((a - b).abs().max()) <= 2e-4 * float(b.abs().max())
+
+
 # ------------------------------------------------------------------- latent attention ----
 LATENT = [
     dict(heads=3, dim=24, vdim=40, q_rank=28, kv_rank=36, scale=0.2),
