@@ -288,6 +288,17 @@ int b200_prefill_attention(const void* query, const void* key, const void* value
                            void* workspace, int64_t workspace_bytes, int32_t* status,
                            void* stream);
 
+/* The causal form on tcgen05 for a portion of a sequence: `tokens` query rows behind `context` earlier
+ * positions, keys and values [B, Hkv, context + tokens, D]; row t sees positions 0 .. context + t. With
+ * sink (bf16 [Hq], NULL for none) the softmax denominator of head h also holds exp(sink[h]): no key, no
+ * value. bf16, head_dim 64 / 128, scale > 0, strides a tensor map can describe; else
+ * B200_ERR_UNSUPPORTED. output memory is B x T x Hq x D. No counterpart in the reference. */
+int b200_context_attention(const void* query, const void* key, const void* value, const void* sink,
+                           void* output, int64_t batch, int64_t q_heads, int64_t kv_heads, int64_t tokens,
+                           int64_t context, int64_t head_dim, const int64_t query_strides[4],
+                           const int64_t key_strides[4], const int64_t value_strides[4], double scale,
+                           int32_t* status, void* stream);
+
 /* ---- Linear ------------------------------------------------------------------
  * y[M,N] = x[M,K] * W[N,K]^T (+ bias[N]) with fp32 accumulation and an optional
  * fused epilogue. Replaces triton_linear (backends/triton_linear.py:87-148) and the

@@ -161,6 +161,8 @@ SIGNATURES = {
     "b200_recurrence_scan": (c_int, [c_void_p] * 11 + [c_int64] * 6 + [c_void_p]),
     "b200_recurrence_chunked_workspace_bytes": (c_int64, [c_int64] * 4 + [c_int]),
     "b200_recurrence_chunked": (c_int, [c_void_p] * 12 + [c_int64] * 7 + [c_void_p, c_int64, c_void_p]),
+    "b200_context_attention": (c_int, [c_void_p] * 5 + [c_int64] * 6 + [_I64P] * 3 +
+                               [c_double, c_void_p, c_void_p]),
     "b200_head_linear": (c_int, [c_void_p] * 3 + [c_int64] * 8 + [c_int, c_void_p]),
     "b200_latent_attention_workspace_bytes": (c_int64, [c_int64] * 6 + [c_int]),
     "b200_latent_attention": (c_int, [c_void_p] * 8 + [c_int64] * 7 + [c_double, c_int, c_void_p, c_int64, c_void_p]),

@@ -51,6 +51,8 @@ struct PrefillTcParams {
   __nv_bfloat16* out;  // [B, T, Hq, D]
   int32_t* status;
   int q_heads, groups, tokens;
+  int context = 0;  // keys in front of the first query row (causal form)
+  const __nv_bfloat16* sink = nullptr;  // [Hq]: exp(sink) joins the row sum (causal form)
   int q_token_dim1, k_token_dim1, v_token_dim1;  // coordinate order of the three tensor maps
   float scale_log2;
   // MASKED: additive fp32 mask with a contiguous last dimension; classes of its 128 x 128 tiles
@@ -143,12 +145,15 @@ prefill_attention_tcgen05_kernel(const PrefillTcParams p, const __grid_constant_
   const int hq = blockIdx.x, b = blockIdx.y;
   const int kvh = hq / p.groups;
   const int q0 = q_block * G * kTile;
-  const int all_tiles = (p.tokens + kTile - 1) / kTile;
+  const int context = MASKED ? 0 : p.context;
+  const int all_tiles = (context + p.tokens + kTile - 1) / kTile;
   // Key tiles are walked from `lo` on; `j` below counts from there (buffer slots and barrier
   // phases follow j, coordinates lo + j). causal: group g (query tile G q_block + g) needs key
-  // tiles 0 .. its own. MASKED: from the first to the last tile that is not all -inf for the
+  // tiles 0 .. the one that holds its last row's own position. MASKED: from the first to the last tile that is not all -inf for the
   // group's query tile (a group without any such tile still walks one, and yields NaN rows).
-  int lo = 0, tiles_0 = min(q_block * G + 1, all_tiles), tiles_1 = min(q_block * G + 2, all_tiles);
+  int lo = 0;
+  int tiles_0 = min((context + q0 + 2 * kTile - 1) / kTile, all_tiles);
+  int tiles_1 = min((context + q0 + 3 * kTile - 1) / kTile, all_tiles);
   const uint8_t* class_row[G] = {nullptr, nullptr};
   if (MASKED) {
     int first[G], last[G];
@@ -324,7 +329,7 @@ prefill_attention_tcgen05_kernel(const PrefillTcParams p, const __grid_constant_
     // rows and split the 128 key columns (and, where O is touched, its D columns) in halves.
     const int g = warp >> 3, half = (warp >> 2) & 1;
     const int row = ((warp & 3) << 5) | lane;
-    const int q_tile = q_block * G + g;
+    const int group_position = context + q0 + g * kTile;  // of the group's first row
     const int my_tiles = tiles_of(g);
     const uint32_t lane_base = static_cast<uint32_t>((warp & 3) * 32) << 16;
     const uint32_t s_taddr = s_column(g) + lane_base + half * 64;
@@ -417,11 +422,13 @@ prefill_attention_tcgen05_kernel(const PrefillTcParams p, const __grid_constant_
           else
             failed = 1;
         }
-        if (!MASKED && j == q_tile) {  // diagonal tile: keys beyond the row's own position are masked
+        if (!MASKED && (j + 1) * kTile - 1 > group_position) {
+          // a tile that reaches past the group's first row: keys beyond a row's own position are masked
+          const int last_key = group_position + row - j * kTile - key0;
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
-            if (key0 + i > row) s0[i] = 0xff800000u;
-            if (key0 + i + 32 > row) s1[i] = 0xff800000u;
+            if (i > last_key) s0[i] = 0xff800000u;
+            if (i + 32 > last_key) s1[i] = 0xff800000u;
           }
         }
         float max0 = -INFINITY, max1 = -INFINITY, max2 = -INFINITY, max3 = -INFINITY;
@@ -519,7 +526,10 @@ prefill_attention_tcgen05_kernel(const PrefillTcParams p, const __grid_constant_
       failed = 1;
     } else {
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-      const float inv = 1.0f / (l_run + row_sum_slot[(half ^ 1) * kTile + row]);
+      float row_sum = l_run + row_sum_slot[(half ^ 1) * kTile + row];
+      if (!MASKED && p.sink != nullptr)  // no key, no value: the denominator alone
+        row_sum += exp2_fast(fmaf(__bfloat162float(p.sink[hq]), kLog2e, -m_ref));
+      const float inv = 1.0f / row_sum;
       __nv_bfloat16* dst = p.out + ((static_cast<int64_t>(b) * p.tokens + q_row) * p.q_heads + hq) * D +
                            half * (D / 2);
 #pragma unroll
@@ -566,12 +576,15 @@ int prefill_attention_tcgen05(const void* query, const void* key, const void* va
                               int64_t head_dim, const int64_t query_strides[4],
                               const int64_t key_strides[4], const int64_t value_strides[4],
                               double scale, int32_t* status, cudaStream_t stream, const void* mask,
-                              const int64_t* mask_strides, void* workspace, int64_t workspace_bytes) {
+                              const int64_t* mask_strides, void* workspace, int64_t workspace_bytes,
+                              int64_t context, const void* sink) {
   if ((launch_mode() & B200_LAUNCH_PREFILL_WARP_LEVEL) != 0) return B200_ERR_UNSUPPORTED;
   const char* path = getenv("B200_PREFILL_ATTENTION_PATH");
   if (path != nullptr && strcmp(path, "mma.sync") == 0) return B200_ERR_UNSUPPORTED;
   if (head_dim != 64 && head_dim != 128) return B200_ERR_UNSUPPORTED;
   if (!(scale > 0.0) || tokens < 1) return B200_ERR_UNSUPPORTED;
+  if (context < 0 || context + tokens > (1 << 30) || (mask != nullptr && (context != 0 || sink != nullptr)))
+    return B200_ERR_UNSUPPORTED;
   const int64_t q_blocks = ceil_div(tokens, static_cast<int64_t>(kTile) * kGroups);
   if (q_blocks > 65535 || batch > 65535) return B200_ERR_UNSUPPORTED;
   const int64_t tiles = ceil_div(tokens, static_cast<int64_t>(kTile));
@@ -586,9 +599,9 @@ int prefill_attention_tcgen05(const void* query, const void* key, const void* va
   bool q_dim1, k_dim1, v_dim1;
   if (!make_bf16_bhtd_map(&q_map, query, batch, q_heads, tokens, head_dim, query_strides[0],
                           query_strides[1], query_strides[2], kTile, &q_dim1) ||
-      !make_bf16_bhtd_map(&k_map, key, batch, kv_heads, tokens, head_dim, key_strides[0],
+      !make_bf16_bhtd_map(&k_map, key, batch, kv_heads, context + tokens, head_dim, key_strides[0],
                           key_strides[1], key_strides[2], kTile, &k_dim1) ||
-      !make_bf16_bhtd_map(&v_map, value, batch, kv_heads, tokens, head_dim, value_strides[0],
+      !make_bf16_bhtd_map(&v_map, value, batch, kv_heads, context + tokens, head_dim, value_strides[0],
                           value_strides[1], value_strides[2], kTile, &v_dim1))
     return B200_ERR_UNSUPPORTED;
   PrefillTcParams p;
@@ -597,6 +610,8 @@ int prefill_attention_tcgen05(const void* query, const void* key, const void* va
   p.q_heads = static_cast<int>(q_heads);
   p.groups = static_cast<int>(q_heads / kv_heads);
   p.tokens = static_cast<int>(tokens);
+  p.context = static_cast<int>(context);
+  p.sink = static_cast<const __nv_bfloat16*>(sink);
   p.q_token_dim1 = q_dim1 ? 1 : 0;
   p.k_token_dim1 = k_dim1 ? 1 : 0;
   p.v_token_dim1 = v_dim1 ? 1 : 0;
@@ -639,3 +654,20 @@ int prefill_attention_tcgen05(const void* query, const void* key, const void* va
 }
 
 }  // namespace b200
+
+using namespace b200;
+
+extern "C" int b200_context_attention(const void* query, const void* key, const void* value, const void* sink,
+                                      void* output, int64_t batch, int64_t q_heads, int64_t kv_heads, int64_t tokens,
+                                      int64_t context, int64_t head_dim, const int64_t query_strides[4],
+                                      const int64_t key_strides[4], const int64_t value_strides[4], double scale,
+                                      int32_t* status, void* stream) {
+  if (!query || !key || !value || !output || !query_strides || !key_strides || !value_strides || batch <= 0 ||
+      q_heads <= 0 || kv_heads <= 0 || q_heads % kv_heads != 0 || tokens <= 0 || context < 0)
+    return B200_ERR_BAD_ARGUMENT;
+  if (query_strides[3] != 1 || key_strides[3] != 1 || value_strides[3] != 1) return B200_ERR_UNSUPPORTED;
+  if (!aligned16(query) || !aligned16(key) || !aligned16(value) || !aligned16(output)) return B200_ERR_ALIGNMENT;
+  return prefill_attention_tcgen05(query, key, value, output, batch, q_heads, kv_heads, tokens, head_dim,
+                                   query_strides, key_strides, value_strides, scale, status,
+                                   static_cast<cudaStream_t>(stream), nullptr, nullptr, nullptr, 0, context, sink);
+}

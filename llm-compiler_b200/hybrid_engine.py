@@ -9,6 +9,7 @@ graph per batch size."""
 
 from __future__ import annotations
 
+import os
 from typing import Dict, List, Optional, Sequence, Tuple
 
 import torch
@@ -49,6 +50,7 @@ class HybridEngine(ServingEngine):
         self._row_starts = torch.arange(batch + 1, **int32)
         self._row_sequence = torch.arange(batch, **int32)
         self._host_slots = torch.zeros(batch, dtype=torch.int32).pin_memory()
+        self.programmatic_launch = os.environ.get("B200_PROGRAMMATIC_LAUNCH", "1") != "0"
         self._row_graphs: Dict[int, Tuple[torch.cuda.CUDAGraph, torch.Tensor]] = {}
 
     # ------------------------------------------------------------------ the layers ----
@@ -96,9 +98,14 @@ class HybridEngine(ServingEngine):
         tokens whose logits are asked for (default: each entry's last). Returns the logits of the
         wanted places in order, [wanted, vocab] in the model dtype, or None if there are none."""
 
-        counts = [len(tokens) for _, tokens in entries]
         slots = [slot for slot, _ in entries]
-        if not entries or min(counts) == 0 or len(set(slots)) != len(slots):
+        counts = [len(tokens) for _, tokens in entries]
+        ids = torch.tensor([t for _, tokens in entries for t in tokens], dtype=torch.int64)
+        return self._forward_ids(ids, slots, counts, want, streams)
+
+    def _forward_ids(self, ids: torch.Tensor, slots: List[int], counts: List[int],
+                     want: Optional[Sequence[Sequence[int]]], streams: Optional[list] = None) -> Optional[torch.Tensor]:
+        if not slots or min(counts) == 0 or len(set(slots)) != len(slots):
             raise ValueError("every entry needs a slot of its own and at least one token")
         for slot, count in zip(slots, counts):
             self.state.require(slot, count)
@@ -106,18 +113,17 @@ class HybridEngine(ServingEngine):
         starts = [0]
         for count in counts:
             starts.append(starts[-1] + count)
-        rows = starts[-1]
-        ids = torch.tensor([t for _, tokens in entries for t in tokens], dtype=torch.int64).to(self.device)
-        packed = torch.tensor([i for i, count in enumerate(counts) for _ in range(count)] + starts + slots + bases,
-                              dtype=torch.int32).to(self.device)
-        n = len(entries)
-        batch = SequenceBatch(rows, n, packed[:rows], packed[rows:rows + n + 1],
-                              packed[rows + n + 1:rows + 2 * n + 1], packed[rows + 2 * n + 1:], counts, bases, slots)
+        rows, n = starts[-1], len(slots)
         if want is None:
             want = [[count - 1] for count in counts]
-        wanted = [starts[i] + place for i, places in enumerate(want) for place in places]
         if any(not 0 <= place < counts[i] for i, places in enumerate(want) for place in places):
             raise ValueError("a wanted place lies outside its entry")
+        wanted = [starts[i] + place for i, places in enumerate(want) for place in places]
+        ids = ids.to(self.device)
+        packed = torch.cat([torch.repeat_interleave(torch.arange(n, dtype=torch.int32), torch.tensor(counts)),
+                            torch.tensor(starts + slots + bases, dtype=torch.int32)]).to(self.device)
+        batch = SequenceBatch(rows, n, packed[:rows], packed[rows:rows + n + 1],
+                              packed[rows + n + 1:rows + 2 * n + 1], packed[rows + 2 * n + 1:], counts, bases, slots)
         x, _ = self._run_layers(ids, batch, None, streams)
         hk.advance_slots(self.state.lengths, batch, self.capacity)
         for slot, count in zip(slots, counts):
@@ -135,9 +141,14 @@ class HybridEngine(ServingEngine):
         before = kernels.launch_count(self.device)
         batch = SequenceBatch(rows, rows, self._row_sequence[:rows], self._row_starts[:rows + 1],
                               self.row_slots[:rows], self._row_bases[:rows])
-        hk.sequence_positions(self.state.lengths, batch.slots, batch.bases)
-        _, h = self._run_layers(self.input_ids[:rows], batch, self.final_norm)
-        logits = self._logits(h)
+        # The step opens with fully serialised launches (positions, embedding), weights are written once,
+        # and a layer's recurrent state by that layer's own step kernel only: the kernels behind may
+        # fetch weights and state before their predecessor has finished.
+        with kernels.launch_mode(programmatic=self.programmatic_launch, constant_weights=self.programmatic_launch,
+                                 stable_kv_prefix=self.programmatic_launch):
+            hk.sequence_positions(self.state.lengths, batch.slots, batch.bases)
+            _, h = self._run_layers(self.input_ids[:rows], batch, self.final_norm)
+            logits = self._logits(h)
         kernels.b200_argmax(logits, self.next_ids[:rows])
         hk.advance_slots(self.state.lengths, batch, self.capacity)
         self.kernels_per_step = kernels.launch_count(self.device) - before
@@ -164,8 +175,8 @@ class HybridEngine(ServingEngine):
             raise ValueError("prompt must be batch x tokens")
         self.state.reset_all()
         self.row_slots.copy_(torch.arange(self.batch, dtype=torch.int32))
-        prompts = input_ids.tolist()
-        self.logits = self.forward(list(enumerate(prompts)))
+        self.logits = self._forward_ids(input_ids.reshape(-1), list(range(self.batch)),
+                                        [input_ids.shape[1]] * self.batch, None)
         kernels.b200_argmax(self.logits, self.next_ids)
         self.input_ids.copy_(self.next_ids)
         return self.logits

@@ -6,7 +6,7 @@ synchronise, and there is no fallback to PyTorch."""
 from __future__ import annotations
 
 from ctypes import byref
-from dataclasses import dataclass
+from dataclasses import dataclass, field
 from typing import List, Optional, Tuple
 
 import torch
@@ -40,11 +40,18 @@ class SequenceBatch:
     counts: Optional[List[int]] = None
     bases_host: Optional[List[int]] = None
     slots_host: Optional[List[int]] = None
+    dense: dict = field(default_factory=dict)  # layer state -> this step's latents side by side
     _chunks: Optional[Tuple[torch.Tensor, int]] = None
 
     @property
     def decode(self) -> bool:
         return self.counts is None or max(self.counts) == 1
+
+    @property
+    def uniform_start(self) -> bool:
+        """Every portion starts its sequence and all are of one length."""
+
+        return self.counts is not None and not any(self.bases_host) and len(set(self.counts)) == 1
 
     def chunk_table(self) -> Tuple[torch.Tensor, int]:
         """First chunk of every sequence (int32 [sequences + 1]) and the number of chunks."""
@@ -365,6 +372,26 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, sink: Optional[torch.
     _check(code, "b200_latent_attention")
     _count(rt, 2 if need else 1)
     return output
+
+
+def context_attention(query: torch.Tensor, key: torch.Tensor, value: torch.Tensor, sink: Optional[torch.Tensor],
+                      output: torch.Tensor, *, context: int, scale: float) -> None:
+    """Causal attention of a portion on the tcgen05 prefill kernel: query B x H x T x D behind `context`
+    earlier positions, key / value B x Hkv x (context + T) x D (views), output memory B x T x H x D."""
+
+    device = _require_cuda(query, key, value, sink, output)
+    batch, heads, tokens, dim = query.shape
+    if key.shape != value.shape or key.shape[2] != context + tokens or key.shape[3] != dim:
+        raise ValueError("keys and values must hold the context and the portion")
+    if output.shape != (batch, tokens, heads, dim) or not output.is_contiguous():
+        raise ValueError("output must be a contiguous B x T x H x D tensor")
+    rt = runtime(device)
+    code = _lib.load().b200_context_attention(
+        query.data_ptr(), key.data_ptr(), value.data_ptr(), _ptr(sink), output.data_ptr(), batch, heads, key.shape[1],
+        tokens, context, dim, _lib.i64_array(query.stride()), _lib.i64_array(key.stride()),
+        _lib.i64_array(value.stride()), float(scale), rt.status.data_ptr(), _stream())
+    _check(code, "b200_context_attention")
+    _count(rt)
 
 
 def sequence_positions(lengths: torch.Tensor, slots: torch.Tensor, positions: torch.Tensor) -> None:

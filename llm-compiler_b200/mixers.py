@@ -17,6 +17,7 @@ from . import hybrid_kernels as hk
 from . import kernels
 from .hybrid_kernels import SequenceBatch, pad8
 
+ABSORBED_ROWS = 16  # longest portion that attends in the latent space (beyond: expanded keys and values)
 PARTIAL_ROWS = 128  # rows up to which a projection in front of a residual leaves split-K partials
 
 
@@ -180,11 +181,17 @@ class LatentAttention(Mixer):
         self.kv_norm = weights["dkv.norm"] if kv_from is None else None
         self.sink = weights["sink"].contiguous()
         self.q_size, self.v_size = pad8(dim), pad8(vdim)
+        # 16-bit prompts run on the tcgen05 prefill kernel where a head fits it: q, k and v of a head
+        # zero-padded to one size of 64 or 128
+        self.expandable = self.w_down.dtype == torch.bfloat16 and max(dim, vdim) <= 128 and scale > 0
+        if self.expandable:
+            self.q_size = self.v_size = 64 if max(dim, vdim) <= 64 else 128
         self.w_q = pad_matrix(pad_heads(weights["uq"], heads, self.q_size), heads * self.q_size, pad8(q_rank))
         key = pad_heads(pad_matrix(weights["uk"], heads * dim, self.rank_row), heads, self.q_size)
         value = pad_heads(pad_matrix(weights["uv"], heads * vdim, self.rank_row), heads, self.v_size)
         self.w_into = key.view(heads, self.q_size, self.rank_row).transpose(1, 2).contiguous()
         self.w_from = value.view(heads, self.v_size, self.rank_row).contiguous()
+        self.w_expand = torch.cat([key, value]).contiguous() if self.expandable else None
         out = pad_heads(weights["o"].t().contiguous(), heads, self.v_size).t()
         self.w_out = pad_matrix(out, pad8(width), heads * self.v_size)
         self.w_out = self.w_out.contiguous()
@@ -197,14 +204,44 @@ class LatentAttention(Mixer):
     def __call__(self, h, batch, state):
         down = kernels.b200_linear(h, self.w_down)
         cache = state["latent"]
-        query_latent, _ = hk.latent_norm(down, self.q_norm, self.kv_norm, cache, batch, kv_column=self.kv_column,
-                                         epsilon=self.epsilon)
+        expand = self.expandable and batch.counts is not None and max(batch.counts) > ABSORBED_ROWS
+        query_latent, dense = hk.latent_norm(down, self.q_norm, self.kv_norm, cache, batch,
+                                             kv_column=self.kv_column, epsilon=self.epsilon,
+                                             dense=expand and batch.uniform_start)
+        if dense is not None:
+            batch.dense[cache.data_ptr()] = dense
         rows = h.shape[0]
         q = kernels.b200_linear(query_latent, self.w_q).view(rows, self.heads, self.q_size)
-        absorbed = hk.head_linear(q, self.w_into)
-        weighted = hk.latent_attention(absorbed, cache, self.sink, batch, scale=self.scale)
-        values = hk.head_linear(weighted, self.w_from)
+        if expand:
+            values = self._attend_expanded(q, cache, batch)
+        else:
+            absorbed = hk.head_linear(q, self.w_into)
+            weighted = hk.latent_attention(absorbed, cache, self.sink, batch, scale=self.scale)
+            values = hk.head_linear(weighted, self.w_from)
         return project_out(values.view(rows, self.heads * self.v_size), self.w_out)
+
+    def _attend_expanded(self, q: torch.Tensor, cache: torch.Tensor, batch: SequenceBatch) -> torch.Tensor:
+        """Keys and values of a portion and everything before it expanded from the latents, then the
+        prefill kernel: one launch for equal whole prompts, else one per sequence."""
+
+        rows, heads, size = q.shape
+        output = torch.empty((rows, heads, size), dtype=q.dtype, device=q.device)
+        dense = batch.dense.get(cache.data_ptr()) if batch.uniform_start else None
+        if dense is not None:
+            groups = [(0, batch.sequences, batch.counts[0], 0, dense)]
+        else:
+            groups, first = [], 0
+            for slot, base, count in zip(batch.slots_host, batch.bases_host, batch.counts):
+                groups.append((first, 1, count, base, cache[slot, :base + count]))
+                first += count
+        for first, sequences, tokens, context, latents in groups:
+            expanded = kernels.b200_linear(latents, self.w_expand).view(sequences, context + tokens, 2 * heads, size)
+            part = slice(first, first + sequences * tokens)
+            hk.context_attention(q[part].view(sequences, tokens, heads, size).transpose(1, 2),
+                                 expanded[:, :, :heads].transpose(1, 2), expanded[:, :, heads:].transpose(1, 2),
+                                 self.sink, output[part].view(sequences, tokens, heads, size), context=context,
+                                 scale=self.scale)
+        return output
 
 
 class GatedMlp:

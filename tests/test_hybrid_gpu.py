@@ -314,6 +314,40 @@ def test_one_key_that_stands_out(dtype, rank, heads, tokens):
             assert seen == (position <= last + t)
 
 
+@pytest.mark.parametrize("size", [64, 128])
+@pytest.mark.parametrize("context", [0, 1, 63, 64, 127, 128, 129, 300])
+def test_portion_attention_on_the_prefill_kernel(size, context):
+    """Rows behind a context of any length: the diagonal crosses two key tiles. One key stands out, at
+    tile borders, at a row's own position and just beyond it; the sink takes its share."""
+    heads, tokens = 3, 150
+    g = torch.Generator().manual_seed(context + size)
+    q = torch.randn(1, heads, tokens, size, generator=g).to(torch.bfloat16)
+    k = (0.1 * torch.randn(1, heads, context + tokens, size, generator=g)).to(torch.bfloat16)
+    v = torch.randn(1, heads, context + tokens, size, generator=g).to(torch.bfloat16)
+    sink = torch.tensor([-20.0, 0.5, 4.0]).to(torch.bfloat16)
+    mark = torch.sign(torch.randn(size, generator=g)).to(torch.bfloat16)
+    q += mark
+    for position in {0, 127, 128, context, context + 1, context + 40, context + 149}:
+        if position >= context + tokens:
+            continue
+        marked = k.clone()
+        marked[0, :, position] = mark
+        for terms in (sink, None):
+            out = torch.empty(1, tokens, heads, size, dtype=torch.bfloat16, device="cuda")
+            hk.context_attention(q.cuda(), marked.cuda(), v.cuda(), None if terms is None else terms.cuda(), out,
+                                 context=context, scale=size ** -0.5)
+            kernels.runtime().check_status()
+            scores = torch.einsum("bhtd,bhkd->bhtk", q.double(), marked.double()) * size ** -0.5
+            seen = torch.arange(context + tokens)[None, :] <= context + torch.arange(tokens)[:, None]
+            scores.masked_fill_(~seen, -torch.inf)
+            extra = torch.full((1, heads, tokens, 1), -torch.inf, dtype=torch.float64)
+            if terms is not None:
+                extra = terms.double()[None, :, None, None].expand_as(extra)
+            weights = torch.softmax(torch.cat([scores, extra], -1), -1)[..., :-1]
+            want = torch.einsum("bhtk,bhkd->bthd", weights, v.double())
+            close(out[0], want[0], torch.bfloat16)
+
+
 @BOTH
 def test_layers_that_share_latents(dtype):
     """A layer that reads another layer's latents: its own W_uk, W_uv and queries on the other's rows."""
@@ -410,6 +444,18 @@ def test_first_tokens(dtype):
         want = oracle.forward(config.to_dict(), weights, tokens)
         close(run_cut(engine, tokens, [length]), want, dtype, MODEL_TOLERANCE[dtype])
         close(run_cut(engine, tokens, [1] * length), want, dtype, MODEL_TOLERANCE[dtype])
+
+
+def test_equal_prompts_in_one_step_equal_each_alone():
+    """Whole prompts of one length take one attention launch over the step's own latents."""
+    config = small_config()
+    engine, weights = model(config, torch.bfloat16)
+    prompts = [tokens_of(config, 140, s) for s in range(3)]
+    slots = [engine.open() for _ in prompts]
+    got = engine.forward(list(zip(slots, prompts)), [list(range(140))] * 3)
+    for i, prompt in enumerate(prompts):
+        close(got[140 * i:140 * (i + 1)], oracle.forward(config.to_dict(), weights, prompt), torch.bfloat16,
+              MODEL_TOLERANCE[torch.bfloat16])
 
 
 @BOTH
