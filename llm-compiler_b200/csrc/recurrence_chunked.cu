@@ -20,7 +20,9 @@ namespace b200 {
 namespace {
 
 constexpr int kChunk = 64, kSub = 16, kSubs = kChunk / kSub;
-constexpr int kIntraThreads = 256, kInterThreads = 256;
+constexpr int kIntraThreads = 512;
+template <int N>
+struct IntConstant { static constexpr int value = N; };
 
 struct ChunkParams {
   const float *q, *k, *v;   // [rows, kv_heads, dim] x 2, [rows, heads, vdim]
@@ -52,89 +54,218 @@ __device__ __forceinline__ void split_bf16x2(float a, float b, uint32_t& high, u
 }
 
 // ---- within the chunks -------------------------------------------------------------------
+constexpr int kTriangle = kChunk + 8;  // row pitch (bf16) of the solve's triangular planes
+constexpr int kInverse = kSub + 8;     // of the inverted 16 x 16 blocks
+
 template <int D>
 constexpr int intra_smem_bytes() {
-  return 4 * kChunk * (D + 4) * 4 + 2 * kChunk * (kChunk + 4) * 4 + (2 * kSub + (kSubs - 1) * kSub) * 2 * (D + 8) * 2;
+  constexpr int blocks = (2 * kSub + (kSubs - 1) * kSub) * 2 * (D + 8) * 2;
+  constexpr int solve = 2 * kChunk * kTriangle * 2 + 2 * kChunk * kInverse * 2;
+  return 4 * kChunk * (D + 4) * 4 + 2 * kChunk * (kChunk + 4) * 4 + 2 * kSubs * D * 4 + (blocks > solve ? blocks : solve);
 }
 
-template <int D, bool DELTA>
-__global__ void __launch_bounds__(kIntraThreads, 1) chunk_intra_kernel(const ChunkParams p) {
+// Which sequence a chunk belongs to, its first row and how many of its 64 rows exist.
+__device__ __forceinline__ int locate_chunk(const ChunkParams& p, int chunk, int64_t& row0) {
+  int sequence = 0;
+  while (sequence + 1 < p.sequences && p.chunk_starts[sequence + 1] <= chunk) ++sequence;
+  row0 = p.batch.starts[sequence] + static_cast<int64_t>(chunk - p.chunk_starts[sequence]) * kChunk;
+  const int64_t left = p.batch.starts[sequence + 1] - row0;
+  return left < kChunk ? static_cast<int>(left) : kChunk;
+}
+
+__device__ __forceinline__ float4 exp2_4(float4 x) {
+  return make_float4(exp2f(x.x), exp2f(x.y), exp2f(x.z), exp2f(x.w));
+}
+__device__ __forceinline__ float4 mul4(float4 a, float4 b) {
+  return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w);
+}
+__device__ __forceinline__ float4 add4(float4 a, float4 b) {
+  return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w);
+}
+__device__ __forceinline__ float dot4(float4 a, float4 b) {
+  return fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, a.w * b.w)));
+}
+__device__ __forceinline__ void split4(float4 v, uint2& high, uint2& low) {
+  split_bf16x2(v.x, v.y, high.x, low.x);
+  split_bf16x2(v.z, v.w, high.y, low.y);
+}
+// Four channels of a row of an operand; zeros outside
+__device__ __forceinline__ float4 load4(const float* source, int c, int dim, bool inside, bool whole) {
+  float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+  if (inside && whole) return *reinterpret_cast<const float4*>(source + c);
+  if (inside) {
+    if (c < dim) v.x = source[c];
+    if (c + 1 < dim) v.y = source[c + 1];
+    if (c + 2 < dim) v.z = source[c + 2];
+    if (c + 3 < dim) v.w = source[c + 3];
+  }
+  return v;
+}
+
+// Retention: one decay per head, so the decayed products are the plain ones times decay^(i - j).
+template <int D>
+__global__ void __launch_bounds__(kIntraThreads) chunk_intra_retention_kernel(const ChunkParams p) {
+  constexpr int PB = (D + 8) * 2;
+  using Layout = ChunkLayout<D>;
+  extern __shared__ __align__(128) unsigned char smem[];
+  unsigned char* q_planes = smem;                          // [2][64][PB]
+  unsigned char* k_planes = smem + 2 * kChunk * PB;
+  const int chunk = blockIdx.x, head = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  int64_t row0;
+  const int count = locate_chunk(p, chunk, row0);
+  const int kv_head = head / (p.heads / p.kv_heads);
+  unsigned char* out = p.workspace + (static_cast<int64_t>(chunk) * p.heads + head) * Layout::bytes(false, p.vdim);
+  const float decay = fmaxf(log2f(p.decay[head]), -126.0f);  // (less than 2^-126 is nothing)
+  const bool whole = p.dim == D;
+#pragma unroll
+  for (int i = 0; i < kChunk * D / 4 / kIntraThreads; ++i) {
+    const int item = threadIdx.x + i * kIntraThreads, t = item / (D / 4), c = item % (D / 4) * 4;
+    const int64_t source = ((row0 + t) * p.kv_heads + kv_head) * p.dim;
+    const float4 q = load4(p.q + source, c, p.dim, t < count, whole), k = load4(p.k + source, c, p.dim, t < count, whole);
+    const float into = exp2f(decay * (t + 1)), rest = t < count ? exp2f(decay * (count - 1 - t)) : 0.0f;
+    uint2 high, low;
+    split4(q, high, low);
+    *reinterpret_cast<uint2*>(q_planes + t * PB + c * 2) = high;
+    *reinterpret_cast<uint2*>(q_planes + (kChunk + t) * PB + c * 2) = low;
+    split4(k, high, low);
+    *reinterpret_cast<uint2*>(k_planes + t * PB + c * 2) = high;
+    *reinterpret_cast<uint2*>(k_planes + (kChunk + t) * PB + c * 2) = low;
+    split4(mul4(q, make_float4(into, into, into, into)), high, low);
+    reinterpret_cast<uint2*>(out + Layout::kQ)[item] = high;
+    reinterpret_cast<uint2*>(out + Layout::kQ + Layout::kPlane)[item] = low;
+    split4(mul4(k, make_float4(rest, rest, rest, rest)), high, low);
+    reinterpret_cast<uint2*>(out + Layout::kK)[item] = high;
+    reinterpret_cast<uint2*>(out + Layout::kK + Layout::kPlane)[item] = low;
+  }
+  if (threadIdx.x < D) reinterpret_cast<float*>(out + Layout::kEnd)[threadIdx.x] = exp2f(decay * count);
+  __syncthreads();
+  // 16 warps: 16 rows x 16 columns each
+  const int m0 = (warp >> 2) * 16, n0 = (warp & 3) * 16;
+  float acc[2][4] = {};
+  if (n0 <= m0) {
+    const uint32_t a_base = smem_u32(q_planes) + (m0 + (lane & 15)) * PB + (lane >> 4) * 16;
+    const uint32_t b_base = smem_u32(k_planes) + (n0 + ((lane >> 4) << 3) + (lane & 7)) * PB + ((lane >> 3) & 1) * 16;
+#pragma unroll
+    for (int step = 0; step < D / 16; ++step) {
+      uint32_t ah[4], al[4], bh[4], bl[4];
+      ldmatrix_x4(ah, a_base + step * 32);
+      ldmatrix_x4(al, a_base + kChunk * PB + step * 32);
+      ldmatrix_x4(bh, b_base + step * 32);
+      ldmatrix_x4(bl, b_base + kChunk * PB + step * 32);
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        mma_bf16_16816(acc[h], ah, bh[h * 2], bh[h * 2 + 1]);
+        mma_bf16_16816(acc[h], ah, bl[h * 2], bl[h * 2 + 1]);
+        mma_bf16_16816(acc[h], al, bh[h * 2], bh[h * 2 + 1]);
+      }
+    }
+  }
+#pragma unroll
+  for (int h = 0; h < 2; ++h)
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int i = m0 + (lane >> 2) + half * 8, j = n0 + h * 8 + (lane & 3) * 2;
+      const float a = i >= j ? acc[h][half * 2] * exp2f(decay * (i - j)) : 0.0f;
+      const float b = i >= j + 1 ? acc[h][half * 2 + 1] * exp2f(decay * (i - j - 1)) : 0.0f;
+      uint32_t high, low;
+      split_bf16x2(a, b, high, low);
+      reinterpret_cast<uint32_t*>(out + Layout::kA)[(i * kChunk + j) / 2] = high;
+      reinterpret_cast<uint32_t*>(out + Layout::kA + Layout::kSquare)[(i * kChunk + j) / 2] = low;
+    }
+}
+
+template <int D>
+__global__ void __launch_bounds__(kIntraThreads, 1) chunk_intra_delta_kernel(const ChunkParams p) {
   constexpr int PD = D + 4, PM = kChunk + 4, PB = (D + 8) * 2;  // pitches: floats, floats, bytes
+  constexpr int kRounds = kChunk * D / 4 / kIntraThreads;        // float4 items of a [64][D] array per thread
   using Layout = ChunkLayout<D>;
   extern __shared__ __align__(128) unsigned char smem[];
   float* ks = reinterpret_cast<float*>(smem);       // [64][PD]
-  float* qs = ks + kChunk * PD;
+  float* qs = ks + kChunk * PD;                     // later the staging of W's planes
   float* xs = qs + kChunk * PD;                     // log2 g, later its running sum within 16 tokens
   float* gs = xs + kChunk * PD;                     // g, later the sum of log2 g over the rest of the 16 tokens
   float* lower = gs + kChunk * PD;                  // [64][PM] beta_i k_i . (P_i / P_j) k_j, j < i
   float* mixed = lower + kChunk * PM;               // [64][PM] q_i . (P_i / P_j) k_j, j <= i
-  unsigned char* planes = reinterpret_cast<unsigned char*>(mixed + kChunk * PM);
+  float* pre = mixed + kChunk * PM;                 // [4][D] log2 of the decay in front of 16 tokens
+  float* post = pre + kSubs * D;                    // [4][D] ... behind them
+  unsigned char* planes = reinterpret_cast<unsigned char*>(post + kSubs * D);
   __shared__ float betas[kChunk];
-  __shared__ int sequence_slot;
   const int chunk = blockIdx.x, head = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  if (threadIdx.x == 0) {
-    int s = 0;
-    while (s + 1 < p.sequences && p.chunk_starts[s + 1] <= chunk) ++s;
-    sequence_slot = s;
-  }
-  __syncthreads();
-  const int sequence = sequence_slot;
-  const int64_t row0 = p.batch.starts[sequence] + static_cast<int64_t>(chunk - p.chunk_starts[sequence]) * kChunk;
-  const int64_t left = p.batch.starts[sequence + 1] - row0;
-  const int count = left < kChunk ? static_cast<int>(left) : kChunk;
+  int64_t row0;
+  const int count = locate_chunk(p, chunk, row0);
   const int kv_head = head / (p.heads / p.kv_heads);
-  unsigned char* out = p.workspace + (static_cast<int64_t>(chunk) * p.heads + head) * Layout::bytes(DELTA, p.vdim);
-  const float head_decay = DELTA ? 0.0f : fmaxf(log2f(p.decay[head]), -126.0f);
-  for (int item = threadIdx.x; item < kChunk * D; item += kIntraThreads) {
-    const int t = item / D, c = item % D;
-    const bool inside = t < count && c < p.dim;
-    const int64_t source = inside ? ((row0 + t) * p.kv_heads + kv_head) * p.dim + c : 0;
-    ks[t * PD + c] = inside ? p.k[source] : 0.0f;
-    qs[t * PD + c] = inside ? p.q[source] : 0.0f;
-    // (a token that keeps less than 2^-126 keeps nothing)
-    float x = 0.0f;
-    if (DELTA) x = inside ? fmaxf(p.decay[((row0 + t) * p.heads + head) * p.dim + c] * 1.4426950408889634f, -126.0f) : 0.0f;
-    else x = t < count ? head_decay : 0.0f;
-    xs[t * PD + c] = x;
-    gs[t * PD + c] = exp2f(x);
+  unsigned char* out = p.workspace + (static_cast<int64_t>(chunk) * p.heads + head) * Layout::bytes(true, p.vdim);
+  const bool whole = p.dim == D;
+  {
+    float4 k[kRounds], q[kRounds], x[kRounds];
+#pragma unroll
+    for (int i = 0; i < kRounds; ++i) {
+      const int item = threadIdx.x + i * kIntraThreads, t = item / (D / 4), c = item % (D / 4) * 4;
+      const int64_t source = ((row0 + t) * p.kv_heads + kv_head) * p.dim;
+      k[i] = load4(p.k + source, c, p.dim, t < count, whole);
+      q[i] = load4(p.q + source, c, p.dim, t < count, whole);
+      x[i] = load4(p.decay + ((row0 + t) * p.heads + head) * p.dim, c, p.dim, t < count, whole);
+    }
+    if (threadIdx.x < kChunk)
+      betas[threadIdx.x] = threadIdx.x < count ? p.beta[(row0 + threadIdx.x) * p.heads + head] : 0.0f;
+    for (int item = threadIdx.x; item < kChunk * PM / 4; item += kIntraThreads)
+      reinterpret_cast<float4*>(mixed)[item] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    constexpr float kLog2e = 1.4426950408889634f;
+#pragma unroll
+    for (int i = 0; i < kRounds; ++i) {
+      const int item = threadIdx.x + i * kIntraThreads, at = item / (D / 4) * PD + item % (D / 4) * 4;
+      // (a token that keeps less than 2^-126 keeps nothing)
+      const float4 l = make_float4(fmaxf(x[i].x * kLog2e, -126.0f), fmaxf(x[i].y * kLog2e, -126.0f),
+                                   fmaxf(x[i].z * kLog2e, -126.0f), fmaxf(x[i].w * kLog2e, -126.0f));
+      *reinterpret_cast<float4*>(ks + at) = k[i];
+      *reinterpret_cast<float4*>(qs + at) = q[i];
+      *reinterpret_cast<float4*>(xs + at) = l;
+      *reinterpret_cast<float4*>(gs + at) = exp2_4(l);
+    }
   }
-  if (threadIdx.x < kChunk)
-    betas[threadIdx.x] = DELTA && threadIdx.x < count ? p.beta[(row0 + threadIdx.x) * p.heads + head] : 0.0f;
-  for (int item = threadIdx.x; item < kChunk * PM; item += kIntraThreads) mixed[item] = 0.0f;
   __syncthreads();
 
   // ---- the 16 x 16 blocks on the diagonal: w = (P_i / P_j) k_j built up token by token ----
-  {
-    const int column = threadIdx.x >> 2, part = threadIdx.x & 3;  // four lanes a column, a quarter of the channels each
-    const int block = column / kSub * kSub, j = column % kSub;
-    float4 w[D / 16];
+  // D / 4 lanes share four columns j of a block, four channels each; their eight sums per row are
+  // reduced together, every exchange halving the number of sums a lane still carries.
+  constexpr int LG = D / 4;
+  if (static_cast<int>(threadIdx.x) / LG < 16) {
+    const int group = threadIdx.x / LG, l = threadIdx.x % LG;
+    const int block = group / 4 * kSub, j0 = group % 4 * 4;
+    float4 w[4];
 #pragma unroll
-    for (int m = 0; m < D / 16; ++m) w[m] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    for (int jj = 0; jj < 4; ++jj) w[jj] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
     for (int i = 0; i < kSub; ++i) {
-      const int at = (block + i) * PD + part * 4;
-      float along_k = 0.0f, along_q = 0.0f;
+      const int at = (block + i) * PD + l * 4;
+      const float4 kk = *reinterpret_cast<const float4*>(ks + at);
+      const float4 qq = *reinterpret_cast<const float4*>(qs + at);
+      const float4 gg = *reinterpret_cast<const float4*>(gs + at);
+      float v[8];
 #pragma unroll
-      for (int m = 0; m < D / 16; ++m) {
-        const float4 kk = *reinterpret_cast<const float4*>(ks + at + m * 16);
-        const float4 qq = *reinterpret_cast<const float4*>(qs + at + m * 16);
-        const float4 gg = *reinterpret_cast<const float4*>(gs + at + m * 16);
-        if (i == j) {
-          w[m] = kk;
-        } else {
-          w[m].x *= gg.x; w[m].y *= gg.y; w[m].z *= gg.z; w[m].w *= gg.w;
-        }
-        if (DELTA) along_k += kk.x * w[m].x + kk.y * w[m].y + kk.z * w[m].z + kk.w * w[m].w;
-        along_q += qq.x * w[m].x + qq.y * w[m].y + qq.z * w[m].z + qq.w * w[m].w;
+      for (int jj = 0; jj < 4; ++jj) {
+        w[jj] = i == j0 + jj ? kk : mul4(w[jj], gg);
+        v[jj] = dot4(kk, w[jj]);
+        v[4 + jj] = dot4(qq, w[jj]);
       }
-      along_q += __shfl_xor_sync(0xffffffffu, along_q, 1);
-      along_q += __shfl_xor_sync(0xffffffffu, along_q, 2);
-      if (DELTA) {
-        along_k += __shfl_xor_sync(0xffffffffu, along_k, 1);
-        along_k += __shfl_xor_sync(0xffffffffu, along_k, 2);
+      const bool is_q = (l & (LG / 2)) != 0, second = (l & (LG / 4)) != 0, odd = (l & (LG / 8)) != 0;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float received = __shfl_xor_sync(0xffffffffu, is_q ? v[e] : v[4 + e], LG / 2);
+        v[e] = (is_q ? v[4 + e] : v[e]) + received;
       }
-      if (part == 0) {
-        if (DELTA) lower[(block + i) * PM + column] = i > j ? along_k * betas[block + i] : 0.0f;
-        mixed[(block + i) * PM + column] = i >= j ? along_q : 0.0f;
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const float received = __shfl_xor_sync(0xffffffffu, second ? v[e] : v[2 + e], LG / 4);
+        v[e] = (second ? v[2 + e] : v[e]) + received;
+      }
+      const float received = __shfl_xor_sync(0xffffffffu, odd ? v[0] : v[1], LG / 8);
+      float sum = (odd ? v[1] : v[0]) + received;
+#pragma unroll
+      for (int o = LG / 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+      if ((l & (LG / 8 - 1)) == 0) {
+        const int j = j0 + (second ? 2 : 0) + (odd ? 1 : 0), at_m = (block + i) * PM + block + j;
+        if (is_q) mixed[at_m] = i >= j ? sum : 0.0f;
+        else lower[at_m] = i > j ? sum * betas[block + i] : 0.0f;
       }
     }
   }
@@ -142,29 +273,39 @@ __global__ void __launch_bounds__(kIntraThreads, 1) chunk_intra_kernel(const Chu
   // ---- running sums of log2 g within 16 tokens, forwards (inclusive) and backwards (exclusive) ----
   for (int item = threadIdx.x; item < kSubs * D; item += kIntraThreads) {
     const int at = item / D * kSub * PD + item % D;
+    float x[kSub];
+#pragma unroll
+    for (int i = 0; i < kSub; ++i) x[i] = xs[at + i * PD];
     float sum = 0.0f;
+#pragma unroll
     for (int i = kSub - 1; i >= 0; --i) {
       gs[at + i * PD] = sum;
-      sum += xs[at + i * PD];
+      sum += x[i];
     }
     sum = 0.0f;
+#pragma unroll
     for (int i = 0; i < kSub; ++i) {
-      sum += xs[at + i * PD];
+      sum += x[i];
       xs[at + i * PD] = sum;
     }
   }
   __syncthreads();
-  auto total = [&](int sub, int c) { return xs[(sub * kSub + kSub - 1) * PD + c]; };
-  auto before = [&](int t, int c) {  // log2 P_t
-    float sum = xs[t * PD + c];
-    for (int s = 0; s < t / kSub; ++s) sum += total(s, c);
-    return sum;
-  };
-  auto after = [&](int t, int c) {  // log2 (P_last / P_t)
-    float sum = gs[t * PD + c];
-    for (int s = t / kSub + 1; s < kSubs; ++s) sum += total(s, c);
-    return sum;
-  };
+  for (int c = threadIdx.x; c < D; c += kIntraThreads) {
+    float total[kSubs], sum = 0.0f;
+#pragma unroll
+    for (int s = 0; s < kSubs; ++s) {
+      total[s] = xs[(s * kSub + kSub - 1) * PD + c];
+      pre[s * D + c] = sum;
+      sum += total[s];
+    }
+    reinterpret_cast<float*>(out + Layout::kEnd)[c] = exp2f(sum);
+    sum = 0.0f;
+#pragma unroll
+    for (int s = kSubs - 1; s >= 0; --s) {
+      post[s * D + c] = sum;
+      sum += total[s];
+    }
+  }
 
   // ---- the blocks below the diagonal, on the tensor cores ----
   unsigned char* rows_k = planes;                      // [2][16][PB] k_i decayed from the block's start
@@ -172,39 +313,35 @@ __global__ void __launch_bounds__(kIntraThreads, 1) chunk_intra_kernel(const Chu
   unsigned char* columns = rows_q + 2 * kSub * PB;     // [2][48][PB] k_j decayed to the block's start
   constexpr int kColumnRows = (kSubs - 1) * kSub;
   for (int block = 1; block < kSubs; ++block) {
-    for (int item = threadIdx.x; item < kSub * D / 2; item += kIntraThreads) {
-      const int i = item / (D / 2), c = item % (D / 2) * 2, at = (block * kSub + i) * PD + c;
-      const float f0 = exp2f(xs[at]), f1 = exp2f(xs[at + 1]);
-      uint32_t high, low;
-      if (DELTA) {
-        split_bf16x2(ks[at] * f0, ks[at + 1] * f1, high, low);
-        *reinterpret_cast<uint32_t*>(rows_k + i * PB + c * 2) = high;
-        *reinterpret_cast<uint32_t*>(rows_k + (kSub + i) * PB + c * 2) = low;
-      }
-      split_bf16x2(qs[at] * f0, qs[at + 1] * f1, high, low);
-      *reinterpret_cast<uint32_t*>(rows_q + i * PB + c * 2) = high;
-      *reinterpret_cast<uint32_t*>(rows_q + (kSub + i) * PB + c * 2) = low;
+    for (int item = threadIdx.x; item < kSub * D / 4; item += kIntraThreads) {
+      const int i = item / (D / 4), c = item % (D / 4) * 4, at = (block * kSub + i) * PD + c;
+      const float4 f = exp2_4(*reinterpret_cast<const float4*>(xs + at));
+      uint2 high, low;
+      split4(mul4(*reinterpret_cast<const float4*>(ks + at), f), high, low);
+      *reinterpret_cast<uint2*>(rows_k + i * PB + c * 2) = high;
+      *reinterpret_cast<uint2*>(rows_k + (kSub + i) * PB + c * 2) = low;
+      split4(mul4(*reinterpret_cast<const float4*>(qs + at), f), high, low);
+      *reinterpret_cast<uint2*>(rows_q + i * PB + c * 2) = high;
+      *reinterpret_cast<uint2*>(rows_q + (kSub + i) * PB + c * 2) = low;
     }
-    for (int item = threadIdx.x; item < block * kSub * D / 2; item += kIntraThreads) {
-      const int j = item / (D / 2), c = item % (D / 2) * 2, at = j * PD + c;
-      float e0 = gs[at], e1 = gs[at + 1];
-      for (int s = j / kSub + 1; s < block; ++s) {
-        e0 += total(s, c);
-        e1 += total(s, c + 1);
-      }
-      uint32_t high, low;
-      split_bf16x2(ks[at] * exp2f(e0), ks[at + 1] * exp2f(e1), high, low);
-      *reinterpret_cast<uint32_t*>(columns + j * PB + c * 2) = high;
-      *reinterpret_cast<uint32_t*>(columns + (kColumnRows + j) * PB + c * 2) = low;
+    for (int item = threadIdx.x; item < block * kSub * D / 4; item += kIntraThreads) {
+      const int j = item / (D / 4), c = item % (D / 4) * 4, at = j * PD + c;
+      float4 e = *reinterpret_cast<const float4*>(gs + at);
+      for (int s = j / kSub + 1; s < block; ++s)
+        e = add4(e, *reinterpret_cast<const float4*>(xs + (s * kSub + kSub - 1) * PD + c));
+      uint2 high, low;
+      split4(mul4(*reinterpret_cast<const float4*>(ks + at), exp2_4(e)), high, low);
+      *reinterpret_cast<uint2*>(columns + j * PB + c * 2) = high;
+      *reinterpret_cast<uint2*>(columns + (kColumnRows + j) * PB + c * 2) = low;
     }
     __syncthreads();
     const int tiles = block * 2;  // n8 tiles of a matrix
-    for (int tile = warp; tile < (DELTA ? 2 : 1) * tiles; tile += kIntraThreads / 32) {
+    for (int tile = warp; tile < 2 * tiles; tile += kIntraThreads / 32) {
       const bool is_q = tile < tiles;
       const int n0 = (is_q ? tile : tile - tiles) * 8;
       const uint32_t a_base = smem_u32(is_q ? rows_q : rows_k) + (lane & 15) * PB + (lane >> 4) * 16;
       const uint32_t b_base = smem_u32(columns) + (n0 + (lane & 7)) * PB + ((lane >> 3) & 1) * 16 + (lane >> 4) * kColumnRows * PB;
-      float acc[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+      float acc[4] = {0.0f, 0.0f, 0.0f, 0.0f}, cross[4] = {0.0f, 0.0f, 0.0f, 0.0f};
 #pragma unroll
       for (int step = 0; step < D / 16; ++step) {
         uint32_t ah[4], al[4], b[4];  // b: high (two registers), low
@@ -212,86 +349,137 @@ __global__ void __launch_bounds__(kIntraThreads, 1) chunk_intra_kernel(const Chu
         ldmatrix_x4(al, a_base + kSub * PB + step * 32);
         ldmatrix_x4(b, b_base + step * 32);
         mma_bf16_16816(acc, ah, b[0], b[1]);
-        mma_bf16_16816(acc, ah, b[2], b[3]);
-        mma_bf16_16816(acc, al, b[0], b[1]);
+        mma_bf16_16816(cross, ah, b[2], b[3]);
+        mma_bf16_16816(cross, al, b[0], b[1]);
       }
       float* matrix = is_q ? mixed : lower;
       const int r0 = block * kSub + (lane >> 2), c0 = n0 + (lane & 3) * 2;
       const float s0 = is_q ? 1.0f : betas[r0], s1 = is_q ? 1.0f : betas[r0 + 8];
-      matrix[r0 * PM + c0] = acc[0] * s0;
-      matrix[r0 * PM + c0 + 1] = acc[1] * s0;
-      matrix[(r0 + 8) * PM + c0] = acc[2] * s1;
-      matrix[(r0 + 8) * PM + c0 + 1] = acc[3] * s1;
+      *reinterpret_cast<float2*>(matrix + r0 * PM + c0) = make_float2((acc[0] + cross[0]) * s0, (acc[1] + cross[1]) * s0);
+      *reinterpret_cast<float2*>(matrix + (r0 + 8) * PM + c0) = make_float2((acc[2] + cross[2]) * s1, (acc[3] + cross[3]) * s1);
     }
     __syncthreads();
   }
 
-  // ---- decayed operands of the second kernel ----
-  for (int item = threadIdx.x; item < kChunk * D / 2; item += kIntraThreads) {
-    const int t = item / (D / 2), c = item % (D / 2) * 2, at = t * PD + c;
-    uint32_t high, low;
-    split_bf16x2(qs[at] * exp2f(before(t, c)), qs[at + 1] * exp2f(before(t, c + 1)), high, low);
-    reinterpret_cast<uint32_t*>(out + Layout::kQ)[item] = high;
-    reinterpret_cast<uint32_t*>(out + Layout::kQ + Layout::kPlane)[item] = low;
-    split_bf16x2(ks[at] * exp2f(after(t, c)), ks[at + 1] * exp2f(after(t, c + 1)), high, low);
-    reinterpret_cast<uint32_t*>(out + Layout::kK)[item] = high;
-    reinterpret_cast<uint32_t*>(out + Layout::kK + Layout::kPlane)[item] = low;
+  // ---- decayed operands of the second kernel; planes of the solve ----
+#pragma unroll
+  for (int i = 0; i < kRounds; ++i) {
+    const int item = threadIdx.x + i * kIntraThreads, t = item / (D / 4), c = item % (D / 4) * 4, at = t * PD + c;
+    const float4 into = add4(*reinterpret_cast<const float4*>(xs + at), *reinterpret_cast<const float4*>(pre + t / kSub * D + c));
+    const float4 rest = add4(*reinterpret_cast<const float4*>(gs + at), *reinterpret_cast<const float4*>(post + t / kSub * D + c));
+    uint2 high, low;
+    split4(mul4(*reinterpret_cast<const float4*>(qs + at), exp2_4(into)), high, low);
+    reinterpret_cast<uint2*>(out + Layout::kQ)[item] = high;
+    reinterpret_cast<uint2*>(out + Layout::kQ + Layout::kPlane)[item] = low;
+    split4(mul4(*reinterpret_cast<const float4*>(ks + at), exp2_4(rest)), high, low);
+    reinterpret_cast<uint2*>(out + Layout::kK)[item] = high;
+    reinterpret_cast<uint2*>(out + Layout::kK + Layout::kPlane)[item] = low;
   }
-  for (int item = threadIdx.x; item < kChunk * kChunk / 2; item += kIntraThreads) {
-    const int i = item / (kChunk / 2), j = item % (kChunk / 2) * 2;
-    uint32_t high, low;
-    split_bf16x2(mixed[i * PM + j], mixed[i * PM + j + 1], high, low);
-    reinterpret_cast<uint32_t*>(out + Layout::kA)[item] = high;
-    reinterpret_cast<uint32_t*>(out + Layout::kA + Layout::kSquare)[item] = low;
-  }
-  for (int c = threadIdx.x; c < D; c += kIntraThreads)
-    reinterpret_cast<float*>(out + Layout::kEnd)[c] = exp2f(before(kChunk - 1, c));
-
-  // ---- triangular solve, one column of (P k | v) a thread ----
-  if (DELTA) {
-    const int v_row = (p.vdim + 31) / 32 * 32;
-    for (int column = threadIdx.x; column < D + v_row; column += kIntraThreads) {
-      float x[kChunk];
-      if (column < D) {
-        float base = 0.0f;
-#pragma unroll
-        for (int i = 0; i < kChunk; ++i) {
-          if (i > 0 && i % kSub == 0) base += total(i / kSub - 1, column);
-          x[i] = betas[i] * ks[i * PD + column] * exp2f(base + xs[i * PD + column]);
-        }
-      } else {
-        const int c = column - D;
-#pragma unroll
-        for (int i = 0; i < kChunk; ++i)
-          x[i] = i < count && c < p.vdim ? betas[i] * p.v[((row0 + i) * p.heads + head) * p.vdim + c] : 0.0f;
-      }
-#pragma unroll
-      for (int i = 1; i < kChunk; ++i) {
-#pragma unroll
-        for (int j = 0; j < i; j += 4) {
-          const float4 l = *reinterpret_cast<const float4*>(lower + i * PM + j);
-          x[i] = fmaf(-l.x, x[j], x[i]);
-          if (j + 1 < i) x[i] = fmaf(-l.y, x[j + 1], x[i]);
-          if (j + 2 < i) x[i] = fmaf(-l.z, x[j + 2], x[i]);
-          if (j + 3 < i) x[i] = fmaf(-l.w, x[j + 3], x[i]);
-        }
-      }
-      if (column < D) {
-        __nv_bfloat16* high = reinterpret_cast<__nv_bfloat16*>(out + Layout::kW) + column;
-        __nv_bfloat16* low = reinterpret_cast<__nv_bfloat16*>(out + Layout::kW + Layout::kPlane) + column;
-#pragma unroll
-        for (int i = 0; i < kChunk; ++i) {
-          const __nv_bfloat16 h = __float2bfloat16_rn(x[i]);
-          high[i * D] = h;
-          low[i * D] = __float2bfloat16_rn(x[i] - __bfloat162float(h));
-        }
-      } else {
-        float* u = reinterpret_cast<float*>(out + Layout::kU) + column - D;
-#pragma unroll
-        for (int i = 0; i < kChunk; ++i) u[i * v_row] = x[i];
-      }
+  __nv_bfloat16* triangle = reinterpret_cast<__nv_bfloat16*>(planes);      // [2][64][kTriangle]: minus the lower blocks
+  __nv_bfloat16* inverse = triangle + 2 * kChunk * kTriangle;             // [2][64][kInverse]: inverted diagonal blocks
+  for (int item = threadIdx.x; item < kChunk * kChunk / 4; item += kIntraThreads) {
+    const int i = item / (kChunk / 4), j = item % (kChunk / 4) * 4;
+    uint2 high, low;
+    split4(*reinterpret_cast<const float4*>(mixed + i * PM + j), high, low);
+    reinterpret_cast<uint2*>(out + Layout::kA)[item] = high;
+    reinterpret_cast<uint2*>(out + Layout::kA + Layout::kSquare)[item] = low;
+    if (j / kSub < i / kSub) {
+      const float4 v = *reinterpret_cast<const float4*>(lower + i * PM + j);
+      split4(make_float4(-v.x, -v.y, -v.z, -v.w), high, low);
+      *reinterpret_cast<uint2*>(triangle + i * kTriangle + j) = high;
+      *reinterpret_cast<uint2*>(triangle + (kChunk + i) * kTriangle + j) = low;
     }
   }
+  if (threadIdx.x >= kIntraThreads - kChunk) {  // (I + N)^-1 of a diagonal block, one column a thread
+    const int column = threadIdx.x - (kIntraThreads - kChunk), block = column / kSub * kSub, own = column % kSub;
+    float x[kSub];
+#pragma unroll
+    for (int i = 0; i < kSub; ++i) {
+      float v = i == own ? 1.0f : 0.0f;
+#pragma unroll
+      for (int j = 0; j < i; ++j) v = fmaf(-lower[(block + i) * PM + block + j], x[j], v);
+      x[i] = v;
+      const __nv_bfloat16 high = __float2bfloat16_rn(v);
+      inverse[(block + i) * kInverse + own] = high;
+      inverse[(kChunk + block + i) * kInverse + own] = __float2bfloat16_rn(v - __bfloat162float(high));
+    }
+  }
+  __syncthreads();
+
+  // ---- triangular solve (I + lower) [W | U] = beta [P k | v] on the tensor cores, transposed: a warp owns
+  // 16 columns, Y_I = (R_I - sum_{J<I} Y_J lower_IJ^T) inverse_I^T stays in its registers throughout ----
+  __nv_bfloat16* staging = reinterpret_cast<__nv_bfloat16*>(qs);  // [2][64][D] planes of W
+  const int v_row = (p.vdim + 31) / 32 * 32;
+  for (int tile = warp; tile < (D + v_row) / 16; tile += kIntraThreads / 32) {
+    const int c0 = tile * 16 + (lane >> 2);  // fragment rows c0 and c0 + 8 are columns of [W | U]
+    float rhs[kSubs][2][4];
+#pragma unroll
+    for (int I = 0; I < kSubs; ++I)
+#pragma unroll
+      for (int h = 0; h < 2; ++h)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int i = I * kSub + h * 8 + (lane & 3) * 2 + (e & 1), c = c0 + (e >> 1) * 8;
+          if (tile < D / 16) {
+            rhs[I][h][e] = betas[i] * ks[i * PD + c] * exp2f(xs[i * PD + c] + pre[I * D + c]);
+          } else {
+            const int vc = c - D;
+            rhs[I][h][e] = i < count && vc < p.vdim ? p.v[((row0 + i) * p.heads + head) * p.vdim + vc] : 0.0f;
+          }
+        }
+    uint32_t yh[kSubs][4], yl[kSubs][4];
+#pragma unroll
+    for (int I = 0; I < kSubs; ++I) {
+      float acc[2][4];
+#pragma unroll
+      for (int h = 0; h < 2; ++h)
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          acc[h][e] = tile < D / 16 ? rhs[I][h][e] : rhs[I][h][e] * betas[I * kSub + h * 8 + (lane & 3) * 2 + (e & 1)];
+      const int n_row = I * kSub + ((lane >> 4) << 3) + (lane & 7), k_half = ((lane >> 3) & 1) * 8;
+      auto multiply = [&](const uint32_t (&ah)[4], const uint32_t (&al)[4], const __nv_bfloat16* plane, int pitch,
+                          int column, float (&to)[2][4]) {
+        uint32_t bh[4], bl[4];
+        ldmatrix_x4(bh, smem_u32(plane + n_row * pitch + column + k_half));
+        ldmatrix_x4(bl, smem_u32(plane + (kChunk + n_row) * pitch + column + k_half));
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          mma_bf16_16816(to[h], ah, bh[h * 2], bh[h * 2 + 1]);
+          mma_bf16_16816(to[h], ah, bl[h * 2], bl[h * 2 + 1]);
+          mma_bf16_16816(to[h], al, bh[h * 2], bh[h * 2 + 1]);
+        }
+      };
+#pragma unroll
+      for (int J = 0; J < I; ++J) multiply(yh[J], yl[J], triangle, kTriangle, J * kSub, acc);
+      uint32_t zh[4], zl[4];
+      split_bf16x2(acc[0][0], acc[0][1], zh[0], zl[0]);
+      split_bf16x2(acc[0][2], acc[0][3], zh[1], zl[1]);
+      split_bf16x2(acc[1][0], acc[1][1], zh[2], zl[2]);
+      split_bf16x2(acc[1][2], acc[1][3], zh[3], zl[3]);
+      float y[2][4] = {};
+      multiply(zh, zl, inverse, kInverse, 0, y);
+      split_bf16x2(y[0][0], y[0][1], yh[I][0], yl[I][0]);
+      split_bf16x2(y[0][2], y[0][3], yh[I][1], yl[I][1]);
+      split_bf16x2(y[1][0], y[1][1], yh[I][2], yl[I][2]);
+      split_bf16x2(y[1][2], y[1][3], yh[I][3], yl[I][3]);
+#pragma unroll
+      for (int h = 0; h < 2; ++h)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int i = I * kSub + h * 8 + (lane & 3) * 2 + (e & 1), c = c0 + (e >> 1) * 8;
+          if (tile < D / 16) {
+            const __nv_bfloat16 high = __float2bfloat16_rn(y[h][e]);
+            staging[i * D + c] = high;
+            staging[(kChunk + i) * D + c] = __float2bfloat16_rn(y[h][e] - __bfloat162float(high));
+          } else {
+            reinterpret_cast<float*>(out + Layout::kU)[i * v_row + c - D] = y[h][e];
+          }
+        }
+    }
+  }
+  __syncthreads();
+  for (int item = threadIdx.x; item < 2 * kChunk * D / 8; item += kIntraThreads)
+    reinterpret_cast<uint4*>(out + Layout::kW)[item] = reinterpret_cast<const uint4*>(staging)[item];
 }
 
 // ---- across the chunks -------------------------------------------------------------------
@@ -300,11 +488,13 @@ constexpr int inter_smem_bytes() {
   return (DELTA ? 6 : 4) * kChunk * (D + 8) * 2 + 2 * kChunk * (kChunk + 8) * 2 + 2 * D * (VB + 8) * 2 + 2 * kChunk * (VB + 8) * 2;
 }
 
+// Warps: H = VB / 16 share the columns of a 16-row tile. First product: 4 H warps on W S, 4 H on Q S;
+// second: D / 16 x H warps on K^T U (their tile of S stays in registers), the last 4 H on A U.
 template <int D, int VB, bool DELTA>
-__global__ void __launch_bounds__(kInterThreads, 1) chunk_inter_kernel(const ChunkParams p) {
+__global__ void __launch_bounds__(VB * 16, 1) chunk_inter_kernel(const ChunkParams p) {
+  constexpr int kThreads = VB * 16, H = VB / 16;
   constexpr int PB = (D + 8) * 2, PA = (kChunk + 8) * 2, PV = (VB + 8) * 2;  // byte pitches
-  constexpr int NT = VB / 8;
-  constexpr int kStateTiles = D / 16;  // warps that own a 16-row tile of S
+  constexpr int kStateTiles = D / 16;
   using Layout = ChunkLayout<D>;
   extern __shared__ __align__(128) unsigned char smem[];
   unsigned char* q_planes = smem;                            // [2][64][PB]
@@ -322,149 +512,154 @@ __global__ void __launch_bounds__(kInterThreads, 1) chunk_inter_kernel(const Chu
   const int chunks = static_cast<int>((last - first + kChunk - 1) / kChunk);
   const unsigned char* in = p.workspace + (static_cast<int64_t>(p.chunk_starts[sequence]) * p.heads + head) * per;
   const int64_t stride = per * p.heads;
-  auto copy = [&](unsigned char* dst, const unsigned char* src, int rows, int row_bytes, int pitch) {
-    const int chunks16 = row_bytes / 16;
-    for (int item = threadIdx.x; item < rows * chunks16; item += kInterThreads) {
+  auto copy = [&](unsigned char* dst, const unsigned char* src, auto row_bytes_constant, int pitch) {
+    constexpr int row_bytes = decltype(row_bytes_constant)::value, chunks16 = row_bytes / 16;
+#pragma unroll
+    for (int item = threadIdx.x; item < 2 * kChunk * chunks16; item += kThreads) {
       const int r = item / chunks16, c = item % chunks16;
-      cp_async16(smem_u32(dst + r * pitch + c * 16), src + static_cast<int64_t>(r) * row_bytes + c * 16);
+      cp_async16(smem_u32(dst + r * pitch + c * 16), src + static_cast<int64_t>(item) * 16);
     }
   };
   auto load_first = [&](int chunk) {  // operands of the products with S
-    copy(q_planes, in + chunk * stride + Layout::kQ, 2 * kChunk, D * 2, PB);
-    if (DELTA) copy(w_planes, in + chunk * stride + Layout::kW, 2 * kChunk, D * 2, PB);
+    copy(q_planes, in + chunk * stride + Layout::kQ, IntConstant<D * 2>{}, PB);
+    if (DELTA) copy(w_planes, in + chunk * stride + Layout::kW, IntConstant<D * 2>{}, PB);
     cp_async_commit();
   };
   auto load_second = [&](int chunk) {  // operands of the products with U
-    copy(k_planes, in + chunk * stride + Layout::kK, 2 * kChunk, D * 2, PB);
-    copy(a_planes, in + chunk * stride + Layout::kA, 2 * kChunk, kChunk * 2, PA);
+    copy(k_planes, in + chunk * stride + Layout::kK, IntConstant<D * 2>{}, PB);
+    copy(a_planes, in + chunk * stride + Layout::kA, IntConstant<kChunk * 2>{}, PA);
     cp_async_commit();
   };
   load_first(0);
   load_second(0);
 
-  // S: warp w owns rows 16 w .. 16 w + 15 of this CTA's columns, as an accumulator fragment
-  float s[NT][4];
-  const int s_row = warp * 16 + (lane >> 2), s_column = v0 + (lane & 3) * 2;
+  const int half = warp % H;                    // which 16 columns of this CTA's VB
+  const int column = half * 16 + (lane & 3) * 2;  // this lane's first column of n8 tile 0
+  const bool reads_out = warp >= 4 * H;         // Q S and A U; else W S and U
+  const int tile = warp / H % 4, t_row = tile * 16 + (lane >> 2);
+  const bool owns_state = warp / H < kStateTiles;
+  const int s_row = warp / H * 16 + (lane >> 2);
   float* state = p.state + (static_cast<int64_t>(slot) * p.heads + head) * p.dim * p.state_row;
   const bool fresh = p.batch.bases[sequence] == 0;
-  auto store_planes = [&](unsigned char* planes_at, int rows, int row, int column, float a, float b) {
-    uint32_t high, low;
-    split_bf16x2(a, b, high, low);
-    *reinterpret_cast<uint32_t*>(planes_at + row * PV + column * 2) = high;
-    *reinterpret_cast<uint32_t*>(planes_at + (rows + row) * PV + column * 2) = low;
-  };
-  if (warp < kStateTiles) {
+  auto store_planes = [&](unsigned char* planes_at, int rows, int row, const float (&v)[2][4]) {
 #pragma unroll
-    for (int t = 0; t < NT; ++t)
+    for (int t = 0; t < 2; ++t)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        uint32_t high, low;
+        split_bf16x2(v[t][e * 2], v[t][e * 2 + 1], high, low);
+        *reinterpret_cast<uint32_t*>(planes_at + (row + e * 8) * PV + (column + t * 8) * 2) = high;
+        *reinterpret_cast<uint32_t*>(planes_at + (rows + row + e * 8) * PV + (column + t * 8) * 2) = low;
+      }
+  };
+  float s[2][4] = {};
+  if (owns_state) {
+#pragma unroll
+    for (int t = 0; t < 2; ++t)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const int r = s_row + (e >> 1) * 8, c = s_column + t * 8 + (e & 1);
+        const int r = s_row + (e >> 1) * 8, c = v0 + column + t * 8 + (e & 1);
         s[t][e] = !fresh && r < p.dim && c < p.vdim ? state[static_cast<int64_t>(r) * p.state_row + c] : 0.0f;
       }
-#pragma unroll
-    for (int t = 0; t < NT; ++t) {
-      store_planes(s_planes, D, s_row, (lane & 3) * 2 + t * 8, s[t][0], s[t][1]);
-      store_planes(s_planes, D, s_row + 8, (lane & 3) * 2 + t * 8, s[t][2], s[t][3]);
-    }
+    store_planes(s_planes, D, s_row, s);
   }
-  cp_async_wait<1>();
-  __syncthreads();
-
-  // acc += A B with A [16 rows][k] K-major planes, B [k][VB] planes (row-major in shared memory)
-  auto product = [&](float (&acc)[NT][4], uint32_t a_high, int a_low_offset, uint32_t b_high, int b_low_offset,
-                     int steps) {
-    for (int step = 0; step < steps; ++step) {
-      uint32_t ah[4], al[4];
-      ldmatrix_x4(ah, a_high + step * 32);
-      ldmatrix_x4(al, a_high + a_low_offset + step * 32);
-#pragma unroll
-      for (int pair = 0; pair < NT / 2; ++pair) {
-        uint32_t bh[4], bl[4];
-        ldmatrix_x4_trans(bh, b_high + step * 16 * PV + pair * 32);
-        ldmatrix_x4_trans(bl, b_high + b_low_offset + step * 16 * PV + pair * 32);
-#pragma unroll
-        for (int half = 0; half < 2; ++half) {
-          mma_bf16_16816(acc[pair * 2 + half], ah, bh[half * 2], bh[half * 2 + 1]);
-          mma_bf16_16816(acc[pair * 2 + half], ah, bl[half * 2], bl[half * 2 + 1]);
-          mma_bf16_16816(acc[pair * 2 + half], al, bh[half * 2], bh[half * 2 + 1]);
-        }
-      }
-    }
-  };
-  const uint32_t b_lane = (lane & 15) * PV + (lane >> 4) * 16;
   const int v_row = (p.vdim + 31) / 32 * 32;
-  for (int chunk = 0; chunk < chunks; ++chunk) {
+  float u0[2][4] = {}, end0 = 0.0f, end1 = 0.0f;  // fetched a chunk ahead
+  auto fetch = [&](int chunk) {
     const int64_t row0 = first + static_cast<int64_t>(chunk) * kChunk;
-    float acc[NT][4] = {};  // warps 0-3: W S, then U; warps 4-7: the read-out
-    const int tile = warp & 3, t_row = tile * 16 + (lane >> 2);
-    if (warp < 4) {
-      float u0[NT][4];
+    if (!reads_out) {
 #pragma unroll
-      for (int t = 0; t < NT; ++t)
+      for (int t = 0; t < 2; ++t)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const int r = t_row + (e >> 1) * 8, c = s_column + t * 8 + (e & 1);
+          const int r = t_row + (e >> 1) * 8, c = v0 + column + t * 8 + (e & 1);
           if (DELTA) u0[t][e] = c < v_row ? reinterpret_cast<const float*>(in + chunk * stride + Layout::kU)[r * v_row + c] : 0.0f;
           else u0[t][e] = row0 + r < last && c < p.vdim ? p.v[((row0 + r) * p.heads + head) * p.vdim + c] : 0.0f;
         }
-      if (DELTA)
-        product(acc, smem_u32(w_planes) + (tile * 16 + (lane & 15)) * PB + (lane >> 4) * 16, kChunk * PB,
-                smem_u32(s_planes) + b_lane, D * PV, D / 16);
-#pragma unroll
-      for (int t = 0; t < NT; ++t) {
-        store_planes(u_planes, kChunk, t_row, (lane & 3) * 2 + t * 8, u0[t][0] - acc[t][0], u0[t][1] - acc[t][1]);
-        store_planes(u_planes, kChunk, t_row + 8, (lane & 3) * 2 + t * 8, u0[t][2] - acc[t][2], u0[t][3] - acc[t][3]);
-      }
-    } else {
-      product(acc, smem_u32(q_planes) + (tile * 16 + (lane & 15)) * PB + (lane >> 4) * 16, kChunk * PB,
-              smem_u32(s_planes) + b_lane, D * PV, D / 16);
     }
+    if (owns_state) {
+      const float* end = reinterpret_cast<const float*>(in + chunk * stride + Layout::kEnd);
+      end0 = end[s_row];
+      end1 = end[s_row + 8];
+    }
+  };
+  fetch(0);
+  cp_async_wait<1>();
+  __syncthreads();
+
+  // acc += A B: A given by its lanes' addresses (planes `a_low` bytes apart, `a_step` bytes a k16 step;
+  // transposed when it lies [k][m]), B [k][VB] planes
+  const uint32_t b_lane = (lane & 15) * PV + (lane >> 4) * 16 + half * 32;
+  auto product = [&](float (&acc)[2][4], auto transposed, uint32_t a, int a_low, int a_step, uint32_t b, int b_low,
+                     auto steps) {
+    float cross[2][4] = {};
+#pragma unroll
+    for (int step = 0; step < decltype(steps)::value; ++step) {
+      uint32_t ah[4], al[4], bh[4], bl[4];
+      if (decltype(transposed)::value != 0) {
+        ldmatrix_x4_trans(ah, a + step * a_step);
+        ldmatrix_x4_trans(al, a + a_low + step * a_step);
+      } else {
+        ldmatrix_x4(ah, a + step * a_step);
+        ldmatrix_x4(al, a + a_low + step * a_step);
+      }
+      ldmatrix_x4_trans(bh, b + step * 16 * PV);
+      ldmatrix_x4_trans(bl, b + b_low + step * 16 * PV);
+#pragma unroll
+      for (int t = 0; t < 2; ++t) {
+        mma_bf16_16816(acc[t], ah, bh[t * 2], bh[t * 2 + 1]);
+        mma_bf16_16816(cross[t], ah, bl[t * 2], bl[t * 2 + 1]);
+        mma_bf16_16816(cross[t], al, bh[t * 2], bh[t * 2 + 1]);
+      }
+    }
+#pragma unroll
+    for (int t = 0; t < 2; ++t)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[t][e] += cross[t][e];
+  };
+  const uint32_t row_lane = (tile * 16 + (lane & 15)) * PB + (lane >> 4) * 16;
+  const uint32_t s_base = smem_u32(s_planes) + b_lane, u_base = smem_u32(u_planes) + b_lane;
+  for (int chunk = 0; chunk < chunks; ++chunk) {
+    const int64_t row0 = first + static_cast<int64_t>(chunk) * kChunk;
+    float acc[2][4] = {};
+    if (reads_out) {
+      product(acc, IntConstant<0>{}, smem_u32(q_planes) + row_lane, kChunk * PB, 32, s_base, D * PV, IntConstant<D / 16>{});
+    } else {
+      if (DELTA)
+        product(acc, IntConstant<0>{}, smem_u32(w_planes) + row_lane, kChunk * PB, 32, s_base, D * PV, IntConstant<D / 16>{});
+#pragma unroll
+      for (int t = 0; t < 2; ++t)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[t][e] = u0[t][e] - acc[t][e];
+      store_planes(u_planes, kChunk, t_row, acc);
+    }
+    const float e0 = end0, e1 = end1;
     cp_async_wait<0>();
     __syncthreads();  // U is written, the second operands have landed, the first are free
-    if (chunk + 1 < chunks) load_first(chunk + 1);
-    if (warp < kStateTiles) {
-      const float* end = reinterpret_cast<const float*>(in + chunk * stride + Layout::kEnd);
-      const float e0 = end[s_row], e1 = end[s_row + 8];
+    if (chunk + 1 < chunks) {
+      load_first(chunk + 1);
+      fetch(chunk + 1);
+    }
+    if (owns_state) {
 #pragma unroll
-      for (int t = 0; t < NT; ++t) {
+      for (int t = 0; t < 2; ++t) {
         s[t][0] *= e0; s[t][1] *= e0;
         s[t][2] *= e1; s[t][3] *= e1;
       }
-      // S += K^T U: the planes hold K [token][channel], so A is read transposed
-      const uint32_t a_base = smem_u32(k_planes) + ((lane & 7) + ((lane >> 4) << 3)) * PB + warp * 32 + ((lane >> 3) & 1) * 16;
-#pragma unroll
-      for (int step = 0; step < kChunk / 16; ++step) {
-        uint32_t ah[4], al[4];
-        ldmatrix_x4_trans(ah, a_base + step * 16 * PB);
-        ldmatrix_x4_trans(al, a_base + kChunk * PB + step * 16 * PB);
-#pragma unroll
-        for (int pair = 0; pair < NT / 2; ++pair) {
-          uint32_t bh[4], bl[4];
-          ldmatrix_x4_trans(bh, smem_u32(u_planes) + b_lane + step * 16 * PV + pair * 32);
-          ldmatrix_x4_trans(bl, smem_u32(u_planes) + b_lane + kChunk * PV + step * 16 * PV + pair * 32);
-#pragma unroll
-          for (int half = 0; half < 2; ++half) {
-            mma_bf16_16816(s[pair * 2 + half], ah, bh[half * 2], bh[half * 2 + 1]);
-            mma_bf16_16816(s[pair * 2 + half], ah, bl[half * 2], bl[half * 2 + 1]);
-            mma_bf16_16816(s[pair * 2 + half], al, bh[half * 2], bh[half * 2 + 1]);
-          }
-        }
-      }
-#pragma unroll
-      for (int t = 0; t < NT; ++t) {
-        store_planes(s_planes, D, s_row, (lane & 3) * 2 + t * 8, s[t][0], s[t][1]);
-        store_planes(s_planes, D, s_row + 8, (lane & 3) * 2 + t * 8, s[t][2], s[t][3]);
-      }
+      // the planes hold K [token][channel], so A = K^T is read transposed
+      product(s, IntConstant<1>{}, smem_u32(k_planes) + ((lane & 7) + ((lane >> 4) << 3)) * PB + warp / H * 32 + ((lane >> 3) & 1) * 16,
+              kChunk * PB, 16 * PB, u_base, kChunk * PV, IntConstant<kChunk / 16>{});
+      store_planes(s_planes, D, s_row, s);
     }
-    if (warp >= 4) {
-      product(acc, smem_u32(a_planes) + (tile * 16 + (lane & 15)) * PA + (lane >> 4) * 16, kChunk * PA,
-              smem_u32(u_planes) + b_lane, kChunk * PV, kChunk / 16);
+    if (reads_out) {
+      product(acc, IntConstant<0>{}, smem_u32(a_planes) + (tile * 16 + (lane & 15)) * PA + (lane >> 4) * 16, kChunk * PA, 32,
+              u_base, kChunk * PV, IntConstant<kChunk / 16>{});
 #pragma unroll
-      for (int t = 0; t < NT; ++t)
+      for (int t = 0; t < 2; ++t)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int64_t row = row0 + t_row + (e >> 1) * 8;
-          const int c = s_column + t * 8 + (e & 1);
+          const int c = v0 + column + t * 8 + (e & 1);
           if (row < last && c < p.vdim) p.output[(row * p.heads + head) * p.vdim + c] = acc[t][e];
         }
     }
@@ -472,12 +667,12 @@ __global__ void __launch_bounds__(kInterThreads, 1) chunk_inter_kernel(const Chu
     __syncthreads();  // S is written, the first operands have landed, the second are free
     if (chunk + 1 < chunks) load_second(chunk + 1);
   }
-  if (warp < kStateTiles) {
+  if (owns_state) {
 #pragma unroll
-    for (int t = 0; t < NT; ++t)
+    for (int t = 0; t < 2; ++t)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const int r = s_row + (e >> 1) * 8, c = s_column + t * 8 + (e & 1);
+        const int r = s_row + (e >> 1) * 8, c = v0 + column + t * 8 + (e & 1);
         if (r < p.dim && c < p.vdim) state[static_cast<int64_t>(r) * p.state_row + c] = s[t][e];
       }
   }
@@ -485,8 +680,9 @@ __global__ void __launch_bounds__(kInterThreads, 1) chunk_inter_kernel(const Chu
 
 template <int D, bool DELTA>
 int launch_chunked(const ChunkParams& p, int64_t chunks, cudaStream_t stream) {
-  auto intra = chunk_intra_kernel<D, DELTA>;
-  constexpr int intra_smem = intra_smem_bytes<D>();
+  auto intra = chunk_intra_delta_kernel<D>;
+  if (!DELTA) intra = chunk_intra_retention_kernel<D>;
+  constexpr int intra_smem = DELTA ? intra_smem_bytes<D>() : 4 * kChunk * (D + 8) * 2;
   static_assert(intra_smem <= 226 * 1024, "the chunk does not fit shared memory");
   if (cudaFuncSetAttribute(intra, cudaFuncAttributeMaxDynamicSharedMemorySize, intra_smem) != cudaSuccess)
     return B200_ERR_LAUNCH;
@@ -495,7 +691,7 @@ int launch_chunked(const ChunkParams& p, int64_t chunks, cudaStream_t stream) {
     if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess)
       return B200_ERR_LAUNCH;
     kernel<<<dim3(static_cast<unsigned>(ceil_div(p.vdim, vb)), static_cast<unsigned>(p.heads),
-                  static_cast<unsigned>(p.sequences)), kInterThreads, smem, stream>>>(p);
+                  static_cast<unsigned>(p.sequences)), vb * 16, smem, stream>>>(p);
     return launch_status();
   };
   // narrow column slices while the wide ones would leave half the SMs without a CTA
