@@ -155,19 +155,19 @@ def kernel_table(engine, config, size, context, batch, hbm_gbs, tflops):
         inputs = hk.delta_inputs(big, big_gates, delta.conv, delta.a_log, delta.dt_bias, ring, prompt, heads=heads,
                                  kv_heads=heads, dim=dim, vdim=dim, columns=delta.columns,
                                  decay_column=delta.decay_column, q_scale=delta.q_scale)
-        operands = hk.delta_prep(inputs, n, torch.bfloat16, device)
+        operands = hk.delta_prep(inputs, prompt, torch.bfloat16, device)
         state = 0.1 * rand(sequences, heads, dim, dim)
         unit = n * heads * dim
         # necessary traffic: the bf16 projections once and the gated result once
         chunk_flops = 2 * n * heads * (64 * dim * 3 + 3 * dim * dim)
 
         def delta_core():
-            o = hk.delta_prep(inputs, n, torch.bfloat16, device)
+            o = hk.delta_prep(inputs, prompt, torch.bfloat16, device)
             out = hk.recurrence(*o, state, prompt, torch.bfloat16)
             hk.gated_head_norm(out, delta.norm, big_gates[:, delta.gate_column:], kind="sigmoid", epsilon=1e-5)
 
         record(name + "delta rule, all launches", [delta_core], unit * 2 * 6, chunk_flops)
-        record(name + "delta prep", [lambda: hk.delta_prep(inputs, n, torch.bfloat16, device)], unit * (8 + 16))
+        record(name + "delta prep", [lambda: hk.delta_prep(inputs, prompt, torch.bfloat16, device)], unit * (8 + 16))
         record(name + "delta chunks", [lambda: hk.recurrence(*operands, state, prompt, torch.bfloat16)],
                unit * (16 + 4), chunk_flops)
         read_out = rand(n, heads, dim)

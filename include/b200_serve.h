@@ -556,7 +556,7 @@ int b200_retention_step(const b200_retention_inputs* inputs, const b200_step_out
 int b200_delta_step(const b200_delta_inputs* inputs, const b200_step_output* output, int64_t sequences,
                     int dtype, void* stream);
 int b200_delta_prep(const b200_delta_inputs* inputs, float* q, float* k, float* v, float* beta,
-                    float* log_decay, int64_t rows, int dtype, void* stream);
+                    float* log_decay, int64_t rows, int64_t sequences, int64_t longest, int dtype, void* stream);
 int b200_conv_tail(const b200_delta_inputs* inputs, int64_t sequences, int dtype, void* stream);
 int b200_recurrence_scan(const float* q, const float* k, const float* v, const float* beta, const float* decay,
                          float* state, float* output, const int32_t* token_sequence, const int32_t* starts,

@@ -156,7 +156,7 @@ SIGNATURES = {
     "b200_retention_prep": (c_int, [_RETENTION] + [c_void_p] * 3 + [c_int64, c_int, c_void_p]),
     "b200_retention_step": (c_int, [_RETENTION, _STEP, c_int64, c_int, c_void_p]),
     "b200_delta_step": (c_int, [_DELTA, _STEP, c_int64, c_int, c_void_p]),
-    "b200_delta_prep": (c_int, [_DELTA] + [c_void_p] * 5 + [c_int64, c_int, c_void_p]),
+    "b200_delta_prep": (c_int, [_DELTA] + [c_void_p] * 5 + [c_int64] * 3 + [c_int, c_void_p]),
     "b200_conv_tail": (c_int, [_DELTA, c_int64, c_int, c_void_p]),
     "b200_recurrence_scan": (c_int, [c_void_p] * 11 + [c_int64] * 6 + [c_void_p]),
     "b200_recurrence_chunked_workspace_bytes": (c_int64, [c_int64] * 4 + [c_int]),

@@ -87,6 +87,100 @@ __global__ void __launch_bounds__(256) residual_norm_kernel(const ResidualNormPa
     Elem<T>::store(h + c, c < p.width ? row_values[c] * factor * (p.weight_offset + Elem<T>::load(w + c)) : 0.0f);
 }
 
+// Four elements of a model-dtype row
+template <typename T>
+__device__ __forceinline__ float4 load_quad(const T* p) {
+  if (sizeof(T) == 4) return *reinterpret_cast<const float4*>(p);
+  const uint2 v = *reinterpret_cast<const uint2*>(p);
+  return make_float4(bf16_lo(v.x), bf16_hi(v.x), bf16_lo(v.y), bf16_hi(v.y));
+}
+template <typename T>
+__device__ __forceinline__ void store_quad(T* p, float4 v) {
+  if (sizeof(T) == 4) *reinterpret_cast<float4*>(p) = v;
+  else *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
+}
+__device__ __forceinline__ float squares_of(float4 v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
+
+// The same for widths that are a multiple of four: four columns an access, the row in registers, every
+// load of the row in flight at once.
+template <typename T, int Q>
+__global__ void __launch_bounds__(Q == 1 ? 1024 : 512) residual_norm_quads_kernel(const ResidualNormParams p) {
+  __shared__ float scratch[32];
+  grid_launch_dependents();
+  const int quads = p.width / 4;
+  const int64_t row = blockIdx.x;
+  float* x = p.x + row * p.width;
+  const T* post = static_cast<const T*>(p.w_post);
+  const T* next = static_cast<const T*>(p.w_next);
+  grid_dependency_wait_cta();
+  float4 v[Q], y[Q];
+  float sum = 0.0f;
+#pragma unroll
+  for (int i = 0; i < Q; ++i) {
+    const int c = threadIdx.x + i * blockDim.x;
+    v[i] = c < quads ? *reinterpret_cast<const float4*>(x + c * 4) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+  }
+  if (p.y != nullptr) {
+    if (p.splits > 0) {
+      const float* partial = static_cast<const float*>(p.y) + row * p.y_row_stride;
+      const int64_t slice = static_cast<int64_t>(p.rows) * p.y_row_stride;
+#pragma unroll
+      for (int i = 0; i < Q; ++i) {
+        const int c = threadIdx.x + i * blockDim.x;
+        y[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (c >= quads) continue;
+        for (int s0 = 0; s0 < p.splits; s0 += 4) {
+          float4 t[4];
+#pragma unroll
+          for (int s = 0; s < 4; ++s)
+            t[s] = s0 + s < p.splits ? __ldcg(reinterpret_cast<const float4*>(partial + (s0 + s) * slice + c * 4))
+                                     : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll
+          for (int s = 0; s < 4; ++s) {
+            y[i].x += t[s].x; y[i].y += t[s].y; y[i].z += t[s].z; y[i].w += t[s].w;
+          }
+        }
+      }
+    } else {
+      const T* in = static_cast<const T*>(p.y) + row * p.y_row_stride;
+#pragma unroll
+      for (int i = 0; i < Q; ++i) {
+        const int c = threadIdx.x + i * blockDim.x;
+        y[i] = c < quads ? load_quad<T>(in + c * 4) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < Q; ++i) sum += squares_of(y[i]);
+    const float factor = 1.0f / sqrtf(block_sum(sum, scratch) / p.width + p.eps);
+#pragma unroll
+    for (int i = 0; i < Q; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      if (c >= quads) continue;
+      const float4 w = load_quad<T>(post + c * 4);
+      v[i].x += y[i].x * factor * (p.weight_offset + w.x);
+      v[i].y += y[i].y * factor * (p.weight_offset + w.y);
+      v[i].z += y[i].z * factor * (p.weight_offset + w.z);
+      v[i].w += y[i].w * factor * (p.weight_offset + w.w);
+      *reinterpret_cast<float4*>(x + c * 4) = v[i];
+    }
+  }
+  if (p.w_next == nullptr) return;
+  sum = 0.0f;
+#pragma unroll
+  for (int i = 0; i < Q; ++i) sum += squares_of(v[i]);
+  const float factor = 1.0f / sqrtf(block_sum(sum, scratch) / p.width + p.eps);
+  T* h = static_cast<T*>(p.h) + row * p.h_row_stride;
+#pragma unroll
+  for (int i = 0; i < Q; ++i) {
+    const int c = threadIdx.x + i * blockDim.x;
+    if (c >= quads) continue;
+    const float4 w = load_quad<T>(next + c * 4);
+    store_quad<T>(h + c * 4, make_float4(v[i].x * factor * (p.weight_offset + w.x), v[i].y * factor * (p.weight_offset + w.y),
+                                         v[i].z * factor * (p.weight_offset + w.z), v[i].w * factor * (p.weight_offset + w.w)));
+  }
+  if (static_cast<int>(threadIdx.x) < p.h_row_stride - p.width) Elem<T>::store(h + p.width + threadIdx.x, 0.0f);
+}
+
 struct LatentNormParams {
   const void* input;  // T [rows, input_row_stride]: query latent at column 0, kv latent at kv_column
   const void* q_weight;
@@ -181,6 +275,33 @@ __global__ void __launch_bounds__(256) gated_head_norm_kernel(const GatedHeadNor
   }
 }
 
+// The same for vdim 64 or 128 (V) and 16-byte rows: V / 4 lanes a (row, head), four columns each.
+template <typename T, int V>
+__global__ void __launch_bounds__(256) gated_head_norm_quads_kernel(const GatedHeadNormParams p) {
+  constexpr int L = V / 4;
+  grid_launch_dependents();
+  grid_dependency_wait_cta();
+  const int64_t unit = (static_cast<int64_t>(blockIdx.x) * 256 + threadIdx.x) / L;
+  const bool inside = unit < static_cast<int64_t>(p.rows) * p.heads;
+  const int64_t row = inside ? unit / p.heads : 0;
+  const int head = inside ? static_cast<int>(unit - row * p.heads) : 0, c = threadIdx.x % L * 4;
+  const int64_t at = static_cast<int64_t>(head) * V + c;
+  float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f), gate = v;
+  if (inside) {
+    v = __ldcs(reinterpret_cast<const float4*>(p.input + unit * V + c));
+    gate = load_quad<T>(static_cast<const T*>(p.gate) + row * p.gate_row_stride + at);
+  }
+  float sum = squares_of(v);
+#pragma unroll
+  for (int o = L / 2; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+  if (!inside) return;
+  const float factor = 1.0f / sqrtf(sum / V + p.eps);
+  const float4 w = p.weight != nullptr ? load_quad<T>(static_cast<const T*>(p.weight) + c) : make_float4(1.0f, 1.0f, 1.0f, 1.0f);
+  store_quad<T>(static_cast<T*>(p.output) + row * p.output_row_stride + at,
+                make_float4(v.x * factor * w.x * gate_value(gate.x, p.gate_kind), v.y * factor * w.y * gate_value(gate.y, p.gate_kind),
+                            v.z * factor * w.z * gate_value(gate.z, p.gate_kind), v.w * factor * w.w * gate_value(gate.w, p.gate_kind)));
+}
+
 // positions[r] and the row's slot: what a replayed step reads; lengths advance behind the step
 __global__ void sequence_positions_kernel(const int64_t* lengths, const int32_t* slots, int32_t* positions,
                                           int rows) {
@@ -215,6 +336,23 @@ extern "C" int b200_residual_norm(void* x, const void* y, const void* post_weigh
   ResidualNormParams p{static_cast<float*>(x), y, post_weight, next_weight, h, static_cast<int>(splits),
                        static_cast<int>(rows), static_cast<int>(width), y_row_stride, h_row_stride,
                        static_cast<float>(epsilon), static_cast<float>(weight_offset)};
+  const int64_t quads = width / 4;
+  if (width % 4 == 0 && quads <= 2048 && y_row_stride % 4 == 0 && h_row_stride % 4 == 0 &&
+      h_row_stride - width < 32 && aligned16(x) && aligned16(y) && aligned16(h) && aligned16(post_weight) &&
+      aligned16(next_weight)) {
+    // few rows: a thread per four columns; many: rows of fewer, longer-working threads
+    const int q = rows <= 2 * kNumSMs && quads <= 1024 ? 1 : quads <= 512 ? 2 : 4;
+    const unsigned threads = static_cast<unsigned>(ceil_div(ceil_div(quads, q), 32) * 32);
+    auto go = [&](auto kernel) {
+      return launch_chained(kernel, dim3(static_cast<unsigned>(rows)), dim3(threads), 0,
+                            static_cast<cudaStream_t>(stream), p) == cudaSuccess ? launch_status() : B200_ERR_LAUNCH;
+    };
+    if (dtype == B200_F32)
+      return q == 1 ? go(residual_norm_quads_kernel<float, 1>) : q == 2 ? go(residual_norm_quads_kernel<float, 2>)
+                                                                        : go(residual_norm_quads_kernel<float, 4>);
+    return q == 1 ? go(residual_norm_quads_kernel<__nv_bfloat16, 1>)
+                  : q == 2 ? go(residual_norm_quads_kernel<__nv_bfloat16, 2>) : go(residual_norm_quads_kernel<__nv_bfloat16, 4>);
+  }
   const size_t smem = width * sizeof(float);
   auto launch = [&](auto kernel) {
     if (smem > 48 * 1024 &&
@@ -265,6 +403,16 @@ extern "C" int b200_gated_head_norm(const void* input, const void* weight, const
   GatedHeadNormParams p{static_cast<const float*>(input), weight, gate, output, static_cast<int>(rows),
                         static_cast<int>(heads), static_cast<int>(vdim), gate_kind, gate_row_stride,
                         output_row_stride, static_cast<float>(epsilon)};
+  if ((vdim == 64 || vdim == 128) && gate_row_stride % 8 == 0 && output_row_stride == heads * vdim && aligned16(input) &&
+      aligned16(gate) && aligned16(output) && aligned16(weight)) {
+    const dim3 blocks(static_cast<unsigned>(ceil_div(rows * heads * (vdim / 4), 256)));
+    auto go = [&](auto kernel) {
+      return launch_chained(kernel, blocks, dim3(256), 0, static_cast<cudaStream_t>(stream), p) == cudaSuccess
+                 ? launch_status() : B200_ERR_LAUNCH;
+    };
+    if (dtype == B200_F32) return vdim == 64 ? go(gated_head_norm_quads_kernel<float, 64>) : go(gated_head_norm_quads_kernel<float, 128>);
+    return vdim == 64 ? go(gated_head_norm_quads_kernel<__nv_bfloat16, 64>) : go(gated_head_norm_quads_kernel<__nv_bfloat16, 128>);
+  }
   const dim3 grid(static_cast<unsigned>(ceil_div(rows * heads, 8)));
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const cudaError_t code = dtype == B200_F32 ? launch_chained(gated_head_norm_kernel<float>, grid, dim3(256), 0, s, p)

@@ -134,12 +134,15 @@ __global__ void __launch_bounds__(128) head_linear_bf16_kernel(const HeadLinearP
 
 // ---- attention on the tensor cores ---------------------------------------------------------
 // Rows of a sequence are its (token, head) pairs. A CTA takes 16 MT rows and one split of the keys, 32
-// keys a step: S = Q C^T (four groups of 8 keys x two halves of the rank per warp), softmax in fp32
-// through shared memory, O += P C with a warp on every eighth of the rank. C, the keys and the values in
-// one, is fetched once per step for both products. The probabilities enter the product as the sum of
-// two bf16 numbers, so that they keep 16 bits of mantissa. Splits leave fp32 partial results and
-// (max, sum) pairs; the combining kernel adds the sink to the denominator, once.
-constexpr int kLatentKeys = 32, kLatentStages = 3, kLatentThreads = 256;
+// keys a step: S = Q C^T (a warp: 8 keys, a quarter of the rank), softmax in fp32 through shared memory,
+// O += P C (a warp: a sixteenth of the rank). C, the keys and the values in one, is fetched once for both
+// products; the scores of the next step are computed in the same phase as the output of this one. The
+// probabilities enter the product as the sum of two bf16 numbers, so that they keep 16 bits of mantissa.
+// Splits leave fp32 partial results and (max, sum) pairs; the combining kernel adds the sink to the
+// denominator, once.
+constexpr int kLatentKeys = 32, kLatentThreads = 512;
+constexpr int kScorePitch = kLatentKeys + 4;                  // floats
+constexpr int kProbabilityPitch = kLatentKeys * 2 + 16;       // bytes
 
 struct LatentSplitParams {
   const __nv_bfloat16* q;      // [rows, heads, rank]
@@ -147,7 +150,7 @@ struct LatentSplitParams {
   float* partial;              // [rows * heads, splits, rank]
   float2* partial_stats;       // [rows * heads, splits]: max (log2 domain), sum
   SequenceBatch batch;
-  int heads, rank, splits, pitch;  // pitch: bytes of a row in shared memory
+  int heads, rank, splits, pitch, stages;  // pitch: bytes of a row in shared memory
   int64_t capacity;
   float scale_log2;
 };
@@ -162,10 +165,8 @@ __device__ __forceinline__ void split_range(int64_t keys, int splits, int split,
 }
 
 template <int MT, int NT>
-__global__ void __launch_bounds__(kLatentThreads) latent_attention_split_kernel(const LatentSplitParams p) {
+__global__ void __launch_bounds__(kLatentThreads, 1) latent_attention_split_kernel(const LatentSplitParams p) {
   constexpr int M = 16 * MT;
-  constexpr int kSPitch = kLatentKeys + 4;           // floats
-  constexpr int kPPitch = kLatentKeys * 2 + 16;      // bytes
   extern __shared__ __align__(128) unsigned char smem[];
   __shared__ float row_factor[M];
   __shared__ float row_max[M], row_sum[M];
@@ -191,8 +192,8 @@ __global__ void __launch_bounds__(kLatentThreads) latent_attention_split_kernel(
   }
   const uint32_t q_tile = smem_u32(smem);
   const uint32_t c_tiles = q_tile + M * p.pitch;
-  float* scores = reinterpret_cast<float*>(smem + M * p.pitch + kLatentStages * kLatentKeys * p.pitch);  // [2][M][kSPitch]
-  unsigned char* probabilities = reinterpret_cast<unsigned char*>(scores + 2 * M * kSPitch);  // [2][M][kPPitch]: high, low
+  float* scores = reinterpret_cast<float*>(smem + (M + p.stages * kLatentKeys) * p.pitch);  // [4][M][kScorePitch]
+  unsigned char* probabilities = reinterpret_cast<unsigned char*>(scores + 4 * M * kScorePitch);  // [2][M]: high, low
   const int chunks = p.rank / 8;
   for (int item = threadIdx.x; item < M * chunks; item += kLatentThreads) {
     const int r = item / chunks, c = item % chunks;
@@ -201,89 +202,94 @@ __global__ void __launch_bounds__(kLatentThreads) latent_attention_split_kernel(
   }
   const __nv_bfloat16* cache = p.cache + static_cast<int64_t>(slot) * p.capacity * p.rank;
   const int steps = static_cast<int>((end - begin + kLatentKeys - 1) / kLatentKeys);
-  auto load = [&](int step) {
-    const uint32_t tile = c_tiles + (step % kLatentStages) * kLatentKeys * p.pitch;
-    const int64_t key0 = begin + static_cast<int64_t>(step) * kLatentKeys;
-    for (int item = threadIdx.x; item < kLatentKeys * chunks; item += kLatentThreads) {
-      const int r = item / chunks, c = item % chunks;
-      const bool inside = key0 + r < end;
-      cp_async16_zfill(tile + r * p.pitch + c * 16, cache + (inside ? (key0 + r) * p.rank + c * 8 : 0), inside ? 16 : 0);
+  // a thread copies chunk `copy_chunk` of every `copy_rows`-th key of a step
+  const int copy_rows = kLatentThreads / chunks, copy_row = threadIdx.x / chunks, copy_chunk = threadIdx.x - copy_row * chunks;
+  auto load = [&](int step, int stage) {
+    if (copy_row < copy_rows) {
+      const uint32_t tile = c_tiles + stage * kLatentKeys * p.pitch + copy_chunk * 16;
+      const int64_t key0 = begin + static_cast<int64_t>(step) * kLatentKeys;
+      const __nv_bfloat16* source = cache + key0 * p.rank + copy_chunk * 8;
+      const int valid = static_cast<int>(end - key0 < kLatentKeys ? end - key0 : kLatentKeys);
+      for (int r = copy_row; r < kLatentKeys; r += copy_rows)
+        cp_async16_zfill(tile + r * p.pitch, r < valid ? source + static_cast<int64_t>(r) * p.rank : cache, r < valid ? 16 : 0);
     }
   };
-#pragma unroll
-  for (int s = 0; s < kLatentStages - 1; ++s) {
-    if (s < steps) load(s);
-    cp_async_commit();  // (the first group holds Q as well)
+  // tiles 0 .. stages - 2 in flight; one group a tile (the first holds Q as well)
+  for (int s = 0; s < p.stages - 1; ++s) {
+    if (s < steps) load(s, s);
+    cp_async_commit();
   }
   for (int r = threadIdx.x; r < M; r += kLatentThreads) {
     row_max[r] = -INFINITY;
     row_sum[r] = 0.0f;
   }
-  float acc[MT][NT][4] = {};
-  const int k_steps = p.rank / 16;
-  const int k_begin = (warp >> 2) ? (k_steps + 1) / 2 : 0, k_end = (warp >> 2) ? k_steps : (k_steps + 1) / 2;
-  for (int step = 0; step < steps; ++step) {
-    cp_async_wait<kLatentStages - 2>();
-    __syncthreads();  // the tile has landed; everyone is done with the one that is refilled now
-    if (step + kLatentStages - 1 < steps) load(step + kLatentStages - 1);
-    cp_async_commit();
-    const uint32_t tile = c_tiles + (step % kLatentStages) * kLatentKeys * p.pitch;
-    // ---- scores: this warp's 8 keys, its half of the rank ----
-    {
-      float s[MT][4] = {};
-      const int key = (warp & 3) * 8 + (lane & 7);
-      for (int ks = k_begin; ks < k_end; ++ks) {
-        uint32_t b[2];
-        asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];\n"
-                     : "=r"(b[0]), "=r"(b[1])
-                     : "r"(tile + key * p.pitch + ks * 32 + ((lane >> 3) & 1) * 16));
-#pragma unroll
-        for (int mt = 0; mt < MT; ++mt) {
-          uint32_t a[4];
-          ldmatrix_x4(a, q_tile + (mt * 16 + (lane & 15)) * p.pitch + ks * 32 + (lane >> 4) * 16);
-          mma_bf16_16816(s[mt], a, b[0], b[1]);
-        }
-      }
-      float* out = scores + (warp >> 2) * M * kSPitch + (warp & 3) * 8 + (lane & 3) * 2;
+  const int k_steps = p.rank / 16, quarter = warp >> 2, per_quarter = (k_steps + 3) / 4;
+  const int k_begin = quarter * per_quarter, k_end = min(k_begin + per_quarter, k_steps);
+  auto compute_scores = [&](uint32_t tile) {
+    float s[MT][4] = {};
+    const uint32_t b_lane = tile + ((warp & 3) * 8 + (lane & 7)) * p.pitch + ((lane >> 3) & 1) * 16;
+    const uint32_t a_lane = q_tile + (lane & 15) * p.pitch + (lane >> 4) * 16;
+#pragma unroll 4
+    for (int ks = k_begin; ks < k_end; ++ks) {
+      uint32_t b[2];
+      asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];\n" : "=r"(b[0]), "=r"(b[1]) : "r"(b_lane + ks * 32));
 #pragma unroll
       for (int mt = 0; mt < MT; ++mt) {
-        *reinterpret_cast<float2*>(out + (mt * 16 + (lane >> 2)) * kSPitch) = make_float2(s[mt][0], s[mt][1]);
-        *reinterpret_cast<float2*>(out + (mt * 16 + (lane >> 2) + 8) * kSPitch) = make_float2(s[mt][2], s[mt][3]);
+        uint32_t a[4];
+        ldmatrix_x4(a, a_lane + mt * 16 * p.pitch + ks * 32);
+        mma_bf16_16816(s[mt], a, b[0], b[1]);
       }
     }
-    __syncthreads();
-    // ---- softmax: 8 lanes a row, 4 keys each ----
-    for (int r = threadIdx.x >> 3; r < M; r += kLatentThreads / 8) {
-      const int c = (threadIdx.x & 7) * 4;
-      const float4 s0 = *reinterpret_cast<const float4*>(scores + r * kSPitch + c);
-      const float4 s1 = *reinterpret_cast<const float4*>(scores + (M + r) * kSPitch + c);
-      float v[4] = {s0.x + s1.x, s0.y + s1.y, s0.z + s1.z, s0.w + s1.w};
+    float* out = scores + quarter * M * kScorePitch + (warp & 3) * 8 + (lane & 3) * 2;
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt) {
+      *reinterpret_cast<float2*>(out + (mt * 16 + (lane >> 2)) * kScorePitch) = make_float2(s[mt][0], s[mt][1]);
+      *reinterpret_cast<float2*>(out + (mt * 16 + (lane >> 2) + 8) * kScorePitch) = make_float2(s[mt][2], s[mt][3]);
+    }
+  };
+  float acc[MT][NT][4] = {};
+  if (p.stages == 3) cp_async_wait<1>();
+  else if (p.stages == 4) cp_async_wait<2>();
+  else cp_async_wait<3>();
+  __syncthreads();  // tile 0 and Q
+  compute_scores(c_tiles);
+  int stage = 0;
+  for (int step = 0; step < steps; ++step) {
+    // tile step + 1 has landed (of the groups behind it, stages - 3 may be in flight)
+    if (p.stages == 3) cp_async_wait<0>();
+    else if (p.stages == 4) cp_async_wait<1>();
+    else cp_async_wait<2>();
+    __syncthreads();  // the scores are written; everyone is done with tile step - 1
+    const int previous = stage == 0 ? p.stages - 1 : stage - 1;
+    if (step + p.stages - 1 < steps) load(step + p.stages - 1, previous);
+    cp_async_commit();
+    // ---- softmax: 16 lanes a row, 2 keys each ----
+    for (int r = threadIdx.x >> 4; r < M; r += kLatentThreads / 16) {
+      const int c = (threadIdx.x & 15) * 2;
+      float v[2] = {0.0f, 0.0f};
+#pragma unroll
+      for (int part = 0; part < 4; ++part) {
+        const float2 t = *reinterpret_cast<const float2*>(scores + (part * M + r) * kScorePitch + c);
+        v[0] += t.x;
+        v[1] += t.y;
+      }
       const int64_t key0 = begin + static_cast<int64_t>(step) * kLatentKeys + c;
       const int64_t limit = min(base + (row0 + r) / p.heads + 1, end);
-      float top = row_max[r];
-      const float before = top;
+      const float before = row_max[r];
+      v[0] = key0 < limit ? v[0] * p.scale_log2 : -INFINITY;
+      v[1] = key0 + 1 < limit ? v[1] * p.scale_log2 : -INFINITY;
+      float top = fmaxf(before, fmaxf(v[0], v[1]));
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        v[i] = key0 + i < limit ? v[i] * p.scale_log2 : -INFINITY;
-        top = fmaxf(top, v[i]);
-      }
-#pragma unroll
-      for (int o = 4; o > 0; o >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
+      for (int o = 8; o > 0; o >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
       const float reference = top == -INFINITY ? 0.0f : top;  // (no visible key so far: all weights are 0)
-      float sum = 0.0f;
-      uint32_t high[2], low[2];
+      const float p0 = exp2f(v[0] - reference), p1 = exp2f(v[1] - reference);
+      const uint32_t high = pack_bf16x2(p0, p1), low = pack_bf16x2(p0 - bf16_lo(high), p1 - bf16_hi(high));
+      float sum = p0 + p1;
 #pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        const float p0 = exp2f(v[2 * i] - reference), p1 = exp2f(v[2 * i + 1] - reference);
-        sum += p0 + p1;
-        high[i] = pack_bf16x2(p0, p1);
-        low[i] = pack_bf16x2(p0 - bf16_lo(high[i]), p1 - bf16_hi(high[i]));
-      }
-#pragma unroll
-      for (int o = 4; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-      *reinterpret_cast<uint2*>(probabilities + r * kPPitch + c * 2) = make_uint2(high[0], high[1]);
-      *reinterpret_cast<uint2*>(probabilities + (M + r) * kPPitch + c * 2) = make_uint2(low[0], low[1]);
-      if ((threadIdx.x & 7) == 0) {
+      for (int o = 8; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+      *reinterpret_cast<uint32_t*>(probabilities + r * kProbabilityPitch + c * 2) = high;
+      *reinterpret_cast<uint32_t*>(probabilities + (M + r) * kProbabilityPitch + c * 2) = low;
+      if ((threadIdx.x & 15) == 0) {
         const float factor = exp2f(before - reference);  // (0 on the first visible key)
         row_factor[r] = factor;
         row_sum[r] = row_sum[r] * factor + sum;
@@ -291,8 +297,11 @@ __global__ void __launch_bounds__(kLatentThreads) latent_attention_split_kernel(
       }
     }
     __syncthreads();
-    // ---- O += P C on this warp's columns ----
-    const uint32_t p_tile = smem_u32(probabilities);
+    const uint32_t tile = c_tiles + stage * kLatentKeys * p.pitch;
+    stage = stage + 1 == p.stages ? 0 : stage + 1;
+    // ---- the next step's scores, and O += P C on this warp's columns ----
+    if (step + 1 < steps) compute_scores(c_tiles + stage * kLatentKeys * p.pitch);
+    const uint32_t p_tile = smem_u32(probabilities) + (lane & 15) * kProbabilityPitch + (lane >> 4) * 16;
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt) {
       const float f0 = row_factor[mt * 16 + (lane >> 2)], f1 = row_factor[mt * 16 + (lane >> 2) + 8];
@@ -307,14 +316,13 @@ __global__ void __launch_bounds__(kLatentThreads) latent_attention_split_kernel(
       uint32_t hi[MT][4], lo[MT][4];
 #pragma unroll
       for (int mt = 0; mt < MT; ++mt) {
-        const uint32_t address = p_tile + (mt * 16 + (lane & 15)) * kPPitch + ks * 32 + (lane >> 4) * 16;
-        ldmatrix_x4(hi[mt], address);
-        ldmatrix_x4(lo[mt], address + M * kPPitch);
+        ldmatrix_x4(hi[mt], p_tile + mt * 16 * kProbabilityPitch + ks * 32);
+        ldmatrix_x4(lo[mt], p_tile + (M + mt * 16) * kProbabilityPitch + ks * 32);
       }
 #pragma unroll
       for (int t = 0; t < NT; ++t) {
         const int n_tile = warp * NT + t;
-        if (n_tile * 8 < p.rank) {
+        if (n_tile < chunks) {
           uint32_t b[2];
           asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];\n"
                        : "=r"(b[0]), "=r"(b[1])
@@ -343,7 +351,7 @@ __global__ void __launch_bounds__(kLatentThreads) latent_attention_split_kernel(
           *reinterpret_cast<float2*>(out + n) = make_float2(acc[mt][t][half * 2], acc[mt][t][half * 2 + 1]);
       }
     }
-  for (int r = threadIdx.x; r <= last_row - row0; r += kLatentThreads)  // (written before the last barrier but one)
+  for (int r = threadIdx.x; r <= last_row - row0; r += kLatentThreads)  // (written before the last barrier)
     p.partial_stats[(unit0 + r) * p.splits + split] = make_float2(row_max[r], row_sum[r]);
 }
 
@@ -384,23 +392,25 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const float* partia
 }
 
 struct LatentPlan {
-  int mt, nt, row_blocks, splits, pitch, smem;
+  int mt, nt, row_blocks, splits, pitch, stages, smem;
 };
 
-// Row tile and split count: about two CTAs a SM (one for the 64-row tile), in whole waves.
+// Row tile, ring depth and split count: as many CTAs as fill the GPU's slots in whole waves.
 LatentPlan plan_latent(int64_t sequences, int64_t longest, int64_t heads, int64_t rank, int64_t context) {
   LatentPlan plan{};
   if (rank % 16 != 0 || rank > 512) return plan;
   const int64_t rows = longest * heads;
   plan.mt = rows <= 16 ? 1 : rows <= 32 ? 2 : 4;
-  const int64_t tiles = (rank / 8 + 7) / 8;
-  plan.nt = tiles <= 1 ? 1 : tiles <= 2 ? 2 : tiles <= 4 ? 4 : 8;
+  plan.nt = rank <= 128 ? 1 : rank <= 256 ? 2 : 4;
   const int m = 16 * plan.mt;
   plan.pitch = static_cast<int>(rank * 2 + 16);
-  plan.smem = (m + kLatentStages * kLatentKeys) * plan.pitch + 2 * m * (kLatentKeys + 4) * 4 + 2 * m * (kLatentKeys * 2 + 16);
+  const int fixed = m * plan.pitch + 4 * m * kScorePitch * 4 + 2 * m * kProbabilityPitch;
+  for (plan.stages = 5; plan.stages > 3; --plan.stages)
+    if (fixed + plan.stages * kLatentKeys * plan.pitch <= 224 * 1024) break;
+  plan.smem = fixed + plan.stages * kLatentKeys * plan.pitch;
+  if (plan.smem > 224 * 1024) return LatentPlan{};
   plan.row_blocks = static_cast<int>(ceil_div(rows, m));
-  const int per_sm = plan.smem <= 112 * 1024 && plan.mt <= 2 ? 2 : 1;
-  const int64_t slots = static_cast<int64_t>(kNumSMs) * per_sm, units = sequences * plan.row_blocks;
+  const int64_t slots = kNumSMs, units = sequences * plan.row_blocks;
   const int64_t most = ceil_div(context, 128);
   double best = -1.0;
   plan.splits = 1;
@@ -430,8 +440,7 @@ int launch_split_nt(const LatentSplitParams& p, const LatentPlan& plan, int64_t 
   switch (plan.nt) {
     case 1: return launch_split<MT, 1>(p, plan, sequences, stream);
     case 2: return launch_split<MT, 2>(p, plan, sequences, stream);
-    case 4: return launch_split<MT, 4>(p, plan, sequences, stream);
-    default: return launch_split<MT, 8>(p, plan, sequences, stream);
+    default: return launch_split<MT, 4>(p, plan, sequences, stream);
   }
 }
 
@@ -612,7 +621,7 @@ extern "C" int b200_latent_attention(const void* q, const void* cache, const voi
       float2* stats = reinterpret_cast<float2*>(partial + rows * heads * plan.splits * rank_row);
       LatentSplitParams p{static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(cache), partial, stats,
                           {token_sequence, starts, slots, bases}, static_cast<int>(heads), static_cast<int>(rank_row),
-                          plan.splits, plan.pitch, capacity, static_cast<float>(scale * 1.4426950408889634)};
+                          plan.splits, plan.pitch, plan.stages, capacity, static_cast<float>(scale * 1.4426950408889634)};
       const int code = plan.mt == 1 ? launch_split_nt<1>(p, plan, sequences, s)
                        : plan.mt == 2 ? launch_split_nt<2>(p, plan, sequences, s)
                                       : launch_split_nt<4>(p, plan, sequences, s);

@@ -81,6 +81,112 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaInputs p, fl
   }
 }
 
+// bf16 prompts with dim = vdim = 32 CPL and at most four taps: a warp walks 32 tokens of one unit (a q,
+// k or v head, or a head's decays) with the convolution's window in registers, CPL channels a lane, eight
+// tokens' loads in flight.
+template <int CPL>
+__device__ __forceinline__ void load_channels(const __nv_bfloat16* p, float (&v)[CPL]) {
+  if (CPL == 4) {
+    const uint2 t = *reinterpret_cast<const uint2*>(p);
+    v[0] = bf16_lo(t.x); v[1] = bf16_hi(t.x); v[CPL - 2] = bf16_lo(t.y); v[CPL - 1] = bf16_hi(t.y);
+  } else {
+    const uint32_t t = *reinterpret_cast<const uint32_t*>(p);
+    v[0] = bf16_lo(t); v[1] = bf16_hi(t);
+  }
+}
+template <int CPL>
+__device__ __forceinline__ void store_channels(float* p, const float (&v)[CPL]) {
+  if (CPL == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[CPL - 2], v[CPL - 1]);
+  else *reinterpret_cast<float2*>(p) = make_float2(v[0], v[1]);
+}
+
+template <int CPL>
+__global__ void __launch_bounds__(256) delta_prep_tiled_kernel(const DeltaInputs p, float* q, float* k, float* v,
+                                                               float* beta, float* log_decay) {
+  constexpr int kDim = 32 * CPL, kTokens = 32, kBatch = 8, kTaps = 4;
+  const int lane = threadIdx.x & 31, sequence = blockIdx.z;
+  const int unit = blockIdx.y * 8 + (threadIdx.x >> 5);
+  const int slot = p.batch.slots[sequence];
+  const int64_t first = p.batch.starts[sequence], last = p.batch.starts[sequence + 1];
+  const int64_t row0 = first + static_cast<int64_t>(blockIdx.x) * kTokens;
+  if (unit >= 2 * p.kv_heads + 2 * p.heads || row0 >= last || slot < 0) return;
+  const int count = last - row0 < kTokens ? static_cast<int>(last - row0) : kTokens;
+  const int c = lane * CPL;
+  if (unit >= 2 * p.kv_heads + p.heads) {  // step size and decays
+    const int head = unit - 2 * p.kv_heads - p.heads;
+    const __nv_bfloat16* in = static_cast<const __nv_bfloat16*>(p.gates) + p.decay_column + head * kDim + c;
+    float bias[CPL];
+    load_channels<CPL>(static_cast<const __nv_bfloat16*>(p.dt_bias) + head * kDim + c, bias);
+    const float rate = -expf(__bfloat162float(static_cast<const __nv_bfloat16*>(p.a_log)[head]));
+    if (lane < count) beta[(row0 + lane) * p.heads + head] = delta_beta<__nv_bfloat16>(p, row0 + lane, head);
+    for (int t0 = 0; t0 < count; t0 += kBatch) {
+      float step[kBatch][CPL];
+#pragma unroll
+      for (int t = 0; t < kBatch; ++t)
+        if (t0 + t < count) load_channels<CPL>(in + (row0 + t0 + t) * p.gate_row_stride, step[t]);
+#pragma unroll
+      for (int t = 0; t < kBatch; ++t) {
+        if (t0 + t >= count) break;
+#pragma unroll
+        for (int i = 0; i < CPL; ++i) step[t][i] = rate * softplus_f32(step[t][i] + bias[i]);
+        store_channels<CPL>(log_decay + ((row0 + t0 + t) * p.heads + head) * kDim + c, step[t]);
+      }
+    }
+    return;
+  }
+  const int which = unit < p.kv_heads ? 0 : unit < 2 * p.kv_heads ? 1 : 2;
+  const int head = unit - which * p.kv_heads;
+  const int channel = head * kDim + c;
+  const __nv_bfloat16* in = static_cast<const __nv_bfloat16*>(p.input) +
+                            (which == 0 ? p.q_column : which == 1 ? p.k_column : p.v_column) + channel;
+  const __nv_bfloat16* taps = static_cast<const __nv_bfloat16*>(which == 0 ? p.q_conv : which == 1 ? p.k_conv : p.v_conv);
+  float weight[CPL][kTaps], window[kTaps - 1][CPL];  // weight[.][b]: of the input b tokens back; window: 1, 2, 3 back
+#pragma unroll
+  for (int i = 0; i < CPL; ++i)
+#pragma unroll
+    for (int b = 0; b < kTaps; ++b)
+      weight[i][b] = b < p.taps ? __bfloat162float(taps[(channel + i) * p.taps + p.taps - 1 - b]) : 0.0f;
+  const int64_t position = p.batch.position(sequence, row0);
+  const int qk = p.kv_heads * p.dim, channels = 2 * qk + p.heads * p.vdim;
+  const __nv_bfloat16* ring = static_cast<const __nv_bfloat16*>(p.ring) + static_cast<int64_t>(slot) * p.taps * channels + which * qk + channel;
+#pragma unroll
+  for (int b = 1; b < kTaps; ++b) {
+#pragma unroll
+    for (int i = 0; i < CPL; ++i) window[b - 1][i] = 0.0f;
+    if (b >= p.taps || b > position) continue;
+    if (row0 - b >= first) load_channels<CPL>(in + (row0 - b) * p.row_stride, window[b - 1]);
+    else load_channels<CPL>(ring + static_cast<int>((position - b) % p.taps) * static_cast<int64_t>(channels), window[b - 1]);
+  }
+  float* out = which == 0 ? q : which == 1 ? k : v;
+  const int out_heads = which == 2 ? p.heads : p.kv_heads;
+  for (int t0 = 0; t0 < count; t0 += kBatch) {
+    float raw[kBatch][CPL];
+#pragma unroll
+    for (int t = 0; t < kBatch; ++t)
+      if (t0 + t < count) load_channels<CPL>(in + (row0 + t0 + t) * p.row_stride, raw[t]);
+#pragma unroll
+    for (int t = 0; t < kBatch; ++t) {
+      if (t0 + t >= count) break;
+      float y[CPL], sum = 0.0f;
+#pragma unroll
+      for (int i = 0; i < CPL; ++i) {
+        y[i] = silu_of(weight[i][0] * raw[t][i] + weight[i][1] * window[0][i] + weight[i][2] * window[1][i] + weight[i][3] * window[2][i]);
+        sum += y[i] * y[i];
+        window[2][i] = window[1][i];
+        window[1][i] = window[0][i];
+        window[0][i] = raw[t][i];
+      }
+      if (which < 2) {
+        float factor = 1.0f / sqrtf(warp_sum(sum) + kUnitEpsilon);
+        if (which == 0) factor *= p.q_scale;
+#pragma unroll
+        for (int i = 0; i < CPL; ++i) y[i] *= factor;
+      }
+      store_channels<CPL>(out + ((row0 + t0 + t) * out_heads + head) * kDim + c, y);
+    }
+  }
+}
+
 // The last taps inputs of every sequence into its ring (entry position % taps), behind the kernels
 // that still read the ring's older entries.
 template <typename T>
@@ -88,6 +194,7 @@ __global__ void __launch_bounds__(256) conv_tail_kernel(const DeltaInputs p) {
   const int sequence = blockIdx.x;
   const int slot = p.batch.slots[sequence];
   if (slot < 0) return;
+  const int c = blockIdx.y * blockDim.x + threadIdx.x;
   const int64_t first = p.batch.starts[sequence], last = p.batch.starts[sequence + 1];
   const int64_t begin = last - first > p.taps ? last - p.taps : first;
   const int channels = 2 * p.kv_heads * p.dim + p.heads * p.vdim;
@@ -95,7 +202,7 @@ __global__ void __launch_bounds__(256) conv_tail_kernel(const DeltaInputs p) {
     const int64_t entry = p.batch.position(sequence, row) % p.taps;
     T* ring = static_cast<T*>(p.ring) + (slot * p.taps + entry) * channels;
     const T* in = static_cast<const T*>(p.input) + row * p.row_stride;
-    for (int c = threadIdx.x; c < channels; c += blockDim.x) {
+    if (c < channels) {
       const int qk = p.kv_heads * p.dim;
       const int column = c < qk ? p.q_column + c : (c < 2 * qk ? p.k_column + c - qk : p.v_column + c - 2 * qk);
       ring[c] = in[column];
@@ -244,14 +351,26 @@ extern "C" int b200_retention_prep(const b200_retention_inputs* inputs, float* q
 }
 
 extern "C" int b200_delta_prep(const b200_delta_inputs* inputs, float* q, float* k, float* v, float* beta,
-                               float* log_decay, int64_t rows, int dtype, void* stream) {
+                               float* log_decay, int64_t rows, int64_t sequences, int64_t longest, int dtype,
+                               void* stream) {
   DeltaInputs p;
-  if (!delta_inputs_from(inputs, &p) || !q || !k || !v || !beta || !log_decay || rows < 0)
+  if (!delta_inputs_from(inputs, &p) || !q || !k || !v || !beta || !log_decay || rows < 0 ||
+      sequences < 0 || longest < 0)
     return B200_ERR_BAD_ARGUMENT;
   if (dtype != B200_F32 && dtype != B200_BF16) return B200_ERR_UNSUPPORTED;
   if (rows == 0) return B200_OK;
   if (rows > INT32_MAX) return B200_ERR_TOO_LARGE;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (dtype == B200_BF16 && (p.dim == 64 || p.dim == 128) && p.vdim == p.dim && p.taps <= 4 && longest >= 16 &&
+      p.row_stride % 8 == 0 && p.gate_row_stride % 8 == 0 && p.q_column % 8 == 0 && p.k_column % 8 == 0 &&
+      p.v_column % 8 == 0 && p.decay_column % 8 == 0 && aligned16(p.input) && aligned16(p.gates) && aligned16(p.ring) &&
+      aligned16(p.dt_bias) && sequences <= 65535) {
+    const dim3 grid(static_cast<unsigned>(ceil_div(longest, 32)), static_cast<unsigned>(ceil_div(2 * p.kv_heads + 2 * p.heads, 8)),
+                    static_cast<unsigned>(sequences));
+    if (p.dim == 64) delta_prep_tiled_kernel<2><<<grid, 256, 0, s>>>(p, q, k, v, beta, log_decay);
+    else delta_prep_tiled_kernel<4><<<grid, 256, 0, s>>>(p, q, k, v, beta, log_decay);
+    return launch_status();
+  }
   if (dtype == B200_F32)
     delta_prep_kernel<float><<<static_cast<unsigned>(rows), 256, 0, s>>>(p, q, k, v, beta, log_decay);
   else
@@ -265,8 +384,9 @@ extern "C" int b200_conv_tail(const b200_delta_inputs* inputs, int64_t sequences
   if (dtype != B200_F32 && dtype != B200_BF16) return B200_ERR_UNSUPPORTED;
   if (sequences == 0 || p.taps <= 1) return B200_OK;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (dtype == B200_F32) conv_tail_kernel<float><<<static_cast<unsigned>(sequences), 256, 0, s>>>(p);
-  else conv_tail_kernel<__nv_bfloat16><<<static_cast<unsigned>(sequences), 256, 0, s>>>(p);
+  const dim3 grid(static_cast<unsigned>(sequences), static_cast<unsigned>(ceil_div(2 * p.kv_heads * p.dim + p.heads * p.vdim, 256)));
+  if (dtype == B200_F32) conv_tail_kernel<float><<<grid, 256, 0, s>>>(p);
+  else conv_tail_kernel<__nv_bfloat16><<<grid, 256, 0, s>>>(p);
   return launch_status();
 }
 

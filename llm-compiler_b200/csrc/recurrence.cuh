@@ -60,12 +60,18 @@ __device__ __forceinline__ float short_conv(const DeltaInputs& p, int which, int
   const int qk = p.kv_heads * p.dim;
   const int channels = 2 * qk + p.heads * p.vdim;
   const T* ring = static_cast<const T*>(p.ring) + static_cast<int64_t>(slot) * p.taps * channels + which * qk + channel;
+  const int entry = static_cast<int>(position) % p.taps;
+  auto value_at = [&](int back) {
+    const int index = entry - back < 0 ? entry - back + p.taps : entry - back;
+    return back <= local ? Elem<T>::load(in - back * p.row_stride)
+                         : Elem<T>::load(ring + static_cast<int64_t>(index) * channels);
+  };
+  const int reach = position < p.taps - 1 ? static_cast<int>(position) : p.taps - 1;
   float sum = 0.0f;
-  for (int back = 0; back < p.taps && back <= position; ++back) {
-    const float value = back <= local ? Elem<T>::load(in - back * p.row_stride)
-                                      : Elem<T>::load(ring + ((position - back) % p.taps) * channels);
-    sum = fmaf(Elem<T>::load(taps + p.taps - 1 - back), value, sum);
-  }
+#pragma unroll
+  for (int back = 0; back < 4; ++back)  // (the loads of the first four do not wait for one another)
+    if (back <= reach) sum = fmaf(Elem<T>::load(taps + p.taps - 1 - back), value_at(back), sum);
+  for (int back = 4; back <= reach; ++back) sum = fmaf(Elem<T>::load(taps + p.taps - 1 - back), value_at(back), sum);
   return sum;
 }
 
@@ -106,43 +112,39 @@ inline bool retention_inputs_from(const b200_retention_inputs* in, RetentionInpu
   return true;
 }
 
-// ---- operands of a single decoded token: q, k (before a unit norm) and the decay of one key channel ----
+// ---- operands of a single decoded token, item by item: q [dim] and k [dim] (before a unit norm), decays
+// [dim], v [vdim] of one head, in this order ----
 template <typename T>
-__device__ __forceinline__ void step_operands(const DeltaInputs& p, int head, int c, int64_t row, int64_t position,
-                                              int slot, float& q, float& k, float& g) {
-  const int channel = head / (p.heads / p.kv_heads) * p.dim + c;
-  q = silu_of(short_conv<T>(p, 0, channel, row, 0, position, slot));
-  k = silu_of(short_conv<T>(p, 1, channel, row, 0, position, slot));
-  g = expf(delta_log_decay<T>(p, row, head, c));
-}
-template <typename T>
-__device__ __forceinline__ void step_operands(const RetentionInputs& p, int head, int c, int64_t row,
-                                              int64_t position, int, float& q, float& k, float& g) {
-  const T* in = static_cast<const T*>(p.input) + row * p.row_stride + head * p.dim + c;
-  const T *qp = in + p.q_column, *kp = in + p.k_column;
-  q = Elem<T>::load(qp);
-  k = Elem<T>::load(kp);
-  const int half = p.rot_dims / 2;
-  if (c < p.rot_dims) {
-    const int i = c < half ? c : c - half;
-    const int other = c < half ? half : -half;
-    float cosine, sine;
-    rotation_of(position, i, p.rot_dims, p.log2_base, cosine, sine);
-    if (c < half) sine = -sine;
-    q = q * cosine + Elem<T>::load(qp + other) * sine;
-    k = k * cosine + Elem<T>::load(kp + other) * sine;
+__device__ __forceinline__ float step_operand(const DeltaInputs& p, int head, int item, int64_t row, int64_t position,
+                                              int slot) {
+  if (item < 2 * p.dim) {
+    const int which = item < p.dim ? 0 : 1;
+    const int channel = head / (p.heads / p.kv_heads) * p.dim + item - which * p.dim;
+    return silu_of(short_conv<T>(p, which, channel, row, 0, position, slot));
   }
-  k *= p.k_scale;
-  g = p.decay[head];
+  if (item < 3 * p.dim) return expf(delta_log_decay<T>(p, row, head, item - 2 * p.dim));
+  return silu_of(short_conv<T>(p, 2, head * p.vdim + item - 3 * p.dim, row, 0, position, slot));
 }
 template <typename T>
-__device__ __forceinline__ float step_value(const DeltaInputs& p, int head, int c, int64_t row, int64_t position,
-                                            int slot) {
-  return silu_of(short_conv<T>(p, 2, head * p.vdim + c, row, 0, position, slot));
-}
-template <typename T>
-__device__ __forceinline__ float step_value(const RetentionInputs& p, int head, int c, int64_t row, int64_t, int) {
-  return Elem<T>::load(static_cast<const T*>(p.input) + row * p.row_stride + p.v_column + head * p.vdim + c);
+__device__ __forceinline__ float step_operand(const RetentionInputs& p, int head, int item, int64_t row,
+                                              int64_t position, int) {
+  const T* in = static_cast<const T*>(p.input) + row * p.row_stride;
+  if (item < 2 * p.dim) {
+    const bool is_k = item >= p.dim;
+    const int c = is_k ? item - p.dim : item;
+    const T* src = in + (is_k ? p.k_column : p.q_column) + head * p.dim + c;
+    float value = Elem<T>::load(src);
+    const int half = p.rot_dims / 2;
+    if (c < p.rot_dims) {
+      const int other = c < half ? half : -half;
+      float cosine, sine;
+      rotation_of(position, c < half ? c : c - half, p.rot_dims, p.log2_base, cosine, sine);
+      value = value * cosine + Elem<T>::load(src + other) * (c < half ? -sine : sine);
+    }
+    return is_k ? value * p.k_scale : value;
+  }
+  if (item < 3 * p.dim) return p.decay[head];
+  return Elem<T>::load(in + p.v_column + head * p.vdim + item - 3 * p.dim);
 }
 template <typename T>
 __device__ __forceinline__ float step_beta(const DeltaInputs& p, int64_t row, int head) {

@@ -65,17 +65,19 @@ __global__ void __launch_bounds__(THREADS) recurrence_step_kernel(const Inputs p
   float beta = 0.0f;
   float q_squares = 0.0f, k_squares = 0.0f, along = 0.0f;  // sums over the key channels
   if (slot >= 0) {
+    // (qs, ks, gs and vs lie side by side in the items' order)
+    for (int item = threadIdx.x; item < 3 * p.dim + p.vdim; item += THREADS)
+      qs[item] = step_operand<T>(p, head, item, row, position, slot);
+    beta = step_beta<T>(p, row, head);
+  }
+  __syncthreads();
+  if (slot >= 0) {
     for (int c = threadIdx.x; c < p.dim; c += THREADS) {
-      float q, k;
-      step_operands<T>(p, head, c, row, position, slot, q, k, gs[c]);
-      qs[c] = q;
-      ks[c] = k;
+      const float q = qs[c], k = ks[c];
       q_squares += q * q;
       k_squares += k * k;
       along += q * k;
     }
-    for (int c = threadIdx.x; c < p.vdim; c += THREADS) vs[c] = step_value<T>(p, head, c, row, position, slot);
-    beta = step_beta<T>(p, row, head);
   }
   q_squares = warp_sum(q_squares);
   k_squares = warp_sum(k_squares);

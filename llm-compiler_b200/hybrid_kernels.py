@@ -63,6 +63,10 @@ class SequenceBatch:
             self._chunks = (torch.tensor(table, dtype=torch.int32).to(self.starts.device), table[-1])
         return self._chunks
 
+    @property
+    def longest(self) -> int:
+        return 1 if self.counts is None else max(self.counts)
+
     def context_bound(self, capacity: int) -> int:
         """Upper bound of the positions any row of this step sees."""
 
@@ -245,10 +249,11 @@ def delta_inputs(projected: torch.Tensor, gates: torch.Tensor, conv: Tuple[torch
     return inputs
 
 
-def delta_prep(inputs: "_lib.DeltaInputs", rows: int, dtype: torch.dtype, device: torch.device):
+def delta_prep(inputs: "_lib.DeltaInputs", batch: SequenceBatch, dtype: torch.dtype, device: torch.device):
     """fp32 operands of the gated delta rule: q, k [rows, kv_heads, dim], v [rows, heads, vdim],
     beta [rows, heads] and log g [rows, heads, dim]."""
 
+    rows = batch.rows
     q = torch.empty((rows, inputs.kv_heads, inputs.dim), dtype=torch.float32, device=device)
     k = torch.empty_like(q)
     v = torch.empty((rows, inputs.heads, inputs.vdim), dtype=torch.float32, device=device)
@@ -256,7 +261,7 @@ def delta_prep(inputs: "_lib.DeltaInputs", rows: int, dtype: torch.dtype, device
     decay = torch.empty((rows, inputs.heads, inputs.dim), dtype=torch.float32, device=device)
     rt = runtime(device)
     code = _lib.load().b200_delta_prep(byref(inputs), q.data_ptr(), k.data_ptr(), v.data_ptr(), beta.data_ptr(),
-                                       decay.data_ptr(), rows, _code(dtype), _stream())
+                                       decay.data_ptr(), rows, batch.sequences, batch.longest, _code(dtype), _stream())
     _check(code, "b200_delta_prep")
     _count(rt)
     return q, k, v, beta, decay
@@ -361,7 +366,7 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, sink: Optional[torch.
     output = torch.empty_like(q)
     rt = runtime(device)
     library = _lib.load()
-    longest = 1 if batch.counts is None else max(batch.counts)
+    longest = batch.longest
     context = batch.context_bound(cache.shape[1])
     need = int(library.b200_latent_attention_workspace_bytes(rows, batch.sequences, longest, heads, row, context,
                                                             _code(q.dtype)))

@@ -158,7 +158,7 @@ class ChannelDelta(Mixer):
             mixed = hk.recurrence_step(inputs, state["state"], gate, self.norm, batch.sequences, kind="sigmoid",
                                        epsilon=self.epsilon)
         if mixed is None:
-            q, k, v, beta, log_decay = hk.delta_prep(inputs, h.shape[0], h.dtype, h.device)
+            q, k, v, beta, log_decay = hk.delta_prep(inputs, batch, h.dtype, h.device)
             read_out = hk.recurrence(q, k, v, beta, log_decay, state["state"], batch, h.dtype)
             hk.conv_tail(inputs, batch.sequences, h.dtype, h.device)
             mixed = hk.gated_head_norm(read_out, self.norm, gate, kind="sigmoid", epsilon=self.epsilon)
