@@ -578,8 +578,9 @@ int64_t b200_latent_attention_workspace_bytes(int64_t rows, int64_t sequences, i
 int b200_latent_attention(const void* q, const void* cache, const void* sink, void* out,
                           const int32_t* token_sequence, const int32_t* starts, const int32_t* slots,
                           const int32_t* bases, int64_t rows, int64_t sequences, int64_t longest,
-                          int64_t heads, int64_t rank_row, int64_t capacity, int64_t context, double scale,
-                          int dtype, void* workspace, int64_t workspace_bytes, void* stream);
+                          int64_t heads, int64_t rank_row, int64_t slot_count, int64_t capacity,
+                          int64_t context, double scale, int dtype, void* workspace,
+                          int64_t workspace_bytes, int32_t* status, void* stream);
 int b200_sequence_positions(const int64_t* lengths, const int32_t* slots, int32_t* positions, int64_t rows,
                             void* stream);
 int b200_advance_slots(int64_t* lengths, const int32_t* slots, const int32_t* starts, int64_t rows,

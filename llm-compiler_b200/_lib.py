@@ -165,7 +165,8 @@ SIGNATURES = {
                                [c_double, c_void_p, c_void_p]),
     "b200_head_linear": (c_int, [c_void_p] * 3 + [c_int64] * 8 + [c_int, c_void_p]),
     "b200_latent_attention_workspace_bytes": (c_int64, [c_int64] * 6 + [c_int]),
-    "b200_latent_attention": (c_int, [c_void_p] * 8 + [c_int64] * 7 + [c_double, c_int, c_void_p, c_int64, c_void_p]),
+    "b200_latent_attention": (c_int, [c_void_p] * 8 + [c_int64] * 8 + [c_double, c_int, c_void_p, c_int64,
+                                                                     c_void_p, c_void_p]),
     "b200_sequence_positions": (c_int, [c_void_p] * 3 + [c_int64, c_void_p]),
     "b200_advance_slots": (c_int, [c_void_p] * 3 + [c_int64, c_int64, c_void_p, c_void_p]),
 }

@@ -3,11 +3,16 @@
 // cached rows themselves, and the weighted sum of the rows is carried out of it (W_uv) behind the
 // attention. The softmax denominator may hold a learned term per head (a sink) beside the keys.
 //
-// This file: the per-head projections in and out of the latent space, attention on warp-level tensor
-// cores with the keys split over CTAs (bf16, rank up to 512), and attention for any rank up to 1024 on
-// the CUDA cores (fp32 models, and shapes the tensor-core kernel does not take).
+// This file: the per-head projections in and out of the latent space; attention on warp-level tensor
+// cores with the keys split over CTAs (bf16, rank up to 512; B200_LATENT_PATH=mma.sync, the default is
+// the tcgen05 kernel of latent_attention_tcgen05.cu), the kernel that combines the splits of either; and
+// attention for any rank up to 1024 on the CUDA cores (fp32 models, and shapes the others do not take).
+#include <stdlib.h>
+#include <string.h>
+
 #include "common.cuh"
 #include "hybrid.cuh"
+#include "latent_attention.cuh"
 
 namespace b200 {
 namespace {
@@ -155,15 +160,6 @@ struct LatentSplitParams {
   float scale_log2;
 };
 
-// The keys of split `split`: equal shares of at least 128 keys, in whole steps.
-__device__ __forceinline__ void split_range(int64_t keys, int splits, int split, int64_t& begin, int64_t& end) {
-  int64_t share = (keys + splits - 1) / splits;
-  if (share < 128) share = 128;
-  share = (share + kLatentKeys - 1) / kLatentKeys * kLatentKeys;
-  begin = share * split;
-  end = begin + share < keys ? begin + share : keys;
-}
-
 template <int MT, int NT>
 __global__ void __launch_bounds__(kLatentThreads, 1) latent_attention_split_kernel(const LatentSplitParams p) {
   constexpr int M = 16 * MT;
@@ -183,7 +179,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_attention_split_kern
   int64_t keys = base + last_row / p.heads + 1;
   if (keys > p.capacity) keys = p.capacity;
   int64_t begin, end;
-  split_range(keys, p.splits, split, begin, end);
+  latent_split_range(keys, p.splits, split, kLatentKeys, begin, end);
   const int64_t unit0 = static_cast<int64_t>(first) * p.heads + row0;  // row of q and of the partials
   if (begin >= end) {
     for (int r = threadIdx.x; r <= last_row - row0; r += kLatentThreads)
@@ -589,53 +585,78 @@ extern "C" int b200_head_linear(const void* x, const void* w, void* y, int64_t m
   return launch_status();
 }
 
+// Which split-KV kernel serves a bf16 call, and with how many splits; splits 0: neither does.
+struct LatentChoice {
+  LatentTcPlan tcgen05;
+  LatentPlan warp_level;
+  int splits;
+};
+static LatentChoice choose_latent(int64_t sequences, int64_t longest, int64_t heads, int64_t rank, int64_t context) {
+  LatentChoice choice{};
+  const char* path = getenv("B200_LATENT_PATH");
+  if (path == nullptr || strcmp(path, "mma.sync") != 0)
+    choice.tcgen05 = plan_latent_tcgen05(sequences, longest, heads, rank, context);
+  choice.splits = choice.tcgen05.splits;
+  if (choice.tcgen05.n == 0) {
+    choice.warp_level = plan_latent(sequences, longest, heads, rank, context);
+    choice.splits = choice.warp_level.mt != 0 ? choice.warp_level.splits : 0;
+  }
+  return choice;
+}
+
 extern "C" int64_t b200_latent_attention_workspace_bytes(int64_t rows, int64_t sequences, int64_t longest,
                                                          int64_t heads, int64_t rank_row, int64_t context,
                                                          int dtype) {
   if (dtype != B200_BF16 || rows <= 0 || sequences <= 0 || longest <= 0 || heads <= 0 || rank_row <= 0 || context <= 0)
     return 0;
-  const LatentPlan plan = plan_latent(sequences, longest, heads, rank_row, context);
-  return plan.mt == 0 ? 0 : rows * heads * plan.splits * (rank_row + 2) * 4;
+  return rows * heads * choose_latent(sequences, longest, heads, rank_row, context).splits * (rank_row + 2) * 4;
 }
 
 extern "C" int b200_latent_attention(const void* q, const void* cache, const void* sink, void* out,
                                      const int32_t* token_sequence, const int32_t* starts, const int32_t* slots,
                                      const int32_t* bases, int64_t rows, int64_t sequences, int64_t longest,
-                                     int64_t heads, int64_t rank_row, int64_t capacity, int64_t context,
-                                     double scale, int dtype, void* workspace, int64_t workspace_bytes,
-                                     void* stream) {
+                                     int64_t heads, int64_t rank_row, int64_t slot_count, int64_t capacity,
+                                     int64_t context, double scale, int dtype, void* workspace,
+                                     int64_t workspace_bytes, int32_t* status, void* stream) {
   if (!q || !cache || !out || !token_sequence || !starts || !slots || !bases || rows < 0 || sequences <= 0 ||
-      longest <= 0 || heads <= 0 || rank_row <= 0 || capacity <= 0 || context <= 0)
+      longest <= 0 || heads <= 0 || rank_row <= 0 || slot_count <= 0 || capacity <= 0 || context <= 0)
     return B200_ERR_BAD_ARGUMENT;
   if (dtype != B200_F32 && dtype != B200_BF16) return B200_ERR_UNSUPPORTED;
   if (rows == 0) return B200_OK;
-  if (rows > INT32_MAX || heads > 65535 || sequences > 65535) return B200_ERR_TOO_LARGE;
+  if (rows * heads > INT32_MAX || heads > 65535 || sequences > 65535) return B200_ERR_TOO_LARGE;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (dtype == B200_BF16) {
-    const LatentPlan plan = plan_latent(sequences, longest, heads, rank_row, context);
-    if (plan.mt != 0 && plan.row_blocks <= 65535) {
-      const int64_t need = rows * heads * plan.splits * (rank_row + 2) * 4;
-      if (!workspace || workspace_bytes < need) return B200_ERR_WORKSPACE;
-      if (!aligned16(q) || !aligned16(cache) || !aligned16(workspace)) return B200_ERR_ALIGNMENT;
-      float* partial = static_cast<float*>(workspace);
-      float2* stats = reinterpret_cast<float2*>(partial + rows * heads * plan.splits * rank_row);
+  const SequenceBatch batch{token_sequence, starts, slots, bases};
+  const LatentChoice choice = dtype == B200_BF16 ? choose_latent(sequences, longest, heads, rank_row, context) : LatentChoice{};
+  if (choice.splits > 0) {
+    const int64_t need = rows * heads * choice.splits * (rank_row + 2) * 4;
+    if (!workspace || workspace_bytes < need) return B200_ERR_WORKSPACE;
+    if (!aligned16(q) || !aligned16(cache) || !aligned16(workspace)) return B200_ERR_ALIGNMENT;
+    float* partial = static_cast<float*>(workspace);
+    float2* stats = reinterpret_cast<float2*>(partial + rows * heads * choice.splits * rank_row);
+    int code;
+    if (choice.tcgen05.n != 0) {
+      if (choice.tcgen05.row_blocks > 65535) return B200_ERR_TOO_LARGE;
+      code = latent_attention_tcgen05(choice.tcgen05, q, cache, partial, stats, batch, rows, sequences, heads, rank_row,
+                                      slot_count, capacity, scale, status, s);
+    } else {
+      const LatentPlan& plan = choice.warp_level;
+      if (plan.row_blocks > 65535) return B200_ERR_TOO_LARGE;
       LatentSplitParams p{static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(cache), partial, stats,
-                          {token_sequence, starts, slots, bases}, static_cast<int>(heads), static_cast<int>(rank_row),
-                          plan.splits, plan.pitch, plan.stages, capacity, static_cast<float>(scale * 1.4426950408889634)};
-      const int code = plan.mt == 1 ? launch_split_nt<1>(p, plan, sequences, s)
-                       : plan.mt == 2 ? launch_split_nt<2>(p, plan, sequences, s)
-                                      : launch_split_nt<4>(p, plan, sequences, s);
-      if (code != B200_OK) return code;
-      const dim3 grid(static_cast<unsigned>(rows), static_cast<unsigned>(heads));
-      const SequenceBatch batch{token_sequence, starts, slots, bases};
-      return launch_chained(latent_combine_kernel, grid, dim3(128), 0, s, static_cast<const float*>(partial),
-                            static_cast<const float2*>(stats), static_cast<const __nv_bfloat16*>(sink),
-                            static_cast<__nv_bfloat16*>(out), batch, static_cast<int>(heads),
-                            static_cast<int>(rank_row), plan.splits) == cudaSuccess
-                 ? launch_status() : B200_ERR_LAUNCH;
+                          batch, static_cast<int>(heads), static_cast<int>(rank_row), plan.splits, plan.pitch, plan.stages,
+                          capacity, static_cast<float>(scale * 1.4426950408889634)};
+      code = plan.mt == 1 ? launch_split_nt<1>(p, plan, sequences, s)
+             : plan.mt == 2 ? launch_split_nt<2>(p, plan, sequences, s)
+                            : launch_split_nt<4>(p, plan, sequences, s);
     }
+    if (code != B200_OK) return code;
+    const dim3 grid(static_cast<unsigned>(rows), static_cast<unsigned>(heads));
+    return launch_chained(latent_combine_kernel, grid, dim3(128), 0, s, static_cast<const float*>(partial),
+                          static_cast<const float2*>(stats), static_cast<const __nv_bfloat16*>(sink),
+                          static_cast<__nv_bfloat16*>(out), batch, static_cast<int>(heads),
+                          static_cast<int>(rank_row), choice.splits) == cudaSuccess
+               ? launch_status() : B200_ERR_LAUNCH;
   }
-  LatentAttentionParams p{q, cache, sink, out, {token_sequence, starts, slots, bases}, static_cast<int>(heads),
+  LatentAttentionParams p{q, cache, sink, out, batch, static_cast<int>(heads),
                           static_cast<int>(rank_row), capacity, static_cast<float>(scale)};
   return dtype == B200_F32 ? launch_generic<float>(p, rows, s) : launch_generic<__nv_bfloat16>(p, rows, s);
 }

@@ -26,10 +26,11 @@ __device__ __forceinline__ uint64_t smem_descriptor_mn_major(uint32_t smem_addr,
          (uint64_t(1) << 46) | (uint64_t(2) << 61);
 }
 
-// Instruction descriptor of kind::f16: fp32 accumulator, bf16 A and B; A K-major, B K-major
-// or (b_mn_major) MN-major.
-__host__ __device__ constexpr uint32_t instruction_descriptor(int m, int n, bool b_mn_major = false) {
-  return (1u << 4) | (1u << 7) | (1u << 10) | (b_mn_major ? (1u << 16) : 0u) |
+// Instruction descriptor of kind::f16: fp32 accumulator, bf16 A and B; each K-major, or MN-major
+// (the transpose bits 15 of A and 16 of B).
+__host__ __device__ constexpr uint32_t instruction_descriptor(int m, int n, bool b_mn_major = false,
+                                                              bool a_mn_major = false) {
+  return (1u << 4) | (1u << 7) | (1u << 10) | (a_mn_major ? (1u << 15) : 0u) | (b_mn_major ? (1u << 16) : 0u) |
          (static_cast<uint32_t>(n >> 3) << 17) | (static_cast<uint32_t>(m >> 4) << 24);
 }
 

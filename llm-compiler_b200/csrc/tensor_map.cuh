@@ -45,6 +45,21 @@ inline bool make_bf16_matrix_map(CUtensorMap* map, const void* base, int64_t row
                 CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
+// bf16 [slots, rows, cols] contiguous, read in boxes of box_rows x 64 columns of one slot (128-byte rows,
+// 128B swizzle); rows past a slot's end and columns past cols give zeros.
+inline bool make_bf16_slot_map(CUtensorMap* map, const void* base, int64_t slots, int64_t rows, int64_t cols,
+                               int box_rows) {
+  EncodeTiledFn encode = tensor_map_encoder();
+  if (encode == nullptr || box_rows > 256 || slots <= 0 || rows <= 0 || cols <= 0 || cols % 8 != 0) return false;
+  const cuuint64_t dims[3] = {static_cast<cuuint64_t>(cols), static_cast<cuuint64_t>(rows), static_cast<cuuint64_t>(slots)};
+  const cuuint64_t strides[2] = {static_cast<cuuint64_t>(cols * 2), static_cast<cuuint64_t>(rows * cols * 2)};
+  const cuuint32_t box[3] = {64, static_cast<cuuint32_t>(box_rows), 1};
+  const cuuint32_t element_strides[3] = {1, 1, 1};
+  return encode(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box,
+                element_strides, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B,
+                CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
+}
+
 // bf16 tensor of logical shape [B, H, T, D] with element strides {sb, sh, st, 1}, read in boxes
 // of `box_tokens` tokens x 64 elements of one (batch, head): a 4-D map whose dimensions are
 // ordered by stride. *token_is_dim1 tells the kernel the coordinate order: {d, t, h, b} when

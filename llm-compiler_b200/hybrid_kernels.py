@@ -373,7 +373,8 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, sink: Optional[torch.
     workspace = rt.workspace("latent_attention", need)
     code = library.b200_latent_attention(
         q.data_ptr(), cache.data_ptr(), _ptr(sink), output.data_ptr(), *batch.pointers(), rows, batch.sequences,
-        longest, heads, row, cache.shape[1], context, float(scale), _code(q.dtype), _ptr(workspace), need, _stream())
+        longest, heads, row, cache.shape[0], cache.shape[1], context, float(scale), _code(q.dtype), _ptr(workspace),
+        need, rt.status.data_ptr(), _stream())
     _check(code, "b200_latent_attention")
     _count(rt, 2 if need else 1)
     return output

@@ -288,12 +288,15 @@ def test_sink_takes_its_share_of_the_denominator(dtype, sink):
 
 
 @pytest.mark.parametrize("dtype,rank,heads", [(torch.float32, 48, 3), (torch.bfloat16, 64, 3),
-                                              (torch.bfloat16, 512, 16), (torch.bfloat16, 80, 70)],
-                         ids=["fp32", "bf16", "bf16-rank512", "bf16-70heads"])
+                                              (torch.bfloat16, 512, 16), (torch.bfloat16, 80, 70),
+                                              (torch.bfloat16, 256, 28), (torch.bfloat16, 512, 40)],
+                         ids=["fp32", "bf16", "rank512", "70heads", "rank256", "rank512-40heads"])
 @pytest.mark.parametrize("tokens", [1, 3])
-def test_one_key_that_stands_out(dtype, rank, heads, tokens):
+@pytest.mark.parametrize("path", ["tcgen05", "mma.sync"])
+def test_one_key_that_stands_out(dtype, rank, heads, tokens, path, monkeypatch):
     """Queries that match one far key: it must be found wherever it lies, and must not be seen one
-    position beyond the row."""
+    position beyond the row. Both split-KV kernels; rows behind the last key hold anything finite."""
+    monkeypatch.setenv("B200_LATENT_PATH", path)
     g = torch.Generator().manual_seed(rank + heads)
     capacity, last = 700, 650  # the rows stand at last .. last + tokens - 1
     cache = (0.05 * torch.randn(2, capacity, rank, generator=g)).to(dtype).cuda()
@@ -312,6 +315,31 @@ def test_one_key_that_stands_out(dtype, rank, heads, tokens):
             close(out[t], want, dtype)
             seen = float((out[t].double().cpu() - rows[position]).abs().max()) < 0.2
             assert seen == (position <= last + t)
+    kernels.runtime().check_status()
+
+
+def test_latent_attention_over_ragged_batches_and_growing_scores():
+    """Contexts of one key to several tiles, an idle row, and scores that grow along the context, so that the
+    running reference has to move again and again."""
+    g = torch.Generator().manual_seed(0)
+    heads, rank, capacity = 20, 192, 1100
+    lengths = [1, 2, 127, 128, 129, 700, 1099, 5]
+    cache = torch.randn(9, capacity, rank, generator=g).to(torch.bfloat16)
+    direction = torch.randn(rank, generator=g)
+    direction /= direction.norm()
+    ramp = torch.linspace(0, 60, capacity)[:, None] * direction
+    cache = (0.3 * cache.float() + ramp).to(torch.bfloat16)
+    q = (torch.randn(8, heads, rank, generator=g) + 4 * direction).to(torch.bfloat16)
+    batch = batch_of([(slot, n - 1, 1) for slot, n in enumerate(lengths)])
+    batch.slots[7] = -1
+    sink = torch.randn(heads, generator=g).to(torch.bfloat16)
+    out = hk.latent_attention(q.cuda(), cache.cuda(), sink.cuda(), batch, scale=0.7)
+    kernels.runtime().check_status()
+    assert torch.all(out[7] == 0)
+    for i, n in enumerate(lengths[:7]):
+        rows = cache[i, :n].double()
+        scores = torch.cat([torch.einsum("hr,kr->hk", q[i].double(), rows) * 0.7, sink.double()[:, None]], -1)
+        close(out[i], torch.softmax(scores, -1)[:, :-1] @ rows, torch.bfloat16)
 
 
 @pytest.mark.parametrize("size", [64, 128])

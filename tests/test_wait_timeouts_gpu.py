@@ -99,3 +99,23 @@ def test_decode_attention_wait_timeout_then_recovery():
     close(b200.b200_decode_attention(q.cuda(), k.cuda(), v.cuda(), lengths.cuda(), None, scale=0.125,
                                      split_tokens=256), ref)
     kernels.runtime().check_status()
+
+
+def test_latent_attention_wait_timeout_then_recovery():
+    from llm_compiler_b200 import hybrid_kernels as hk
+
+    g = torch.Generator().manual_seed(9)
+    q = torch.randn(2, 16, 256, generator=g).bfloat16()
+    cache = torch.randn(2, 400, 256, generator=g).bfloat16()
+    vector = lambda values: torch.tensor(values, dtype=torch.int32, device="cuda")
+    batch = hk.SequenceBatch(2, 2, vector([0, 1]), vector([0, 1, 2]), vector([0, 1]), vector([299, 399]))
+    call = lambda: hk.latent_attention(q.cuda(), cache.cuda(), None, batch, scale=0.05)
+    for _ in range(3):
+        with waits_that_run_out():
+            call()
+        expect_timeout()
+    out = call()
+    for i, n in enumerate((300, 400)):
+        weights = torch.softmax(torch.einsum("hr,kr->hk", q[i].float(), cache[i, :n].float()) * 0.05, -1)
+        close(out[i], weights @ cache[i, :n].float())
+    kernels.runtime().check_status()
