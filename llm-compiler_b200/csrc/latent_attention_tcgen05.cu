@@ -5,12 +5,14 @@
 //   S^T [128 keys x N]       = C Q^T        C tile K-major (as TMA lays it down), Q K-major
 //   O^T [128 rank x N] each  = C^T P^T      the same C tile read MN-major, P [N x 128 keys] K-major
 //
-// One fetch of a latent therefore serves as key and as value. The tile is cut into pairs of 64-column
-// panels (32 KB) that move through a ring: a pair is free as soon as its block of O^T has been issued and
-// retired, while the next tile's pairs stream in. One thread issues the TMA boxes, one the MMAs; four warps
+// so one read of HBM serves as key and as value. The tile is cut into pairs of 64-column panels (32 KB) that
+// stream through a ring. Where the ring holds two tiles, a tile's pairs stay until its output product has
+// read them. Where it does not (rank above 256), every pair is fetched twice, once per product (the second
+// time from L2, a few microseconds later), so that the stream never waits for a softmax: the scores of tile
+// j + 1 are computed before the output of tile j. One thread issues the TMA boxes, one the MMAs; four warps
 // hold a key per thread, take the column maxima with warp reductions, and write the probabilities as two
-// bf16 planes whose sum keeps 16 bits of mantissa (the tensor core has room for both products: the kernel
-// is bound by the fetch). The reference maximum is lazy: O^T is rescaled in tensor memory only when a row's
+// bf16 numbers whose sum keeps 16 bits of mantissa: both are rows of one operand (2 N columns of O^T, added at
+// the end), because a product of this shape costs what reading its M operand costs. The reference maximum is lazy: O^T is rescaled in tensor memory only when a row's
 // maximum rises by more than 8 in the log2 domain. Every wait is bounded.
 #include "common.cuh"
 #include "hybrid.cuh"
@@ -31,7 +33,7 @@ struct LatentTcParams {
   float2* partial_stats;  // [rows * heads, splits]: reference (log2 domain), sum
   SequenceBatch batch;
   int32_t* status;
-  int heads, rank, splits, pairs, ring;
+  int heads, rank, splits, pairs, ring, refetch;
   int64_t capacity;
   float scale_log2;
   uint32_t wait_limit;
@@ -57,9 +59,9 @@ __global__ void __launch_bounds__(kThreads, 1)
 latent_attention_tcgen05_kernel(const LatentTcParams p, const __grid_constant__ CUtensorMap q_map,
                                 const __grid_constant__ CUtensorMap c_map) {
   constexpr int kGroups = N / 32;                        // 32-column groups of a row of S^T
-  constexpr uint32_t kQPanel = N * 128, kPPanel = N * 128, kPPlane = 2 * kPPanel;
+  constexpr uint32_t kQPanel = N * 128, kPPanel = 2 * N * 128, kPLow = N * 128;
   extern __shared__ __align__(1024) unsigned char smem[];
-  __shared__ __align__(8) uint64_t q_full, s_full, p_full, o_done, pair_full[kMaxRing], pair_empty[kMaxRing];
+  __shared__ __align__(8) uint64_t q_full, s_full[2], p_full, o_done, pair_full[kMaxRing], pair_empty[kMaxRing];
   __shared__ float warp_tops[2][kSoftmaxWarps][N];
   __shared__ int limits[N];
   __shared__ uint32_t tmem_slot;
@@ -67,11 +69,12 @@ latent_attention_tcgen05_kernel(const LatentTcParams p, const __grid_constant__ 
   grid_launch_dependents();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int split = blockIdx.x, sequence = blockIdx.z, row0 = blockIdx.y * N;
-  const uint32_t columns = (p.pairs + 1) * N <= 128 ? 128u : (p.pairs + 1) * N <= 256 ? 256u : 512u;
+  const uint32_t columns = (p.pairs + 1) * 2 * N <= 128 ? 128u : (p.pairs + 1) * 2 * N <= 256 ? 256u : 512u;
   if (threadIdx.x == 0) {
     failed = 0;
     mbarrier_init(smem_u32(&q_full), 1);
-    mbarrier_init(smem_u32(&s_full), 1);
+    mbarrier_init(smem_u32(&s_full[0]), 1);
+    mbarrier_init(smem_u32(&s_full[1]), 1);
     mbarrier_init(smem_u32(&p_full), kSoftmaxWarps);
     mbarrier_init(smem_u32(&o_done), 1);
     for (int i = 0; i < kMaxRing; ++i) {
@@ -79,6 +82,10 @@ latent_attention_tcgen05_kernel(const LatentTcParams p, const __grid_constant__ 
       mbarrier_init(smem_u32(&pair_empty[i]), 1);
     }
     fence_mbarrier_init();
+  }
+  if (warp == kTmaWarp && lane == 0) {
+    asm volatile("prefetch.tensormap [%0];" ::"l"(reinterpret_cast<uint64_t>(&q_map)) : "memory");
+    asm volatile("prefetch.tensormap [%0];" ::"l"(reinterpret_cast<uint64_t>(&c_map)) : "memory");
   }
   if (warp == kMmaWarp) {
     asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;"
@@ -105,8 +112,8 @@ latent_attention_tcgen05_kernel(const LatentTcParams p, const __grid_constant__ 
   const int tiles = (span + kTileKeys - 1) / kTileKeys;
   const uint32_t ring_smem = smem_u32(smem);
   const uint32_t q_smem = ring_smem + p.ring * kPairBytes;             // [2 pairs] panels of N rows
-  const uint32_t p_smem = q_smem + 2 * p.pairs * kQPanel;              // [high, low][2 panels of 64 keys][N rows]
-  const uint32_t o_column = tmem + N;
+  const uint32_t p_smem = q_smem + 2 * p.pairs * kQPanel;              // [2 panels of 64 keys][N high, N low rows]
+  const uint32_t o_column = tmem + 2 * N;  // behind two buffers of S^T
   if (active && threadIdx.x < N)  // first key, counted from begin, that a row does not see
     limits[threadIdx.x] = row0 + static_cast<int>(threadIdx.x) <= last_row
                               ? static_cast<int>(min(base + (row0 + static_cast<int>(threadIdx.x)) / p.heads + 1, end) - begin)
@@ -123,17 +130,24 @@ latent_attention_tcgen05_kernel(const LatentTcParams p, const __grid_constant__ 
     for (int panel = 0; panel < 2 * p.pairs; ++panel)
       tma_load_2d(q_smem + panel * kQPanel, &q_map, smem_u32(&q_full), panel * 64, static_cast<int>(unit0));
     bool ok = true;
-    int index = 0;  // pair number over all tiles
-    for (int j = 0; ok && j < tiles; ++j)
-      for (int m = 0; ok && m < p.pairs; ++m, ++index) {
+    int index = 0;  // pairs fetched so far
+    auto push = [&](int j) {
+      for (int m = 0; ok && m < p.pairs; ++m) {
         const int place = index % p.ring, use = index / p.ring;
         ok = use == 0 || mbarrier_wait_bounded(smem_u32(&pair_empty[place]), (use - 1) & 1, p.wait_limit);
-        if (!ok) break;
+        if (!ok) return;
         mbarrier_arrive_expect_tx(smem_u32(&pair_full[place]), kPairBytes);
         for (int half = 0; half < 2; ++half)
           tma_load_3d(ring_smem + place * kPairBytes + half * kPanelBytes, &c_map, smem_u32(&pair_full[place]),
                       m * 128 + half * 64, static_cast<int>(begin) + j * kTileKeys, slot);
+        ++index;
       }
+    };
+    push(0);
+    for (int j = 0; ok && j < tiles; ++j) {
+      if (j + 1 < tiles) push(j + 1);
+      if (p.refetch) push(j);
+    }
     if (!ok) failed = 1;
     // nothing of this CTA's is in flight when it ends
     mbarrier_wait_bounded(smem_u32(&q_full), 0, p.wait_limit);
@@ -142,43 +156,49 @@ latent_attention_tcgen05_kernel(const LatentTcParams p, const __grid_constant__ 
   } else if (warp == kMmaWarp && lane == 0) {
     // ---- MMA issuer ----
     constexpr uint32_t idesc_s = instruction_descriptor(128, N);
-    constexpr uint32_t idesc_o = instruction_descriptor(128, N, false, true);
+    constexpr uint32_t idesc_o = instruction_descriptor(128, 2 * N, false, true);
     const uint64_t q_desc = smem_descriptor(q_smem), p_desc = smem_descriptor(p_smem);
     bool ok = mbarrier_wait_bounded(smem_u32(&q_full), 0, p.wait_limit);
+    int index = 0;  // pairs taken so far (refetch)
+    auto next_pair = [&](int j, int m) { return p.refetch ? index++ : j * p.pairs + m; };
+    auto landed = [&](int pair) {
+      ok = mbarrier_wait_bounded(smem_u32(&pair_full[pair % p.ring]), (pair / p.ring) & 1, p.wait_limit);
+      asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+      return ok;
+    };
     auto issue_scores = [&](int j) {
-      for (int m = 0; ok && m < p.pairs; ++m) {
-        const int index = j * p.pairs + m, place = index % p.ring;
-        ok = mbarrier_wait_bounded(smem_u32(&pair_full[place]), (index / p.ring) & 1, p.wait_limit);
-        if (!ok) return;
-        asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-        const uint64_t c_desc = smem_descriptor(ring_smem + place * kPairBytes);
+      for (int m = 0; m < p.pairs; ++m) {
+        const int pair = next_pair(j, m);
+        if (!landed(pair)) return;
+        const uint64_t c_desc = smem_descriptor(ring_smem + pair % p.ring * kPairBytes);
 #pragma unroll
         for (int ks = 0; ks < 8; ++ks)
-          umma_bf16(tmem, descriptor_advance(c_desc, (ks / 4) * kPanelBytes + (ks % 4) * 32),
+          umma_bf16(tmem + (j & 1) * N, descriptor_advance(c_desc, (ks / 4) * kPanelBytes + (ks % 4) * 32),
                     descriptor_advance(q_desc, (2 * m + ks / 4) * kQPanel + (ks % 4) * 32), idesc_s,
                     m > 0 || ks > 0 ? 1u : 0u);
+        if (p.refetch) umma_commit(smem_u32(&pair_empty[pair % p.ring]));
       }
-      umma_commit(smem_u32(&s_full));
+      umma_commit(smem_u32(&s_full[j & 1]));
     };
     if (ok) issue_scores(0);
     for (int j = 0; ok && j < tiles; ++j) {
-      ok = mbarrier_wait_bounded(smem_u32(&p_full), j & 1, p.wait_limit);
+      if (j + 1 < tiles) issue_scores(j + 1);  // (its buffer's scores, of tile j - 1, were read before p_full of j - 1)
+      ok = ok && mbarrier_wait_bounded(smem_u32(&p_full), j & 1, p.wait_limit);
       if (!ok) break;
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       for (int m = 0; m < p.pairs; ++m) {
-        const int place = (j * p.pairs + m) % p.ring;
-        const uint64_t c_desc = smem_descriptor_mn_major(ring_smem + place * kPairBytes, kPanelBytes);
+        const int pair = next_pair(j, m);
+        if (p.refetch && !landed(pair)) break;
+        const uint64_t c_desc = smem_descriptor_mn_major(ring_smem + pair % p.ring * kPairBytes, kPanelBytes);
 #pragma unroll
         for (int ks = 0; ks < 8; ++ks) {  // 16 keys a step
           const uint32_t at = (ks / 4) * kPPanel + (ks % 4) * 32;
-          const uint64_t a = descriptor_advance(c_desc, ks * 2048);
-          umma_bf16(o_column + m * N, a, descriptor_advance(p_desc, at), idesc_o, j > 0 || ks > 0 ? 1u : 0u);
-          umma_bf16(o_column + m * N, a, descriptor_advance(p_desc, kPPlane + at), idesc_o, 1u);
+          umma_bf16(o_column + m * 2 * N, descriptor_advance(c_desc, ks * 2048), descriptor_advance(p_desc, at), idesc_o,
+                    j > 0 || ks > 0 ? 1u : 0u);
         }
-        umma_commit(smem_u32(&pair_empty[place]));
+        umma_commit(smem_u32(&pair_empty[pair % p.ring]));
       }
-      umma_commit(smem_u32(&o_done));
-      if (j + 1 < tiles) issue_scores(j + 1);  // (the scores of tile j were read before its p_full)
+      if (ok) umma_commit(smem_u32(&o_done));
     }
     if (!ok) failed = 1;
   } else if (warp < kSoftmaxWarps) {
@@ -197,7 +217,7 @@ latent_attention_tcgen05_kernel(const LatentTcParams p, const __grid_constant__ 
     const uint32_t chunk = (row & 63) >> 3;
     bool ok = true;
     for (int j = 0; j < tiles; ++j) {
-      ok = ok && __all_sync(0xffffffffu, mbarrier_wait_ready_first(smem_u32(&s_full), j & 1, p.wait_limit));
+      ok = ok && __all_sync(0xffffffffu, mbarrier_wait_ready_first(smem_u32(&s_full[j & 1]), (j >> 1) & 1, p.wait_limit));
       float s[N];
       const int key = j * kTileKeys + row;
       if (ok) {
@@ -205,7 +225,7 @@ latent_attention_tcgen05_kernel(const LatentTcParams p, const __grid_constant__ 
 #pragma unroll
         for (int g = 0; g < kGroups; ++g) {
           float t[32];
-          tmem_load_32x32(tmem + lane_base + g * 32, t);
+          tmem_load_32x32(tmem + (j & 1) * N + lane_base + g * 32, t);
 #pragma unroll
           for (int i = 0; i < 32; ++i) s[g * 32 + i] = t[i] * p.scale_log2;
         }
@@ -255,7 +275,7 @@ latent_attention_tcgen05_kernel(const LatentTcParams p, const __grid_constant__ 
             f[i] = __shfl_sync(0xffffffffu, factor[g], i);
             sums[g * 32 + i] *= f[i];
           }
-          for (int m = 0; m < p.pairs; ++m) {
+          for (int m = 0; m < 2 * p.pairs; ++m) {  // high and low parts
             float t[32];
             tmem_load_32x32(o_column + m * N + lane_base + g * 32, t);
 #pragma unroll
@@ -273,17 +293,23 @@ latent_attention_tcgen05_kernel(const LatentTcParams p, const __grid_constant__ 
         const uint16_t high = f32_to_bf16_bits(value), low = f32_to_bf16_bits(value - bf16_to_f32(high));
         const uint32_t at = p_row + n * 128 + ((chunk ^ (n & 7)) << 4);
         asm volatile("st.shared.u16 [%0], %1;" ::"r"(at), "h"(high) : "memory");
-        asm volatile("st.shared.u16 [%0], %1;" ::"r"(at + kPPlane), "h"(low) : "memory");
+        asm volatile("st.shared.u16 [%0], %1;" ::"r"(at + kPLow), "h"(low) : "memory");
       }
-      if (key >= span) {  // rows behind the split's end carry weight 0: make them 0 as values, too
+      if ((j + 1) * kTileKeys > span) {  // rows behind the split's end carry weight 0: make them 0 as values, too
         for (int m = 0; m < p.pairs; ++m) {
-          const uint32_t at = ring_smem + ((j * p.pairs + m) % p.ring) * kPairBytes + row * 128;
+          const int pair = p.refetch ? (2 * tiles - 1) * p.pairs + m : j * p.pairs + m;
+          if (p.refetch)
+            ok = ok && __all_sync(0xffffffffu, mbarrier_wait_ready_first(smem_u32(&pair_full[pair % p.ring]),
+                                                                         (pair / p.ring) & 1, p.wait_limit));
+          if (!ok || key < span) continue;
+          const uint32_t at = ring_smem + pair % p.ring * kPairBytes + row * 128;
 #pragma unroll
           for (int i = 0; i < 8; ++i) {
             asm volatile("st.shared.v4.b32 [%0], {%1, %1, %1, %1};" ::"r"(at + i * 16), "r"(0u) : "memory");
             asm volatile("st.shared.v4.b32 [%0], {%1, %1, %1, %1};" ::"r"(at + kPanelBytes + i * 16), "r"(0u) : "memory");
           }
         }
+        if (!ok) continue;
       }
       asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -298,13 +324,14 @@ latent_attention_tcgen05_kernel(const LatentTcParams p, const __grid_constant__ 
       for (int m = 0; m < p.pairs; ++m)
 #pragma unroll
         for (int g = 0; g < kGroups; ++g) {
-          float t[32];
-          tmem_load_32x32(o_column + m * N + lane_base + g * 32, t);
+          float t[32], low[32];
+          tmem_load_32x32(o_column + m * 2 * N + lane_base + g * 32, t);
+          tmem_load_32x32(o_column + m * 2 * N + N + lane_base + g * 32, low);
           if (m * 128 + row < p.rank) {
             float* out = p.partial + ((unit0 + g * 32) * p.splits + split) * p.rank + m * 128 + row;
 #pragma unroll
             for (int i = 0; i < 32; ++i)
-              if (row0 + g * 32 + i <= last_row) out[static_cast<int64_t>(i) * p.splits * p.rank] = t[i];
+              if (row0 + g * 32 + i <= last_row) out[static_cast<int64_t>(i) * p.splits * p.rank] = t[i] + low[i];
           }
         }
     }
@@ -347,24 +374,23 @@ LatentTcPlan plan_latent_tcgen05(int64_t sequences, int64_t longest, int64_t hea
   const int64_t rows = longest * heads;
   plan.pairs = static_cast<int>(ceil_div(rank, 128));
   int n = rows <= 32 ? 32 : 64, fixed = 0;
-  for (;; n = 32) {  // 64 rows where a whole tile fits beside them
+  for (;; n = 32) {  // 64 rows where a whole tile fits beside them, and the output in tensor memory
     fixed = 2 * plan.pairs * n * 128 + 4 * n * 128;  // Q, P
     plan.ring = (222 * 1024 - fixed) / kPairBytes;
-    if (plan.ring >= plan.pairs || n == 32) break;
+    if ((plan.ring >= plan.pairs && (plan.pairs + 1) * 2 * n <= 512) || n == 32) break;
   }
   if (plan.ring > kMaxRing) plan.ring = kMaxRing;
   if (plan.ring < plan.pairs) return plan;
   plan.n = n;
   plan.smem = fixed + plan.ring * kPairBytes;
   plan.row_blocks = static_cast<int>(ceil_div(rows, n));
-  const int64_t units = sequences * plan.row_blocks, most = ceil_div(context, 2 * kTileKeys);
-  double best = -1.0;
-  plan.splits = 1;
-  for (int64_t s = 1; s <= 64 && s <= most; ++s) {
-    const int64_t ctas = units * s;
-    const double fill = static_cast<double>(ctas) / (ceil_div(ctas, static_cast<int64_t>(kNumSMs)) * kNumSMs) - 0.01 * s;
-    if (fill > best) {
-      best = fill;
+  // whole waves of CTAs, each of which costs its tiles and about five more for its start and its end
+  const int64_t units = sequences * plan.row_blocks, all = ceil_div(context, static_cast<int64_t>(kTileKeys));
+  int64_t best = -1;
+  for (int64_t s = 1; s <= 64 && (s == 1 || 2 * s <= all); ++s) {
+    const int64_t cost = ceil_div(units * s, static_cast<int64_t>(kNumSMs)) * (ceil_div(all, s) + 5);
+    if (best < 0 || cost < best) {
+      best = cost;
       plan.splits = static_cast<int>(s);
     }
   }
@@ -379,7 +405,7 @@ int latent_attention_tcgen05(const LatentTcPlan& plan, const void* q, const void
       !make_bf16_slot_map(&c_map, cache, slots, capacity, rank, kTileKeys))
     return B200_ERR_UNSUPPORTED;
   LatentTcParams p{partial, stats, batch, status, static_cast<int>(heads), static_cast<int>(rank), plan.splits,
-                   plan.pairs, plan.ring, capacity, static_cast<float>(scale * 1.4426950408889634), wait_limit(),
+                   plan.pairs, plan.ring, plan.ring < 2 * plan.pairs ? 1 : 0, capacity, static_cast<float>(scale * 1.4426950408889634), wait_limit(),
                    drop_loads()};
   const dim3 grid(static_cast<unsigned>(plan.splits), static_cast<unsigned>(plan.row_blocks),
                   static_cast<unsigned>(sequences));
