@@ -69,7 +69,7 @@ latent_attention_tcgen05_kernel(const LatentTcParams p, const __grid_constant__ 
   grid_launch_dependents();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int split = blockIdx.x, sequence = blockIdx.z, row0 = blockIdx.y * N;
-  const uint32_t columns = (p.pairs + 1) * 2 * N <= 128 ? 128u : (p.pairs + 1) * 2 * N <= 256 ? 256u : 512u;
+  const uint32_t columns = (p.pairs + 2) * 2 * N <= 256 ? 256u : 512u;
   if (threadIdx.x == 0) {
     failed = 0;
     mbarrier_init(smem_u32(&q_full), 1);
@@ -113,7 +113,7 @@ latent_attention_tcgen05_kernel(const LatentTcParams p, const __grid_constant__ 
   const uint32_t ring_smem = smem_u32(smem);
   const uint32_t q_smem = ring_smem + p.ring * kPairBytes;             // [2 pairs] panels of N rows
   const uint32_t p_smem = q_smem + 2 * p.pairs * kQPanel;              // [2 panels of 64 keys][N high, N low rows]
-  const uint32_t o_column = tmem + 2 * N;  // behind two buffers of S^T
+  const uint32_t o_column = tmem + 4 * N;  // behind two buffers of two partial S^T
   if (active && threadIdx.x < N)  // first key, counted from begin, that a row does not see
     limits[threadIdx.x] = row0 + static_cast<int>(threadIdx.x) <= last_row
                               ? static_cast<int>(min(base + (row0 + static_cast<int>(threadIdx.x)) / p.heads + 1, end) - begin)
@@ -173,9 +173,9 @@ latent_attention_tcgen05_kernel(const LatentTcParams p, const __grid_constant__ 
         const uint64_t c_desc = smem_descriptor(ring_smem + pair % p.ring * kPairBytes);
 #pragma unroll
         for (int ks = 0; ks < 8; ++ks)
-          umma_bf16(tmem + (j & 1) * N, descriptor_advance(c_desc, (ks / 4) * kPanelBytes + (ks % 4) * 32),
+          umma_bf16(tmem + ((j & 1) * 2 + (ks & 1)) * N, descriptor_advance(c_desc, (ks / 4) * kPanelBytes + (ks % 4) * 32),
                     descriptor_advance(q_desc, (2 * m + ks / 4) * kQPanel + (ks % 4) * 32), idesc_s,
-                    m > 0 || ks > 0 ? 1u : 0u);
+                    m > 0 || ks > 1 ? 1u : 0u);
         if (p.refetch) umma_commit(smem_u32(&pair_empty[pair % p.ring]));
       }
       umma_commit(smem_u32(&s_full[j & 1]));
@@ -186,17 +186,24 @@ latent_attention_tcgen05_kernel(const LatentTcParams p, const __grid_constant__ 
       ok = ok && mbarrier_wait_bounded(smem_u32(&p_full), j & 1, p.wait_limit);
       if (!ok) break;
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-      for (int m = 0; m < p.pairs; ++m) {
-        const int pair = next_pair(j, m);
-        if (p.refetch && !landed(pair)) break;
-        const uint64_t c_desc = smem_descriptor_mn_major(ring_smem + pair % p.ring * kPairBytes, kPanelBytes);
+      // Products with one accumulator follow one another at the latency of a product: two blocks of O^T
+      // take turns.
+      for (int m = 0; ok && m < p.pairs; m += 2) {
+        const bool two = m + 1 < p.pairs;
+        const int pair0 = next_pair(j, m), pair1 = two ? next_pair(j, m + 1) : pair0;
+        if (p.refetch && (!landed(pair0) || (two && !landed(pair1)))) break;
+        const uint64_t c0 = smem_descriptor_mn_major(ring_smem + pair0 % p.ring * kPairBytes, kPanelBytes);
+        const uint64_t c1 = smem_descriptor_mn_major(ring_smem + pair1 % p.ring * kPairBytes, kPanelBytes);
 #pragma unroll
         for (int ks = 0; ks < 8; ++ks) {  // 16 keys a step
-          const uint32_t at = (ks / 4) * kPPanel + (ks % 4) * 32;
-          umma_bf16(o_column + m * 2 * N, descriptor_advance(c_desc, ks * 2048), descriptor_advance(p_desc, at), idesc_o,
-                    j > 0 || ks > 0 ? 1u : 0u);
+          const uint32_t at = (ks / 4) * kPPanel + (ks % 4) * 32, accumulate = j > 0 || ks > 0 ? 1u : 0u;
+          umma_bf16(o_column + m * 2 * N, descriptor_advance(c0, ks * 2048), descriptor_advance(p_desc, at), idesc_o, accumulate);
+          if (two)
+            umma_bf16(o_column + (m + 1) * 2 * N, descriptor_advance(c1, ks * 2048), descriptor_advance(p_desc, at), idesc_o,
+                      accumulate);
         }
-        umma_commit(smem_u32(&pair_empty[pair % p.ring]));
+        umma_commit(smem_u32(&pair_empty[pair0 % p.ring]));
+        if (two) umma_commit(smem_u32(&pair_empty[pair1 % p.ring]));
       }
       if (ok) umma_commit(smem_u32(&o_done));
     }
@@ -224,10 +231,11 @@ latent_attention_tcgen05_kernel(const LatentTcParams p, const __grid_constant__ 
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
 #pragma unroll
         for (int g = 0; g < kGroups; ++g) {
-          float t[32];
-          tmem_load_32x32(tmem + (j & 1) * N + lane_base + g * 32, t);
+          float t[32], u[32];  // the sums over even and odd k-steps
+          tmem_load_32x32(tmem + (j & 1) * 2 * N + lane_base + g * 32, t);
+          tmem_load_32x32(tmem + (j & 1) * 2 * N + N + lane_base + g * 32, u);
 #pragma unroll
-          for (int i = 0; i < 32; ++i) s[g * 32 + i] = t[i] * p.scale_log2;
+          for (int i = 0; i < 32; ++i) s[g * 32 + i] = (t[i] + u[i]) * p.scale_log2;
         }
         asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
         if ((j + 1) * kTileKeys > seen_by_all) {
@@ -377,7 +385,7 @@ LatentTcPlan plan_latent_tcgen05(int64_t sequences, int64_t longest, int64_t hea
   for (;; n = 32) {  // 64 rows where a whole tile fits beside them, and the output in tensor memory
     fixed = 2 * plan.pairs * n * 128 + 4 * n * 128;  // Q, P
     plan.ring = (222 * 1024 - fixed) / kPairBytes;
-    if ((plan.ring >= plan.pairs && (plan.pairs + 1) * 2 * n <= 512) || n == 32) break;
+    if ((plan.ring >= plan.pairs && (plan.pairs + 2) * 2 * n <= 512) || n == 32) break;
   }
   if (plan.ring > kMaxRing) plan.ring = kMaxRing;
   if (plan.ring < plan.pairs) return plan;
