@@ -463,6 +463,7 @@ int b200_argmax(const void* logits, int64_t* ids, int64_t rows, int64_t vocab,
  * starts from an empty state whatever the slot held before. dtype is B200_F32 or B200_BF16 (weights,
  * projections, cached latents); state, decays, gates, norms and the residual are fp32.
  *
+ *   b200_embedding_residual  x[r, :] = table[ids[r], :] widened to fp32
  *   b200_residual_norm   x += norm(y) * (weight_offset + post_weight); h = norm(x) * (weight_offset +
  *                        next_weight). x fp32 [rows, width]; y of the model dtype, or fp32 split-K
  *                        partials [splits, rows, y_row_stride] when splits > 0; y NULL: h only;
@@ -537,6 +538,8 @@ typedef struct b200_step_output {
   int64_t gate_kind;
   double epsilon;
 } b200_step_output;
+int b200_embedding_residual(const void* table, const int64_t* ids, float* x, int64_t rows, int64_t width,
+                            int64_t vocab, int dtype, int32_t* status, void* stream);
 int b200_residual_norm(void* x, const void* y, const void* post_weight, const void* next_weight, void* h,
                        int64_t rows, int64_t width, int64_t splits, int64_t y_row_stride,
                        int64_t h_row_stride, double epsilon, double weight_offset, int dtype, void* stream);

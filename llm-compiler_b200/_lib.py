@@ -150,6 +150,7 @@ SIGNATURES = {
     "b200_advance_lengths": (c_int, [c_void_p, c_int64, c_int64, c_int64, c_int64, c_void_p,
                                      c_void_p]),
     "b200_argmax": (c_int, [c_void_p, c_void_p, c_int64, c_int64, c_int64, c_int, c_void_p]),
+    "b200_embedding_residual": (c_int, [c_void_p] * 3 + [c_int64] * 3 + [c_int, c_void_p, c_void_p]),
     "b200_residual_norm": (c_int, [c_void_p] * 5 + [c_int64] * 5 + [c_double, c_double, c_int, c_void_p]),
     "b200_latent_norm": (c_int, [c_void_p] * 10 + [c_int64] * 8 + [c_double, c_int, c_void_p, c_void_p]),
     "b200_gated_head_norm": (c_int, [c_void_p] * 4 + [c_int64] * 5 + [c_int, c_double, c_int, c_void_p]),

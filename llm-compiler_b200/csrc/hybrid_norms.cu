@@ -302,6 +302,23 @@ __global__ void __launch_bounds__(256) gated_head_norm_quads_kernel(const GatedH
                             v.z * factor * w.z * gate_value(gate.z, p.gate_kind), v.w * factor * w.w * gate_value(gate.w, p.gate_kind)));
 }
 
+// The residual stream's first rows: a row of the table per id, widened to fp32
+template <typename T>
+__global__ void __launch_bounds__(256) embedding_residual_kernel(const T* table, const int64_t* ids, float* x, int width,
+                                                                 int64_t vocab, int32_t* status) {
+  const int64_t row = blockIdx.x, id = ids[row];
+  const bool known = id >= 0 && id < vocab;
+  if (!known && threadIdx.x == 0) atomicOr(status, B200_STATUS_BAD_TOKEN_ID);
+  const T* source = table + (known ? id : 0) * width;
+  float* out = x + row * width;
+  if (width % 4 == 0) {
+    for (int c = threadIdx.x * 4; c < width; c += blockDim.x * 4)
+      *reinterpret_cast<float4*>(out + c) = known ? load_quad<T>(source + c) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+  } else {
+    for (int c = threadIdx.x; c < width; c += blockDim.x) out[c] = known ? Elem<T>::load(source + c) : 0.0f;
+  }
+}
+
 // positions[r] and the row's slot: what a replayed step reads; lengths advance behind the step
 __global__ void sequence_positions_kernel(const int64_t* lengths, const int32_t* slots, int32_t* positions,
                                           int rows) {
@@ -418,6 +435,23 @@ extern "C" int b200_gated_head_norm(const void* input, const void* weight, const
   const cudaError_t code = dtype == B200_F32 ? launch_chained(gated_head_norm_kernel<float>, grid, dim3(256), 0, s, p)
                                              : launch_chained(gated_head_norm_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, p);
   return code == cudaSuccess ? launch_status() : B200_ERR_LAUNCH;
+}
+
+extern "C" int b200_embedding_residual(const void* table, const int64_t* ids, float* x, int64_t rows, int64_t width,
+                                       int64_t vocab, int dtype, int32_t* status, void* stream) {
+  if (!table || !ids || !x || !status || rows < 0 || width <= 0 || vocab <= 0) return B200_ERR_BAD_ARGUMENT;
+  if (dtype != B200_F32 && dtype != B200_BF16) return B200_ERR_UNSUPPORTED;
+  if (rows == 0) return B200_OK;
+  if (rows > INT32_MAX || width > INT32_MAX) return B200_ERR_TOO_LARGE;
+  if (!aligned16(table) || !aligned16(x)) return B200_ERR_ALIGNMENT;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (dtype == B200_F32)
+    embedding_residual_kernel<float><<<static_cast<unsigned>(rows), 256, 0, s>>>(
+        static_cast<const float*>(table), ids, x, static_cast<int>(width), vocab, status);
+  else
+    embedding_residual_kernel<__nv_bfloat16><<<static_cast<unsigned>(rows), 256, 0, s>>>(
+        static_cast<const __nv_bfloat16*>(table), ids, x, static_cast<int>(width), vocab, status);
+  return launch_status();
 }
 
 extern "C" int b200_sequence_positions(const int64_t* lengths, const int32_t* slots, int32_t* positions,

@@ -62,9 +62,7 @@ class HybridEngine(ServingEngine):
                     streams: Optional[list] = None) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
         """Residual stream behind the last layer, and its rows normed with `last_norm`."""
 
-        x = kernels.b200_embedding(self.embed, ids)
-        if x.dtype != torch.float32:
-            x = kernels.b200_contiguous(x, torch.float32)
+        x = hk.embedding_residual(self.embed, ids)
         h = self._norm_step(x, None, None, self.layers[0].norm_in)
         for index, layer in enumerate(self.layers):
             after = self.layers[index + 1].norm_in if index + 1 < len(self.layers) else last_norm

@@ -84,6 +84,23 @@ def _require_rows(tensor: torch.Tensor, what: str) -> None:
         raise ValueError(f"{what} must be a matrix with contiguous rows")
 
 
+def embedding_residual(table: torch.Tensor, ids: torch.Tensor) -> torch.Tensor:
+    """Rows of `table` gathered by int64 ids and widened to fp32: the start of the residual stream."""
+
+    device = _require_cuda(table, ids)
+    if table.ndim != 2 or not table.is_contiguous() or ids.dtype != torch.int64 or ids.ndim != 1 or \
+            not ids.is_contiguous():
+        raise ValueError("embedding needs a contiguous V x H table and a vector of int64 ids")
+    x = torch.empty((ids.shape[0], table.shape[1]), dtype=torch.float32, device=device)
+    rt = runtime(device)
+    code = _lib.load().b200_embedding_residual(table.data_ptr(), ids.data_ptr(), x.data_ptr(), ids.shape[0],
+                                               table.shape[1], table.shape[0], _code(table.dtype),
+                                               rt.status.data_ptr(), _stream())
+    _check(code, "b200_embedding_residual")
+    _count(rt)
+    return x
+
+
 def residual_norm(x: torch.Tensor, y: Optional[torch.Tensor], post_weight: Optional[torch.Tensor],
                   next_weight: Optional[torch.Tensor], *, epsilon: float, weight_offset: float,
                   dtype: torch.dtype) -> Optional[torch.Tensor]:

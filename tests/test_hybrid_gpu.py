@@ -6,15 +6,23 @@ fp32 runs are compared tightly; bf16 runs (16-bit projections, fp32 recurrences,
 a few rounding errors of the same bf16 weights in double precision.
 """
 
+import io
+import json
+
+import numpy as np
 import pytest
 import torch
 
 from llm_compiler_b200 import bazirax, kernels
 from llm_compiler_b200 import hybrid_kernels as hk
+from llm_compiler_b200.cli import main
 from llm_compiler_b200.hybrid_engine import HybridEngine
 from llm_compiler_b200.kv_state import ExecutionError
 from llm_compiler_b200.mixers import ChannelDelta, LatentAttention, Retention
+from llm_compiler_b200.registry import load_model
+from llm_compiler_b200.safetensors_io import save_safetensors
 from llm_compiler_b200.scheduler import RequestScheduler
+from llm_compiler_b200.trace import replay
 from oracle import hybrid_model as oracle
 
 pytestmark = pytest.mark.gpu
@@ -107,6 +115,19 @@ def test_residual_norm(dtype, width):
                             dtype=dtype) is None
     want = x.double() + oracle.rms_norm(parts.double().sum(0), post.double(), EPS)
     assert float((residual.double().cpu() - want).abs().max()) < 1e-5
+
+
+@BOTH
+@pytest.mark.parametrize("width", [36, 50])
+def test_embedding_residual(dtype, width):
+    table = torch.randn(11, width, generator=torch.Generator().manual_seed(0)).to(dtype).cuda()
+    ids = torch.tensor([3, 0, 10, 3], device="cuda")
+    assert torch.equal(hk.embedding_residual(table, ids), table.float()[ids])
+    kernels.runtime().check_status()
+    x = hk.embedding_residual(table, torch.tensor([11, 2], device="cuda"))
+    with pytest.raises(kernels.KernelStatusError, match="token id"):
+        kernels.runtime().check_status()
+    assert torch.all(x[0] == 0) and torch.equal(x[1], table.float()[2])
 
 
 # -------------------------------------------------------------------------- retention ----
@@ -613,3 +634,49 @@ def test_idle_rows_leave_no_trace():
         for name, tensor in layer.items():
             assert torch.equal(tensor[slots[3]], saved[name])
     assert engine.state.lengths.tolist() == [6, 7, 8, 8]
+
+
+# ---------------------------------------------------------------- files and command line ----
+def stored_model(folder, config, seed=0):
+    weights = bazirax.make_weights(config, seed=seed, dtype=torch.bfloat16, gate_rank=12)
+    (folder / "config.json").write_text(json.dumps(config.to_dict()))
+    save_safetensors(weights, folder / "model.safetensors")
+    return weights
+
+
+@BOTH
+def test_trace_replay(dtype, tmp_path):
+    """A stored model loaded through the registry and driven step by step: portions, a step without wanted
+    places, a second sequence in the slot of the first."""
+    config = small_config(1)
+    weights = stored_model(tmp_path, config)
+    first, second = tokens_of(config, 60, 1), tokens_of(config, 25, 2)
+    steps = [{"step": 0, "entries": [{"id": "a", "tokens": first[:50], "want": [0, 49]}], "end": []},
+             {"step": 1, "entries": [{"id": "a", "tokens": first[50:58], "want": []}], "end": []},
+             {"step": 2, "entries": [{"id": "a", "tokens": first[58:], "want": [1, 0]}], "end": ["a"]},
+             {"step": 3, "entries": [{"id": "b", "tokens": second, "want": [24]}], "end": ["b"]}]
+    output = io.StringIO()
+    engine = load_model(tmp_path, dtype=dtype, batch=1, capacity=64)
+    replay(engine, [json.dumps(step) for step in steps], tmp_path, output)
+    assert output.getvalue().split("\n")[:-1] == [f"done {n}" for n in range(4)]
+    assert not (tmp_path / "1.f32").exists() and engine.state.slots_in_use() == 0
+    a, b = (oracle.forward(config.to_dict(), weights, t) for t in (first, second))
+    for step, want in ((0, a[[0, 49]]), (2, a[[59, 58]]), (3, b[[24]])):
+        got = np.fromfile(tmp_path / f"{step}.f32", dtype="<f4").reshape(len(want), config.vocab_size)
+        close(torch.from_numpy(got), want, dtype, MODEL_TOLERANCE[dtype])
+
+
+def test_command_line_generates_from_a_stored_model(tmp_path, capsys):
+    config = small_config(1)
+    stored_model(tmp_path, config, seed=3)
+    prompts = [tokens_of(config, n, n) for n in (5, 30, 11)]
+    arguments = [x for p in prompts for x in ("--prompt", ",".join(map(str, p)))]
+    assert main(["generate", "--model", str(tmp_path), "--new-tokens", "4", "--max-batch", "2", "--max-portion", "8",
+                 *arguments]) == 0
+    lines = [json.loads(line) for line in capsys.readouterr().out.strip().splitlines()]
+    assert [line["prompt"] for line in lines] == prompts
+    engine, _ = model(config, torch.bfloat16, batch=2, capacity=34, seed=3)
+    scheduler = RequestScheduler(engine, max_portion=8)
+    requests = [scheduler.submit(p, 4) for p in prompts]
+    scheduler.run()
+    assert [line["output"] for line in lines] == [r.output for r in requests]
