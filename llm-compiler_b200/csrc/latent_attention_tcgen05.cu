@@ -67,7 +67,7 @@ latent_attention_tcgen05_kernel(const LatentTcParams p, const __grid_constant__ 
   __shared__ uint32_t tmem_slot;
   __shared__ int failed;
   grid_launch_dependents();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int warp = __shfl_sync(0xffffffffu, threadIdx.x >> 5, 0), lane = threadIdx.x & 31;
   const int split = blockIdx.x, sequence = blockIdx.z, row0 = blockIdx.y * N;
   const uint32_t columns = (p.pairs + 2) * 2 * N <= 256 ? 256u : 512u;
   if (threadIdx.x == 0) {
@@ -153,16 +153,17 @@ latent_attention_tcgen05_kernel(const LatentTcParams p, const __grid_constant__ 
     mbarrier_wait_bounded(smem_u32(&q_full), 0, p.wait_limit);
     for (int i = max(0, index - p.ring); i < index; ++i)
       mbarrier_wait_bounded(smem_u32(&pair_full[i % p.ring]), (i / p.ring) & 1, p.wait_limit);
-  } else if (warp == kMmaWarp && lane == 0) {
-    // ---- MMA issuer ----
+  } else if (warp == kMmaWarp) {
+    // ---- MMA issuer: the whole warp walks the loops (the descriptors stay in uniform registers), one lane issues ----
+    const uint32_t leader = lane == 0 ? 1u : 0u;
     constexpr uint32_t idesc_s = instruction_descriptor(128, N);
     constexpr uint32_t idesc_o = instruction_descriptor(128, 2 * N, false, true);
     const uint64_t q_desc = smem_descriptor(q_smem), p_desc = smem_descriptor(p_smem);
-    bool ok = mbarrier_wait_bounded(smem_u32(&q_full), 0, p.wait_limit);
+    bool ok = __all_sync(0xffffffffu, mbarrier_wait_bounded(smem_u32(&q_full), 0, p.wait_limit));
     int index = 0;  // pairs taken so far (refetch)
     auto next_pair = [&](int j, int m) { return p.refetch ? index++ : j * p.pairs + m; };
     auto landed = [&](int pair) {
-      ok = mbarrier_wait_bounded(smem_u32(&pair_full[pair % p.ring]), (pair / p.ring) & 1, p.wait_limit);
+      ok = __all_sync(0xffffffffu, mbarrier_wait_bounded(smem_u32(&pair_full[pair % p.ring]), (pair / p.ring) & 1, p.wait_limit));
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       return ok;
     };
@@ -173,17 +174,17 @@ latent_attention_tcgen05_kernel(const LatentTcParams p, const __grid_constant__ 
         const uint64_t c_desc = smem_descriptor(ring_smem + pair % p.ring * kPairBytes);
 #pragma unroll
         for (int ks = 0; ks < 8; ++ks)
-          umma_bf16(tmem + ((j & 1) * 2 + (ks & 1)) * N, descriptor_advance(c_desc, (ks / 4) * kPanelBytes + (ks % 4) * 32),
+          umma_bf16_if(leader, tmem + ((j & 1) * 2 + (ks & 1)) * N, descriptor_advance(c_desc, (ks / 4) * kPanelBytes + (ks % 4) * 32),
                     descriptor_advance(q_desc, (2 * m + ks / 4) * kQPanel + (ks % 4) * 32), idesc_s,
                     m > 0 || ks > 1 ? 1u : 0u);
-        if (p.refetch) umma_commit(smem_u32(&pair_empty[pair % p.ring]));
+        if (p.refetch) umma_commit_if(leader, smem_u32(&pair_empty[pair % p.ring]));
       }
-      umma_commit(smem_u32(&s_full[j & 1]));
+      umma_commit_if(leader, smem_u32(&s_full[j & 1]));
     };
     if (ok) issue_scores(0);
     for (int j = 0; ok && j < tiles; ++j) {
       if (j + 1 < tiles) issue_scores(j + 1);  // (its buffer's scores, of tile j - 1, were read before p_full of j - 1)
-      ok = ok && mbarrier_wait_bounded(smem_u32(&p_full), j & 1, p.wait_limit);
+      ok = ok && __all_sync(0xffffffffu, mbarrier_wait_bounded(smem_u32(&p_full), j & 1, p.wait_limit));
       if (!ok) break;
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       // Products with one accumulator follow one another at the latency of a product: two blocks of O^T
@@ -197,15 +198,15 @@ latent_attention_tcgen05_kernel(const LatentTcParams p, const __grid_constant__ 
 #pragma unroll
         for (int ks = 0; ks < 8; ++ks) {  // 16 keys a step
           const uint32_t at = (ks / 4) * kPPanel + (ks % 4) * 32, accumulate = j > 0 || ks > 0 ? 1u : 0u;
-          umma_bf16(o_column + m * 2 * N, descriptor_advance(c0, ks * 2048), descriptor_advance(p_desc, at), idesc_o, accumulate);
+          umma_bf16_if(leader, o_column + m * 2 * N, descriptor_advance(c0, ks * 2048), descriptor_advance(p_desc, at), idesc_o, accumulate);
           if (two)
-            umma_bf16(o_column + (m + 1) * 2 * N, descriptor_advance(c1, ks * 2048), descriptor_advance(p_desc, at), idesc_o,
+            umma_bf16_if(leader, o_column + (m + 1) * 2 * N, descriptor_advance(c1, ks * 2048), descriptor_advance(p_desc, at), idesc_o,
                       accumulate);
         }
-        umma_commit(smem_u32(&pair_empty[pair0 % p.ring]));
-        if (two) umma_commit(smem_u32(&pair_empty[pair1 % p.ring]));
+        umma_commit_if(leader, smem_u32(&pair_empty[pair0 % p.ring]));
+        if (two) umma_commit_if(leader, smem_u32(&pair_empty[pair1 % p.ring]));
       }
-      if (ok) umma_commit(smem_u32(&o_done));
+      if (ok) umma_commit_if(leader, smem_u32(&o_done));
     }
     if (!ok) failed = 1;
   } else if (warp < kSoftmaxWarps) {

@@ -49,6 +49,24 @@ __device__ __forceinline__ void umma_commit(uint32_t bar) {
                ::"r"(bar) : "memory");
 }
 
+// The same for a warp that walks its loops as a whole: only the lane that passes a leader other than 0 issues
+// (always the same one: a commit covers its own thread's products).
+__device__ __forceinline__ void umma_bf16_if(uint32_t leader, uint32_t tmem_d, uint64_t a_desc, uint64_t b_desc,
+                                             uint32_t idesc, uint32_t accumulate) {
+  asm volatile(
+      "{\n\t.reg .pred p, q;\n\t"
+      "setp.ne.b32 p, %4, 0;\n\t"
+      "setp.ne.b32 q, %6, 0;\n\t"
+      "@q tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, {%5, %5, %5, %5}, p;\n\t}"
+      ::"r"(tmem_d), "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(accumulate), "r"(0u), "r"(leader)
+      : "memory");
+}
+__device__ __forceinline__ void umma_commit_if(uint32_t leader, uint32_t bar) {
+  asm volatile("{\n\t.reg .pred q;\n\tsetp.ne.b32 q, %1, 0;\n\t"
+               "@q tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];\n\t}"
+               ::"r"(bar), "r"(leader) : "memory");
+}
+
 __device__ __forceinline__ void tmem_load_32x32(uint32_t taddr, float (&v)[32]) {
   uint32_t r[32];
   asm volatile(
