@@ -504,7 +504,7 @@ int b200_argmax(const void* logits, int64_t* ids, int64_t rows, int64_t vocab,
 typedef struct b200_delta_inputs {
   const void* input;  /* [rows, row_stride]: projections of h; *_column: where an operand starts */
   const void* gates;  /* [rows, gate_row_stride]: decay projections from decay_column on */
-  const void* q_conv; /* [kv_heads * dim, taps], last column: the current token */
+  const void* q_conv; /* [kv_heads * dim, taps] in time order: the newest input meets the last tap */
   const void* k_conv;
   const void* v_conv; /* [heads * vdim, taps] */
   const void* a_log;  /* [heads] */

@@ -14,7 +14,7 @@ import torch
 from .mixers import ChannelDelta, GatedMlp, LatentAttention, Mixer, Retention
 
 ARCHITECTURE = "Bazirax"
-NORM_OFFSET = 1.0  # the residual norms' weights are stored around zero
+NORM_OFFSET = 1.0  # the residual norms scale by 1 + their weight
 
 
 class ConfigError(ValueError):

@@ -1,6 +1,6 @@
 // Linear recurrences with a matrix state per head, S [dim, vdim] in fp32:
-//   retention      S <- decay_h S + k v^T;                                     o = S^T q
-//   channel delta  S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T;       o = S^T q
+//   retention      S' = gamma_h S + k v^T,                                      read-out S'^T q
+//   channel delta  P = diag(g) S, S' = P + k (beta (v - P^T k))^T,             read-out S'^T q
 // The columns of S are independent of each other, so a CTA owns a slice of them and walks the tokens.
 //
 // This file: the operand preparation (rotation, short convolution, unit norm, decays) and the token by

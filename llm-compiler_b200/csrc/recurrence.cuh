@@ -20,7 +20,7 @@ struct DeltaInputs {
   static constexpr bool kDelta = true;
   const void* input;   // T [rows, row_stride]: the projections of h
   const void* gates;   // T [rows, gate_row_stride]: decay columns [heads * dim] from decay_column
-  const void *q_conv, *k_conv, *v_conv;  // T [channels, taps], last column: the current token
+  const void *q_conv, *k_conv, *v_conv;  // T [channels, taps] in time order
   const void* a_log;   // T [heads]
   const void* dt_bias; // T [heads * dim]
   void* ring;          // T [slots, taps, 2 kv_heads dim + heads vdim]: inputs by position % taps

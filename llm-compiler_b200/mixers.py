@@ -89,7 +89,7 @@ class Mixer:
 
 
 class Retention(Mixer):
-    """q, k, v and a silu gate; S <- decay_h S + k v^T, o = S^T q, read-out normed per head."""
+    """q, k, v and a silu gate; S' = gamma_h S + k v^T, read-out S'^T q normed per head."""
 
     def __init__(self, weights: Dict[str, torch.Tensor], *, width: int, heads: int, dim: int, vdim: int,
                  decay: Sequence[float], rot_dims: int, rot_base: float, epsilon: float) -> None:
@@ -166,7 +166,7 @@ class ChannelDelta(Mixer):
 
 
 class LatentAttention(Mixer):
-    """Attention without positions over one cached latent per token; `kv_from` reads the latents that
+    """Attention over one cached latent per token (no rotation); `kv_from` reads the latents that
     an earlier layer keeps."""
 
     def __init__(self, weights: Dict[str, torch.Tensor], *, width: int, heads: int, dim: int, vdim: int,

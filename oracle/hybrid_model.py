@@ -68,7 +68,7 @@ def unit(x: Tensor, eps: float = 1e-6) -> Tensor:
 
 
 def retention_scan(q: Tensor, k: Tensor, v: Tensor, decay: List[float]) -> Tensor:
-    """S <- decay_h S + k v^T; o = S^T q. q, k [T, H, D], v [T, H, V] -> [T, H, V]."""
+    """S' = gamma_h S + k v^T, read-out S'^T q. q, k [T, H, D], v [T, H, V] -> [T, H, V]."""
     tokens, heads, dim = q.shape
     out = torch.zeros(tokens, heads, v.shape[2], dtype=q.dtype)
     for h in range(heads):
@@ -80,7 +80,7 @@ def retention_scan(q: Tensor, k: Tensor, v: Tensor, decay: List[float]) -> Tenso
 
 
 def delta_scan(q: Tensor, k: Tensor, v: Tensor, g: Tensor, beta: Tensor) -> Tensor:
-    """S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q.
+    """P = diag(g) S, S' = P + k (beta (v - P^T k))^T, read-out S'^T q.
     q, k, g [T, H, D], v [T, H, V], beta [T, H] -> [T, H, V]."""
     tokens, heads, dim = q.shape
     out = torch.zeros(tokens, heads, v.shape[2], dtype=q.dtype)
