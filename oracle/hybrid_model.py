@@ -203,3 +203,101 @@ def greedy(config: dict, weights: Dict[str, Tensor], prompt: List[int], steps: i
     for _ in range(steps):
         tokens.append(int(forward(config, weights, tokens)[-1].argmax()))
     return tokens[len(prompt):]
+
+
+# ------------------------------------------------------------- mechanisms of Lozanex ----
+def chunk_attention(q: Tensor, k: Tensor, v: Tensor, scale: float, chunk: Optional[int]) -> Tensor:
+    """Causal softmax attention with grouped heads (H query heads on G key heads); with `chunk` a row sees
+    only the keys of its own chunk of `chunk` positions. q [T, H, D], k [T, G, D], v [T, G, V]."""
+    tokens, heads, _ = q.shape
+    group = heads // k.shape[1]
+    out = torch.zeros(tokens, heads, v.shape[2], dtype=q.dtype)
+    for h in range(heads):
+        keys, values = k[:, h // group], v[:, h // group]
+        for i in range(tokens):
+            first = 0 if chunk is None else i // chunk * chunk
+            scores = (keys[first:i + 1] @ q[i, h]) * scale
+            weights = torch.exp(scores - scores.max())
+            out[i, h] = (weights / weights.sum()) @ values[first:i + 1]
+    return out
+
+
+def attention_keys(w: Dict[str, Tensor], spec: dict, h: Tensor, eps: float):
+    """Keys (normed over the whole projection, then rotated) and values of every token."""
+    tokens, groups = h.shape[0], spec["kv_heads"]
+    k = rms_norm(h @ w["k"].T + w["k.b"], w["k.norm"], eps).view(tokens, groups, spec["dim"])
+    rot = spec.get("rot")
+    if rot is not None:
+        k = rotate_half(k, rot["base"], rot["dims"])
+    return k, (h @ w["v"].T + w["v.b"]).view(tokens, groups, spec["vdim"])
+
+
+def attention(w: Dict[str, Tensor], spec: dict, h: Tensor, keys: Tensor, values: Tensor, eps: float) -> Tensor:
+    tokens, heads = h.shape[0], spec["heads"]
+    q = rms_norm(h @ w["q"].T + w["q.b"], w["q.norm"], eps).view(tokens, heads, spec["dim"])
+    rot, mask = spec.get("rot"), spec.get("mask")
+    if rot is not None:
+        q = rotate_half(q, rot["base"], rot["dims"])
+    o = chunk_attention(q, keys, values, spec["scale"], None if mask is None else mask["size"])
+    return o.reshape(tokens, heads * spec["vdim"]) @ w["o"].T + w["o.b"]
+
+
+def head_delta(w: Dict[str, Tensor], spec: dict, h: Tensor, eps: float) -> Tensor:
+    """The gated delta rule with one decay per head and a silu gate on the normed read-out."""
+    tokens = h.shape[0]
+    heads, kv_heads, dim, vdim = spec["heads"], spec["kv_heads"], spec["dim"], spec["vdim"]
+    q = silu(causal_conv(h @ w["q"].T, w["q.conv"])).view(tokens, kv_heads, dim)
+    k = silu(causal_conv(h @ w["k"].T, w["k.conv"])).view(tokens, kv_heads, dim)
+    v = silu(causal_conv(h @ w["v"].T, w["v.conv"])).view(tokens, heads, vdim)
+    shared = heads // kv_heads
+    q = (unit(q) * dim ** -0.5).repeat_interleave(shared, dim=1)
+    k = unit(k).repeat_interleave(shared, dim=1)
+    beta = sigmoid(h @ w["b"].T)
+    g = torch.exp(-torch.exp(w["A_log"]) * softplus(h @ w["a"].T + w["dt_bias"]))
+    o = rms_norm(delta_scan(q, k, v, g[:, :, None].expand(tokens, heads, dim), beta), w["norm"], eps)
+    gate = silu(h @ w["g"].T).view(tokens, heads, vdim)
+    return (o * gate).reshape(tokens, heads * vdim) @ w["o"].T
+
+
+def route(router: Tensor, h: Tensor, top: int):
+    """The `top` experts of every token with the largest sigmoid scores, and the scores themselves."""
+    scores = sigmoid(h @ router.T)
+    return torch.topk(scores, top, dim=-1)
+
+
+def expert_mlp(w: Dict[str, Tensor], spec: dict, h: Tensor) -> Tensor:
+    """Every token's chosen experts run on the token scaled by the expert's score; their results are added
+    to the shared expert's."""
+    scores, chosen = route(w["router"], h, spec["router"]["top"])
+    out = torch.zeros_like(h)
+    for t in range(h.shape[0]):
+        for score, expert in zip(scores[t], chosen[t].tolist()):
+            out[t] += dense_mlp(_under(w, f"e{expert}."), (score * h[t])[None])[0]
+    return out if spec.get("shared") is None else out + dense_mlp(_under(w, "shared."), h)
+
+
+def lozanex_forward(config: dict, weights: Dict[str, Tensor], tokens: List[int], *,
+                    streams: Optional[list] = None, dtype: torch.dtype = torch.float64) -> Tensor:
+    """Logits [T, vocab] of one sequence from the start; `streams` receives the residual stream
+    after every layer."""
+    w = {name: value.to(dtype) for name, value in weights.items()}
+    eps = config["norm"]["eps"]
+    x = rms_norm(w["embed"][torch.tensor(tokens, dtype=torch.int64)], w["embed.norm"], eps)
+    cached: Dict[int, tuple] = {}
+    for i, layer in enumerate(config["layers"]):
+        p, spec = f"l{i}.", layer["mixer"]
+        mix = _under(w, p + "mix.")
+        if layer["type"] == "delta":
+            y = head_delta(mix, spec, x, eps)
+        elif layer["type"] == "attention":
+            source = spec.get("kv_from")
+            cached[i] = attention_keys(mix, spec, x, eps) if source is None else cached[source]
+            y = attention(mix, spec, x, *cached[i], eps)
+        else:
+            raise ValueError(f"unknown mixer {layer['type']!r}")
+        x = x + rms_norm(y, w[p + "norm1"], eps)
+        if layer.get("mlp") is not None:
+            x = x + rms_norm(expert_mlp(_under(w, p + "mlp."), layer["mlp"], x), w[p + "norm2"], eps)
+        if streams is not None:
+            streams.append(x)
+    return rms_norm(x, w["final.norm"], eps) @ w["head"].T
