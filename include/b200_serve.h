@@ -291,11 +291,12 @@ int b200_prefill_attention(const void* query, const void* key, const void* value
 /* The causal form on tcgen05 for a portion of a sequence: `tokens` query rows behind `context` earlier
  * positions, keys and values [B, Hkv, context + tokens, D]; row t sees positions 0 .. context + t. With
  * sink (bf16 [Hq], NULL for none) the softmax denominator of head h also holds exp(sink[h]): no key, no
- * value. bf16, head_dim 64 / 128, scale > 0, strides a tensor map can describe; else
+ * value. With chunk > 0 a position sees only the earlier positions of its own chunk of `chunk` keys (chunks
+ * counted from key 0). bf16, head_dim 64 / 128, scale > 0, strides a tensor map can describe; else
  * B200_ERR_UNSUPPORTED. output memory is B x T x Hq x D. No counterpart in the reference. */
 int b200_context_attention(const void* query, const void* key, const void* value, const void* sink,
                            void* output, int64_t batch, int64_t q_heads, int64_t kv_heads, int64_t tokens,
-                           int64_t context, int64_t head_dim, const int64_t query_strides[4],
+                           int64_t context, int64_t chunk, int64_t head_dim, const int64_t query_strides[4],
                            const int64_t key_strides[4], const int64_t value_strides[4], double scale,
                            int32_t* status, void* stream);
 
@@ -331,7 +332,8 @@ int b200_linear(const void* input, const void* weight, const void* bias, const v
  * input (fixed slice order: deterministic). These entry points stand for the op sequences of
  * one decoder layer of the reference graph (qwen2.py:152-304 after the passes):
  *   b200_linear_partial            serve.linear without its epilogue: partials[s, m, n] (fp32),
- *                                  s < b200_linear_partial_splits(m, k, n); with row_squares
+ *                                  s < b200_linear_partial_splits(m, k, n), M <= 128 (any M with
+ *                                  splits 1: an fp32 result); with row_squares
  *                                  (fp32 [splits, m], M <= 128; may be NULL) also the sum of
  *                                  squares of every input row over each K slice, for a consumer
  *                                  that applies an RMSNorm folded into this projection
@@ -453,8 +455,10 @@ int b200_argmax(const void* logits, int64_t* ids, int64_t rows, int64_t vocab,
 
 /* ---- Hybrid layers -------------------------------------------------------------------
  * Operators of decoder layers whose mixers are recurrences with a matrix state (retention, the
- * gated delta rule with a decay per key channel) or attention over cached latents, with an RMS norm
- * before and after every sublayer and an fp32 residual stream. No counterpart in the reference.
+ * gated delta rule with a decay per key channel or per head), attention over cached latents or over
+ * cached keys and values (of a whole sequence or of chunks of it), and whose feed-forward may be a
+ * mixture of experts, on an fp32 residual stream with an RMS norm behind every sublayer and, in some
+ * designs, one in front of it. No counterpart in the reference.
  *
  * The rows of a step are the tokens of `sequences` sequences side by side: sequence s owns rows
  * starts[s] .. starts[s + 1] - 1 (int32 [sequences + 1]), its first row stands at position bases[s]
@@ -463,11 +467,14 @@ int b200_argmax(const void* logits, int64_t* ids, int64_t rows, int64_t vocab,
  * starts from an empty state whatever the slot held before. dtype is B200_F32 or B200_BF16 (weights,
  * projections, cached latents); state, decays, gates, norms and the residual are fp32.
  *
- *   b200_embedding_residual  x[r, :] = table[ids[r], :] widened to fp32
+ *   b200_embedding_residual  x[r, :] = table[ids[r], :] widened to fp32; with weight, norm(row) *
+ *                        (weight_offset + weight); with h the same rows in the model dtype too
  *   b200_residual_norm   x += norm(y) * (weight_offset + post_weight); h = norm(x) * (weight_offset +
- *                        next_weight). x fp32 [rows, width]; y of the model dtype, or fp32 split-K
- *                        partials [splits, rows, y_row_stride] when splits > 0; y NULL: h only;
- *                        next_weight NULL: no h. Columns of h from width to h_row_stride are zeroed.
+ *                        next_weight), or h = x with next_weight NULL. x fp32 [rows, width]; y of the
+ *                        model dtype, or fp32 split-K partials [splits, rows, y_row_stride] when splits >
+ *                        0, y_bias [width] or NULL is added to it; with top > 0 the rows places[row, 0 .. top - 1] (int32) of summands are added
+ *                        to y (y may then be NULL); y NULL and top 0: h only; h NULL: none. Columns of h
+ *                        from width to h_row_stride are zeroed.
  *   b200_latent_norm     RMS norms (plain weights) of the query latent (columns 0 .. q_rank - 1 of
  *                        input) and the kv latent (from kv_column); the latter goes to the cache row of
  *                        the token's position, and to dense [rows, cache_row] when given. kv_weight
@@ -480,7 +487,8 @@ int b200_argmax(const void* logits, int64_t* ids, int64_t rows, int64_t vocab,
  *                        silu), beta and log g as fp32 operands
  *   b200_conv_tail       keeps the last `taps` inputs of every sequence for the next portion
  *   b200_recurrence_scan token by token recurrence on prepared operands. beta NULL: retention, decay
- *                        is [heads]; otherwise the delta rule, decay is log g [rows, heads, dim]. State
+ *                        is [heads]; otherwise the delta rule, decay is log g [rows, heads, decay_dim],
+ *                        decay_dim being dim or 1 (one decay for all channels of a head). State
  *                        [slots, heads, dim, state_row] is read, and written behind the last token.
  *   b200_recurrence_chunked  the same results in chunks of 64 tokens on the tensor cores (operands split
  *                        into two bf16 numbers each); chunk_starts (int32 [sequences + 1]): the first chunk
@@ -497,18 +505,38 @@ int b200_argmax(const void* logits, int64_t* ids, int64_t rows, int64_t vocab,
  *                        most rows of one sequence; context: an upper bound of the keys (they choose the
  *                        row tile and the split count; every sequence's keys are then shared out among the
  *                        splits on the device)
+ *   b200_attention_prep  what stands between the projections of attention and the scores: bias (of
+ *                        partial sums; q and k and v columns of one stacked projection), RMS norms over
+ *                        the whole q and the whole k, rotation of the first rot_dims dimensions of every
+ *                        head (pair (i, i + rot_dims / 2), turns[i] turns per position), then q to
+ *                        q_out [rows, heads, row_size] and k, v to the slots' caches [slots, capacity,
+ *                        kv_heads, row_size] at the tokens' positions, zeros behind dim / vdim. keys NULL:
+ *                        q only
+ *   b200_slot_decode_attention  one token per sequence (row r at position bases[r] of slot slots[r])
+ *                        over the caches, bf16, row_size 64 or 128; chunk > 0: only the keys of the
+ *                        position's own chunk of `chunk` positions. context: upper bound of the keys
+ *   b200_slot_attention  the same for any rows, sizes and dtype, on the CUDA cores
+ *   b200_expert_route    the top experts of every row from router logits (fp32, split-K partials
+ *                        [splits, rows, logit_stride]): expert ids and sigmoid scores [rows, top], and
+ *                        each choice's number among its expert's; counts [experts] must be zero before
+ *   b200_expert_place    choices to rows of an expert-sorted matrix whose experts start at multiples of
+ *                        tile rows: places [rows, top], sorted (rows of h, copied), scores [sorted rows],
+ *                        tiles [max_tiles, 2]: a tile's expert (-1: none) and how many rows it holds
+ *   b200_grouped_linear  out[r, :] = w[expert of r's tile] x[r, :] over the sorted rows; with SwiGLU (rows
+ *                        of w: gate_j, up_j alternating) silu(s_r g) (s_r u), s the scores (NULL: 1).
+ *                        clear: int32 [clear_count] set to zero (the counts of b200_expert_route)
  *   b200_sequence_positions  positions[r] = lengths[slots[r]] (0 for an idle row)
  *   b200_advance_slots   lengths[slots[r]] += starts[r + 1] - starts[r], clamped with a status bit */
 #define B200_GATE_SILU 0
 #define B200_GATE_SIGMOID 1
 typedef struct b200_delta_inputs {
   const void* input;  /* [rows, row_stride]: projections of h; *_column: where an operand starts */
-  const void* gates;  /* [rows, gate_row_stride]: decay projections from decay_column on */
+  const void* gates;  /* [rows, gate_row_stride]: decay projections [heads * decay_dim] from decay_column on */
   const void* q_conv; /* [kv_heads * dim, taps] in time order: the newest input meets the last tap */
   const void* k_conv;
   const void* v_conv; /* [heads * vdim, taps] */
   const void* a_log;  /* [heads] */
-  const void* dt_bias; /* [heads * dim] */
+  const void* dt_bias; /* [heads * decay_dim] */
   void* ring;         /* [slots, taps, 2 kv_heads dim + heads vdim]: inputs by position % taps */
   const int32_t* token_sequence;
   const int32_t* starts;
@@ -517,6 +545,7 @@ typedef struct b200_delta_inputs {
   int64_t heads, kv_heads, dim, vdim, taps;
   int64_t q_column, k_column, v_column, beta_column, decay_column;
   int64_t row_stride, gate_row_stride;
+  int64_t decay_dim;  /* dim: a decay per key channel; 1: one per head */
   double q_scale;
 } b200_delta_inputs;
 typedef struct b200_retention_inputs {
@@ -538,11 +567,52 @@ typedef struct b200_step_output {
   int64_t gate_kind;
   double epsilon;
 } b200_step_output;
-int b200_embedding_residual(const void* table, const int64_t* ids, float* x, int64_t rows, int64_t width,
-                            int64_t vocab, int dtype, int32_t* status, void* stream);
-int b200_residual_norm(void* x, const void* y, const void* post_weight, const void* next_weight, void* h,
-                       int64_t rows, int64_t width, int64_t splits, int64_t y_row_stride,
-                       int64_t h_row_stride, double epsilon, double weight_offset, int dtype, void* stream);
+typedef struct b200_attention_prep_inputs {
+  const void* input;    /* [rows, row_stride], or fp32 partials [splits, rows, row_stride] */
+  const void* bias;     /* [row_stride] added to the partials; NULL: none */
+  const void* q_weight; /* [heads * dim] */
+  const void* k_weight; /* [kv_heads * dim] */
+  const double* turns;  /* [rot_dims / 2] */
+  void* q_out;
+  void* keys;
+  void* values;
+  const int32_t* token_sequence;
+  const int32_t* starts;
+  const int32_t* slots;
+  const int32_t* bases;
+  int64_t rows, heads, kv_heads, dim, vdim, row_size, rot_dims;
+  int64_t q_column, k_column, v_column, row_stride, splits, capacity;
+  double epsilon;
+} b200_attention_prep_inputs;
+int b200_embedding_residual(const void* table, const void* weight, const int64_t* ids, float* x, void* h,
+                            int64_t rows, int64_t width, int64_t vocab, int64_t h_row_stride, double epsilon,
+                            double weight_offset, int dtype, int32_t* status, void* stream);
+int b200_residual_norm(void* x, const void* y, const void* y_bias, const void* post_weight,
+                       const void* next_weight, void* h, const void* summands, const int32_t* places, int64_t rows, int64_t width, int64_t splits,
+                       int64_t top, int64_t y_row_stride, int64_t h_row_stride, int64_t summand_row_stride,
+                       double epsilon, double weight_offset, int dtype, void* stream);
+int b200_attention_prep(const b200_attention_prep_inputs* inputs, int dtype, int32_t* status, void* stream);
+int64_t b200_slot_decode_attention_workspace_bytes(int64_t rows, int64_t heads, int64_t kv_heads,
+                                                   int64_t row_size, int64_t context);
+int b200_slot_decode_attention(const void* q, const void* keys, const void* values, void* out,
+                               const int32_t* slots, const int32_t* bases, int64_t rows, int64_t heads,
+                               int64_t kv_heads, int64_t row_size, int64_t slot_count, int64_t capacity,
+                               int64_t chunk, int64_t context, double scale, void* workspace,
+                               int64_t workspace_bytes, int32_t* status, void* stream);
+int b200_slot_attention(const void* q, const void* keys, const void* values, void* out,
+                        const int32_t* token_sequence, const int32_t* starts, const int32_t* slots,
+                        const int32_t* bases, int64_t rows, int64_t heads, int64_t kv_heads, int64_t row_size,
+                        int64_t capacity, int64_t chunk, double scale, int dtype, void* stream);
+int b200_expert_route(const float* logits, int32_t* chosen, float* scores, int32_t* numbers, int32_t* counts,
+                      int64_t rows, int64_t experts, int64_t top, int64_t splits, int64_t logit_stride,
+                      void* stream);
+int b200_expert_place(const void* h, const int32_t* chosen, const float* scores, const int32_t* numbers,
+                      const int32_t* counts, int32_t* places, void* sorted, float* sorted_scores, int32_t* tiles,
+                      int64_t rows, int64_t experts, int64_t top, int64_t tile, int64_t max_tiles, int64_t columns,
+                      int64_t h_row_stride, int dtype, void* stream);
+int b200_grouped_linear(const void* x, const void* w, const int32_t* tiles, const float* scores, void* out,
+                        int32_t* clear, int64_t clear_count, int64_t experts, int64_t tile, int64_t max_tiles,
+                        int64_t k, int64_t n, int epilogue, int dtype, int32_t* status, void* stream);
 int b200_latent_norm(const void* input, const void* q_weight, const void* kv_weight, void* q_out,
                      void* cache, void* dense, const int32_t* token_sequence, const int32_t* starts,
                      const int32_t* slots, const int32_t* bases, int64_t rows, int64_t q_rank,
@@ -564,15 +634,16 @@ int b200_conv_tail(const b200_delta_inputs* inputs, int64_t sequences, int dtype
 int b200_recurrence_scan(const float* q, const float* k, const float* v, const float* beta, const float* decay,
                          float* state, float* output, const int32_t* token_sequence, const int32_t* starts,
                          const int32_t* slots, const int32_t* bases, int64_t sequences, int64_t heads,
-                         int64_t kv_heads, int64_t dim, int64_t vdim, int64_t state_row, void* stream);
+                         int64_t kv_heads, int64_t dim, int64_t vdim, int64_t state_row, int64_t decay_dim,
+                         void* stream);
 int64_t b200_recurrence_chunked_workspace_bytes(int64_t chunks, int64_t heads, int64_t dim, int64_t vdim,
                                                 int delta);
 int b200_recurrence_chunked(const float* q, const float* k, const float* v, const float* beta,
                             const float* decay, float* state, float* output, const int32_t* token_sequence,
                             const int32_t* starts, const int32_t* slots, const int32_t* bases,
                             const int32_t* chunk_starts, int64_t chunks, int64_t sequences, int64_t heads,
-                            int64_t kv_heads, int64_t dim, int64_t vdim, int64_t state_row, void* workspace,
-                            int64_t workspace_bytes, void* stream);
+                            int64_t kv_heads, int64_t dim, int64_t vdim, int64_t state_row, int64_t decay_dim,
+                            void* workspace, int64_t workspace_bytes, void* stream);
 int b200_head_linear(const void* x, const void* w, void* y, int64_t m, int64_t heads, int64_t k, int64_t n,
                      int64_t x_row_stride, int64_t x_head_stride, int64_t y_row_stride,
                      int64_t y_head_stride, int dtype, void* stream);

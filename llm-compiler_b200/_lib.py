@@ -52,7 +52,7 @@ class DeltaInputs(ctypes.Structure):
                  "token_sequence", "starts", "slots", "bases")] + \
                [(name, c_int64) for name in
                 ("heads", "kv_heads", "dim", "vdim", "taps", "q_column", "k_column", "v_column",
-                 "beta_column", "decay_column", "row_stride", "gate_row_stride")] + \
+                 "beta_column", "decay_column", "row_stride", "gate_row_stride", "decay_dim")] + \
                [("q_scale", c_double)]
 
 
@@ -64,6 +64,18 @@ class RetentionInputs(ctypes.Structure):
                [(name, c_int64) for name in
                 ("heads", "dim", "vdim", "q_column", "k_column", "v_column", "row_stride", "rot_dims")] + \
                [("rot_base", c_double), ("k_scale", c_double)]
+
+
+class AttentionPrepInputs(ctypes.Structure):
+    """b200_attention_prep_inputs of include/b200_serve.h."""
+
+    _fields_ = [(name, c_void_p) for name in
+                ("input", "bias", "q_weight", "k_weight", "turns", "q_out", "keys", "values",
+                 "token_sequence", "starts", "slots", "bases")] + \
+               [(name, c_int64) for name in
+                ("rows", "heads", "kv_heads", "dim", "vdim", "row_size", "rot_dims",
+                 "q_column", "k_column", "v_column", "row_stride", "splits", "capacity")] + \
+               [("epsilon", c_double)]
 
 
 class StepOutput(ctypes.Structure):
@@ -78,7 +90,7 @@ class StepOutput(ctypes.Structure):
 _DELTA, _RETENTION, _STEP = POINTER(DeltaInputs), POINTER(RetentionInputs), POINTER(StepOutput)
 
 # What b200_abi_version() of a matching library returns (bumped with every signature change).
-ABI_VERSION = 105
+ABI_VERSION = 106
 
 # name -> (restype, argtypes); mirrors include/b200_serve.h one to one
 SIGNATURES = {
@@ -150,8 +162,16 @@ SIGNATURES = {
     "b200_advance_lengths": (c_int, [c_void_p, c_int64, c_int64, c_int64, c_int64, c_void_p,
                                      c_void_p]),
     "b200_argmax": (c_int, [c_void_p, c_void_p, c_int64, c_int64, c_int64, c_int, c_void_p]),
-    "b200_embedding_residual": (c_int, [c_void_p] * 3 + [c_int64] * 3 + [c_int, c_void_p, c_void_p]),
-    "b200_residual_norm": (c_int, [c_void_p] * 5 + [c_int64] * 5 + [c_double, c_double, c_int, c_void_p]),
+    "b200_embedding_residual": (c_int, [c_void_p] * 5 + [c_int64] * 4 + [c_double, c_double, c_int, c_void_p, c_void_p]),
+    "b200_residual_norm": (c_int, [c_void_p] * 8 + [c_int64] * 7 + [c_double, c_double, c_int, c_void_p]),
+    "b200_attention_prep": (c_int, [POINTER(AttentionPrepInputs), c_int, c_void_p, c_void_p]),
+    "b200_slot_decode_attention_workspace_bytes": (c_int64, [c_int64] * 5),
+    "b200_slot_decode_attention": (c_int, [c_void_p] * 6 + [c_int64] * 8 + [c_double, c_void_p, c_int64, c_void_p,
+                                                                          c_void_p]),
+    "b200_slot_attention": (c_int, [c_void_p] * 8 + [c_int64] * 6 + [c_double, c_int, c_void_p]),
+    "b200_expert_route": (c_int, [c_void_p] * 5 + [c_int64] * 5 + [c_void_p]),
+    "b200_expert_place": (c_int, [c_void_p] * 9 + [c_int64] * 7 + [c_int, c_void_p]),
+    "b200_grouped_linear": (c_int, [c_void_p] * 6 + [c_int64] * 6 + [c_int, c_int, c_void_p, c_void_p]),
     "b200_latent_norm": (c_int, [c_void_p] * 10 + [c_int64] * 8 + [c_double, c_int, c_void_p, c_void_p]),
     "b200_gated_head_norm": (c_int, [c_void_p] * 4 + [c_int64] * 5 + [c_int, c_double, c_int, c_void_p]),
     "b200_retention_prep": (c_int, [_RETENTION] + [c_void_p] * 3 + [c_int64, c_int, c_void_p]),
@@ -159,10 +179,10 @@ SIGNATURES = {
     "b200_delta_step": (c_int, [_DELTA, _STEP, c_int64, c_int, c_void_p]),
     "b200_delta_prep": (c_int, [_DELTA] + [c_void_p] * 5 + [c_int64] * 3 + [c_int, c_void_p]),
     "b200_conv_tail": (c_int, [_DELTA, c_int64, c_int, c_void_p]),
-    "b200_recurrence_scan": (c_int, [c_void_p] * 11 + [c_int64] * 6 + [c_void_p]),
+    "b200_recurrence_scan": (c_int, [c_void_p] * 11 + [c_int64] * 7 + [c_void_p]),
     "b200_recurrence_chunked_workspace_bytes": (c_int64, [c_int64] * 4 + [c_int]),
-    "b200_recurrence_chunked": (c_int, [c_void_p] * 12 + [c_int64] * 7 + [c_void_p, c_int64, c_void_p]),
-    "b200_context_attention": (c_int, [c_void_p] * 5 + [c_int64] * 6 + [_I64P] * 3 +
+    "b200_recurrence_chunked": (c_int, [c_void_p] * 12 + [c_int64] * 8 + [c_void_p, c_int64, c_void_p]),
+    "b200_context_attention": (c_int, [c_void_p] * 5 + [c_int64] * 7 + [_I64P] * 3 +
                                [c_double, c_void_p, c_void_p]),
     "b200_head_linear": (c_int, [c_void_p] * 3 + [c_int64] * 8 + [c_int, c_void_p]),
     "b200_latent_attention_workspace_bytes": (c_int64, [c_int64] * 6 + [c_int]),

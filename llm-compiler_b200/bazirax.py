@@ -11,14 +11,10 @@ from typing import Dict, Iterator, List, Optional, Tuple
 
 import torch
 
-from .mixers import ChannelDelta, GatedMlp, LatentAttention, Mixer, Retention
+from .hybrid_config import ConfigError
+from .mixers import ChannelDelta, GatedMlp, HybridLayer, LatentAttention, Mixer, Retention
 
 ARCHITECTURE = "Bazirax"
-NORM_OFFSET = 1.0  # the residual norms scale by 1 + their weight
-
-
-class ConfigError(ValueError):
-    """config.json asks for something the design does not have, or contradicts itself."""
 
 
 @dataclass(frozen=True)
@@ -34,6 +30,11 @@ class BaziraxConfig:
     hidden_size: int
     norm_eps: float
     layers: Tuple[LayerSpec, ...]
+
+    norm_offset = 1.0  # the residual norms scale by 1 + their weight
+
+    def build_layers(self, weights: Dict[str, torch.Tensor]) -> List[HybridLayer]:
+        return build_layers(self, weights)
 
     @property
     def num_layers(self) -> int:
@@ -161,18 +162,6 @@ def check_weights(config: BaziraxConfig, weights: Dict[str, torch.Tensor]) -> No
             shape = (shape[0], ranks[low])
         if tuple(weights[name].shape) != shape:
             raise ConfigError(f"tensor {name} has shape {tuple(weights[name].shape)}, expected {shape}")
-
-
-@dataclass
-class HybridLayer:
-    """What HybridEngine runs: a mixer between its two norms, and a feed-forward between its own."""
-
-    mixer: Mixer
-    norm_in: torch.Tensor
-    norm_out: torch.Tensor
-    mlp: Optional[GatedMlp] = None
-    mlp_norm_in: Optional[torch.Tensor] = None
-    mlp_norm_out: Optional[torch.Tensor] = None
 
 
 def build_layers(config: BaziraxConfig, weights: Dict[str, torch.Tensor]) -> List[HybridLayer]:

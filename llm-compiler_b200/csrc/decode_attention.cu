@@ -85,6 +85,12 @@ struct DecodeParams {
   // longest-first scheduling when the grid is several waves of CTAs.
   const int32_t* order = nullptr;
   int block_size = 0, table_stride = 0;
+  // Slot form (slots != nullptr): kbuf / vbuf are [slots, capacity, Hkv, D], row b of the batch stands at
+  // position bases[b] of slot slots[b] (-1: an idle row, its output is zero) and sees the positions up to
+  // its own, with chunk > 0 those of its own chunk of `chunk` positions only. lengths is not read.
+  const int32_t* slots = nullptr;
+  const int32_t* bases = nullptr;
+  int chunk = 0, slot_count = 0;
   int64_t pool_rows = 0;  // blocks x block_size: the extent of the pools' tensor maps
   uint32_t wait_limit = 4000000u;  // polls of a bounded wait
   int drop_loads = 0;              // debug: no KV copy is issued (every wait runs out)
@@ -135,7 +141,7 @@ __device__ __forceinline__ bool stream_segment(const DecodeParams& p, const CUte
                                                int stable_end = -1, TraceScope* trace = nullptr,
                                                const __nv_bfloat16* qbase = nullptr,
                                                int64_t q_row_stride = 0,
-                                               Prepare prepare = Prepare()) {
+                                               Prepare prepare = Prepare(), int64_t slot_row = -1) {
   constexpr int kChunksPerRow = D / 8;
   constexpr int kTileBytes = TOK * D * 2;  // one of K or V, one stage
   constexpr int kStageBytes = 2 * kTileBytes;
@@ -155,6 +161,7 @@ __device__ __forceinline__ bool stream_segment(const DecodeParams& p, const CUte
   const __nv_bfloat16* vglob = p.vbuf + (static_cast<int64_t>(b) * p.capacity * p.kv_heads + kvh) * D;
   // first buffer row of the TOK tokens that start at token t0 of this sequence
   auto first_row = [&](int t0) -> int64_t {
+    if (slot_row >= 0) return slot_row + t0;
     if (p.block_table == nullptr) return static_cast<int64_t>(b) * p.capacity + t0;
     const int block = __ldg(p.block_table + static_cast<int64_t>(b) * p.table_stride + t0 / p.block_size);
     return static_cast<int64_t>(block) * p.block_size + t0 % p.block_size;
@@ -512,7 +519,17 @@ decode_attention_kernel(const DecodeParams p, const __grid_constant__ CUtensorMa
     grid_dependency_wait();  // lengths, q and the newest KV row come from kernels before this one
     trace.mark(0);
   }
-  int64_t len = p.lengths[b] + p.length_bias;
+  int64_t len = 0, slot_row = -1;  // slot_row: the buffer row of the first key this row sees
+  if (p.slots != nullptr) {
+    const int slot = p.slots[b], position = p.bases[b];
+    if (slot >= 0) {
+      const int first = p.chunk > 0 ? position / p.chunk * p.chunk : 0;
+      slot_row = static_cast<int64_t>(slot) * p.capacity + first;
+      len = min(position, p.capacity - 1) - first + 1;
+    }
+  } else {
+    len = p.lengths[b] + p.length_bias;
+  }
   if (len > p.mask_len) {
     if (threadIdx.x == 0 && split == 0 && head_block == 0 && p.status != nullptr)
       atomicOr(p.status, B200_STATUS_LENGTH_OVER_MASK);
@@ -623,7 +640,8 @@ decode_attention_kernel(const DecodeParams p, const __grid_constant__ CUtensorMa
         static_cast<int64_t>(D), prepare_fused);
   else
     stream_segment<D, TOK, WIDE, FAST, TMA, NoPrepare, WARPS>(
-        p, kmap, vmap, smem, bar0, b, kvh, g0, rows, start, end, it_base, stable_end, &trace);
+        p, kmap, vmap, smem, bar0, b, kvh, g0, rows, start, end, it_base, stable_end, &trace, nullptr, 0,
+        NoPrepare(), slot_row);
   trace.mark_middle();
   if (owner) {
     // the newest token as one more partial: max = its score (log2 domain), sum = 1, O = its V row
@@ -661,6 +679,7 @@ decode_attention_kernel(const DecodeParams p, const __grid_constant__ CUtensorMa
       o_all += new_v[col] * wgt;
     }
     const int hq = kvh * p.groups + g0 + row;
+    if (p.slots != nullptr && n_tokens == 0) l_all = 1.0f;  // an idle row: zeros
     if (p.num_splits == 1) {
       p.out[(static_cast<int64_t>(b) * p.q_heads + hq) * D + col] =
           __float2bfloat16_rn(o_all / l_all);  // 0/0 = NaN for an empty sequence, as the oracle
@@ -701,6 +720,7 @@ decode_attention_kernel(const DecodeParams p, const __grid_constant__ CUtensorMa
           l_all += load_cluster_f32(staging + (16 * D + row * 2 + 1) * 4, s) * wgt;
           o_all += load_cluster_f32(staging + idx * 4, s) * wgt;
         }
+        if (p.slots != nullptr && n_tokens == 0) l_all = 1.0f;
         const int hq = kvh * p.groups + g0 + row;
         p.out[(static_cast<int64_t>(b) * p.q_heads + hq) * D + col] =
             __float2bfloat16_rn(o_all / l_all);
@@ -755,6 +775,7 @@ decode_attention_kernel(const DecodeParams p, const __grid_constant__ CUtensorMa
       l_all += __ldcg(p.ws_ml + (base + s) * 2 + 1) * wgt;
       o_all += __ldcg(p.ws_o + (base + s) * D + col) * wgt;
     }
+    if (p.slots != nullptr && n_tokens == 0) l_all = 1.0f;
     p.out[(static_cast<int64_t>(b) * p.q_heads + hq) * D + col] = __float2bfloat16_rn(o_all / l_all);
   }
 }
@@ -1214,8 +1235,8 @@ int launch_bf16(const DecodeParams& p, cudaStream_t stream, int flat_grid = 0) {
     tma = p.block_table != nullptr
               ? make_kv_tensor_map(&kmap, p.kbuf, 1, p.pool_rows, p.kv_heads, D, box_tokens) &&
                     make_kv_tensor_map(&vmap, p.vbuf, 1, p.pool_rows, p.kv_heads, D, box_tokens)
-              : make_kv_tensor_map(&kmap, p.kbuf, p.batch, p.capacity, p.kv_heads, D, box_tokens) &&
-                    make_kv_tensor_map(&vmap, p.vbuf, p.batch, p.capacity, p.kv_heads, D, box_tokens);
+              : make_kv_tensor_map(&kmap, p.kbuf, p.slots != nullptr ? p.slot_count : p.batch, p.capacity, p.kv_heads, D, box_tokens) &&
+                    make_kv_tensor_map(&vmap, p.vbuf, p.slots != nullptr ? p.slot_count : p.batch, p.capacity, p.kv_heads, D, box_tokens);
   int code;
   if (p.qkv_partials != nullptr) {
     // the fused form (q|k|v reduction, RoPE and KV store in front of the streaming) is its own
@@ -1505,6 +1526,77 @@ extern "C" int b200_decode_attention_ordered(
                                mask_batch_stride, mask_dtype, scale, dtype, mode, split_tokens,
                                max_length_hint, workspace, workspace_bytes, status, stream,
                                sequence_order);
+}
+
+// ---- Slot layout ---------------------------------------------------------------------------
+// The same kernel over the caches of sequences that come and go: every row of a step has its slot and
+// position, and sees its whole sequence or its own chunk of it. `context`: upper bound of the keys seen.
+extern "C" int64_t b200_slot_decode_attention_workspace_bytes(int64_t rows, int64_t heads, int64_t kv_heads,
+                                                              int64_t row_size, int64_t context) {
+  if (rows <= 0 || heads <= 0 || kv_heads <= 0 || row_size <= 0 || context <= 0) return 0;
+  const int64_t split_tokens = round_up(default_split_tokens(rows, kv_heads * ceil_div(heads / kv_heads, 16), context), 32);
+  const int64_t splits = ceil_div(context, split_tokens);
+  return splits <= 1 ? 0 : workspace_bytes_for(rows, heads, row_size, splits);
+}
+
+extern "C" int b200_slot_decode_attention(const void* q, const void* keys, const void* values, void* out,
+                                          const int32_t* slots, const int32_t* bases, int64_t rows, int64_t heads,
+                                          int64_t kv_heads, int64_t row_size, int64_t slot_count, int64_t capacity,
+                                          int64_t chunk, int64_t context, double scale, void* workspace,
+                                          int64_t workspace_bytes, int32_t* status, void* stream) {
+  if (!q || !keys || !values || !out || !slots || !bases || !status || rows < 0 || heads <= 0 || kv_heads <= 0 ||
+      heads % kv_heads != 0 || slot_count <= 0 || capacity <= 0 || chunk < 0 || context <= 0)
+    return B200_ERR_BAD_ARGUMENT;
+  if ((row_size != 64 && row_size != 128) || !(scale > 0.0)) return B200_ERR_UNSUPPORTED;
+  if (rows == 0) return B200_OK;
+  if (rows > 65535 || capacity > INT32_MAX / 2 || slot_count * capacity > INT32_MAX) return B200_ERR_TOO_LARGE;
+  if (!aligned16(keys) || !aligned16(values) || !aligned16(q)) return B200_ERR_ALIGNMENT;
+  const int64_t head_blocks = kv_heads * ceil_div(heads / kv_heads, 16);
+  const int64_t split_tokens = round_up(default_split_tokens(rows, head_blocks, context), 32);
+  const int64_t splits = ceil_div(context, split_tokens);
+  if (splits > 65535 || split_tokens > INT32_MAX) return B200_ERR_TOO_LARGE;
+  DecodeParams p;
+  p.q = static_cast<const __nv_bfloat16*>(q);
+  p.kbuf = static_cast<const __nv_bfloat16*>(keys);
+  p.vbuf = static_cast<const __nv_bfloat16*>(values);
+  p.lengths = nullptr;
+  p.mask = nullptr;
+  p.out = static_cast<__nv_bfloat16*>(out);
+  p.status = status;
+  p.q_batch_stride = heads * row_size;
+  p.q_head_stride = row_size;
+  p.mask_batch_stride = 0;
+  p.batch = static_cast<int>(rows);
+  p.q_heads = static_cast<int>(heads);
+  p.kv_heads = static_cast<int>(kv_heads);
+  p.groups = static_cast<int>(heads / kv_heads);
+  p.capacity = static_cast<int>(capacity);
+  p.mask_len = static_cast<int>(context);
+  p.split_tokens = static_cast<int>(split_tokens);
+  p.num_splits = static_cast<int>(splits);
+  p.mask_dtype = B200_F32;
+  p.compat = 0;
+  p.early_kv = (launch_mode() & B200_LAUNCH_STABLE_KV_PREFIX) != 0 ? 1 : 0;
+  p.scale = static_cast<float>(scale);
+  p.ws_o = nullptr;
+  p.ws_ml = nullptr;
+  p.counters = nullptr;
+  p.slots = slots;
+  p.bases = bases;
+  p.chunk = static_cast<int>(chunk < capacity ? chunk : 0);
+  p.slot_count = static_cast<int>(slot_count);
+  p.wait_limit = wait_limit();
+  p.drop_loads = drop_loads();
+  const GridPlan plan = plan_grid(splits, split_tokens, rows, head_blocks);
+  if (plan.splits > 1 && !plan.cluster) {
+    if (!workspace || workspace_bytes < workspace_bytes_for(rows, heads, row_size, splits)) return B200_ERR_WORKSPACE;
+    if (rows * head_blocks > kMaxCounters) return B200_ERR_TOO_LARGE;
+    p.counters = static_cast<int*>(workspace);
+    p.ws_o = reinterpret_cast<float*>(static_cast<char*>(workspace) + kCounterBytes);
+    p.ws_ml = p.ws_o + rows * heads * splits * row_size;
+  }
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  return row_size == 64 ? launch_bf16<64>(p, s) : launch_bf16<128>(p, s);
 }
 
 // ---- Paged KV layout ---------------------------------------------------------------------

@@ -1,8 +1,8 @@
-// Normalisation steps of the hybrid layers (recurrent mixers and latent attention beside each
-// other, every sublayer normed before and after), all arithmetic in fp32:
-//   residual_norm   x += norm_post(y); h = norm_next(x): the step between two sublayers in one
-//                   launch. x is the fp32 residual stream; y the sublayer's result, in the model
-//                   dtype or as fp32 split-K partial sums.
+// Normalisation steps of the hybrid layers (recurrent mixers and attention beside each other, a norm
+// behind every sublayer, in some designs one in front of it as well), all arithmetic in fp32:
+//   residual_norm   x += norm_post(y); h = norm_next(x), or x itself: the step between two sublayers
+//                   in one launch. x is the fp32 residual stream; y the sublayer's result, in the model
+//                   dtype or as fp32 split-K partial sums, plus the rows that a token's experts left.
 //   latent_norm     the two RMS norms behind the down projections of latent attention; the
 //                   latent of every token goes straight into its cache row.
 //   gated_head_norm per-head RMS norm of a recurrence's read-out, times a weight and a gate.
@@ -28,12 +28,19 @@ struct ResidualNormParams {
   float* x;             // [rows, width]: read, and written when there is a y
   const void* y;        // T [rows, y_row_stride], or fp32 partials [splits, rows, y_row_stride]; may be NULL
   const void* w_post;   // T [width]
-  const void* w_next;   // T [width]; NULL: no h
-  void* h;              // T [rows, h_row_stride]; columns from width on are zeroed
+  const void* w_next;   // T [width]; NULL: h is x itself, without a norm
+  void* h;              // T [rows, h_row_stride]; columns from width on are zeroed; NULL: no h
   int splits;           // 0: y has dtype T
   int rows, width;
   int64_t y_row_stride, h_row_stride;
   float eps, weight_offset;
+  // y also takes the sum of rows places[row, 0 .. top - 1] of this matrix (top 0: none)
+  const void* summands; // T [any, summand_row_stride]
+  const int32_t* places;
+  int top;
+  int64_t summand_row_stride;
+  const void* y_bias;   // T [width] added to every y, or NULL
+  __device__ __forceinline__ bool adds() const { return y != nullptr || top > 0; }
 };
 
 // One CTA per row; a row's fp32 values stay in shared memory between the two norms.
@@ -46,22 +53,18 @@ __global__ void __launch_bounds__(256) residual_norm_kernel(const ResidualNormPa
   const int64_t row = blockIdx.x;
   float* x = p.x + row * p.width;
   float sum = 0.0f;
-  if (p.y != nullptr) {
-    if (p.splits > 0) {
-      const float* y = static_cast<const float*>(p.y) + row * p.y_row_stride;
-      const int64_t slice = static_cast<int64_t>(p.rows) * p.y_row_stride;
-      for (int c = threadIdx.x; c < p.width; c += blockDim.x) {
-        const float v = sum_slices(y + c, slice, p.splits);
-        row_values[c] = v;
-        sum += v * v;
-      }
-    } else {
-      const T* y = static_cast<const T*>(p.y) + row * p.y_row_stride;
-      for (int c = threadIdx.x; c < p.width; c += blockDim.x) {
-        const float v = Elem<T>::load(y + c);
-        row_values[c] = v;
-        sum += v * v;
-      }
+  if (p.adds()) {
+    const int64_t slice = static_cast<int64_t>(p.rows) * p.y_row_stride;
+    for (int c = threadIdx.x; c < p.width; c += blockDim.x) {
+      float v = 0.0f;
+      if (p.y != nullptr)
+        v = p.splits > 0 ? sum_slices(static_cast<const float*>(p.y) + row * p.y_row_stride + c, slice, p.splits)
+                         : Elem<T>::load(static_cast<const T*>(p.y) + row * p.y_row_stride + c);
+      if (p.y_bias != nullptr) v += Elem<T>::load(static_cast<const T*>(p.y_bias) + c);
+      for (int k = 0; k < p.top; ++k)
+        v += Elem<T>::load(static_cast<const T*>(p.summands) + p.places[row * p.top + k] * p.summand_row_stride + c);
+      row_values[c] = v;
+      sum += v * v;
     }
     const float factor = 1.0f / sqrtf(block_sum(sum, scratch) / p.width + p.eps);
     const T* w = static_cast<const T*>(p.w_post);
@@ -79,10 +82,14 @@ __global__ void __launch_bounds__(256) residual_norm_kernel(const ResidualNormPa
       sum += v * v;
     }
   }
-  if (p.w_next == nullptr) return;
-  const float factor = 1.0f / sqrtf(block_sum(sum, scratch) / p.width + p.eps);
-  const T* w = static_cast<const T*>(p.w_next);
+  if (p.h == nullptr) return;
   T* h = static_cast<T*>(p.h) + row * p.h_row_stride;
+  const T* w = static_cast<const T*>(p.w_next);
+  if (w == nullptr) {
+    for (int c = threadIdx.x; c < p.h_row_stride; c += blockDim.x) Elem<T>::store(h + c, c < p.width ? row_values[c] : 0.0f);
+    return;
+  }
+  const float factor = 1.0f / sqrtf(block_sum(sum, scratch) / p.width + p.eps);
   for (int c = threadIdx.x; c < p.h_row_stride; c += blockDim.x)
     Elem<T>::store(h + c, c < p.width ? row_values[c] * factor * (p.weight_offset + Elem<T>::load(w + c)) : 0.0f);
 }
@@ -120,14 +127,15 @@ __global__ void __launch_bounds__(Q == 1 ? 1024 : 512) residual_norm_quads_kerne
     const int c = threadIdx.x + i * blockDim.x;
     v[i] = c < quads ? *reinterpret_cast<const float4*>(x + c * 4) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
   }
-  if (p.y != nullptr) {
-    if (p.splits > 0) {
+  if (p.adds()) {
+#pragma unroll
+    for (int i = 0; i < Q; ++i) y[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    if (p.y != nullptr && p.splits > 0) {
       const float* partial = static_cast<const float*>(p.y) + row * p.y_row_stride;
       const int64_t slice = static_cast<int64_t>(p.rows) * p.y_row_stride;
 #pragma unroll
       for (int i = 0; i < Q; ++i) {
         const int c = threadIdx.x + i * blockDim.x;
-        y[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
         if (c >= quads) continue;
         for (int s0 = 0; s0 < p.splits; s0 += 4) {
           float4 t[4];
@@ -141,12 +149,32 @@ __global__ void __launch_bounds__(Q == 1 ? 1024 : 512) residual_norm_quads_kerne
           }
         }
       }
-    } else {
+    } else if (p.y != nullptr) {
       const T* in = static_cast<const T*>(p.y) + row * p.y_row_stride;
 #pragma unroll
       for (int i = 0; i < Q; ++i) {
         const int c = threadIdx.x + i * blockDim.x;
-        y[i] = c < quads ? load_quad<T>(in + c * 4) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (c < quads) y[i] = load_quad<T>(in + c * 4);
+      }
+    }
+    if (p.y_bias != nullptr) {
+#pragma unroll
+      for (int i = 0; i < Q; ++i) {
+        const int c = threadIdx.x + i * blockDim.x;
+        if (c >= quads) continue;
+        const float4 t = load_quad<T>(static_cast<const T*>(p.y_bias) + c * 4);
+        y[i].x += t.x; y[i].y += t.y; y[i].z += t.z; y[i].w += t.w;
+      }
+    }
+#pragma unroll 2
+    for (int k = 0; k < p.top; ++k) {
+      const T* in = static_cast<const T*>(p.summands) + p.places[row * p.top + k] * p.summand_row_stride;
+#pragma unroll
+      for (int i = 0; i < Q; ++i) {
+        const int c = threadIdx.x + i * blockDim.x;
+        if (c >= quads) continue;
+        const float4 t = load_quad<T>(in + c * 4);
+        y[i].x += t.x; y[i].y += t.y; y[i].z += t.z; y[i].w += t.w;
       }
     }
 #pragma unroll
@@ -164,12 +192,21 @@ __global__ void __launch_bounds__(Q == 1 ? 1024 : 512) residual_norm_quads_kerne
       *reinterpret_cast<float4*>(x + c * 4) = v[i];
     }
   }
-  if (p.w_next == nullptr) return;
+  if (p.h == nullptr) return;
+  T* h = static_cast<T*>(p.h) + row * p.h_row_stride;
+  if (static_cast<int>(threadIdx.x) < p.h_row_stride - p.width) Elem<T>::store(h + p.width + threadIdx.x, 0.0f);
+  if (p.w_next == nullptr) {
+#pragma unroll
+    for (int i = 0; i < Q; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      if (c < quads) store_quad<T>(h + c * 4, v[i]);
+    }
+    return;
+  }
   sum = 0.0f;
 #pragma unroll
   for (int i = 0; i < Q; ++i) sum += squares_of(v[i]);
   const float factor = 1.0f / sqrtf(block_sum(sum, scratch) / p.width + p.eps);
-  T* h = static_cast<T*>(p.h) + row * p.h_row_stride;
 #pragma unroll
   for (int i = 0; i < Q; ++i) {
     const int c = threadIdx.x + i * blockDim.x;
@@ -178,7 +215,6 @@ __global__ void __launch_bounds__(Q == 1 ? 1024 : 512) residual_norm_quads_kerne
     store_quad<T>(h + c * 4, make_float4(v[i].x * factor * (p.weight_offset + w.x), v[i].y * factor * (p.weight_offset + w.y),
                                          v[i].z * factor * (p.weight_offset + w.z), v[i].w * factor * (p.weight_offset + w.w)));
   }
-  if (static_cast<int>(threadIdx.x) < p.h_row_stride - p.width) Elem<T>::store(h + p.width + threadIdx.x, 0.0f);
 }
 
 struct LatentNormParams {
@@ -302,21 +338,58 @@ __global__ void __launch_bounds__(256) gated_head_norm_quads_kernel(const GatedH
                             v.z * factor * w.z * gate_value(gate.z, p.gate_kind), v.w * factor * w.w * gate_value(gate.w, p.gate_kind)));
 }
 
-// The residual stream's first rows: a row of the table per id, widened to fp32
+// The residual stream's first rows: a row of the table per id, widened to fp32; with `weight` normed (RMS,
+// times weight_offset + weight), and with `h` also in the model dtype.
+struct EmbeddingParams {
+  const void* table;  // T [vocab, width]
+  const void* weight; // T [width] or NULL
+  const int64_t* ids;
+  float* x;           // [rows, width]
+  void* h;            // T [rows, h_row_stride] or NULL, zeros from width on
+  int width;
+  int64_t vocab, h_row_stride;
+  float eps, weight_offset;
+  int32_t* status;
+};
 template <typename T>
-__global__ void __launch_bounds__(256) embedding_residual_kernel(const T* table, const int64_t* ids, float* x, int width,
-                                                                 int64_t vocab, int32_t* status) {
-  const int64_t row = blockIdx.x, id = ids[row];
-  const bool known = id >= 0 && id < vocab;
-  if (!known && threadIdx.x == 0) atomicOr(status, B200_STATUS_BAD_TOKEN_ID);
-  const T* source = table + (known ? id : 0) * width;
-  float* out = x + row * width;
-  if (width % 4 == 0) {
-    for (int c = threadIdx.x * 4; c < width; c += blockDim.x * 4)
-      *reinterpret_cast<float4*>(out + c) = known ? load_quad<T>(source + c) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-  } else {
-    for (int c = threadIdx.x; c < width; c += blockDim.x) out[c] = known ? Elem<T>::load(source + c) : 0.0f;
+__global__ void __launch_bounds__(256) embedding_residual_kernel(const EmbeddingParams p) {
+  __shared__ float scratch[32];
+  const int64_t row = blockIdx.x, id = p.ids[row];
+  const bool known = id >= 0 && id < p.vocab;
+  if (!known && threadIdx.x == 0) atomicOr(p.status, B200_STATUS_BAD_TOKEN_ID);
+  const T* source = static_cast<const T*>(p.table) + (known ? id : 0) * p.width;
+  const T* weight = static_cast<const T*>(p.weight);
+  float* out = p.x + row * p.width;
+  T* h = p.h != nullptr ? static_cast<T*>(p.h) + row * p.h_row_stride : nullptr;
+  float factor = 1.0f;
+  const bool quads = p.width % 4 == 0;
+  if (weight != nullptr) {
+    float sum = 0.0f;
+    if (quads) {
+      for (int c = threadIdx.x * 4; c < p.width; c += blockDim.x * 4) sum += squares_of(load_quad<T>(source + c));
+    } else {
+      for (int c = threadIdx.x; c < p.width; c += blockDim.x) sum += Elem<T>::load(source + c) * Elem<T>::load(source + c);
+    }
+    factor = 1.0f / sqrtf(block_sum(sum, scratch) / p.width + p.eps);
   }
+  if (!known) factor = 0.0f;
+  auto scale_at = [&](int c) { return weight != nullptr ? factor * (p.weight_offset + Elem<T>::load(weight + c)) : factor; };
+  if (quads) {
+    for (int c = threadIdx.x * 4; c < p.width; c += blockDim.x * 4) {
+      float4 v = load_quad<T>(source + c);
+      v = make_float4(v.x * scale_at(c), v.y * scale_at(c + 1), v.z * scale_at(c + 2), v.w * scale_at(c + 3));
+      *reinterpret_cast<float4*>(out + c) = v;
+      if (h != nullptr) store_quad<T>(h + c, v);
+    }
+  } else {
+    for (int c = threadIdx.x; c < p.width; c += blockDim.x) {
+      const float v = Elem<T>::load(source + c) * scale_at(c);
+      out[c] = v;
+      if (h != nullptr) Elem<T>::store(h + c, v);
+    }
+  }
+  if (h != nullptr)
+    for (int64_t c = p.width + threadIdx.x; c < p.h_row_stride; c += blockDim.x) Elem<T>::store(h + c, 0.0f);
 }
 
 // positions[r] and the row's slot: what a replayed step reads; lengths advance behind the step
@@ -340,23 +413,27 @@ __global__ void advance_slots_kernel(int64_t* lengths, const int32_t* slots, con
 
 using namespace b200;
 
-extern "C" int b200_residual_norm(void* x, const void* y, const void* post_weight, const void* next_weight,
-                                  void* h, int64_t rows, int64_t width, int64_t splits,
-                                  int64_t y_row_stride, int64_t h_row_stride, double epsilon,
-                                  double weight_offset, int dtype, void* stream) {
-  if (!x || rows < 0 || width <= 0 || splits < 0 || (y && (!post_weight || y_row_stride < width)) ||
-      (next_weight && (!h || h_row_stride < width)) || (!y && !next_weight))
+extern "C" int b200_residual_norm(void* x, const void* y, const void* y_bias, const void* post_weight,
+                                  const void* next_weight, void* h, const void* summands, const int32_t* places, int64_t rows, int64_t width,
+                                  int64_t splits, int64_t top, int64_t y_row_stride, int64_t h_row_stride,
+                                  int64_t summand_row_stride, double epsilon, double weight_offset, int dtype,
+                                  void* stream) {
+  const bool adds = y != nullptr || top > 0;
+  if (!x || rows < 0 || width <= 0 || splits < 0 || top < 0 || (adds && !post_weight) || (y && y_row_stride < width) ||
+      (top > 0 && (!summands || !places || summand_row_stride < width)) || (h && h_row_stride < width) ||
+      (next_weight && !h) || (!adds && !h))
     return B200_ERR_BAD_ARGUMENT;
   if (dtype != B200_F32 && dtype != B200_BF16) return B200_ERR_UNSUPPORTED;
   if (rows == 0) return B200_OK;
-  if (width > 48 * 1024 || rows > INT32_MAX || splits > INT32_MAX) return B200_ERR_TOO_LARGE;
+  if (width > 48 * 1024 || rows > INT32_MAX || splits > INT32_MAX || top > INT32_MAX) return B200_ERR_TOO_LARGE;
   ResidualNormParams p{static_cast<float*>(x), y, post_weight, next_weight, h, static_cast<int>(splits),
                        static_cast<int>(rows), static_cast<int>(width), y_row_stride, h_row_stride,
-                       static_cast<float>(epsilon), static_cast<float>(weight_offset)};
+                       static_cast<float>(epsilon), static_cast<float>(weight_offset), summands, places,
+                       static_cast<int>(top), summand_row_stride, y_bias};
   const int64_t quads = width / 4;
-  if (width % 4 == 0 && quads <= 2048 && y_row_stride % 4 == 0 && h_row_stride % 4 == 0 &&
+  if (width % 4 == 0 && quads <= 2048 && y_row_stride % 4 == 0 && h_row_stride % 4 == 0 && summand_row_stride % 4 == 0 &&
       h_row_stride - width < 32 && aligned16(x) && aligned16(y) && aligned16(h) && aligned16(post_weight) &&
-      aligned16(next_weight)) {
+      aligned16(next_weight) && aligned16(summands) && aligned16(y_bias)) {
     // few rows: a thread per four columns; many: rows of fewer, longer-working threads
     const int q = rows <= 2 * kNumSMs && quads <= 1024 ? 1 : quads <= 512 ? 2 : 4;
     const unsigned threads = static_cast<unsigned>(ceil_div(ceil_div(quads, q), 32) * 32);
@@ -437,20 +514,20 @@ extern "C" int b200_gated_head_norm(const void* input, const void* weight, const
   return code == cudaSuccess ? launch_status() : B200_ERR_LAUNCH;
 }
 
-extern "C" int b200_embedding_residual(const void* table, const int64_t* ids, float* x, int64_t rows, int64_t width,
-                                       int64_t vocab, int dtype, int32_t* status, void* stream) {
-  if (!table || !ids || !x || !status || rows < 0 || width <= 0 || vocab <= 0) return B200_ERR_BAD_ARGUMENT;
+extern "C" int b200_embedding_residual(const void* table, const void* weight, const int64_t* ids, float* x, void* h,
+                                       int64_t rows, int64_t width, int64_t vocab, int64_t h_row_stride,
+                                       double epsilon, double weight_offset, int dtype, int32_t* status, void* stream) {
+  if (!table || !ids || !x || !status || rows < 0 || width <= 0 || vocab <= 0 || (h && h_row_stride < width))
+    return B200_ERR_BAD_ARGUMENT;
   if (dtype != B200_F32 && dtype != B200_BF16) return B200_ERR_UNSUPPORTED;
   if (rows == 0) return B200_OK;
   if (rows > INT32_MAX || width > INT32_MAX) return B200_ERR_TOO_LARGE;
-  if (!aligned16(table) || !aligned16(x)) return B200_ERR_ALIGNMENT;
+  if (!aligned16(table) || !aligned16(x) || !aligned16(h) || h_row_stride % 4 != 0) return B200_ERR_ALIGNMENT;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (dtype == B200_F32)
-    embedding_residual_kernel<float><<<static_cast<unsigned>(rows), 256, 0, s>>>(
-        static_cast<const float*>(table), ids, x, static_cast<int>(width), vocab, status);
-  else
-    embedding_residual_kernel<__nv_bfloat16><<<static_cast<unsigned>(rows), 256, 0, s>>>(
-        static_cast<const __nv_bfloat16*>(table), ids, x, static_cast<int>(width), vocab, status);
+  EmbeddingParams p{table, weight, ids, x, h, static_cast<int>(width), vocab, h_row_stride, static_cast<float>(epsilon),
+                    static_cast<float>(weight_offset), status};
+  if (dtype == B200_F32) embedding_residual_kernel<float><<<static_cast<unsigned>(rows), 256, 0, s>>>(p);
+  else embedding_residual_kernel<__nv_bfloat16><<<static_cast<unsigned>(rows), 256, 0, s>>>(p);
   return launch_status();
 }
 

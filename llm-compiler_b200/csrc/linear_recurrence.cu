@@ -1,6 +1,7 @@
 // Linear recurrences with a matrix state per head, S [dim, vdim] in fp32:
 //   retention      S' = gamma_h S + k v^T,                                      read-out S'^T q
-//   channel delta  P = diag(g) S, S' = P + k (beta (v - P^T k))^T,             read-out S'^T q
+//   gated delta    P = diag(g) S, S' = P + k (beta (v - P^T k))^T,             read-out S'^T q
+//                  (g: a decay per key channel, or one for all channels of a head)
 // The columns of S are independent of each other, so a CTA owns a slice of them and walks the tokens.
 //
 // This file: the operand preparation (rotation, short convolution, unit norm, decays) and the token by
@@ -75,8 +76,8 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaInputs p, fl
     } else {
       const int head = unit - 2 * p.kv_heads - p.heads;
       if (lane == 0) beta[row * p.heads + head] = delta_beta<T>(p, row, head);
-      for (int c = lane; c < p.dim; c += 32)
-        log_decay[(row * p.heads + head) * p.dim + c] = delta_log_decay<T>(p, row, head, c);
+      for (int c = lane; c < p.decay_dim; c += 32)
+        log_decay[(row * p.heads + head) * p.decay_dim + c] = delta_log_decay<T>(p, row, head, c);
     }
   }
 }
@@ -114,11 +115,15 @@ __global__ void __launch_bounds__(256) delta_prep_tiled_kernel(const DeltaInputs
   const int c = lane * CPL;
   if (unit >= 2 * p.kv_heads + p.heads) {  // step size and decays
     const int head = unit - 2 * p.kv_heads - p.heads;
+    if (lane < count) beta[(row0 + lane) * p.heads + head] = delta_beta<__nv_bfloat16>(p, row0 + lane, head);
+    if (p.decay_dim == 1) {
+      if (lane < count) log_decay[(row0 + lane) * p.heads + head] = delta_log_decay<__nv_bfloat16>(p, row0 + lane, head, 0);
+      return;
+    }
     const __nv_bfloat16* in = static_cast<const __nv_bfloat16*>(p.gates) + p.decay_column + head * kDim + c;
     float bias[CPL];
     load_channels<CPL>(static_cast<const __nv_bfloat16*>(p.dt_bias) + head * kDim + c, bias);
     const float rate = -expf(__bfloat162float(static_cast<const __nv_bfloat16*>(p.a_log)[head]));
-    if (lane < count) beta[(row0 + lane) * p.heads + head] = delta_beta<__nv_bfloat16>(p, row0 + lane, head);
     for (int t0 = 0; t0 < count; t0 += kBatch) {
       float step[kBatch][CPL];
 #pragma unroll
@@ -216,11 +221,11 @@ constexpr int kScanThreads = 128, kScanColumns = 8, kScanTokens = 16;
 struct ScanParams {
   const float *q, *k, *v;     // [rows, kv_heads, dim] x 2, [rows, heads, vdim]
   const float* beta;          // [rows, heads]            (delta)
-  const float* log_decay;     // [rows, heads, dim] natural log (delta); [heads] decay itself (retention)
+  const float* log_decay;     // [rows, heads, decay_dim] natural log (delta); [heads] decay itself (retention)
   float* state;               // [slots, heads, dim, state_row]
   float* output;              // [rows, heads, vdim]
   SequenceBatch batch;
-  int heads, kv_heads, dim, vdim, state_row;
+  int heads, kv_heads, dim, vdim, state_row, decay_dim;
 };
 
 // 16 lanes share a column: lane g holds rows g, g + 16, ... A column's sums are four shuffles.
@@ -255,7 +260,7 @@ __global__ void __launch_bounds__(kScanThreads) recurrence_scan_kernel(const Sca
       const int64_t source = ((row0 + t) * p.kv_heads + kv_head) * p.dim + c;
       tile[t * stride + c] = p.k[source];
       tile[t * stride + p.dim + c] = p.q[source];
-      if (DELTA) tile[t * stride + 2 * p.dim + c] = expf(p.log_decay[((row0 + t) * p.heads + head) * p.dim + c]);
+      if (DELTA) tile[t * stride + 2 * p.dim + c] = expf(p.log_decay[((row0 + t) * p.heads + head) * p.decay_dim + (p.decay_dim == 1 ? 0 : c)]);
     }
     for (int item = threadIdx.x; item < count * (kScanColumns + 1); item += kScanThreads) {
       const int t = item / (kScanColumns + 1), c = item % (kScanColumns + 1);
@@ -363,8 +368,8 @@ extern "C" int b200_delta_prep(const b200_delta_inputs* inputs, float* q, float*
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (dtype == B200_BF16 && (p.dim == 64 || p.dim == 128) && p.vdim == p.dim && p.taps <= 4 && longest >= 16 &&
       p.row_stride % 8 == 0 && p.gate_row_stride % 8 == 0 && p.q_column % 8 == 0 && p.k_column % 8 == 0 &&
-      p.v_column % 8 == 0 && p.decay_column % 8 == 0 && aligned16(p.input) && aligned16(p.gates) && aligned16(p.ring) &&
-      aligned16(p.dt_bias) && sequences <= 65535) {
+      p.v_column % 8 == 0 && (p.decay_dim == 1 || (p.decay_column % 8 == 0 && aligned16(p.gates) && aligned16(p.dt_bias))) &&
+      aligned16(p.input) && aligned16(p.ring) && sequences <= 65535) {
     const dim3 grid(static_cast<unsigned>(ceil_div(longest, 32)), static_cast<unsigned>(ceil_div(2 * p.kv_heads + 2 * p.heads, 8)),
                     static_cast<unsigned>(sequences));
     if (p.dim == 64) delta_prep_tiled_kernel<2><<<grid, 256, 0, s>>>(p, q, k, v, beta, log_decay);
@@ -394,15 +399,16 @@ extern "C" int b200_recurrence_scan(const float* q, const float* k, const float*
                                     const float* decay, float* state, float* output,
                                     const int32_t* token_sequence, const int32_t* starts, const int32_t* slots,
                                     const int32_t* bases, int64_t sequences, int64_t heads, int64_t kv_heads,
-                                    int64_t dim, int64_t vdim, int64_t state_row, void* stream) {
+                                    int64_t dim, int64_t vdim, int64_t state_row, int64_t decay_dim, void* stream) {
   if (!q || !k || !v || !decay || !state || !output || !starts || !slots || !bases || sequences < 0 ||
-      heads <= 0 || kv_heads <= 0 || heads % kv_heads != 0 || dim <= 0 || vdim <= 0 || state_row < vdim)
+      heads <= 0 || kv_heads <= 0 || heads % kv_heads != 0 || dim <= 0 || vdim <= 0 || state_row < vdim ||
+      (decay_dim != 1 && decay_dim != dim))
     return B200_ERR_BAD_ARGUMENT;
   if (sequences == 0) return B200_OK;
   if (sequences > 65535 || heads > 65535) return B200_ERR_TOO_LARGE;
   ScanParams p{q, k, v, beta, decay, state, output, {token_sequence, starts, slots, bases},
                static_cast<int>(heads), static_cast<int>(kv_heads), static_cast<int>(dim),
-               static_cast<int>(vdim), static_cast<int>(state_row)};
+               static_cast<int>(vdim), static_cast<int>(state_row), static_cast<int>(decay_dim)};
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   return beta != nullptr ? dispatch_scan<true>(p, sequences, s) : dispatch_scan<false>(p, sequences, s);
 }

@@ -1328,7 +1328,8 @@ extern "C" int b200_linear_partial(const void* input, const void* weight, void* 
   if (!input || !weight || !partials || m <= 0 || k <= 0 || n <= 0 || input_row_stride < k ||
       splits <= 0)
     return B200_ERR_BAD_ARGUMENT;
-  if (m > 128 || splits > ceil_div(k, kBK) || splits > 65535) return B200_ERR_TOO_LARGE;
+  if ((m > 128 && splits != 1) || ceil_div(m, kBM) > 65535 || splits > ceil_div(k, kBK) || splits > 65535)
+    return B200_ERR_TOO_LARGE;
   if (k % 8 != 0 || input_row_stride % 8 != 0 || n % 4 != 0) return B200_ERR_UNSUPPORTED;
   if (!aligned16(input) || !aligned16(weight) || !aligned16(partials)) return B200_ERR_ALIGNMENT;
   if (row_squares != nullptr && m > 128) return B200_ERR_TOO_LARGE;

@@ -335,7 +335,7 @@ int prefill_attention_tcgen05(const void* query, const void* key, const void* va
                               const int64_t key_strides[4], const int64_t value_strides[4],
                               double scale, int32_t* status, cudaStream_t stream, const void* mask,
                               const int64_t* mask_strides, void* workspace, int64_t workspace_bytes,
-                              int64_t context, const void* sink);
+                              int64_t context, const void* sink, int64_t chunk);
 int64_t prefill_attention_tcgen05_workspace_bytes(int64_t batch, int64_t tokens);
 }  // namespace b200
 
@@ -411,7 +411,7 @@ extern "C" int b200_prefill_attention(const void* query, const void* key, const 
     const int code = prefill_attention_tcgen05(query, key, value, output, batch, q_heads, kv_heads,
                                                tokens, head_dim, query_strides, key_strides,
                                                value_strides, scale, status, s, mask, mask_strides,
-                                               workspace, workspace_bytes, 0, nullptr);
+                                               workspace, workspace_bytes, 0, nullptr, 0);
     if (code != B200_ERR_UNSUPPORTED) return code;
   }
 

@@ -52,6 +52,7 @@ struct PrefillTcParams {
   int32_t* status;
   int q_heads, groups, tokens;
   int context = 0;  // keys in front of the first query row (causal form)
+  int chunk = 0;    // CHUNKED: position i sees j <= i with i / chunk == j / chunk
   const __nv_bfloat16* sink = nullptr;  // [Hq]: exp(sink) joins the row sum (causal form)
   int q_token_dim1, k_token_dim1, v_token_dim1;  // coordinate order of the three tensor maps
   float scale_log2;
@@ -112,7 +113,7 @@ constexpr float kRescaleThreshold = 8.0f;  // log2 domain
 constexpr uint32_t kSpinLimit = 2000000u;   // polls of an MMA thread before it gives up (about 0.1 s)
 
 // 18 warps: five on one of the four 16 K-register sub-partitions, so at most 96 registers each.
-template <int D, bool MASKED>
+template <int D, bool MASKED, bool CHUNKED = false>
 __global__ void __launch_bounds__(640, 1)
 prefill_attention_tcgen05_kernel(const PrefillTcParams p, const __grid_constant__ CUtensorMap q_map,
                                  const __grid_constant__ CUtensorMap k_map,
@@ -155,6 +156,11 @@ prefill_attention_tcgen05_kernel(const PrefillTcParams p, const __grid_constant_
   int tiles_0 = min((context + q0 + 2 * kTile - 1) / kTile, all_tiles);
   int tiles_1 = min((context + q0 + 3 * kTile - 1) / kTile, all_tiles);
   const uint8_t* class_row[G] = {nullptr, nullptr};
+  if (CHUNKED) {  // both groups start with the tile that holds the first key of the first row's chunk
+    lo = (context + q0) / p.chunk * p.chunk / kTile;
+    tiles_0 -= lo;
+    tiles_1 -= lo;
+  }
   if (MASKED) {
     int first[G], last[G];
 #pragma unroll
@@ -331,6 +337,9 @@ prefill_attention_tcgen05_kernel(const PrefillTcParams p, const __grid_constant_
     const int row = ((warp & 3) << 5) | lane;
     const int group_position = context + q0 + g * kTile;  // of the group's first row
     const int my_tiles = tiles_of(g);
+    // CHUNKED: first key of this row's chunk, and of the chunk of the group's last row
+    const int chunk_first = CHUNKED ? (group_position + row) / p.chunk * p.chunk : 0;
+    const int group_end = CHUNKED ? (group_position + kTile - 1) / p.chunk * p.chunk : 0;
     const uint32_t lane_base = static_cast<uint32_t>((warp & 3) * 32) << 16;
     const uint32_t s_taddr = s_column(g) + lane_base + half * 64;
     const uint32_t o_taddr = o_column(g) + lane_base + half * (D / 2);
@@ -422,13 +431,22 @@ prefill_attention_tcgen05_kernel(const PrefillTcParams p, const __grid_constant_
           else
             failed = 1;
         }
-        if (!MASKED && (j + 1) * kTile - 1 > group_position) {
+        if (!MASKED && ((CHUNKED ? lo + j : j) + 1) * kTile - 1 > group_position) {
           // a tile that reaches past the group's first row: keys beyond a row's own position are masked
-          const int last_key = group_position + row - j * kTile - key0;
+          const int last_key = group_position + row - (CHUNKED ? lo + j : j) * kTile - key0;
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
             if (i > last_key) s0[i] = 0xff800000u;
             if (i + 32 > last_key) s1[i] = 0xff800000u;
+          }
+        }
+        if (CHUNKED && (lo + j) * kTile < group_end) {
+          // a tile with keys in front of the chunk of the group's last row
+          const int first_key = chunk_first - (lo + j) * kTile - key0;
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {
+            if (i < first_key) s0[i] = 0xff800000u;
+            if (i + 32 < first_key) s1[i] = 0xff800000u;
           }
         }
         float max0 = -INFINITY, max1 = -INFINITY, max2 = -INFINITY, max3 = -INFINITY;
@@ -474,7 +492,7 @@ prefill_attention_tcgen05_kernel(const PrefillTcParams p, const __grid_constant_
       }
       if (!ok) continue;
       // (a reference of -inf, every key so far masked, must not turn -inf - -inf into NaN)
-      const float neg_ref = MASKED && m_ref == -INFINITY ? 0.0f : -m_ref;
+      const float neg_ref = (MASKED || CHUNKED) && m_ref == -INFINITY ? 0.0f : -m_ref;
       float sum0 = 0.0f, sum1 = 0.0f;
       auto emit = [&](const uint32_t (&s)[32], int c0) {  // 32 probabilities: exp2, sum, bf16, store
         uint32_t packed[16];
@@ -577,13 +595,14 @@ int prefill_attention_tcgen05(const void* query, const void* key, const void* va
                               const int64_t key_strides[4], const int64_t value_strides[4],
                               double scale, int32_t* status, cudaStream_t stream, const void* mask,
                               const int64_t* mask_strides, void* workspace, int64_t workspace_bytes,
-                              int64_t context, const void* sink) {
+                              int64_t context, const void* sink, int64_t chunk) {
   if ((launch_mode() & B200_LAUNCH_PREFILL_WARP_LEVEL) != 0) return B200_ERR_UNSUPPORTED;
   const char* path = getenv("B200_PREFILL_ATTENTION_PATH");
   if (path != nullptr && strcmp(path, "mma.sync") == 0) return B200_ERR_UNSUPPORTED;
   if (head_dim != 64 && head_dim != 128) return B200_ERR_UNSUPPORTED;
   if (!(scale > 0.0) || tokens < 1) return B200_ERR_UNSUPPORTED;
-  if (context < 0 || context + tokens > (1 << 30) || (mask != nullptr && (context != 0 || sink != nullptr)))
+  if (context < 0 || context + tokens > (1 << 30) ||
+      (mask != nullptr && (context != 0 || sink != nullptr || chunk != 0)))
     return B200_ERR_UNSUPPORTED;
   const int64_t q_blocks = ceil_div(tokens, static_cast<int64_t>(kTile) * kGroups);
   if (q_blocks > 65535 || batch > 65535) return B200_ERR_UNSUPPORTED;
@@ -611,6 +630,7 @@ int prefill_attention_tcgen05(const void* query, const void* key, const void* va
   p.groups = static_cast<int>(q_heads / kv_heads);
   p.tokens = static_cast<int>(tokens);
   p.context = static_cast<int>(context);
+  p.chunk = chunk < context + tokens ? static_cast<int>(chunk) : 0;  // (a chunk that holds every key is no limit)
   p.sink = static_cast<const __nv_bfloat16*>(sink);
   p.q_token_dim1 = q_dim1 ? 1 : 0;
   p.k_token_dim1 = k_dim1 ? 1 : 0;
@@ -646,6 +666,9 @@ int prefill_attention_tcgen05(const void* query, const void* key, const void* va
   if (mask != nullptr)
     launched = head_dim == 64 ? launch(prefill_attention_tcgen05_kernel<64, true>)
                               : launch(prefill_attention_tcgen05_kernel<128, true>);
+  else if (p.chunk > 0)
+    launched = head_dim == 64 ? launch(prefill_attention_tcgen05_kernel<64, false, true>)
+                              : launch(prefill_attention_tcgen05_kernel<128, false, true>);
   else
     launched = head_dim == 64 ? launch(prefill_attention_tcgen05_kernel<64, false>)
                               : launch(prefill_attention_tcgen05_kernel<128, false>);
@@ -659,15 +682,15 @@ using namespace b200;
 
 extern "C" int b200_context_attention(const void* query, const void* key, const void* value, const void* sink,
                                       void* output, int64_t batch, int64_t q_heads, int64_t kv_heads, int64_t tokens,
-                                      int64_t context, int64_t head_dim, const int64_t query_strides[4],
+                                      int64_t context, int64_t chunk, int64_t head_dim, const int64_t query_strides[4],
                                       const int64_t key_strides[4], const int64_t value_strides[4], double scale,
                                       int32_t* status, void* stream) {
   if (!query || !key || !value || !output || !query_strides || !key_strides || !value_strides || batch <= 0 ||
-      q_heads <= 0 || kv_heads <= 0 || q_heads % kv_heads != 0 || tokens <= 0 || context < 0)
+      q_heads <= 0 || kv_heads <= 0 || q_heads % kv_heads != 0 || tokens <= 0 || context < 0 || chunk < 0)
     return B200_ERR_BAD_ARGUMENT;
   if (query_strides[3] != 1 || key_strides[3] != 1 || value_strides[3] != 1) return B200_ERR_UNSUPPORTED;
   if (!aligned16(query) || !aligned16(key) || !aligned16(value) || !aligned16(output)) return B200_ERR_ALIGNMENT;
   return prefill_attention_tcgen05(query, key, value, output, batch, q_heads, kv_heads, tokens, head_dim,
                                    query_strides, key_strides, value_strides, scale, status,
-                                   static_cast<cudaStream_t>(stream), nullptr, nullptr, nullptr, 0, context, sink);
+                                   static_cast<cudaStream_t>(stream), nullptr, nullptr, nullptr, 0, context, sink, chunk);
 }

@@ -19,23 +19,24 @@ __device__ __forceinline__ void rotation_of(int64_t position, int i, int dims, d
 struct DeltaInputs {
   static constexpr bool kDelta = true;
   const void* input;   // T [rows, row_stride]: the projections of h
-  const void* gates;   // T [rows, gate_row_stride]: decay columns [heads * dim] from decay_column
+  const void* gates;   // T [rows, gate_row_stride]: decay columns [heads * decay_dim] from decay_column
   const void *q_conv, *k_conv, *v_conv;  // T [channels, taps] in time order
   const void* a_log;   // T [heads]
-  const void* dt_bias; // T [heads * dim]
+  const void* dt_bias; // T [heads * decay_dim]
   void* ring;          // T [slots, taps, 2 kv_heads dim + heads vdim]: inputs by position % taps
   SequenceBatch batch;
   int heads, kv_heads, dim, vdim, taps;
   int q_column, k_column, v_column, beta_column, decay_column;
   int64_t row_stride, gate_row_stride;
   float q_scale;
+  int decay_dim;       // decays of a head: dim (one per key channel) or 1
 };
 
 inline bool delta_inputs_from(const b200_delta_inputs* in, DeltaInputs* out) {
   if (in == nullptr || !in->input || !in->gates || !in->q_conv || !in->k_conv || !in->v_conv || !in->a_log ||
       !in->dt_bias || !in->ring || !in->token_sequence || !in->starts || !in->slots || !in->bases ||
       in->heads <= 0 || in->kv_heads <= 0 || in->heads % in->kv_heads != 0 || in->dim <= 0 || in->vdim <= 0 ||
-      in->taps <= 0)
+      in->taps <= 0 || (in->decay_dim != 1 && in->decay_dim != in->dim))
     return false;
   *out = DeltaInputs{in->input, in->gates, in->q_conv, in->k_conv, in->v_conv, in->a_log, in->dt_bias, in->ring,
                      {in->token_sequence, in->starts, in->slots, in->bases},
@@ -43,7 +44,7 @@ inline bool delta_inputs_from(const b200_delta_inputs* in, DeltaInputs* out) {
                      static_cast<int>(in->vdim), static_cast<int>(in->taps), static_cast<int>(in->q_column),
                      static_cast<int>(in->k_column), static_cast<int>(in->v_column),
                      static_cast<int>(in->beta_column), static_cast<int>(in->decay_column), in->row_stride,
-                     in->gate_row_stride, static_cast<float>(in->q_scale)};
+                     in->gate_row_stride, static_cast<float>(in->q_scale), static_cast<int>(in->decay_dim)};
   return true;
 }
 
@@ -80,11 +81,12 @@ __device__ __forceinline__ float delta_beta(const DeltaInputs& p, int64_t row, i
   return sigmoid_f32(Elem<T>::load(static_cast<const T*>(p.input) + row * p.row_stride + p.beta_column + head));
 }
 
-// log g of one key channel
+// log g of one key channel (of the head, where it has one decay)
 template <typename T>
 __device__ __forceinline__ float delta_log_decay(const DeltaInputs& p, int64_t row, int head, int c) {
-  const float step = Elem<T>::load(static_cast<const T*>(p.gates) + row * p.gate_row_stride + p.decay_column + head * p.dim + c) +
-                     Elem<T>::load(static_cast<const T*>(p.dt_bias) + head * p.dim + c);
+  const int at = p.decay_dim == 1 ? head : head * p.dim + c;
+  const float step = Elem<T>::load(static_cast<const T*>(p.gates) + row * p.gate_row_stride + p.decay_column + at) +
+                     Elem<T>::load(static_cast<const T*>(p.dt_bias) + at);
   return -expf(Elem<T>::load(static_cast<const T*>(p.a_log) + head)) * softplus_f32(step);
 }
 

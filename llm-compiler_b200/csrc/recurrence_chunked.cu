@@ -12,7 +12,9 @@
 // Precision: decays stay logarithms until they are differences of one sign (products of decays are taken
 // as sums over the tokens between, never as quotients), the triangular solve is fp32, and every product
 // on the tensor cores splits its fp32 operands into two bf16 numbers (hi hi + hi lo + lo hi), which keeps
-// 16 bits of mantissa. Within 16 tokens the decayed products are built up token by token instead.
+// 16 bits of mantissa. Within 16 tokens the decayed products are built up token by token instead. Where a
+// head has one decay, P_i / P_j is a factor of the plain product k_i . k_j: 2 to a difference of running
+// sums, which are kept in double.
 #include "common.cuh"
 #include "hybrid.cuh"
 
@@ -27,7 +29,7 @@ struct IntConstant { static constexpr int value = N; };
 struct ChunkParams {
   const float *q, *k, *v;   // [rows, kv_heads, dim] x 2, [rows, heads, vdim]
   const float* beta;        // [rows, heads] (delta)
-  const float* decay;       // log g [rows, heads, dim] (delta); decay [heads] (retention)
+  const float* decay;       // log g [rows, heads, dim] or [rows, heads] (delta); decay [heads] (retention)
   float* state;             // [slots, heads, dim, state_row]
   float* output;            // [rows, heads, vdim]
   SequenceBatch batch;
@@ -102,6 +104,106 @@ __device__ __forceinline__ float4 load4(const float* source, int c, int dim, boo
   return v;
 }
 
+// Triangular solve (I + lower) [W | U] = beta [P k | v] on the tensor cores, transposed: a warp owns 16
+// columns, Y_I = (R_I - sum_{J<I} Y_J lower_IJ^T) inverse_I^T stays in its registers throughout.
+// triangle: [2][64][kTriangle] planes of minus the blocks below the diagonal; inverse: [2][64][kInverse]
+// inverted diagonal blocks; decayed_key(i, c): entry c of P_i k_i; staging: [2][64][D] planes of W.
+template <int D, typename DecayedKey>
+__device__ __forceinline__ void solve_chunk(const ChunkParams& p, const __nv_bfloat16* triangle,
+                                            const __nv_bfloat16* inverse, const float* betas, __nv_bfloat16* staging,
+                                            unsigned char* out, int64_t row0, int count, int head, int warp, int lane,
+                                            DecayedKey decayed_key) {
+  using Layout = ChunkLayout<D>;
+  const int v_row = (p.vdim + 31) / 32 * 32;
+  for (int tile = warp; tile < (D + v_row) / 16; tile += kIntraThreads / 32) {
+    const int c0 = tile * 16 + (lane >> 2);  // fragment rows c0 and c0 + 8 are columns of [W | U]
+    float rhs[kSubs][2][4];
+#pragma unroll
+    for (int I = 0; I < kSubs; ++I)
+#pragma unroll
+      for (int h = 0; h < 2; ++h)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int i = I * kSub + h * 8 + (lane & 3) * 2 + (e & 1), c = c0 + (e >> 1) * 8;
+          if (tile < D / 16) {
+            rhs[I][h][e] = betas[i] * decayed_key(i, c);
+          } else {
+            const int vc = c - D;
+            rhs[I][h][e] = i < count && vc < p.vdim ? p.v[((row0 + i) * p.heads + head) * p.vdim + vc] : 0.0f;
+          }
+        }
+    uint32_t yh[kSubs][4], yl[kSubs][4];
+#pragma unroll
+    for (int I = 0; I < kSubs; ++I) {
+      float acc[2][4];
+#pragma unroll
+      for (int h = 0; h < 2; ++h)
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          acc[h][e] = tile < D / 16 ? rhs[I][h][e] : rhs[I][h][e] * betas[I * kSub + h * 8 + (lane & 3) * 2 + (e & 1)];
+      const int n_row = I * kSub + ((lane >> 4) << 3) + (lane & 7), k_half = ((lane >> 3) & 1) * 8;
+      auto multiply = [&](const uint32_t (&ah)[4], const uint32_t (&al)[4], const __nv_bfloat16* plane, int pitch,
+                          int column, float (&to)[2][4]) {
+        uint32_t bh[4], bl[4];
+        ldmatrix_x4(bh, smem_u32(plane + n_row * pitch + column + k_half));
+        ldmatrix_x4(bl, smem_u32(plane + (kChunk + n_row) * pitch + column + k_half));
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          mma_bf16_16816(to[h], ah, bh[h * 2], bh[h * 2 + 1]);
+          mma_bf16_16816(to[h], ah, bl[h * 2], bl[h * 2 + 1]);
+          mma_bf16_16816(to[h], al, bh[h * 2], bh[h * 2 + 1]);
+        }
+      };
+#pragma unroll
+      for (int J = 0; J < I; ++J) multiply(yh[J], yl[J], triangle, kTriangle, J * kSub, acc);
+      uint32_t zh[4], zl[4];
+      split_bf16x2(acc[0][0], acc[0][1], zh[0], zl[0]);
+      split_bf16x2(acc[0][2], acc[0][3], zh[1], zl[1]);
+      split_bf16x2(acc[1][0], acc[1][1], zh[2], zl[2]);
+      split_bf16x2(acc[1][2], acc[1][3], zh[3], zl[3]);
+      float y[2][4] = {};
+      multiply(zh, zl, inverse, kInverse, 0, y);
+      split_bf16x2(y[0][0], y[0][1], yh[I][0], yl[I][0]);
+      split_bf16x2(y[0][2], y[0][3], yh[I][1], yl[I][1]);
+      split_bf16x2(y[1][0], y[1][1], yh[I][2], yl[I][2]);
+      split_bf16x2(y[1][2], y[1][3], yh[I][3], yl[I][3]);
+#pragma unroll
+      for (int h = 0; h < 2; ++h)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int i = I * kSub + h * 8 + (lane & 3) * 2 + (e & 1), c = c0 + (e >> 1) * 8;
+          if (tile < D / 16) {
+            const __nv_bfloat16 high = __float2bfloat16_rn(y[h][e]);
+            staging[i * D + c] = high;
+            staging[(kChunk + i) * D + c] = __float2bfloat16_rn(y[h][e] - __bfloat162float(high));
+          } else {
+            reinterpret_cast<float*>(out + Layout::kU)[i * v_row + c - D] = y[h][e];
+          }
+        }
+    }
+  }
+  __syncthreads();
+  for (int item = threadIdx.x; item < 2 * kChunk * D / 8; item += kIntraThreads)
+    reinterpret_cast<uint4*>(out + Layout::kW)[item] = reinterpret_cast<const uint4*>(staging)[item];
+}
+
+// (I + N)^-1 of the 16 x 16 diagonal blocks, one column a thread of the CTA's last 64
+__device__ __forceinline__ void invert_diagonal_blocks(const float* lower, int pitch, __nv_bfloat16* inverse) {
+  if (threadIdx.x < kIntraThreads - kChunk) return;
+  const int column = threadIdx.x - (kIntraThreads - kChunk), block = column / kSub * kSub, own = column % kSub;
+  float x[kSub];
+#pragma unroll
+  for (int i = 0; i < kSub; ++i) {
+    float v = i == own ? 1.0f : 0.0f;
+#pragma unroll
+    for (int j = 0; j < i; ++j) v = fmaf(-lower[(block + i) * pitch + block + j], x[j], v);
+    x[i] = v;
+    const __nv_bfloat16 high = __float2bfloat16_rn(v);
+    inverse[(block + i) * kInverse + own] = high;
+    inverse[(kChunk + block + i) * kInverse + own] = __float2bfloat16_rn(v - __bfloat162float(high));
+  }
+}
+
 // Retention: one decay per head, so the decayed products are the plain ones times decay^(i - j).
 template <int D>
 __global__ void __launch_bounds__(kIntraThreads) chunk_intra_retention_kernel(const ChunkParams p) {
@@ -172,6 +274,145 @@ __global__ void __launch_bounds__(kIntraThreads) chunk_intra_retention_kernel(co
       reinterpret_cast<uint32_t*>(out + Layout::kA)[(i * kChunk + j) / 2] = high;
       reinterpret_cast<uint32_t*>(out + Layout::kA + Layout::kSquare)[(i * kChunk + j) / 2] = low;
     }
+}
+
+// The delta rule with one decay per head: both triangular matrices are plain products times 2^(x_i - x_j),
+// x the running sum of log2 g.
+template <int D>
+constexpr int intra_head_delta_smem_bytes() {
+  return 4 * kChunk * (D + 8) * 2 + kChunk * (kChunk + 4) * 4 + 2 * kChunk * kTriangle * 2 + 2 * kChunk * kInverse * 2;
+}
+template <int D>
+__global__ void __launch_bounds__(kIntraThreads) chunk_intra_head_delta_kernel(const ChunkParams p) {
+  constexpr int PM = kChunk + 4, PB = (D + 8) * 2;
+  using Layout = ChunkLayout<D>;
+  extern __shared__ __align__(128) unsigned char smem[];
+  unsigned char* q_planes = smem;                          // [2][64][PB], later the staging of W's planes
+  unsigned char* k_planes = smem + 2 * kChunk * PB;
+  float* lower = reinterpret_cast<float*>(k_planes + 2 * kChunk * PB);  // [64][PM]
+  __nv_bfloat16* triangle = reinterpret_cast<__nv_bfloat16*>(lower + kChunk * PM);
+  __nv_bfloat16* inverse = triangle + 2 * kChunk * kTriangle;
+  __shared__ float betas[kChunk], into[kChunk];   // into: 2^x
+  __shared__ double sums[kChunk];                 // x
+  const int chunk = blockIdx.x, head = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  int64_t row0;
+  const int count = locate_chunk(p, chunk, row0);
+  const int kv_head = head / (p.heads / p.kv_heads);
+  unsigned char* out = p.workspace + (static_cast<int64_t>(chunk) * p.heads + head) * Layout::bytes(true, p.vdim);
+  const bool whole = p.dim == D;
+  constexpr int kRounds = kChunk * D / 4 / kIntraThreads;
+  float4 q[kRounds], k[kRounds];
+#pragma unroll
+  for (int i = 0; i < kRounds; ++i) {
+    const int item = threadIdx.x + i * kIntraThreads, t = item / (D / 4), c = item % (D / 4) * 4;
+    const int64_t source = ((row0 + t) * p.kv_heads + kv_head) * p.dim;
+    q[i] = load4(p.q + source, c, p.dim, t < count, whole);
+    k[i] = load4(p.k + source, c, p.dim, t < count, whole);
+  }
+  if (warp == 0) {  // two tokens a lane
+    double x[2];
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int t = lane * 2 + e;
+      const int64_t unit = (row0 + t) * p.heads + head;
+      betas[t] = t < count ? p.beta[unit] : 0.0f;
+      // (a token that keeps less than 2^-126 keeps nothing)
+      x[e] = t < count ? static_cast<double>(fmaxf(p.decay[unit] * 1.4426950408889634f, -126.0f)) : 0.0;
+    }
+    x[1] += x[0];
+    double total = x[1];
+#pragma unroll
+    for (int o = 1; o < 32; o *= 2) {
+      const double before = __shfl_up_sync(0xffffffffu, total, o);
+      if (lane >= o) total += before;
+    }
+    const double front = total - x[1];
+    sums[lane * 2] = front + x[0];
+    sums[lane * 2 + 1] = total;
+    into[lane * 2] = exp2f(static_cast<float>(front + x[0]));
+    into[lane * 2 + 1] = exp2f(static_cast<float>(total));
+  }
+  __syncthreads();
+  const double end = sums[kChunk - 1];
+#pragma unroll
+  for (int i = 0; i < kRounds; ++i) {
+    const int item = threadIdx.x + i * kIntraThreads, t = item / (D / 4), c = item % (D / 4) * 4;
+    const float in = into[t], rest = exp2f(static_cast<float>(end - sums[t]));
+    uint2 high, low;
+    split4(q[i], high, low);
+    *reinterpret_cast<uint2*>(q_planes + t * PB + c * 2) = high;
+    *reinterpret_cast<uint2*>(q_planes + (kChunk + t) * PB + c * 2) = low;
+    split4(k[i], high, low);
+    *reinterpret_cast<uint2*>(k_planes + t * PB + c * 2) = high;
+    *reinterpret_cast<uint2*>(k_planes + (kChunk + t) * PB + c * 2) = low;
+    split4(mul4(q[i], make_float4(in, in, in, in)), high, low);
+    reinterpret_cast<uint2*>(out + Layout::kQ)[item] = high;
+    reinterpret_cast<uint2*>(out + Layout::kQ + Layout::kPlane)[item] = low;
+    split4(mul4(k[i], make_float4(rest, rest, rest, rest)), high, low);
+    reinterpret_cast<uint2*>(out + Layout::kK)[item] = high;
+    reinterpret_cast<uint2*>(out + Layout::kK + Layout::kPlane)[item] = low;
+  }
+  if (threadIdx.x < D) reinterpret_cast<float*>(out + Layout::kEnd)[threadIdx.x] = into[kChunk - 1];
+  __syncthreads();
+  // 16 warps: 16 rows x 16 columns of K K^T and of Q K^T each
+  const int m0 = (warp >> 2) * 16, n0 = (warp & 3) * 16;
+  float kk[2][4] = {}, qk[2][4] = {};
+  if (n0 <= m0) {
+    const uint32_t row_lane = (m0 + (lane & 15)) * PB + (lane >> 4) * 16;
+    const uint32_t ka_base = smem_u32(k_planes) + row_lane, qa_base = smem_u32(q_planes) + row_lane;
+    const uint32_t b_base = smem_u32(k_planes) + (n0 + ((lane >> 4) << 3) + (lane & 7)) * PB + ((lane >> 3) & 1) * 16;
+#pragma unroll
+    for (int step = 0; step < D / 16; ++step) {
+      uint32_t kh[4], kl[4], qh[4], ql[4], bh[4], bl[4];
+      ldmatrix_x4(kh, ka_base + step * 32);
+      ldmatrix_x4(kl, ka_base + kChunk * PB + step * 32);
+      ldmatrix_x4(qh, qa_base + step * 32);
+      ldmatrix_x4(ql, qa_base + kChunk * PB + step * 32);
+      ldmatrix_x4(bh, b_base + step * 32);
+      ldmatrix_x4(bl, b_base + kChunk * PB + step * 32);
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        mma_bf16_16816(kk[h], kh, bh[h * 2], bh[h * 2 + 1]);
+        mma_bf16_16816(qk[h], qh, bh[h * 2], bh[h * 2 + 1]);
+        mma_bf16_16816(kk[h], kh, bl[h * 2], bl[h * 2 + 1]);
+        mma_bf16_16816(qk[h], qh, bl[h * 2], bl[h * 2 + 1]);
+        mma_bf16_16816(kk[h], kl, bh[h * 2], bh[h * 2 + 1]);
+        mma_bf16_16816(qk[h], ql, bh[h * 2], bh[h * 2 + 1]);
+      }
+    }
+  }
+#pragma unroll
+  for (int h = 0; h < 2; ++h)
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int i = m0 + (lane >> 2) + half * 8, j = n0 + h * 8 + (lane & 3) * 2;
+      float a[2], l[2];
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const float f = i >= j + e ? exp2f(static_cast<float>(sums[i] - sums[j + e])) : 0.0f;
+        a[e] = qk[h][half * 2 + e] * f;
+        l[e] = i > j + e ? kk[h][half * 2 + e] * f * betas[i] : 0.0f;
+      }
+      uint32_t high, low;
+      split_bf16x2(a[0], a[1], high, low);
+      reinterpret_cast<uint32_t*>(out + Layout::kA)[(i * kChunk + j) / 2] = high;
+      reinterpret_cast<uint32_t*>(out + Layout::kA + Layout::kSquare)[(i * kChunk + j) / 2] = low;
+      if (n0 == m0) *reinterpret_cast<float2*>(lower + i * PM + j) = make_float2(l[0], l[1]);
+      if (n0 < m0) {
+        split_bf16x2(-l[0], -l[1], high, low);
+        *reinterpret_cast<uint32_t*>(triangle + i * kTriangle + j) = high;
+        *reinterpret_cast<uint32_t*>(triangle + (kChunk + i) * kTriangle + j) = low;
+      }
+    }
+  __syncthreads();
+  invert_diagonal_blocks(lower, PM, inverse);
+  __syncthreads();
+  const __nv_bfloat16* keys = reinterpret_cast<const __nv_bfloat16*>(k_planes);
+  solve_chunk<D>(p, triangle, inverse, betas, reinterpret_cast<__nv_bfloat16*>(q_planes), out, row0, count, head, warp,
+                 lane, [&](int i, int c) {
+                   return (__bfloat162float(keys[i * (D + 8) + c]) + __bfloat162float(keys[(kChunk + i) * (D + 8) + c])) *
+                          into[i];
+                 });
 }
 
 template <int D>
@@ -390,96 +631,12 @@ __global__ void __launch_bounds__(kIntraThreads, 1) chunk_intra_delta_kernel(con
       *reinterpret_cast<uint2*>(triangle + (kChunk + i) * kTriangle + j) = low;
     }
   }
-  if (threadIdx.x >= kIntraThreads - kChunk) {  // (I + N)^-1 of a diagonal block, one column a thread
-    const int column = threadIdx.x - (kIntraThreads - kChunk), block = column / kSub * kSub, own = column % kSub;
-    float x[kSub];
-#pragma unroll
-    for (int i = 0; i < kSub; ++i) {
-      float v = i == own ? 1.0f : 0.0f;
-#pragma unroll
-      for (int j = 0; j < i; ++j) v = fmaf(-lower[(block + i) * PM + block + j], x[j], v);
-      x[i] = v;
-      const __nv_bfloat16 high = __float2bfloat16_rn(v);
-      inverse[(block + i) * kInverse + own] = high;
-      inverse[(kChunk + block + i) * kInverse + own] = __float2bfloat16_rn(v - __bfloat162float(high));
-    }
-  }
+  invert_diagonal_blocks(lower, PM, inverse);
   __syncthreads();
 
-  // ---- triangular solve (I + lower) [W | U] = beta [P k | v] on the tensor cores, transposed: a warp owns
-  // 16 columns, Y_I = (R_I - sum_{J<I} Y_J lower_IJ^T) inverse_I^T stays in its registers throughout ----
   __nv_bfloat16* staging = reinterpret_cast<__nv_bfloat16*>(qs);  // [2][64][D] planes of W
-  const int v_row = (p.vdim + 31) / 32 * 32;
-  for (int tile = warp; tile < (D + v_row) / 16; tile += kIntraThreads / 32) {
-    const int c0 = tile * 16 + (lane >> 2);  // fragment rows c0 and c0 + 8 are columns of [W | U]
-    float rhs[kSubs][2][4];
-#pragma unroll
-    for (int I = 0; I < kSubs; ++I)
-#pragma unroll
-      for (int h = 0; h < 2; ++h)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int i = I * kSub + h * 8 + (lane & 3) * 2 + (e & 1), c = c0 + (e >> 1) * 8;
-          if (tile < D / 16) {
-            rhs[I][h][e] = betas[i] * ks[i * PD + c] * exp2f(xs[i * PD + c] + pre[I * D + c]);
-          } else {
-            const int vc = c - D;
-            rhs[I][h][e] = i < count && vc < p.vdim ? p.v[((row0 + i) * p.heads + head) * p.vdim + vc] : 0.0f;
-          }
-        }
-    uint32_t yh[kSubs][4], yl[kSubs][4];
-#pragma unroll
-    for (int I = 0; I < kSubs; ++I) {
-      float acc[2][4];
-#pragma unroll
-      for (int h = 0; h < 2; ++h)
-#pragma unroll
-        for (int e = 0; e < 4; ++e)
-          acc[h][e] = tile < D / 16 ? rhs[I][h][e] : rhs[I][h][e] * betas[I * kSub + h * 8 + (lane & 3) * 2 + (e & 1)];
-      const int n_row = I * kSub + ((lane >> 4) << 3) + (lane & 7), k_half = ((lane >> 3) & 1) * 8;
-      auto multiply = [&](const uint32_t (&ah)[4], const uint32_t (&al)[4], const __nv_bfloat16* plane, int pitch,
-                          int column, float (&to)[2][4]) {
-        uint32_t bh[4], bl[4];
-        ldmatrix_x4(bh, smem_u32(plane + n_row * pitch + column + k_half));
-        ldmatrix_x4(bl, smem_u32(plane + (kChunk + n_row) * pitch + column + k_half));
-#pragma unroll
-        for (int h = 0; h < 2; ++h) {
-          mma_bf16_16816(to[h], ah, bh[h * 2], bh[h * 2 + 1]);
-          mma_bf16_16816(to[h], ah, bl[h * 2], bl[h * 2 + 1]);
-          mma_bf16_16816(to[h], al, bh[h * 2], bh[h * 2 + 1]);
-        }
-      };
-#pragma unroll
-      for (int J = 0; J < I; ++J) multiply(yh[J], yl[J], triangle, kTriangle, J * kSub, acc);
-      uint32_t zh[4], zl[4];
-      split_bf16x2(acc[0][0], acc[0][1], zh[0], zl[0]);
-      split_bf16x2(acc[0][2], acc[0][3], zh[1], zl[1]);
-      split_bf16x2(acc[1][0], acc[1][1], zh[2], zl[2]);
-      split_bf16x2(acc[1][2], acc[1][3], zh[3], zl[3]);
-      float y[2][4] = {};
-      multiply(zh, zl, inverse, kInverse, 0, y);
-      split_bf16x2(y[0][0], y[0][1], yh[I][0], yl[I][0]);
-      split_bf16x2(y[0][2], y[0][3], yh[I][1], yl[I][1]);
-      split_bf16x2(y[1][0], y[1][1], yh[I][2], yl[I][2]);
-      split_bf16x2(y[1][2], y[1][3], yh[I][3], yl[I][3]);
-#pragma unroll
-      for (int h = 0; h < 2; ++h)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int i = I * kSub + h * 8 + (lane & 3) * 2 + (e & 1), c = c0 + (e >> 1) * 8;
-          if (tile < D / 16) {
-            const __nv_bfloat16 high = __float2bfloat16_rn(y[h][e]);
-            staging[i * D + c] = high;
-            staging[(kChunk + i) * D + c] = __float2bfloat16_rn(y[h][e] - __bfloat162float(high));
-          } else {
-            reinterpret_cast<float*>(out + Layout::kU)[i * v_row + c - D] = y[h][e];
-          }
-        }
-    }
-  }
-  __syncthreads();
-  for (int item = threadIdx.x; item < 2 * kChunk * D / 8; item += kIntraThreads)
-    reinterpret_cast<uint4*>(out + Layout::kW)[item] = reinterpret_cast<const uint4*>(staging)[item];
+  solve_chunk<D>(p, triangle, inverse, betas, staging, out, row0, count, head, warp, lane,
+                 [&](int i, int c) { return ks[i * PD + c] * exp2f(xs[i * PD + c] + pre[i / kSub * D + c]); });
 }
 
 // ---- across the chunks -------------------------------------------------------------------
@@ -679,11 +836,12 @@ __global__ void __launch_bounds__(VB * 16, 1) chunk_inter_kernel(const ChunkPara
 }
 
 template <int D, bool DELTA>
-int launch_chunked(const ChunkParams& p, int64_t chunks, cudaStream_t stream) {
-  auto intra = chunk_intra_delta_kernel<D>;
-  if (!DELTA) intra = chunk_intra_retention_kernel<D>;
-  constexpr int intra_smem = DELTA ? intra_smem_bytes<D>() : 4 * kChunk * (D + 8) * 2;
-  static_assert(intra_smem <= 226 * 1024, "the chunk does not fit shared memory");
+int launch_chunked(const ChunkParams& p, int64_t chunks, bool head_decay, cudaStream_t stream) {
+  auto intra = !DELTA ? chunk_intra_retention_kernel<D> : head_decay ? chunk_intra_head_delta_kernel<D>
+                                                                     : chunk_intra_delta_kernel<D>;
+  static_assert(intra_smem_bytes<D>() <= 226 * 1024, "the chunk does not fit shared memory");
+  const int intra_smem = !DELTA ? 4 * kChunk * (D + 8) * 2 : head_decay ? intra_head_delta_smem_bytes<D>()
+                                                                        : intra_smem_bytes<D>();
   if (cudaFuncSetAttribute(intra, cudaFuncAttributeMaxDynamicSharedMemorySize, intra_smem) != cudaSuccess)
     return B200_ERR_LAUNCH;
   intra<<<dim3(static_cast<unsigned>(chunks), static_cast<unsigned>(p.heads)), kIntraThreads, intra_smem, stream>>>(p);
@@ -717,10 +875,11 @@ extern "C" int b200_recurrence_chunked(const float* q, const float* k, const flo
                                        const float* decay, float* state, float* output, const int32_t* token_sequence,
                                        const int32_t* starts, const int32_t* slots, const int32_t* bases,
                                        const int32_t* chunk_starts, int64_t chunks, int64_t sequences, int64_t heads,
-                                       int64_t kv_heads, int64_t dim, int64_t vdim, int64_t state_row,
+                                       int64_t kv_heads, int64_t dim, int64_t vdim, int64_t state_row, int64_t decay_dim,
                                        void* workspace, int64_t workspace_bytes, void* stream) {
   if (!q || !k || !v || !decay || !state || !output || !starts || !slots || !bases || !chunk_starts || chunks < 0 ||
-      sequences < 0 || heads <= 0 || kv_heads <= 0 || heads % kv_heads != 0 || dim <= 0 || vdim <= 0 || state_row < vdim)
+      sequences < 0 || heads <= 0 || kv_heads <= 0 || heads % kv_heads != 0 || dim <= 0 || vdim <= 0 || state_row < vdim ||
+      (decay_dim != 1 && decay_dim != dim))
     return B200_ERR_BAD_ARGUMENT;
   if (dim > 128 || vdim > 1024) return B200_ERR_UNSUPPORTED;
   if (chunks == 0 || sequences == 0) return B200_OK;
@@ -732,6 +891,8 @@ extern "C" int b200_recurrence_chunked(const float* q, const float* k, const flo
                 static_cast<int>(sequences), static_cast<int>(heads), static_cast<int>(kv_heads), static_cast<int>(dim),
                 static_cast<int>(vdim), static_cast<int>(state_row), static_cast<unsigned char*>(workspace)};
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (dim <= 64) return beta ? launch_chunked<64, true>(p, chunks, s) : launch_chunked<64, false>(p, chunks, s);
-  return beta ? launch_chunked<128, true>(p, chunks, s) : launch_chunked<128, false>(p, chunks, s);
+  const bool head_decay = decay_dim != dim || dim == 1;
+  if (dim <= 64)
+    return beta ? launch_chunked<64, true>(p, chunks, head_decay, s) : launch_chunked<64, false>(p, chunks, false, s);
+  return beta ? launch_chunked<128, true>(p, chunks, head_decay, s) : launch_chunked<128, false>(p, chunks, false, s);
 }

@@ -1,5 +1,5 @@
-"""Serving engine of the hybrid designs: layers whose mixers keep recurrent state or cached latents in
-slots, an fp32 residual stream, portions of prompts and decoded tokens through one step function.
+"""Serving engine of the hybrid designs: layers whose mixers keep recurrent state, cached latents or
+keys and values in slots, an fp32 residual stream, portions of prompts and decoded tokens through one step function.
 
 `forward` is the step: it takes, for any number of sequences, the next tokens of each (a whole prompt, a
 portion of one, or one decoded token) and runs them from the state that earlier steps left. `prefill`,
@@ -14,7 +14,6 @@ from typing import Dict, List, Optional, Sequence, Tuple
 
 import torch
 
-from . import bazirax
 from . import hybrid_kernels as hk
 from . import kernels
 from .engine import ServingEngine
@@ -24,10 +23,11 @@ from .mixers import pad_matrix
 
 
 class HybridEngine(ServingEngine):
-    def __init__(self, config: "bazirax.BaziraxConfig", weights: Dict[str, torch.Tensor], *, batch: int,
+    def __init__(self, config, weights: Dict[str, torch.Tensor], *, batch: int,
                  capacity: int, device: Optional[torch.device] = None) -> None:
-        """`batch` slots of `capacity` tokens each. The weights' dtype (fp32 or bf16) is the dtype of
-        projections and cached latents; they must be on the device."""
+        """`batch` slots of `capacity` tokens each. `config`: a hybrid design's (bazirax, lozanex): sizes,
+        norm_eps, norm_offset and build_layers(weights). The weights' dtype (fp32 or bf16) is the dtype of
+        projections and caches; they must be on the device."""
 
         for name, tensor in weights.items():
             if not tensor.is_cuda:
@@ -36,9 +36,9 @@ class HybridEngine(ServingEngine):
         self.config = config
         self.capacity = capacity
         self.dtype = weights["embed"].dtype
-        self.epsilon, self.norm_offset = config.norm_eps, bazirax.NORM_OFFSET
-        self.layers = bazirax.build_layers(config, weights)
-        self.embed = weights["embed"]
+        self.epsilon, self.norm_offset = config.norm_eps, config.norm_offset
+        self.layers = config.build_layers(weights)
+        self.embed, self.embed_norm = weights["embed"], weights.get("embed.norm")
         self.final_norm = weights["final.norm"]
         self.head = pad_matrix(weights["head"], pad8(config.vocab_size), pad8(config.hidden_size))
         self.state = SlotState([layer.mixer.state_spec(capacity) for layer in self.layers], slots=batch,
@@ -54,25 +54,31 @@ class HybridEngine(ServingEngine):
         self._row_graphs: Dict[int, Tuple[torch.cuda.CUDAGraph, torch.Tensor]] = {}
 
     # ------------------------------------------------------------------ the layers ----
-    def _norm_step(self, x, y, post_weight, next_weight):
+    def _norm_step(self, x, y, post_weight, next_weight, narrow=False):
         return hk.residual_norm(x, y, post_weight, next_weight, epsilon=self.epsilon,
-                                weight_offset=self.norm_offset, dtype=self.dtype)
+                                weight_offset=self.norm_offset, dtype=self.dtype, narrow=narrow)
 
     def _run_layers(self, ids: torch.Tensor, batch: SequenceBatch, last_norm: Optional[torch.Tensor],
                     streams: Optional[list] = None) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
         """Residual stream behind the last layer, and its rows normed with `last_norm`."""
 
-        x = hk.embedding_residual(self.embed, ids)
-        h = self._norm_step(x, None, None, self.layers[0].norm_in)
+        first = self.layers[0].norm_in
+        x = hk.embedding_residual(self.embed, ids, self.embed_norm, epsilon=self.epsilon,
+                                  weight_offset=self.norm_offset, narrow=first is None)
+        if first is None:
+            x, h = x
+        else:
+            h = self._norm_step(x, None, None, first)
         for index, layer in enumerate(self.layers):
-            after = self.layers[index + 1].norm_in if index + 1 < len(self.layers) else last_norm
+            last = index + 1 == len(self.layers)
+            after = last_norm if last else self.layers[index + 1].norm_in
             source = layer.mixer.shared_state
             y = layer.mixer(h, batch, self.state.layers[index if source is None else source])
             if layer.mlp is not None:
-                h = self._norm_step(x, y, layer.norm_out, layer.mlp_norm_in)
-                h = self._norm_step(x, layer.mlp(h), layer.mlp_norm_out, after)
+                h = self._norm_step(x, y, layer.norm_out, layer.mlp_norm_in, narrow=layer.mlp_norm_in is None)
+                h = self._norm_step(x, layer.mlp(h), layer.mlp_norm_out, after, narrow=not last and after is None)
             else:
-                h = self._norm_step(x, y, layer.norm_out, after)
+                h = self._norm_step(x, y, layer.norm_out, after, narrow=not last and after is None)
             if streams is not None:
                 streams.append(x.clone())
         return x, h

@@ -1,5 +1,6 @@
 """Python wrappers over the C ABI for the hybrid layers' operators (include/b200_serve.h, "Hybrid
-layers"): recurrent mixers, latent attention and the fp32 residual stream. Same rules as kernels.py:
+layers"): recurrent mixers, attention over cached latents or keys and values, mixtures of experts and the
+fp32 residual stream. Same rules as kernels.py:
 preconditions raise before anything is launched, launches go to torch's current stream and never
 synchronise, and there is no fallback to PyTorch."""
 
@@ -84,35 +85,56 @@ def _require_rows(tensor: torch.Tensor, what: str) -> None:
         raise ValueError(f"{what} must be a matrix with contiguous rows")
 
 
-def embedding_residual(table: torch.Tensor, ids: torch.Tensor) -> torch.Tensor:
-    """Rows of `table` gathered by int64 ids and widened to fp32: the start of the residual stream."""
+@dataclass
+class Summands:
+    """A sublayer's result in the parts that residual_norm adds up: y (as there) plus `bias` [width], and
+    for every row the rows `places` [rows, top] of the matrix `rows` (the experts' results)."""
 
-    device = _require_cuda(table, ids)
+    y: Optional[torch.Tensor]
+    bias: Optional[torch.Tensor] = None
+    rows: Optional[torch.Tensor] = None
+    places: Optional[torch.Tensor] = None
+
+
+def embedding_residual(table: torch.Tensor, ids: torch.Tensor, weight: Optional[torch.Tensor] = None, *,
+                       epsilon: float = 0.0, weight_offset: float = 0.0, narrow: bool = False):
+    """Rows of `table` gathered by int64 ids and widened to fp32: the start of the residual stream. With
+    `weight` the rows are normed and scaled by weight_offset + weight; with `narrow` also returns them in
+    the table's dtype (padded to 8 elements)."""
+
+    device = _require_cuda(table, ids, weight)
     if table.ndim != 2 or not table.is_contiguous() or ids.dtype != torch.int64 or ids.ndim != 1 or \
             not ids.is_contiguous():
         raise ValueError("embedding needs a contiguous V x H table and a vector of int64 ids")
+    if weight is not None and (weight.shape != (table.shape[1],) or weight.dtype != table.dtype):
+        raise ValueError("the norm weight must be a vector of the table's width")
     x = torch.empty((ids.shape[0], table.shape[1]), dtype=torch.float32, device=device)
+    h = torch.empty((ids.shape[0], pad8(table.shape[1])), dtype=table.dtype, device=device) if narrow else None
     rt = runtime(device)
-    code = _lib.load().b200_embedding_residual(table.data_ptr(), ids.data_ptr(), x.data_ptr(), ids.shape[0],
-                                               table.shape[1], table.shape[0], _code(table.dtype),
+    code = _lib.load().b200_embedding_residual(table.data_ptr(), _ptr(weight), ids.data_ptr(), x.data_ptr(), _ptr(h),
+                                               ids.shape[0], table.shape[1], table.shape[0], pad8(table.shape[1]),
+                                               float(epsilon), float(weight_offset), _code(table.dtype),
                                                rt.status.data_ptr(), _stream())
     _check(code, "b200_embedding_residual")
     _count(rt)
-    return x
+    return (x, h) if narrow else x
 
 
-def residual_norm(x: torch.Tensor, y: Optional[torch.Tensor], post_weight: Optional[torch.Tensor],
+def residual_norm(x: torch.Tensor, y, post_weight: Optional[torch.Tensor],
                   next_weight: Optional[torch.Tensor], *, epsilon: float, weight_offset: float,
-                  dtype: torch.dtype) -> Optional[torch.Tensor]:
+                  dtype: torch.dtype, narrow: bool = False) -> Optional[torch.Tensor]:
     """x += norm(y) * (weight_offset + post_weight) in place on the fp32 residual x [rows, width], then
-    h = norm(x) * (weight_offset + next_weight), returned in `dtype` with rows padded to 8 elements.
-    y: [rows, >= width] in `dtype`, or fp32 split-K partials [splits, rows, >= width]; None: h only."""
+    h = norm(x) * (weight_offset + next_weight), returned in `dtype` with rows padded to 8 elements; without
+    next_weight h is x itself (narrow) or nothing. y: [rows, >= width] in `dtype`, fp32 split-K partials
+    [splits, rows, >= width], or Summands; None: h only."""
 
-    device = _require_cuda(x, y, post_weight, next_weight)
+    parts = y if isinstance(y, Summands) else Summands(y)
+    y = parts.y
+    device = _require_cuda(x, y, post_weight, next_weight, parts.bias, parts.rows, parts.places)
     if x.ndim != 2 or x.dtype != torch.float32 or not x.is_contiguous():
         raise ValueError("the residual is a contiguous fp32 matrix")
     rows, width = x.shape
-    splits = y_stride = 0
+    splits = y_stride = top = summand_stride = 0
     if y is not None:
         if y.ndim == 3:
             if y.dtype != torch.float32 or not y.is_contiguous() or y.shape[1] != rows:
@@ -123,18 +145,28 @@ def residual_norm(x: torch.Tensor, y: Optional[torch.Tensor], post_weight: Optio
             if y.dtype != dtype or y.shape[0] != rows:
                 raise ValueError("the sublayer's result does not match the residual")
             y_stride = y.stride(0)
-        if y.shape[-1] < width or post_weight is None or post_weight.shape != (width,) or \
-                post_weight.dtype != dtype:
-            raise ValueError("the norm behind a sublayer needs a weight and a result of the residual's width")
+        if y.shape[-1] < width:
+            raise ValueError("the sublayer's result is narrower than the residual")
+    if parts.rows is not None:
+        _require_rows(parts.rows, "the summands")
+        if parts.rows.dtype != dtype or parts.rows.shape[1] < width or parts.places is None or \
+                parts.places.dtype != torch.int32 or parts.places.shape[0] != rows or not parts.places.is_contiguous():
+            raise ValueError("summands must be rows of the residual's width with int32 places for every row")
+        top, summand_stride = parts.places.shape[1], parts.rows.stride(0)
+    if parts.bias is not None and (parts.bias.shape[0] < width or parts.bias.dtype != dtype):
+        raise ValueError("the bias must be a vector of the residual's width")
+    if (y is not None or top) and (post_weight is None or post_weight.shape != (width,) or post_weight.dtype != dtype):
+        raise ValueError("the norm behind a sublayer needs a weight and a result of the residual's width")
     h = None
-    if next_weight is not None:
-        if next_weight.shape != (width,) or next_weight.dtype != dtype:
+    if next_weight is not None or narrow:
+        if next_weight is not None and (next_weight.shape != (width,) or next_weight.dtype != dtype):
             raise ValueError("the norm weight must be a vector of the residual's width")
         h = torch.empty((rows, pad8(width)), dtype=dtype, device=device)
     rt = runtime(device)
     code = _lib.load().b200_residual_norm(
-        x.data_ptr(), _ptr(y), _ptr(post_weight), _ptr(next_weight), _ptr(h), rows, width, splits, y_stride,
-        pad8(width), float(epsilon), float(weight_offset), _code(dtype), _stream())
+        x.data_ptr(), _ptr(y), _ptr(parts.bias), _ptr(post_weight), _ptr(next_weight), _ptr(h), _ptr(parts.rows),
+        _ptr(parts.places), rows, width, splits, top, y_stride, pad8(width), summand_stride, float(epsilon),
+        float(weight_offset), _code(dtype), _stream())
     _check(code, "b200_residual_norm")
     _count(rt)
     return h
@@ -248,7 +280,8 @@ def delta_inputs(projected: torch.Tensor, gates: torch.Tensor, conv: Tuple[torch
                  heads: int, kv_heads: int, dim: int, vdim: int, columns: Tuple[int, int, int, int],
                  decay_column: int, q_scale: float) -> "_lib.DeltaInputs":
     """The argument block of the gated delta rule's kernels: projections (columns of q, k, v and beta),
-    decay projections, convolution taps, and the ring of earlier inputs [slots, taps, channels]."""
+    decay projections, convolution taps, and the ring of earlier inputs [slots, taps, channels]. dt_bias has
+    heads * dim elements (a decay per key channel) or heads (one per head)."""
 
     _require_cuda(projected, gates, *conv, a_log, dt_bias, ring)
     _require_rows(projected, "the projection")
@@ -258,24 +291,26 @@ def delta_inputs(projected: torch.Tensor, gates: torch.Tensor, conv: Tuple[torch
         raise ValueError("the ring must hold `taps` inputs of every channel")
     if len({t.dtype for t in (projected, gates, *conv, a_log, dt_bias, ring)}) != 1:
         raise ValueError("projections, weights and ring must share one dtype")
+    if dt_bias.numel() not in (heads, heads * dim):
+        raise ValueError("decays are per head or per key channel")
     inputs = _lib.DeltaInputs(
         projected.data_ptr(), gates.data_ptr(), conv[0].data_ptr(), conv[1].data_ptr(), conv[2].data_ptr(),
         a_log.data_ptr(), dt_bias.data_ptr(), ring.data_ptr(), *batch.pointers(), heads, kv_heads, dim, vdim, taps,
-        *columns, decay_column, projected.stride(0), gates.stride(0), float(q_scale))
+        *columns, decay_column, projected.stride(0), gates.stride(0), dt_bias.numel() // heads, float(q_scale))
     inputs.tensors = (projected, gates, conv, a_log, dt_bias, ring, batch)
     return inputs
 
 
 def delta_prep(inputs: "_lib.DeltaInputs", batch: SequenceBatch, dtype: torch.dtype, device: torch.device):
     """fp32 operands of the gated delta rule: q, k [rows, kv_heads, dim], v [rows, heads, vdim],
-    beta [rows, heads] and log g [rows, heads, dim]."""
+    beta [rows, heads] and log g [rows, heads, dim or 1]."""
 
     rows = batch.rows
     q = torch.empty((rows, inputs.kv_heads, inputs.dim), dtype=torch.float32, device=device)
     k = torch.empty_like(q)
     v = torch.empty((rows, inputs.heads, inputs.vdim), dtype=torch.float32, device=device)
     beta = torch.empty((rows, inputs.heads), dtype=torch.float32, device=device)
-    decay = torch.empty((rows, inputs.heads, inputs.dim), dtype=torch.float32, device=device)
+    decay = torch.empty((rows, inputs.heads, inputs.decay_dim), dtype=torch.float32, device=device)
     rt = runtime(device)
     code = _lib.load().b200_delta_prep(byref(inputs), q.data_ptr(), k.data_ptr(), v.data_ptr(), beta.data_ptr(),
                                        decay.data_ptr(), rows, batch.sequences, batch.longest, _code(dtype), _stream())
@@ -296,7 +331,7 @@ def recurrence_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta: Opt
                     decay: torch.Tensor, state: torch.Tensor, batch: SequenceBatch) -> torch.Tensor:
     """Token by token recurrence over prepared fp32 operands; state [slots, heads, dim, row] is updated
     in place. beta None: retention with `decay` [heads]; else the delta rule, `decay` is log g
-    [rows, heads, dim]. Returns the read-out [rows, heads, vdim]."""
+    [rows, heads, dim or 1]. Returns the read-out [rows, heads, vdim]."""
 
     device = _require_cuda(q, k, v, beta, decay, state)
     rows, kv_heads, dim = q.shape
@@ -308,7 +343,8 @@ def recurrence_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta: Opt
     rt = runtime(device)
     code = _lib.load().b200_recurrence_scan(
         q.data_ptr(), k.data_ptr(), v.data_ptr(), _ptr(beta), decay.data_ptr(), state.data_ptr(), output.data_ptr(),
-        *batch.pointers(), batch.sequences, heads, kv_heads, dim, vdim, state.shape[3], _stream())
+        *batch.pointers(), batch.sequences, heads, kv_heads, dim, vdim, state.shape[3],
+        dim if beta is None else decay.shape[2], _stream())
     _check(code, "b200_recurrence_scan")
     _count(rt)
     return output
@@ -335,7 +371,7 @@ def recurrence_chunked(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta: 
     code = library.b200_recurrence_chunked(
         q.data_ptr(), k.data_ptr(), v.data_ptr(), _ptr(beta), decay.data_ptr(), state.data_ptr(), output.data_ptr(),
         *batch.pointers(), starts.data_ptr(), chunks, batch.sequences, heads, kv_heads, dim, vdim, state.shape[3],
-        _ptr(workspace), need, _stream())
+        dim if beta is None else decay.shape[2], _ptr(workspace), need, _stream())
     _check(code, "b200_recurrence_chunked")
     _count(rt, 2)
     return output
@@ -398,9 +434,10 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, sink: Optional[torch.
 
 
 def context_attention(query: torch.Tensor, key: torch.Tensor, value: torch.Tensor, sink: Optional[torch.Tensor],
-                      output: torch.Tensor, *, context: int, scale: float) -> None:
+                      output: torch.Tensor, *, context: int, scale: float, chunk: int = 0) -> None:
     """Causal attention of a portion on the tcgen05 prefill kernel: query B x H x T x D behind `context`
-    earlier positions, key / value B x Hkv x (context + T) x D (views), output memory B x T x H x D."""
+    earlier positions, key / value B x Hkv x (context + T) x D (views), output memory B x T x H x D. With
+    `chunk` a position sees only its own chunk of that many positions, counted from key 0."""
 
     device = _require_cuda(query, key, value, sink, output)
     batch, heads, tokens, dim = query.shape
@@ -411,10 +448,178 @@ def context_attention(query: torch.Tensor, key: torch.Tensor, value: torch.Tenso
     rt = runtime(device)
     code = _lib.load().b200_context_attention(
         query.data_ptr(), key.data_ptr(), value.data_ptr(), _ptr(sink), output.data_ptr(), batch, heads, key.shape[1],
-        tokens, context, dim, _lib.i64_array(query.stride()), _lib.i64_array(key.stride()),
+        tokens, context, chunk, dim, _lib.i64_array(query.stride()), _lib.i64_array(key.stride()),
         _lib.i64_array(value.stride()), float(scale), rt.status.data_ptr(), _stream())
     _check(code, "b200_context_attention")
     _count(rt)
+
+
+def attention_prep(projected: torch.Tensor, bias: Optional[torch.Tensor], q_weight: torch.Tensor,
+                   k_weight: Optional[torch.Tensor], turns: torch.Tensor, keys: Optional[torch.Tensor],
+                   values: Optional[torch.Tensor], batch: SequenceBatch, *, heads: int, kv_heads: int, dim: int,
+                   vdim: int, row_size: int, columns: Tuple[int, int, int], epsilon: float) -> torch.Tensor:
+    """Queries [rows, heads, row_size] of a stacked projection (columns: where q, k and v start), normed over
+    the whole projection and rotated; with k_weight, keys and values go to the caches [slots, capacity,
+    kv_heads, row_size]. projected: [rows, columns], or fp32 partials [splits, rows, columns] to which `bias`
+    is added. turns (fp64): turns per position of every rotated pair."""
+
+    device = _require_cuda(projected, bias, q_weight, k_weight, turns, keys, values)
+    partial = projected.ndim == 3
+    rows = projected.shape[-2]
+    if partial:
+        if projected.dtype != torch.float32 or not projected.is_contiguous():
+            raise ValueError("partial sums must be a contiguous fp32 [splits, rows, columns] tensor")
+    else:
+        _require_rows(projected, "the projection")
+        if projected.dtype != q_weight.dtype or bias is not None:
+            raise ValueError("a finished projection has the weights' dtype and its bias")
+    if turns.dtype != torch.float64 or q_weight.shape != (heads * dim,):
+        raise ValueError("turns are fp64, the query norm's weight spans the projection")
+    if k_weight is not None and (keys is None or values is None or keys.shape != values.shape or
+                                 keys.shape[2:] != (kv_heads, row_size) or keys.dtype != q_weight.dtype or
+                                 k_weight.shape != (kv_heads * dim,) or
+                                 not (keys.is_contiguous() and values.is_contiguous())):
+        raise ValueError("caches must be contiguous [slots, capacity, kv_heads, row_size] in the weights' dtype")
+    own = k_weight is not None
+    q = torch.empty((rows, heads, row_size), dtype=q_weight.dtype, device=device)
+    inputs = _lib.AttentionPrepInputs(
+        projected.data_ptr(), _ptr(bias), q_weight.data_ptr(), _ptr(k_weight), turns.data_ptr(), q.data_ptr(),
+        _ptr(keys) if own else None, _ptr(values) if own else None, *batch.pointers(), rows, heads, kv_heads, dim, vdim,
+        row_size, 2 * turns.shape[0], *columns, projected.stride(-2), projected.shape[0] if partial else 0,
+        keys.shape[1] if own else 0, float(epsilon))
+    rt = runtime(device)
+    _check(_lib.load().b200_attention_prep(byref(inputs), _code(q_weight.dtype), rt.status.data_ptr(), _stream()),
+           "b200_attention_prep")
+    _count(rt)
+    return q
+
+
+def _check_caches(q: torch.Tensor, keys: torch.Tensor, values: torch.Tensor) -> None:
+    if not (q.is_contiguous() and keys.is_contiguous() and values.is_contiguous()) or q.ndim != 3 or \
+            keys.shape != values.shape or keys.shape[3] != q.shape[2] or len({q.dtype, keys.dtype, values.dtype}) != 1 or \
+            q.shape[1] % keys.shape[2]:
+        raise ValueError("queries [rows, heads, size] and caches [slots, capacity, kv_heads, size] must fit")
+
+
+def slot_decode_attention(q: torch.Tensor, keys: torch.Tensor, values: torch.Tensor, batch: SequenceBatch, *,
+                          scale: float, chunk: int = 0) -> torch.Tensor:
+    """Attention of one token per sequence over its slot's cache (bf16, rows of 64 or 128), with `chunk`
+    over the token's own chunk of positions; returns [rows, heads, size]."""
+
+    device = _require_cuda(q, keys, values)
+    _check_caches(q, keys, values)
+    rows, heads, size = q.shape
+    if rows != batch.sequences or q.dtype != torch.bfloat16:
+        raise ValueError("decode attention takes one bf16 row per sequence")
+    context = batch.context_bound(keys.shape[1])
+    if chunk:
+        context = min(context, chunk)
+    output = torch.empty_like(q)
+    rt = runtime(device)
+    library = _lib.load()
+    need = int(library.b200_slot_decode_attention_workspace_bytes(rows, heads, keys.shape[2], size, context))
+    workspace = rt.workspace("decode_attention", need)
+    code = library.b200_slot_decode_attention(
+        q.data_ptr(), keys.data_ptr(), values.data_ptr(), output.data_ptr(), batch.slots.data_ptr(),
+        batch.bases.data_ptr(), rows, heads, keys.shape[2], size, keys.shape[0], keys.shape[1], chunk, context,
+        float(scale), _ptr(workspace), need, rt.status.data_ptr(), _stream())
+    _check(code, "b200_slot_decode_attention")
+    _count(rt)
+    return output
+
+
+def slot_attention(q: torch.Tensor, keys: torch.Tensor, values: torch.Tensor, batch: SequenceBatch, *,
+                   scale: float, chunk: int = 0) -> torch.Tensor:
+    """The same for any rows, sizes and dtype, on the CUDA cores."""
+
+    device = _require_cuda(q, keys, values)
+    _check_caches(q, keys, values)
+    rows, heads, size = q.shape
+    output = torch.empty_like(q)
+    rt = runtime(device)
+    code = _lib.load().b200_slot_attention(
+        q.data_ptr(), keys.data_ptr(), values.data_ptr(), output.data_ptr(), *batch.pointers(), rows, heads,
+        keys.shape[2], size, keys.shape[1], chunk, float(scale), _code(q.dtype), _stream())
+    _check(code, "b200_slot_attention")
+    _count(rt)
+    return output
+
+
+@dataclass
+class SortedRows:
+    """Rows of a step sorted by the experts they go to: `rows` [sorted rows, columns], the choices' scores,
+    the table of tiles (expert, rows held) and, for every choice of every row, its place."""
+
+    rows: torch.Tensor
+    scores: torch.Tensor
+    tiles: torch.Tensor
+    places: torch.Tensor
+    tile: int
+
+
+def expert_route(logits: torch.Tensor, counts: torch.Tensor, *, top: int):
+    """The `top` experts of every row and their sigmoid scores (both [rows, top]), and each choice's number
+    among its expert's. logits: fp32 [rows, >= experts] or split-K partials of them; counts: int32
+    [experts], zero before."""
+
+    device = _require_cuda(logits, counts)
+    if logits.dtype != torch.float32 or not logits.is_contiguous() or counts.dtype != torch.int32:
+        raise ValueError("the router's logits are contiguous fp32, the counts int32")
+    splits = logits.shape[0] if logits.ndim == 3 else 1
+    rows = logits.shape[-2]
+    chosen = torch.empty((rows, top), dtype=torch.int32, device=device)
+    scores = torch.empty((rows, top), dtype=torch.float32, device=device)
+    numbers = torch.empty_like(chosen)
+    rt = runtime(device)
+    code = _lib.load().b200_expert_route(logits.data_ptr(), chosen.data_ptr(), scores.data_ptr(), numbers.data_ptr(),
+                                         counts.data_ptr(), rows, counts.shape[0], top, splits, logits.shape[-1], _stream())
+    _check(code, "b200_expert_route")
+    _count(rt)
+    return chosen, scores, numbers
+
+
+def expert_place(h: torch.Tensor, chosen: torch.Tensor, scores: torch.Tensor, numbers: torch.Tensor,
+                 counts: torch.Tensor, *, tile: int) -> SortedRows:
+    """The rows of h sorted by expert, every expert starting at a multiple of `tile` rows."""
+
+    device = _require_cuda(h, chosen, scores, numbers, counts)
+    _require_rows(h, "the rows")
+    rows, top = chosen.shape
+    experts, columns = counts.shape[0], h.shape[1]
+    max_tiles = rows * top // tile + min(experts, rows * top)
+    placed = SortedRows(torch.empty((max_tiles * tile, columns), dtype=h.dtype, device=device),
+                        torch.empty(max_tiles * tile, dtype=torch.float32, device=device),
+                        torch.empty((max_tiles, 2), dtype=torch.int32, device=device), torch.empty_like(chosen), tile)
+    rt = runtime(device)
+    code = _lib.load().b200_expert_place(
+        h.data_ptr(), chosen.data_ptr(), scores.data_ptr(), numbers.data_ptr(), counts.data_ptr(),
+        placed.places.data_ptr(), placed.rows.data_ptr(), placed.scores.data_ptr(), placed.tiles.data_ptr(), rows,
+        experts, top, tile, max_tiles, columns, h.stride(0), _code(h.dtype), _stream())
+    _check(code, "b200_expert_place")
+    _count(rt)
+    return placed
+
+
+def grouped_linear(x: torch.Tensor, weight: torch.Tensor, placed: SortedRows, *, swiglu: bool = False,
+                   clear: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """out[r] = weight[expert of r] x[r] over sorted rows; weight [experts, n, k]. swiglu: the rows of a
+    weight alternate gate and up, and the result is silu(s gate) * (s up) with the row's score s. `clear`: an
+    int32 vector set to zero on the way."""
+
+    device = _require_cuda(x, weight, placed.tiles, clear)
+    experts, n, k = weight.shape
+    if not (x.is_contiguous() and weight.is_contiguous()) or x.shape != (placed.rows.shape[0], k) or x.dtype != weight.dtype:
+        raise ValueError("grouped_linear needs contiguous sorted rows and weights [experts, n, k] of one dtype")
+    output = torch.empty((x.shape[0], n // 2 if swiglu else n), dtype=x.dtype, device=device)
+    rt = runtime(device)
+    code = _lib.load().b200_grouped_linear(
+        x.data_ptr(), weight.data_ptr(), placed.tiles.data_ptr(), placed.scores.data_ptr() if swiglu else None,
+        output.data_ptr(), _ptr(clear), 0 if clear is None else clear.numel(), experts, placed.tile,
+        placed.tiles.shape[0], k, n, _lib.EPILOGUE_SWIGLU if swiglu else _lib.EPILOGUE_NONE, _code(x.dtype),
+        rt.status.data_ptr(), _stream())
+    _check(code, "b200_grouped_linear")
+    _count(rt)
+    return output
 
 
 def sequence_positions(lengths: torch.Tensor, slots: torch.Tensor, positions: torch.Tensor) -> None:

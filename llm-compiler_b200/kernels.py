@@ -916,7 +916,8 @@ def linear_partial_splits(m: int, k: int, n: int) -> int:
 def b200_linear_partial(tensor: torch.Tensor, weight: torch.Tensor,
                         partials: Optional[torch.Tensor] = None, *, row_squares: bool = False):
     """Decode-size projection without its epilogue: fp32 partial sums [splits, M, N] over K
-    slices, to be reduced by the operator that follows (b200_reduce_*). M <= 128, bf16.
+    slices, to be reduced by the operator that follows (b200_reduce_*). bf16; beyond 128 rows one
+    slice, an fp32 result.
     row_squares=True (M <= 128) also returns fp32 [splits, M]: the sum of squares of every input
     row over each K slice, for a consumer that applies an RMSNorm folded into this projection."""
 
@@ -930,7 +931,7 @@ def b200_linear_partial(tensor: torch.Tensor, weight: torch.Tensor,
     m, k = tensor.shape
     n = weight.shape[0]
     library = _lib.load()
-    splits = int(library.b200_linear_partial_splits(m, k, n))
+    splits = int(library.b200_linear_partial_splits(m, k, n)) if m <= 128 else 1
     if partials is None:
         partials = torch.empty((splits, m, n), dtype=torch.float32, device=device)
     elif partials.shape != (splits, m, n) or partials.dtype != torch.float32 or \

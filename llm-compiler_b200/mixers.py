@@ -1,7 +1,8 @@
-"""Sequence mixers of hybrid decoder layers on the sm_100a kernels: retention, latent attention and the
-gated delta rule with a decay per key channel. Each takes its sizes and constants from a spec, packs its
-weights once, says what state a sequence keeps, and maps normed rows h to the sublayer's result for any
-mix of portions and decoded tokens.
+"""The sublayers of hybrid decoder layers on the sm_100a kernels: the mixers (retention, latent attention,
+attention over cached keys and values, the gated delta rule with a decay per key channel or per head) and
+the feed-forwards (gated MLP, mixture of experts). Each takes its sizes and constants from a spec, packs its
+weights once, says what state a sequence keeps, and maps rows h to the sublayer's result for any mix of
+portions and decoded tokens.
 
 Packing: all projections of h are one stacked matrix; every operand starts at a multiple of 8 columns,
 and extents are padded with zero rows / columns to multiples of 8, so that the 16-bit GEMMs take any size.
@@ -9,13 +10,15 @@ and extents are padded with zero rows / columns to multiples of 8, so that the 1
 
 from __future__ import annotations
 
-from typing import Dict, List, Optional, Sequence, Tuple
+import math
+from dataclasses import dataclass
+from typing import Callable, Dict, List, Optional, Sequence, Tuple
 
 import torch
 
 from . import hybrid_kernels as hk
 from . import kernels
-from .hybrid_kernels import SequenceBatch, pad8
+from .hybrid_kernels import SequenceBatch, Summands, pad8
 
 ABSORBED_ROWS = 16  # longest portion that attends in the latent space (beyond: expanded keys and values)
 PARTIAL_ROWS = 128  # rows up to which a projection in front of a residual leaves split-K partials
@@ -84,7 +87,9 @@ class Mixer:
     def state_spec(self, capacity: int) -> Dict[str, tuple]:
         return {}
 
-    def __call__(self, h: torch.Tensor, batch: SequenceBatch, state: Dict[str, torch.Tensor]) -> torch.Tensor:
+    def __call__(self, h: torch.Tensor, batch: SequenceBatch, state: Dict[str, torch.Tensor]):
+        """A tensor or Summands: what residual_norm takes."""
+
         raise NotImplementedError
 
 
@@ -122,20 +127,18 @@ class Retention(Mixer):
         return project_out(mixed, self.w_out)
 
 
-class ChannelDelta(Mixer):
-    """Gated delta rule: short convolutions on q, k, v, unit q and k, one decay per head and key
-    channel, a sigmoid gate on the normed read-out."""
+class GatedDelta(Mixer):
+    """Gated delta rule: short convolutions on q, k, v, unit q and k, decays from a_log, dt_bias and a
+    projection of h, and a gate on the normed read-out. A subclass packs the projections and says where the
+    decays (`decay_column`) and the gate (`gate_column`) stand in the matrix that `_gates` returns."""
 
-    def __init__(self, weights: Dict[str, torch.Tensor], *, width: int, heads: int, kv_heads: int, dim: int,
-                 vdim: int, epsilon: float) -> None:
+    gate_kind: str
+    decay_column: int
+    gate_column: int
+
+    def __init__(self, weights: Dict[str, torch.Tensor], *, heads: int, kv_heads: int, dim: int, vdim: int,
+                 width: int, epsilon: float) -> None:
         self.heads, self.kv_heads, self.dim, self.vdim, self.epsilon = heads, kv_heads, dim, vdim, epsilon
-        self.w_in, offsets = stack_projections(
-            [weights[name] for name in ("q", "k", "v", "b", "a1", "g1")], pad8(width))
-        self.columns = tuple(offsets[:4])
-        self.low_column = offsets[4]  # a1 and g1 side by side: the input of the two up projections
-        low = self.w_in.shape[0] - self.low_column
-        self.w_gates, (self.decay_column, self.gate_column) = block_diagonal(
-            [(weights["a2"], 0), (weights["g2"], offsets[5] - offsets[4])], low)
         self.w_out = pad_matrix(weights["o"], pad8(width), pad8(heads * vdim))
         self.conv = tuple(weights[name].contiguous() for name in ("q.conv", "k.conv", "v.conv"))
         self.a_log, self.dt_bias, self.norm = weights["A_log"], weights["dt_bias"], weights["norm"]
@@ -146,23 +149,135 @@ class ChannelDelta(Mixer):
         return {"state": ((self.heads, self.dim, (self.vdim + 3) // 4 * 4), torch.float32),
                 "ring": ((self.taps, 2 * self.kv_heads * self.dim + self.heads * self.vdim), self.w_in.dtype)}
 
+    def _gates(self, projected: torch.Tensor) -> torch.Tensor:
+        raise NotImplementedError
+
     def __call__(self, h, batch, state):
         projected = kernels.b200_linear(h, self.w_in)
-        gates = kernels.b200_linear(projected[:, self.low_column:], self.w_gates)
+        gates = self._gates(projected)
         inputs = hk.delta_inputs(projected, gates, self.conv, self.a_log, self.dt_bias, state["ring"], batch,
                                  heads=self.heads, kv_heads=self.kv_heads, dim=self.dim, vdim=self.vdim,
                                  columns=self.columns, decay_column=self.decay_column, q_scale=self.q_scale)
         gate = gates[:, self.gate_column:]
         mixed = None
         if batch.decode:
-            mixed = hk.recurrence_step(inputs, state["state"], gate, self.norm, batch.sequences, kind="sigmoid",
+            mixed = hk.recurrence_step(inputs, state["state"], gate, self.norm, batch.sequences, kind=self.gate_kind,
                                        epsilon=self.epsilon)
         if mixed is None:
             q, k, v, beta, log_decay = hk.delta_prep(inputs, batch, h.dtype, h.device)
             read_out = hk.recurrence(q, k, v, beta, log_decay, state["state"], batch, h.dtype)
             hk.conv_tail(inputs, batch.sequences, h.dtype, h.device)
-            mixed = hk.gated_head_norm(read_out, self.norm, gate, kind="sigmoid", epsilon=self.epsilon)
+            mixed = hk.gated_head_norm(read_out, self.norm, gate, kind=self.gate_kind, epsilon=self.epsilon)
         return project_out(mixed, self.w_out)
+
+
+class ChannelDelta(GatedDelta):
+    """One decay per head and key channel, decays and a sigmoid gate from low-rank projections."""
+
+    gate_kind = "sigmoid"
+
+    def __init__(self, weights: Dict[str, torch.Tensor], *, width: int, **sizes) -> None:
+        super().__init__(weights, width=width, **sizes)
+        self.w_in, offsets = stack_projections(
+            [weights[name] for name in ("q", "k", "v", "b", "a1", "g1")], pad8(width))
+        self.columns = tuple(offsets[:4])
+        self.low_column = offsets[4]  # a1 and g1 side by side: the input of the two up projections
+        low = self.w_in.shape[0] - self.low_column
+        self.w_gates, (self.decay_column, self.gate_column) = block_diagonal(
+            [(weights["a2"], 0), (weights["g2"], offsets[5] - offsets[4])], low)
+
+    def _gates(self, projected):
+        return kernels.b200_linear(projected[:, self.low_column:], self.w_gates)
+
+
+class HeadDelta(GatedDelta):
+    """One decay per head, a full silu gate."""
+
+    gate_kind = "silu"
+
+    def __init__(self, weights: Dict[str, torch.Tensor], *, width: int, **sizes) -> None:
+        super().__init__(weights, width=width, **sizes)
+        self.w_in, offsets = stack_projections(
+            [weights[name] for name in ("q", "k", "v", "b", "a", "g")], pad8(width))
+        self.columns = tuple(offsets[:4])
+        self.decay_column, self.gate_column = offsets[4:]
+
+    def _gates(self, projected):
+        return projected
+
+
+class Attention(Mixer):
+    """Grouped softmax attention over cached keys and values, with biases, RMS norms over the whole query and
+    the whole key projection and a rotation of the first dimensions of every head; with `chunk` a position
+    sees only its own chunk of that many positions. `kv_from` reads the caches that an earlier layer keeps."""
+
+    def __init__(self, weights: Dict[str, torch.Tensor], *, width: int, heads: int, kv_heads: int, dim: int,
+                 vdim: int, scale: float, rot_dims: int, rot_base: float, epsilon: float, chunk: Optional[int] = None,
+                 kv_from: Optional[int] = None) -> None:
+        self.heads, self.kv_heads, self.dim, self.vdim = heads, kv_heads, dim, vdim
+        self.scale, self.epsilon, self.chunk, self.shared_state = scale, epsilon, chunk or 0, kv_from
+        names = ("q", "k", "v") if kv_from is None else ("q",)
+        self.w_in, offsets = stack_projections([weights[name] for name in names], pad8(width))
+        self.columns = tuple(offsets) if kv_from is None else (0, 0, 0)
+        self.bias = torch.zeros(self.w_in.shape[0], dtype=self.w_in.dtype, device=self.w_in.device)
+        for name, offset in zip(names, offsets):
+            self.bias[offset:offset + weights[name].shape[0]].copy_(weights[name + ".b"])
+        self.q_norm, self.k_norm = weights["q.norm"], weights["k.norm"] if kv_from is None else None
+        # 16-bit models run on the tensor-core kernels where a head fits them: q, k and v of a head
+        # zero-padded to one size of 64 or 128
+        self.dense = self.w_in.dtype == torch.bfloat16 and max(dim, vdim) <= 128 and scale > 0
+        self.size = (64 if max(dim, vdim) <= 64 else 128) if self.dense else pad8(max(dim, vdim))
+        self.w_out = pad_matrix(pad_heads(weights["o"].t().contiguous(), heads, self.size).t(), pad8(width),
+                                heads * self.size)
+        self.out_bias = weights["o.b"].contiguous()
+        self.turns = torch.tensor([rot_base ** (-2.0 * i / rot_dims) / (2.0 * math.pi) for i in range(rot_dims // 2)],
+                                  dtype=torch.float64, device=self.w_in.device)
+
+    def state_spec(self, capacity):
+        if self.shared_state is not None:
+            return {}
+        row = (capacity, self.kv_heads, self.size)
+        return {"keys": (row, self.w_in.dtype), "values": (row, self.w_in.dtype)}
+
+    def __call__(self, h, batch, state):
+        rows = h.shape[0]
+        keys, values = state["keys"], state["values"]
+        partial = h.dtype == torch.bfloat16 and rows <= PARTIAL_ROWS
+        projected = kernels.b200_linear_partial(h, self.w_in) if partial else kernels.b200_linear(h, self.w_in, self.bias)
+        q = hk.attention_prep(projected, self.bias if partial else None, self.q_norm, self.k_norm, self.turns, keys,
+                              values, batch, heads=self.heads, kv_heads=self.kv_heads, dim=self.dim, vdim=self.vdim,
+                              row_size=self.size, columns=self.columns, epsilon=self.epsilon)
+        if not self.dense:
+            mixed = hk.slot_attention(q, keys, values, batch, scale=self.scale, chunk=self.chunk)
+        elif batch.decode:
+            mixed = hk.slot_decode_attention(q, keys, values, batch, scale=self.scale, chunk=self.chunk)
+        else:
+            mixed = self._attend_portions(q, keys, values, batch)
+        return Summands(project_out(mixed.view(rows, self.heads * self.size), self.w_out), self.out_bias)
+
+    def _attend_portions(self, q, keys, values, batch):
+        """The prefill kernel over the caches: one launch for equal whole prompts in neighbouring slots, else
+        one per sequence, from the first key of the chunk that the portion starts in."""
+
+        heads, size = q.shape[1:]
+        output = torch.empty_like(q)
+        slots = batch.slots_host
+        if batch.uniform_start and slots == list(range(slots[0], slots[0] + len(slots))):
+            groups = [(0, slots[0], len(slots), batch.counts[0], 0)]
+        else:
+            groups, first = [], 0
+            for slot, base, count in zip(slots, batch.bases_host, batch.counts):
+                groups.append((first, slot, 1, count, base))
+                first += count
+        for first, slot, sequences, tokens, base in groups:
+            start = base // self.chunk * self.chunk if self.chunk else 0
+            part = slice(first, first + sequences * tokens)
+            seen = (slice(slot, slot + sequences), slice(start, base + tokens))
+            hk.context_attention(q[part].view(sequences, tokens, heads, size).transpose(1, 2),
+                                 keys[seen].transpose(1, 2), values[seen].transpose(1, 2), None,
+                                 output[part].view(sequences, tokens, heads, size), context=base - start,
+                                 scale=self.scale, chunk=self.chunk)
+        return output
 
 
 class LatentAttention(Mixer):
@@ -255,3 +370,52 @@ class GatedMlp:
 
     def __call__(self, h: torch.Tensor) -> torch.Tensor:
         return project_out(kernels.b200_linear(h, self.w_in, epilogue="swiglu"), self.w_out)
+
+
+class ExpertMlp:
+    """Mixture of experts: sigmoid scores of a router, the `top` best experts per token, every expert a gated
+    MLP on the token scaled by its score; a shared gated MLP (None: none) runs for every token."""
+
+    def __init__(self, router: torch.Tensor, experts: Sequence[Dict[str, torch.Tensor]], *, width: int, top: int,
+                 shared: Optional["GatedMlp"] = None) -> None:
+        self.top, self.shared, self.experts = top, shared, len(experts)
+        self.w_router = pad_matrix(router, pad8(len(experts)), pad8(width))
+        ff = pad8(experts[0]["gate"].shape[0])
+        like = dict(dtype=router.dtype, device=router.device)
+        self.w_in = torch.empty((len(experts), 2 * ff, pad8(width)), **like)
+        self.w_out = torch.empty((len(experts), pad8(width), ff), **like)
+        for i, expert in enumerate(experts):
+            self.w_in[i].copy_(kernels.interleave_gate_up(pad_matrix(expert["gate"], ff, pad8(width)),
+                                                          pad_matrix(expert["up"], ff, pad8(width))))
+            self.w_out[i].copy_(pad_matrix(expert["down"], pad8(width), ff))
+        self.counts = torch.zeros(len(experts), dtype=torch.int32, device=router.device)  # zero between calls
+
+    def tile_of(self, rows: int) -> int:
+        """Rows of a tile: near the average number of rows an expert gets."""
+
+        average = rows * self.top / self.experts
+        return next((tile for tile, most in ((16, 12), (32, 24), (64, 56), (128, 160)) if average <= most), 256)
+
+    def __call__(self, h: torch.Tensor) -> Summands:
+        if h.dtype == torch.bfloat16:  # (fp32 results either way)
+            logits = kernels.b200_linear_partial(h, self.w_router)
+        else:
+            logits = kernels.b200_linear(h, self.w_router)
+        placed = hk.expert_place(h, *hk.expert_route(logits, self.counts, top=self.top), self.counts,
+                                 tile=self.tile_of(h.shape[0]))
+        inner = hk.grouped_linear(placed.rows, self.w_in, placed, swiglu=True, clear=self.counts)
+        return Summands(None if self.shared is None else self.shared(h), None,
+                        hk.grouped_linear(inner, self.w_out, placed), placed.places)
+
+
+@dataclass
+class HybridLayer:
+    """What HybridEngine runs: a mixer and a feed-forward (or none), a norm behind each and, in designs whose
+    sublayers do not read the residual itself, one in front of each."""
+
+    mixer: Mixer
+    norm_in: Optional[torch.Tensor]
+    norm_out: torch.Tensor
+    mlp: Optional[Callable[[torch.Tensor], object]] = None
+    mlp_norm_in: Optional[torch.Tensor] = None
+    mlp_norm_out: Optional[torch.Tensor] = None

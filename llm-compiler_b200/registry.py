@@ -61,11 +61,13 @@ def load_model(folder: str | Path, *, dtype: torch.dtype = torch.bfloat16, batch
 
 
 def _register_builtin() -> None:
-    from . import bazirax, qwen2
+    from . import bazirax, lozanex, qwen2
     from .engine import Qwen2Engine
     from .hybrid_engine import HybridEngine
 
     register(ModelEntry(bazirax.ARCHITECTURE, bazirax.BaziraxConfig.from_dict, lambda config, stored: stored,
+                        HybridEngine, portions=True))
+    register(ModelEntry(lozanex.ARCHITECTURE, lozanex.LozanexConfig.from_dict, lambda config, stored: stored,
                         HybridEngine, portions=True))
     register(ModelEntry("Qwen2ForCausalLM", qwen2.config_from_dict, qwen2.weights_from_checkpoint, Qwen2Engine,
                         dtypes=(torch.float32, torch.bfloat16, torch.float16)))
