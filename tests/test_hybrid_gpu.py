@@ -23,57 +23,11 @@ from llm_compiler_b200.registry import load_model
 from llm_compiler_b200.safetensors_io import save_safetensors
 from llm_compiler_b200.scheduler import RequestScheduler
 from llm_compiler_b200.trace import replay
+from hybrid_helpers import (BOTH, CUTS, EPS, MODEL_TOLERANCE, TOLERANCE, batch_of, close, cuda, double, random_rows,
+                            run_cut, run_mixer, tokens_of)
 from oracle import hybrid_model as oracle
 
 pytestmark = pytest.mark.gpu
-EPS = 1e-5
-TOLERANCE = {torch.float32: 3e-5, torch.bfloat16: 3e-2}
-
-
-def batch_of(portions):
-    """SequenceBatch of (slot, first position, count) portions."""
-    counts = [count for _, _, count in portions]
-    starts = [sum(counts[:i]) for i in range(len(counts) + 1)]
-    vector = lambda values: torch.tensor(values, dtype=torch.int32, device="cuda")
-    return hk.SequenceBatch(starts[-1], len(portions),
-                            vector([i for i, c in enumerate(counts) for _ in range(c)]), vector(starts),
-                            vector([slot for slot, _, _ in portions]), vector([base for _, base, _ in portions]),
-                            counts, [base for _, base, _ in portions], [slot for slot, _, _ in portions])
-
-
-def close(actual, expected, dtype, factor=1.0):
-    """Root mean square error per row, relative to the largest row."""
-    actual, expected = actual.double().cpu(), expected.double()
-    error = (actual - expected).pow(2).mean(-1).sqrt()
-    scale = expected.pow(2).mean(-1).sqrt().max()
-    worst = float((error / scale).max())
-    assert worst <= TOLERANCE[dtype] * factor, f"relative error {worst} at row {int(error.argmax())}"
-
-
-def summed(y):
-    return y.sum(0) if y.ndim == 3 else y.float()
-
-
-def run_mixer(mixer, h, cuts, *, slot=1, slots=3, capacity=512, state=None, garbage=True):
-    """The mixer's rows for one sequence, run in portions of the given sizes."""
-    if state is None:
-        state = {name: torch.zeros((slots, *shape), dtype=dtype, device="cuda")
-                 for name, (shape, dtype) in mixer.state_spec(capacity).items()}
-        if garbage:  # what a former sequence left: nothing of it may be read
-            for tensor in state.values():
-                tensor.fill_(3.0)
-    rows, first = [], 0
-    for cut in cuts:
-        piece = torch.zeros((cut, hk.pad8(h.shape[1])), dtype=h.dtype, device="cuda")
-        piece[:, :h.shape[1]] = h[first:first + cut].cuda()
-        rows.append(summed(mixer(piece, batch_of([(slot, first, cut)]), state))[:, :h.shape[1]])
-        first += cut
-    kernels.runtime().check_status()
-    return torch.cat(rows)
-
-
-def random_rows(tokens, width, dtype, seed):
-    return torch.randn(tokens, width, generator=torch.Generator().manual_seed(seed)).to(dtype)
 
 
 def mixer_weights(kind, spec, width, dtype, *, gate_rank=12, seed=0):
@@ -81,18 +35,6 @@ def mixer_weights(kind, spec, width, dtype, *, gate_rank=12, seed=0):
                                    layers=(bazirax.LayerSpec(kind, spec, None),))
     weights = bazirax.make_weights(config, seed=seed, dtype=dtype, gate_rank=gate_rank)
     return {name[len("l0.mix."):]: w for name, w in weights.items() if name.startswith("l0.mix.")}
-
-
-def cuda(weights):
-    return {name: w.cuda() for name, w in weights.items()}
-
-
-def double(weights):
-    return {name: w.double() for name, w in weights.items()}
-
-
-CUTS = [[150], [1] * 150, [2, 3, 61, 64, 20], [63, 2, 65, 2, 18], [128, 22], [7, 1, 1, 1, 90, 50]]
-BOTH = pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16], ids=["fp32", "bf16"])
 
 
 # ------------------------------------------------------------------------------ norms ----
@@ -427,25 +369,6 @@ def small_config(variant=0):
 def model(config, dtype, *, batch=3, capacity=256, seed=0):
     weights = bazirax.make_weights(config, seed=seed, dtype=dtype, gate_rank=12)
     return HybridEngine(config, cuda(weights), batch=batch, capacity=capacity), weights
-
-
-def tokens_of(config, count, seed):
-    return torch.randint(0, config.vocab_size, (count,), generator=torch.Generator().manual_seed(seed)).tolist()
-
-
-def run_cut(engine, tokens, cuts):
-    slot, rows, first = engine.open(), [], 0
-    for cut in cuts:
-        rows.append(engine.forward([(slot, tokens[first:first + cut])], [list(range(cut))]))
-        first += cut
-    engine.state.check()
-    engine.close(slot)
-    return torch.cat(rows)
-
-
-# A single row of a bf16 model may sit where a small read-out is normed to size one and its rounding
-# errors with it (the same row passes in fp32): the worst row gets more room than a mechanism alone.
-MODEL_TOLERANCE = {torch.float32: 1.0, torch.bfloat16: 5.0}
 
 
 def check_model(config, dtype, lengths, cut_lists):

@@ -119,3 +119,43 @@ def test_latent_attention_wait_timeout_then_recovery():
         weights = torch.softmax(torch.einsum("hr,kr->hk", q[i].float(), cache[i, :n].float()) * 0.05, -1)
         close(out[i], weights @ cache[i, :n].float())
     kernels.runtime().check_status()
+
+
+@pytest.mark.parametrize("tile", [16, 128])
+def test_grouped_linear_wait_timeout_then_recovery(tile):
+    from llm_compiler_b200 import hybrid_kernels as hk
+
+    g = torch.Generator().manual_seed(tile)
+    x = torch.randn(40, 136, generator=g).bfloat16()
+    w = (0.1 * torch.randn(3, 400, 136, generator=g)).bfloat16()
+    chosen = torch.arange(40, dtype=torch.int32).remainder(3)[:, None]
+    numbers = (torch.arange(40, dtype=torch.int32) // 3)[:, None].contiguous()
+    counts = torch.bincount(chosen[:, 0], minlength=3).to(torch.int32)
+    placed = hk.expert_place(x.cuda(), chosen.cuda(), torch.ones(40, 1).cuda(), numbers.cuda(), counts.cuda(), tile=tile)
+    for _ in range(3):
+        with waits_that_run_out():
+            hk.grouped_linear(placed.rows, w.cuda(), placed)
+        expect_timeout()
+    out = hk.grouped_linear(placed.rows, w.cuda(), placed)[placed.places[:, 0].long()]
+    close(out, torch.einsum("rnk,rk->rn", w.float()[chosen[:, 0].long()], x.float()))
+    kernels.runtime().check_status()
+
+
+def test_slot_attention_wait_timeout_then_recovery():
+    from llm_compiler_b200 import hybrid_kernels as hk
+
+    g = torch.Generator().manual_seed(11)
+    q = torch.randn(2, 4, 64, generator=g).bfloat16()
+    keys, values = torch.randn(2, 3, 700, 2, 64, generator=g).bfloat16()
+    vector = lambda v: torch.tensor(v, dtype=torch.int32, device="cuda")
+    batch = hk.SequenceBatch(2, 2, vector([0, 1]), vector([0, 1, 2]), vector([2, 0]), vector([650, 310]))
+    call = lambda: hk.slot_decode_attention(q.cuda(), keys.cuda(), values.cuda(), batch, scale=0.125, chunk=300)
+    with waits_that_run_out():
+        call()
+    expect_timeout()
+    out = call()
+    for i, (slot, first, last) in enumerate(((2, 600, 650), (0, 300, 310))):
+        k, v = (t[slot, first:last + 1].float().repeat_interleave(2, 1) for t in (keys, values))
+        weights = torch.softmax(torch.einsum("hd,khd->hk", q[i].float(), k) * 0.125, -1)
+        close(out[i], torch.einsum("hk,khd->hd", weights, v))
+    kernels.runtime().check_status()
