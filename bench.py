@@ -87,11 +87,12 @@ def parse_args():
     parser.add_argument("--cpu-sample-batch", type=int, default=8)
     parser.add_argument("--skip-cpu-baseline", action="store_true")
     parser.add_argument("--skip-parity", action="store_true")
-    parser.add_argument("--model", default="qwen2-0.5b", choices=["qwen2-0.5b", "qwen2-7b", "bazirax-0.5b", "bazirax-1.5b",
-                                                                        "bazirax-7b"],
-                        help="architecture (the headline metric is quoted on qwen2-0.5b); bazirax-*: prefill and "
-                             "decode of a few Bazirax layers of that size beside as many Qwen2 layers of equal "
-                             "width, with the roofline fraction of every kernel (bench_hybrid.py)")
+    parser.add_argument("--model", default="qwen2-0.5b",
+                        choices=["qwen2-0.5b", "qwen2-7b", *(f"{design}-{size}" for design in ("bazirax", "lozanex")
+                                                             for size in ("0.5b", "1.5b", "7b"))],
+                        help="architecture (the headline metric is quoted on qwen2-0.5b); bazirax-* and lozanex-*: "
+                             "prefill and decode of a few layers of that design and size beside as many Qwen2 layers "
+                             "of equal width, with the roofline fraction of every kernel (bench_hybrid.py)")
     parser.add_argument("--context-min", type=int, default=-1,
                         help="with --context-source synthetic: per-sequence contexts uniform in "
                              "[context-min, context] instead of all at --context")
@@ -786,7 +787,7 @@ def main():
     sys.stdout.flush()
     RESULT_STREAM = os.fdopen(os.dup(1), "w")
     os.dup2(2, 1)
-    if args.model.startswith("bazirax"):
+    if args.model.startswith(("bazirax", "lozanex")):
         import bench_hybrid
 
         with ClockSampler(0) as clocks:

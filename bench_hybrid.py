@@ -1,9 +1,11 @@
-"""Bazirax layers beside Qwen2 layers of equal width: `python bench.py --model bazirax-0.5b` (or -1.5b, -7b).
+"""Layers of a hybrid design beside Qwen2 layers of equal width: `python bench.py --model bazirax-0.5b` or
+`lozanex-0.5b` (also -1.5b, -7b).
 
-Both models have the same width, feed-forward, head count and size, layer count and vocabulary, random bf16
-weights; decode is a captured step of `--batch` sequences at `--context` tokens, prefill whole prompts. Then
-every kernel of the new layers alone, over copies of its data that together exceed L2, against the measured
-copy bandwidth and GEMM throughput, with the like kernels of the Qwen2 layers. CUDA events throughout."""
+Both models have the same width, feed-forward (of a mixture of experts: what a token uses of it), head count
+and size, layer count and vocabulary, random bf16 weights; decode is a captured step of `--batch` sequences at
+`--context` tokens, prefill whole prompts. Then every kernel of the new layers alone, over copies of its data
+that together exceed L2, against the measured copy bandwidth and GEMM throughput, with the like kernels of
+the existing layers. CUDA events throughout."""
 
 from __future__ import annotations
 
@@ -18,6 +20,10 @@ SIZES = {
     "bazirax-1.5b": dict(width=2048, ff=8192, heads=16, dim=128, kv_heads=2, q_rank=768, kv_rank=512),
     "bazirax-7b": dict(width=3584, ff=18944, heads=28, dim=128, kv_heads=4, q_rank=1536, kv_rank=512),
 }
+# `active` of `experts` experts and a shared one per token, which together are as wide as the dense feed-forward
+EXPERTS = {"0.5b": dict(experts=16, active=2), "1.5b": dict(experts=32, active=4), "7b": dict(experts=32, active=4)}
+for _name, _experts in EXPERTS.items():
+    SIZES["lozanex-" + _name] = {**SIZES["bazirax-" + _name], **_experts}
 VOCAB = 32768
 PEAKS = Path(__file__).resolve().parent / "MEASURED_PEAKS.json"
 
@@ -34,6 +40,21 @@ def bazirax_config(size):
     layers = [bazirax.LayerSpec(kind, spec, size["ff"]) for kind, spec in kinds * 2]
     layers[5] = bazirax.LayerSpec("latent_attention", dict(latent, kv_from=2), size["ff"])
     return bazirax.BaziraxConfig(vocab_size=VOCAB, hidden_size=size["width"], norm_eps=1e-5, layers=tuple(layers))
+
+
+def lozanex_config(size):
+    from llm_compiler_b200 import lozanex
+
+    heads, dim = size["heads"], size["dim"]
+    delta = dict(heads=heads, kv_heads=heads, dim=dim, vdim=dim, conv=4)
+    attention = dict(heads=heads, kv_heads=size["kv_heads"], dim=dim, vdim=dim, scale=dim ** -0.5,
+                     rot=dict(base=1e6, dims=dim), mask=dict(size=8192))
+    mlp = dict(kind="moe", expert=dict(ff=size["ff"] // 2 // size["active"]),
+               router=dict(experts=size["experts"], top=size["active"]), shared=dict(ff=size["ff"] // 2))
+    layers = [lozanex.LayerSpec(*spec, mlp) for spec in (
+        ("delta", delta), ("attention", attention), ("delta", delta), ("delta", delta),
+        ("attention", dict(attention, kv_from=1)), ("delta", delta))]
+    return lozanex.LozanexConfig(vocab_size=VOCAB, hidden_size=size["width"], norm_eps=1e-5, layers=tuple(layers))
 
 
 def qwen_config(size, layers):
@@ -87,7 +108,7 @@ def decode_ms(engine, context, batch):
     return time
 
 
-def kernel_table(engine, config, size, context, batch, hbm_gbs, tflops):
+def bazirax_kernels(engine, config, size, context, batch, hbm_gbs, tflops):
     """Every kernel of the hybrid layers alone. bytes: what must cross HBM; flops: matrix products."""
     from llm_compiler_b200 import hybrid_kernels as hk, kernels
 
@@ -202,26 +223,183 @@ def kernel_table(engine, config, size, context, batch, hbm_gbs, tflops):
     return rows
 
 
+def lozanex_kernels(engine, config, size, context, batch, hbm_gbs, tflops):
+    """Every kernel of the Lozanex layers alone, and the like kernels of Bazirax and Qwen2 layers on the same
+    shapes. bytes: what must cross HBM; flops: matrix products."""
+    from llm_compiler_b200 import hybrid_kernels as hk, kernels
+
+    rows = {}
+
+    def record(name, calls, nbytes=0, flops=0):
+        ms = graph_milliseconds(calls)
+        floor = max(nbytes / (hbm_gbs * 1e6), flops / (tflops * 1e9))
+        rows[name] = {"us": round(ms * 1e3, 2), "of_roofline": round(floor / ms, 3),
+                      "bound": "memory" if nbytes / (hbm_gbs * 1e6) >= flops / (tflops * 1e9) else "tensor"}
+
+    device = engine.device
+    heads, kv_heads, dim, width = size["heads"], size["kv_heads"], size["dim"], size["width"]
+    delta, attention, mlp = engine.layers[0].mixer, engine.layers[1].mixer, engine.layers[0].mlp
+    experts, top = size["experts"], size["active"]
+    ff, shared_ff = mlp.w_out.shape[2], mlp.shared.w_out.shape[1]
+    rand = lambda *shape: torch.randn(*shape, device=device)
+    bf16 = lambda *shape: (0.5 * rand(*shape)).to(torch.bfloat16)
+    vector = lambda values: torch.tensor(values, dtype=torch.int32, device=device)
+    copies_of = lambda nbytes: max(2, int(3e8 / nbytes))
+
+    def delta_block(projected, ring, part):
+        return hk.delta_inputs(projected, projected, delta.conv, delta.a_log, delta.dt_bias, ring, part, heads=heads,
+                               kv_heads=heads, dim=dim, vdim=dim, columns=delta.columns,
+                               decay_column=delta.decay_column, q_scale=delta.q_scale)
+
+    def prepare(projected, bias, keys, values, part):
+        return hk.attention_prep(projected, bias, attention.q_norm, attention.k_norm, attention.turns, keys, values, part,
+                                 heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, row_size=dim,
+                                 columns=attention.columns, epsilon=1e-5)
+
+    def expert_rows(name, n):
+        """The mixture of experts on n rows, launch by launch, and dense projections of the same size."""
+        h = bf16(n, width)
+        logits = kernels.b200_linear_partial(h, mlp.w_router)
+        used = min(experts, n * top)
+        weight_sets = copies_of(mlp.w_in.numel() * 2)
+        w_in = [mlp.w_in] + [mlp.w_in.clone() for _ in range(weight_sets - 1)]
+        w_out = [mlp.w_out] + [mlp.w_out.clone() for _ in range(weight_sets - 1)]
+        counts = torch.zeros_like(mlp.counts)
+        routed = hk.expert_route(logits, counts, top=top)
+        placed = hk.expert_place(h, *routed, counts, tile=mlp.tile_of(n))
+        inner = hk.grouped_linear(placed.rows, mlp.w_in, placed, swiglu=True)
+        record(name + "router logits", [lambda: kernels.b200_linear_partial(h, mlp.w_router)] * 8,
+               (h.numel() + mlp.w_router.numel()) * 2 + n * mlp.w_router.shape[0] * 4, 2 * n * mlp.w_router.numel())
+        record(name + "routing", [lambda: hk.expert_route(logits, torch.zeros_like(counts), top=top)] * 8, logits.numel() * 4)
+        record(name + "sorting rows", [lambda: hk.expert_place(h, *routed, counts, tile=placed.tile)] * 8,
+               h.numel() * 2 * (1 + top))
+        record(name + "experts, gate and up", [lambda w=w: hk.grouped_linear(placed.rows, w, placed, swiglu=True) for w in w_in],
+               (used * 2 * ff * width + n * top * (width + ff)) * 2, 4 * n * top * ff * width)
+        record(name + "experts, down", [lambda w=w: hk.grouped_linear(inner, w, placed) for w in w_out],
+               (used * ff * width + n * top * (width + ff)) * 2, 2 * n * top * ff * width)
+        dense = bf16(top * n, width)
+        sets = copies_of(4 * ff * width)
+        w_dense = [bf16(2 * ff, width) for _ in range(sets)]
+        record(name + f"dense gate and up, {top * n} rows (Qwen2's)",
+               [lambda w=w: kernels.b200_linear(dense, w, epilogue="swiglu") for w in w_dense],
+               (2 * ff * width + n * top * (width + ff)) * 2, 4 * n * top * ff * width)
+        w_down = [bf16(width, ff) for _ in range(sets)]
+        dense = bf16(top * n, ff)
+        record(name + f"dense down, {top * n} rows (Qwen2's)", [lambda w=w: kernels.b200_linear(dense, w) for w in w_down],
+               (ff * width + n * top * (width + ff)) * 2, 2 * n * top * ff * width)
+        x, norm = rand(n, width), bf16(width)
+        y = hk.Summands(rand(4, n, width) if n <= 128 else bf16(n, width), None,
+                        hk.grouped_linear(inner, mlp.w_out, placed), placed.places)
+        record(name + "residual norm over experts", [lambda: hk.residual_norm(
+            x, y, norm, None, epsilon=1e-5, weight_offset=0.0, dtype=torch.bfloat16, narrow=True)] * 8,
+            n * width * (8 + 2 + 2 * top + (16 if n <= 128 else 2)))
+
+    # ---- decode, `batch` sequences ----
+    step = hk.SequenceBatch(batch, batch, vector(range(batch)), vector(range(batch + 1)), vector(range(batch)),
+                            vector([context] * batch))
+    states = [0.1 * rand(batch, heads, dim, dim) for _ in range(copies_of(batch * heads * dim * dim * 4))]
+    projected, ring = bf16(batch, delta.w_in.shape[0]), bf16(batch, delta.taps, 3 * heads * dim)
+    inputs, gate = delta_block(projected, ring, step), projected[:, delta.gate_column:]
+    record("decode: delta step", [lambda s=s: hk.recurrence_step(inputs, s, gate, delta.norm, batch, kind="silu", epsilon=1e-5)
+                                  for s in states], batch * heads * (2 * dim * dim * 4 + 5 * dim * 2))
+    gates = bf16(batch, 2 * heads * dim)
+    channel = hk.delta_inputs(projected, gates, delta.conv, delta.a_log, bf16(heads * dim), ring, step, heads=heads,
+                              kv_heads=heads, dim=dim, vdim=dim, columns=delta.columns, decay_column=0, q_scale=delta.q_scale)
+    record("decode: delta step (Bazirax's)", [lambda s=s: hk.recurrence_step(
+        channel, s, gates[:, heads * dim:], delta.norm, batch, kind="sigmoid", epsilon=1e-5) for s in states],
+        batch * heads * (2 * dim * dim * 4 + 5 * dim * 2))
+    del states
+    cache_bytes = 2 * batch * context * kv_heads * dim * 2
+    caches = [(bf16(batch, context + 64, kv_heads, dim), bf16(batch, context + 64, kv_heads, dim))
+              for _ in range(copies_of(cache_bytes))]
+    parts = rand(4, batch, attention.w_in.shape[0])
+    record("decode: attention prep", [lambda c=c: prepare(parts, attention.bias, *c, step) for c in caches],
+           parts.numel() * 4 + batch * (heads + 2 * kv_heads) * dim * 2)
+    q = bf16(batch, heads, dim)
+    record("decode: attention", [lambda c=c: hk.slot_decode_attention(q, *c, step, scale=0.1, chunk=8192) for c in caches],
+           cache_bytes)
+    record("decode: attention, chunks of 1024", [lambda c=c: hk.slot_decode_attention(
+        q, *c, hk.SequenceBatch(batch, batch, step.token_sequence, step.starts, step.slots, late), scale=0.1, chunk=1024)
+        for late in (vector([context - 1] * batch),) for c in caches], cache_bytes // context * 1024)
+    lengths = torch.full((batch,), context + 1, dtype=torch.int64, device=device)
+    record("decode: attention (Qwen2's)", [lambda c=c: kernels.b200_decode_attention(
+        q.view(batch, heads, 1, dim), *c, lengths, None, scale=0.1) for c in caches], cache_bytes)
+    del caches
+    expert_rows("decode: ", batch)
+
+    # ---- one prompt of 4096 tokens, and four ----
+    for sequences in (1, 4):
+        tokens = 4096
+        n = sequences * tokens
+        name = f"prefill {sequences} x {tokens}: "
+        slots = list(range(sequences))
+        prompt = hk.SequenceBatch(n, sequences, vector([i for i in slots for _ in range(tokens)]),
+                                  vector([i * tokens for i in range(sequences + 1)]), vector(slots),
+                                  vector([0] * sequences), [tokens] * sequences, [0] * sequences, slots)
+        prompt.chunk_table()
+        big = bf16(n, delta.w_in.shape[0])
+        inputs = delta_block(big, ring, prompt)
+        state = 0.1 * rand(sequences, heads, dim, dim)
+        unit = n * heads * dim
+        chunk_flops = 2 * n * heads * (64 * dim * 3 + 3 * dim * dim)
+
+        def delta_core():
+            o = hk.delta_prep(inputs, prompt, torch.bfloat16, device)
+            out = hk.recurrence(*o, state, prompt, torch.bfloat16)
+            hk.gated_head_norm(out, delta.norm, big[:, delta.gate_column:], kind="silu", epsilon=1e-5)
+
+        record(name + "delta rule, all launches", [delta_core], unit * 2 * 5, chunk_flops)
+        operands = hk.delta_prep(inputs, prompt, torch.bfloat16, device)
+        record(name + "delta prep", [lambda: hk.delta_prep(inputs, prompt, torch.bfloat16, device)], unit * (6 + 12))
+        record(name + "delta chunks", [lambda: hk.recurrence(*operands, state, prompt, torch.bfloat16)],
+               unit * (12 + 4), chunk_flops)
+        per_channel = (*operands[:4], operands[4].expand(-1, -1, dim).contiguous())
+        record(name + "delta chunks (Bazirax's)", [lambda: hk.recurrence(*per_channel, state, prompt, torch.bfloat16)],
+               unit * (16 + 4), chunk_flops)
+        del operands, per_channel, big
+        keys, values = bf16(sequences, tokens, kv_heads, dim), bf16(sequences, tokens, kv_heads, dim)
+        big = bf16(n, attention.w_in.shape[0])
+        record(name + "attention prep", [lambda: prepare(big, None, keys, values, prompt)],
+               n * 2 * (heads + 2 * kv_heads) * dim * 2)
+        q = bf16(sequences, tokens, heads, dim)
+        out = torch.empty_like(q)
+        attend = lambda chunk: hk.context_attention(q.transpose(1, 2), keys.transpose(1, 2), values.transpose(1, 2), None,
+                                                    out, context=0, scale=0.1, chunk=chunk)
+        flops = 2 * sequences * heads * tokens * dim
+        record(name + "attention", [lambda: attend(8192)], 0, flops * tokens)
+        record(name + "attention, chunks of 1024", [lambda: attend(1024)], 0, flops * 1024)
+        record(name + "attention (Qwen2's)", [lambda: kernels.b200_prefill_attention(
+            q.transpose(1, 2), keys.transpose(1, 2), values.transpose(1, 2), None, scale=0.1, causal=True)], 0, flops * tokens)
+        expert_rows(name, n)
+        h, norm = bf16(n, width), bf16(width)
+        record(name + "RMS norm (Qwen2's)", [lambda: kernels.b200_rms_norm(h, norm, epsilon=1e-5)], n * width * 4)
+    return rows
+
+
 def run(args, hbm_gbs):
-    from llm_compiler_b200 import bazirax, qwen2
+    from llm_compiler_b200 import bazirax, lozanex, qwen2
     from llm_compiler_b200.engine import Qwen2Engine
     from llm_compiler_b200.hybrid_engine import HybridEngine
 
     torch.manual_seed(0)
     size = SIZES[args.model]
-    config = bazirax_config(size)
+    design = args.model.split("-")[0]
+    module, make_config, kernel_table = {"bazirax": (bazirax, bazirax_config, bazirax_kernels),
+                                         "lozanex": (lozanex, lozanex_config, lozanex_kernels)}[design]
+    config = make_config(size)
     other = qwen_config(size, config.num_layers)
     batch, context = args.batch, args.context
     peaks = json.loads(PEAKS.read_text()) if PEAKS.exists() else {}
     tflops = peaks.get("bf16_tflops", 1590.0)
     result = {}
     engines = {
-        "bazirax": lambda b, c: HybridEngine(config, weights, batch=b, capacity=c),
+        design: lambda b, c: HybridEngine(config, weights, batch=b, capacity=c),
         "qwen2": lambda b, c: Qwen2Engine(other, weights, batch=b, capacity=c),
     }
     for name, build in engines.items():
-        if name == "bazirax":
-            weights = bazirax.make_weights(config, dtype=torch.bfloat16, device="cuda", gate_rank=size["dim"])
+        if name == design:
+            more = dict(gate_rank=size["dim"]) if design == "bazirax" else {}
+            weights = module.make_weights(config, dtype=torch.bfloat16, device="cuda", **more)
         else:
             weights = qwen2.make_weights(other, dtype=torch.bfloat16, device="cuda", reproducible=False)
         entry = result[name] = {"parameters": sum(w.numel() for w in weights.values())}
@@ -235,11 +413,11 @@ def run(args, hbm_gbs):
         ms = decode_ms(engine, context, batch)
         entry[f"decode {batch} x {context}"] = {"ms": round(ms, 4), "tokens_per_s": round(batch / ms * 1e3),
                                                 "kernels": engine.kernels_per_step}
-        if name == "bazirax":
+        if name == design:
             entry["kernels"] = kernel_table(engine, config, size, context, batch, hbm_gbs, tflops)
         del engine, weights
         torch.cuda.empty_cache()
-    decode = result["bazirax"][f"decode {batch} x {context}"]
+    decode = result[design][f"decode {batch} x {context}"]
     return {"metric": f"{args.model}_layers_decode_tokens_per_s", "value": decode["tokens_per_s"], "unit": "tokens/s",
             "n_gpus": 1, "ms_per_step": decode["ms"], "higher_is_better": True, "vs_baseline": None, "dtype": "bf16",
             "data": "synthetic", "config": {"model": args.model, "layers": config.num_layers, "vocab": VOCAB,
