@@ -259,24 +259,28 @@ def lozanex_kernels(engine, config, size, context, batch, hbm_gbs, tflops):
     def expert_rows(name, n):
         """The mixture of experts on n rows, launch by launch, and dense projections of the same size."""
         h = bf16(n, width)
-        logits = kernels.b200_linear_partial(h, mlp.w_router)
-        used = min(experts, n * top)
+        few, tile = n <= 128, mlp.tile_of(n)
+        always = mlp.slices if few else 0  # the shared expert in slices
+        used, each = min(experts, n * top) + always, top + always
         weight_sets = copies_of(mlp.w_in.numel() * 2)
         w_in = [mlp.w_in] + [mlp.w_in.clone() for _ in range(weight_sets - 1)]
         w_out = [mlp.w_out] + [mlp.w_out.clone() for _ in range(weight_sets - 1)]
-        counts = torch.zeros_like(mlp.counts)
-        routed = hk.expert_route(logits, counts, top=top)
-        placed = hk.expert_place(h, *routed, counts, tile=mlp.tile_of(n))
-        inner = hk.grouped_linear(placed.rows, mlp.w_in, placed, swiglu=True)
-        record(name + "router logits", [lambda: kernels.b200_linear_partial(h, mlp.w_router)] * 8,
-               (h.numel() + mlp.w_router.numel()) * 2 + n * mlp.w_router.shape[0] * 4, 2 * n * mlp.w_router.numel())
-        record(name + "routing", [lambda: hk.expert_route(logits, torch.zeros_like(counts), top=top)] * 8, logits.numel() * 4)
-        record(name + "sorting rows", [lambda: hk.expert_place(h, *routed, counts, tile=placed.tile)] * 8,
-               h.numel() * 2 * (1 + top))
-        record(name + "experts, gate and up", [lambda w=w: hk.grouped_linear(placed.rows, w, placed, swiglu=True) for w in w_in],
-               (used * 2 * ff * width + n * top * (width + ff)) * 2, 4 * n * top * ff * width)
-        record(name + "experts, down", [lambda w=w: hk.grouped_linear(inner, w, placed) for w in w_out],
-               (used * ff * width + n * top * (width + ff)) * 2, 2 * n * top * ff * width)
+        if few:
+            choose = lambda: hk.expert_select(h, mlp.w_router, mlp.counters, top=top, always=always, tile=tile)
+            record(name + "choice of experts", [choose] * 8, (h.numel() + mlp.w_router.numel()) * 2)
+        else:
+            logits = kernels.b200_linear_partial(h, mlp.w_router)
+            choose = lambda: hk.expert_route(logits, h, mlp.counters, top=top, always=0, tile=tile)
+            record(name + "router logits", [lambda: kernels.b200_linear_partial(h, mlp.w_router)] * 8,
+                   (h.numel() + mlp.w_router.numel()) * 2 + n * mlp.w_router.shape[0] * 4, 2 * n * mlp.w_router.numel())
+            record(name + "choice of experts, rows in order", [choose] * 8, logits.numel() * 4 + h.numel() * 2 * (1 + top))
+        order, ordered = (choose(), h) if few else choose()
+        inner = hk.grouped_linear(ordered, mlp.w_in, order, gather=few, swiglu=True)
+        record(name + "experts, gate and up", [lambda w=w: hk.grouped_linear(ordered, w, order, gather=few, swiglu=True)
+                                               for w in w_in],
+               (used * 2 * ff * width + n * width + n * each * ff) * 2, 4 * n * each * ff * width)
+        record(name + "experts, down", [lambda w=w: hk.grouped_linear(inner, w, order) for w in w_out],
+               (used * ff * width + n * each * (width + ff)) * 2, 2 * n * each * ff * width)
         dense = bf16(top * n, width)
         sets = copies_of(4 * ff * width)
         w_dense = [bf16(2 * ff, width) for _ in range(sets)]
@@ -288,11 +292,10 @@ def lozanex_kernels(engine, config, size, context, batch, hbm_gbs, tflops):
         record(name + f"dense down, {top * n} rows (Qwen2's)", [lambda w=w: kernels.b200_linear(dense, w) for w in w_down],
                (ff * width + n * top * (width + ff)) * 2, 2 * n * top * ff * width)
         x, norm = rand(n, width), bf16(width)
-        y = hk.Summands(rand(4, n, width) if n <= 128 else bf16(n, width), None,
-                        hk.grouped_linear(inner, mlp.w_out, placed), placed.places)
+        y = hk.Summands(None if few else bf16(n, width), None, hk.grouped_linear(inner, mlp.w_out, order), order.places)
         record(name + "residual norm over experts", [lambda: hk.residual_norm(
             x, y, norm, None, epsilon=1e-5, weight_offset=0.0, dtype=torch.bfloat16, narrow=True)] * 8,
-            n * width * (8 + 2 + 2 * top + (16 if n <= 128 else 2)))
+            n * width * (8 + 2 + 2 * each + (0 if few else 2)))
 
     # ---- decode, `batch` sequences ----
     step = hk.SequenceBatch(batch, batch, vector(range(batch)), vector(range(batch + 1)), vector(range(batch)),

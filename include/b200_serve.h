@@ -516,15 +516,15 @@ int b200_argmax(const void* logits, int64_t* ids, int64_t rows, int64_t vocab,
  *                        over the caches, bf16, row_size 64 or 128; chunk > 0: only the keys of the
  *                        position's own chunk of `chunk` positions. context: upper bound of the keys
  *   b200_slot_attention  the same for any rows, sizes and dtype, on the CUDA cores
- *   b200_expert_route    the top experts of every row from router logits (fp32, split-K partials
- *                        [splits, rows, logit_stride]): expert ids and sigmoid scores [rows, top], and
- *                        each choice's number among its expert's; counts [experts] must be zero before
- *   b200_expert_place    choices to rows of an expert-sorted matrix whose experts start at multiples of
- *                        tile rows: places [rows, top], sorted (rows of h, copied), scores [sorted rows],
- *                        tiles [max_tiles, 2]: a tile's expert (-1: none) and how many rows it holds
- *   b200_grouped_linear  out[r, :] = w[expert of r's tile] x[r, :] over the sorted rows; with SwiGLU (rows
- *                        of w: gate_j, up_j alternating) silu(s_r g) (s_r u), s the scores (NULL: 1).
- *                        clear: int32 [clear_count] set to zero (the counts of b200_expert_route)
+ *   b200_expert_select   a mixture of experts' choices for a few rows, from h and the router's weights
+ *                        [experts, width] (fp32 sums): the top experts of every row by their logits, with
+ *                        sigmoid scores, and the expert-sorted order of the choices (b200_expert_order)
+ *   b200_expert_route, b200_expert_place  the same in two launches from finished logits (fp32, split-K
+ *                        partials [splits, rows, logit_stride]) for many rows; the second also copies the
+ *                        rows of h (columns elements of each) into their order, unless h is NULL
+ *   b200_grouped_linear  out[r, :] = w[expert of r's tile] x[r, :] over sorted rows r; with index, x is not
+ *                        sorted itself: row index[r] of it (bf16: x_rows <= tile). With SwiGLU (rows of w: gate_j, up_j alternating)
+ *                        silu(s_r g) (s_r u), s the scores (NULL: 1). Rows that no tile holds stay unwritten
  *   b200_sequence_positions  positions[r] = lengths[slots[r]] (0 for an idle row)
  *   b200_advance_slots   lengths[slots[r]] += starts[r + 1] - starts[r], clamped with a status bit */
 #define B200_GATE_SILU 0
@@ -567,6 +567,19 @@ typedef struct b200_step_output {
   int64_t gate_kind;
   double epsilon;
 } b200_step_output;
+typedef struct b200_expert_order {
+  int32_t* chosen;      /* [rows, top] */
+  float* scores;        /* [rows, top] */
+  int32_t* numbers;     /* [rows, top]: a choice's number among those of its expert */
+  int32_t* counters;    /* [experts + 1], zero before a choice and zero again behind its order */
+  int32_t* places;      /* [rows, always + top]: the sorted rows of a row */
+  int32_t* index;       /* [max_tiles * tile]: the row of a sorted row */
+  float* sorted_scores; /* [max_tiles * tile] */
+  int32_t* tiles;       /* [max_tiles][2]: expert of a tile (-1: none) and rows it holds */
+  int64_t experts, top;
+  int64_t always;       /* experts, numbered from `experts` on, that take every row with score 1 */
+  int64_t tile, max_tiles; /* always * ceil(rows / tile) + rows * top / tile + min(experts, rows * top) tiles */
+} b200_expert_order;
 typedef struct b200_attention_prep_inputs {
   const void* input;    /* [rows, row_stride], or fp32 partials [splits, rows, row_stride] */
   const void* bias;     /* [row_stride] added to the partials; NULL: none */
@@ -603,16 +616,16 @@ int b200_slot_attention(const void* q, const void* keys, const void* values, voi
                         const int32_t* token_sequence, const int32_t* starts, const int32_t* slots,
                         const int32_t* bases, int64_t rows, int64_t heads, int64_t kv_heads, int64_t row_size,
                         int64_t capacity, int64_t chunk, double scale, int dtype, void* stream);
-int b200_expert_route(const float* logits, int32_t* chosen, float* scores, int32_t* numbers, int32_t* counts,
-                      int64_t rows, int64_t experts, int64_t top, int64_t splits, int64_t logit_stride,
-                      void* stream);
-int b200_expert_place(const void* h, const int32_t* chosen, const float* scores, const int32_t* numbers,
-                      const int32_t* counts, int32_t* places, void* sorted, float* sorted_scores, int32_t* tiles,
-                      int64_t rows, int64_t experts, int64_t top, int64_t tile, int64_t max_tiles, int64_t columns,
+int b200_expert_select(const void* h, const void* router, const b200_expert_order* order, int64_t rows,
+                       int64_t width, int64_t h_row_stride, int dtype, void* stream);
+int b200_expert_route(const float* logits, const b200_expert_order* order, int64_t rows, int64_t splits,
+                      int64_t logit_stride, void* stream);
+int b200_expert_place(const b200_expert_order* order, const void* h, void* sorted, int64_t rows, int64_t columns,
                       int64_t h_row_stride, int dtype, void* stream);
-int b200_grouped_linear(const void* x, const void* w, const int32_t* tiles, const float* scores, void* out,
-                        int32_t* clear, int64_t clear_count, int64_t experts, int64_t tile, int64_t max_tiles,
-                        int64_t k, int64_t n, int epilogue, int dtype, int32_t* status, void* stream);
+int b200_grouped_linear(const void* x, const void* w, const int32_t* tiles, const int32_t* index,
+                        const float* scores, void* out, int64_t experts, int64_t tile, int64_t max_tiles,
+                        int64_t x_rows, int64_t k, int64_t n, int epilogue, int dtype, int32_t* status,
+                        void* stream);
 int b200_latent_norm(const void* input, const void* q_weight, const void* kv_weight, void* q_out,
                      void* cache, void* dense, const int32_t* token_sequence, const int32_t* starts,
                      const int32_t* slots, const int32_t* bases, int64_t rows, int64_t q_rank,

@@ -78,6 +78,14 @@ class AttentionPrepInputs(ctypes.Structure):
                [("epsilon", c_double)]
 
 
+class ExpertOrder(ctypes.Structure):
+    """b200_expert_order of include/b200_serve.h."""
+
+    _fields_ = [(name, c_void_p) for name in
+                ("chosen", "scores", "numbers", "counters", "places", "index", "sorted_scores", "tiles")] + \
+               [(name, c_int64) for name in ("experts", "top", "always", "tile", "max_tiles")]
+
+
 class StepOutput(ctypes.Structure):
     """b200_step_output of include/b200_serve.h."""
 
@@ -169,8 +177,9 @@ SIGNATURES = {
     "b200_slot_decode_attention": (c_int, [c_void_p] * 6 + [c_int64] * 8 + [c_double, c_void_p, c_int64, c_void_p,
                                                                           c_void_p]),
     "b200_slot_attention": (c_int, [c_void_p] * 8 + [c_int64] * 6 + [c_double, c_int, c_void_p]),
-    "b200_expert_route": (c_int, [c_void_p] * 5 + [c_int64] * 5 + [c_void_p]),
-    "b200_expert_place": (c_int, [c_void_p] * 9 + [c_int64] * 7 + [c_int, c_void_p]),
+    "b200_expert_select": (c_int, [c_void_p, c_void_p, POINTER(ExpertOrder)] + [c_int64] * 3 + [c_int, c_void_p]),
+    "b200_expert_route": (c_int, [c_void_p, POINTER(ExpertOrder)] + [c_int64] * 3 + [c_void_p]),
+    "b200_expert_place": (c_int, [POINTER(ExpertOrder), c_void_p, c_void_p] + [c_int64] * 3 + [c_int, c_void_p]),
     "b200_grouped_linear": (c_int, [c_void_p] * 6 + [c_int64] * 6 + [c_int, c_int, c_void_p, c_void_p]),
     "b200_latent_norm": (c_int, [c_void_p] * 10 + [c_int64] * 8 + [c_double, c_int, c_void_p, c_void_p]),
     "b200_gated_head_norm": (c_int, [c_void_p] * 4 + [c_int64] * 5 + [c_int, c_double, c_int, c_void_p]),

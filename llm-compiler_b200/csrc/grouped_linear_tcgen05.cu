@@ -6,6 +6,10 @@
 // accumulator has an output feature per TMEM lane and a row per column; the epilogue turns 32 x 32 blocks
 // through shared memory into row segments.
 //
+// Sorted rows come in boxes of up to 64, only those that a tile holds. At decode sizes x is not sorted at all
+// (index given): every item multiplies all of the step's rows, which costs the tensor core nothing beside the
+// weights' stream, and the epilogue reads the columns of the rows that the tile holds.
+//
 // A persistent CTA per SM walks (tile, 128 features) items, features fastest: the CTAs at work at one time
 // share a tile's rows, and an expert's weights are read from HBM once and from L2 by its further tiles. The
 // tile table is made on the device; how many of its entries are used is known only there (the used ones come
@@ -30,8 +34,14 @@ struct Shape {
   static constexpr int kStages = TILE == 256 ? 4 : TILE == 128 ? 6 : 8;
   static constexpr int kColumns = TILE < 32 ? 32 : TILE;  // TMEM columns of an accumulator
   static constexpr int kStaging = 4 * 2048;               // 32 x 32 bf16 per epilogue warp
+  static constexpr int kBox = TILE <= 64 ? 16 : 64;       // rows of a box of sorted rows
   static constexpr int kSmem = kStages * kStageBytes + kStaging + 1024;
 };
+
+// One column of the warp's 32 TMEM lanes, without a wait
+__device__ __forceinline__ void tmem_load_column_issue(uint32_t taddr, uint32_t& r) {
+  asm volatile("tcgen05.ld.sync.aligned.32x32b.x1.b32 {%0}, [%1];" : "=r"(r) : "r"(taddr));
+}
 
 struct Params : GroupedLinearParams {
   uint32_t wait_limit;
@@ -44,7 +54,6 @@ grouped_linear_tcgen05_kernel(const Params p, const __grid_constant__ CUtensorMa
                               const __grid_constant__ CUtensorMap x_map) {
   using S = Shape<TILE>;
   constexpr int STAGES = S::kStages;
-  constexpr uint32_t idesc = instruction_descriptor(kFeatures, TILE);
   extern __shared__ __align__(1024) unsigned char smem[];
   __shared__ __align__(8) uint64_t full_bar[STAGES], empty_bar[STAGES], acc_full[2], acc_empty[2];
   __shared__ uint32_t tmem_base_slot;
@@ -80,6 +89,8 @@ grouped_linear_tcgen05_kernel(const Params p, const __grid_constant__ CUtensorMa
   asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
   const uint32_t tmem_base = tmem_base_slot;
 
+  const int all_rows = p.index != nullptr ? p.x_rows : 0;  // 0: x is sorted
+
   if (warp == 4 && lane == 0 && !p.drop_loads) {
     // ---- TMA producer ----
     grid_dependency_wait();
@@ -87,8 +98,10 @@ grouped_linear_tcgen05_kernel(const Params p, const __grid_constant__ CUtensorMa
     bool ok = true;
     for (int item = blockIdx.x; ok && item < items; item += gridDim.x) {
       const int tile = item / features, feature = (item - tile * features) * kFeatures;
-      const int expert = p.tiles[tile * 2];
+      const int expert = p.tiles[tile * 2], held = min(p.tiles[tile * 2 + 1], TILE);
       if (expert < 0 || expert >= p.experts) break;
+      const int first = all_rows > 0 ? 0 : tile * TILE;
+      const int boxes = ((all_rows > 0 ? all_rows : held) + S::kBox - 1) / S::kBox;
       for (int kb = 0; kb < nkb; ++kb, ++round) {
         const int s = round % STAGES;
         if (round >= STAGES &&
@@ -98,9 +111,10 @@ grouped_linear_tcgen05_kernel(const Params p, const __grid_constant__ CUtensorMa
         }
         const uint32_t bar = smem_u32(&full_bar[s]);
         const uint32_t w_dst = smem_base + s * S::kStageBytes;
-        mbarrier_arrive_expect_tx(bar, static_cast<uint32_t>(S::kStageBytes));
+        mbarrier_arrive_expect_tx(bar, static_cast<uint32_t>(S::kWeightBytes + boxes * S::kBox * 128));
         tma_load_3d(w_dst, &w_map, bar, kb * kDepth, feature, expert);
-        tma_load_2d(w_dst + S::kWeightBytes, &x_map, bar, kb * kDepth, tile * TILE);
+        for (int box = 0; box < boxes; ++box)
+          tma_load_2d(w_dst + S::kWeightBytes + box * S::kBox * 128, &x_map, bar, kb * kDepth, first + box * S::kBox);
       }
     }
     if (!ok) {  // the copies still in flight get a bounded chance to land before the CTA retires
@@ -114,8 +128,9 @@ grouped_linear_tcgen05_kernel(const Params p, const __grid_constant__ CUtensorMa
     int round = 0, local = 0;
     bool ok = true;
     for (int item = blockIdx.x; ok && item < items; item += gridDim.x, ++local) {
-      const int expert = p.tiles[item / features * 2];
+      const int expert = p.tiles[item / features * 2], held = min(p.tiles[item / features * 2 + 1], TILE);
       if (expert < 0 || expert >= p.experts) break;
+      const uint32_t idesc = instruction_descriptor(kFeatures, ((all_rows > 0 ? all_rows : held) + 15) / 16 * 16);
       const int acc = local & 1;
       if (local >= 2 && !mbarrier_wait_bounded(smem_u32(&acc_empty[acc]), ((local >> 1) - 1) & 1, p.wait_limit)) {
         ok = false;
@@ -144,8 +159,6 @@ grouped_linear_tcgen05_kernel(const Params p, const __grid_constant__ CUtensorMa
   } else if (warp < 4) {
     // ---- epilogue ----
     grid_dependency_wait();
-    if (p.clear != nullptr && blockIdx.x == 0)
-      for (int i = threadIdx.x; i < p.clear_count; i += 128) p.clear[i] = 0;
     const uint32_t staging = smem_base + STAGES * S::kStageBytes + warp * 2048;
     __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out);
     const int out_columns = p.swiglu ? p.n / 2 : p.n;
@@ -153,7 +166,7 @@ grouped_linear_tcgen05_kernel(const Params p, const __grid_constant__ CUtensorMa
     bool ok = true;
     for (int item = blockIdx.x; item < items; item += gridDim.x, ++local) {
       const int tile = item / features, feature = (item - tile * features) * kFeatures;
-      const int expert = p.tiles[tile * 2], held = p.tiles[tile * 2 + 1];
+      const int expert = p.tiles[tile * 2], held = min(p.tiles[tile * 2 + 1], TILE);
       if (expert < 0 || expert >= p.experts) break;
       const int acc = local & 1;
       // (the wait's outcome is made warp-uniform: tcgen05.ld is a warp-wide instruction)
@@ -167,7 +180,21 @@ grouped_linear_tcgen05_kernel(const Params p, const __grid_constant__ CUtensorMa
       for (int c0 = 0; c0 < held; c0 += 32) {
         if (own >= p.n) break;  // warp-uniform
         float v[32];
-        tmem_load_32x32(t_addr + c0, v);
+        if (all_rows > 0) {
+          const int mine = p.index[row0 + min(c0 + lane, held - 1)];  // the row that stands in column c0 + lane
+          uint32_t raw[32];
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {
+            const int column = __shfl_sync(0xffffffffu, mine, i);
+            raw[i] = 0;
+            if (c0 + i < held) tmem_load_column_issue(t_addr + min(max(column, 0), all_rows - 1), raw[i]);
+          }
+          tmem_load_wait(raw);
+#pragma unroll
+          for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(raw[i]);
+        } else {
+          tmem_load_32x32(t_addr + c0, v);
+        }
         __syncwarp();  // the previous block's reads of the staging tile are done
         if (p.swiglu) {
           // lanes 2 j and 2 j + 1 hold gate and up of output j: each turns one of two neighbouring rows out
@@ -242,12 +269,13 @@ int launch(const Params& p, const CUtensorMap& w_map, const CUtensorMap& x_map, 
 }  // namespace
 
 int grouped_linear_tcgen05(const GroupedLinearParams& in, const void* x, const void* w, cudaStream_t stream) {
+  if (in.index != nullptr && in.x_rows > in.tile) return B200_ERR_UNSUPPORTED;
   if (in.k % 8 != 0 || in.n % (in.swiglu ? 16 : 8) != 0) return B200_ERR_UNSUPPORTED;
   if (!aligned16(x) || !aligned16(w) || !aligned16(in.out)) return B200_ERR_ALIGNMENT;
   if (ceil_div(in.n, kFeatures) * in.max_tiles > INT32_MAX) return B200_ERR_TOO_LARGE;
   CUtensorMap w_map, x_map;
   if (!make_bf16_slot_map(&w_map, w, in.experts, in.n, in.k, kFeatures) ||
-      !make_bf16_matrix_map(&x_map, x, static_cast<int64_t>(in.max_tiles) * in.tile, in.k, in.k, in.tile))
+      !make_bf16_matrix_map(&x_map, x, in.x_rows, in.k, in.k, in.tile <= 64 ? 16 : 64))
     return B200_ERR_UNSUPPORTED;
   Params p;
   static_cast<GroupedLinearParams&>(p) = in;

@@ -1112,7 +1112,7 @@ int linear_tcgen05(const void* input, const void* weight, const void* bias, cons
         bn = candidate;
       }
     }
-    if (best < 0.8 && !fold_norm) return B200_ERR_UNSUPPORTED;
+    if (best < 0.5 && !fold_norm) return B200_ERR_UNSUPPORTED;
     // A folded-norm projection at decode sizes (gate|up: 17 MB of weights) is a chain of
     // latencies, not a stream: 64-column tiles with short rings put two or three CTAs on an SM,
     // whose ring round trips and two-warp SwiGLU epilogues overlap. Measured on the Qwen2-0.5B

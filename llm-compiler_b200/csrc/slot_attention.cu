@@ -26,9 +26,8 @@ struct AttentionPrepParams {
   int32_t* status;
 };
 
-// grid (rows, 1 or 2): y = 0 the queries, y = 1 keys and values. E consecutive elements a thread (4 where
-// the sizes allow it, else 1).
-template <typename T, int E>
+// grid (rows, 1 or 2): y = 0 the queries, y = 1 keys and values. Any sizes.
+template <typename T>
 __global__ void __launch_bounds__(256) attention_prep_kernel(const AttentionPrepParams p) {
   extern __shared__ float values[];  // the projection [heads * dim], then cos, sin [rot_dims / 2] each
   __shared__ float scratch[8];
@@ -42,47 +41,11 @@ __global__ void __launch_bounds__(256) attention_prep_kernel(const AttentionPrep
   const int sequence = p.batch.token_sequence[row];
   const int slot = p.batch.slots[sequence];
   const int64_t position = p.batch.position(sequence, row);
-  auto load = [&](int column, float (&v)[E]) {
-    if (p.splits > 0) {
-      const float* in = static_cast<const float*>(p.input) + row * p.row_stride + column;
-      const int64_t slice = static_cast<int64_t>(p.rows) * p.row_stride;
-#pragma unroll
-      for (int e = 0; e < E; ++e) v[e] = p.bias != nullptr ? Elem<T>::load(static_cast<const T*>(p.bias) + column + e) : 0.0f;
-      for (int s = 0; s < p.splits; s += 4) {
-        float t[4][E];
-#pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          if constexpr (E == 4) {
-            const float4 f = s + j < p.splits ? __ldcg(reinterpret_cast<const float4*>(in + (s + j) * slice))
-                                              : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-            t[j][0] = f.x; t[j][1] = f.y; t[j][2] = f.z; t[j][3] = f.w;
-          } else {
-            t[j][0] = s + j < p.splits ? __ldcg(in + (s + j) * slice) : 0.0f;
-          }
-        }
-#pragma unroll
-        for (int j = 0; j < 4; ++j)
-#pragma unroll
-          for (int e = 0; e < E; ++e) v[e] += t[j][e];
-      }
-    } else {
-      const T* in = static_cast<const T*>(p.input) + row * p.row_stride + column;
-      if constexpr (E == 4 && sizeof(T) == 2) {
-        const uint2 t = *reinterpret_cast<const uint2*>(in);
-        v[0] = bf16_lo(t.x); v[1] = bf16_hi(t.x); v[2] = bf16_lo(t.y); v[3] = bf16_hi(t.y);
-      } else {
-#pragma unroll
-        for (int e = 0; e < E; ++e) v[e] = Elem<T>::load(in + e);
-      }
-    }
-  };
-  auto store = [&](T* out, const float (&v)[E]) {
-    if constexpr (E == 4 && sizeof(T) == 2) {
-      *reinterpret_cast<uint2*>(out) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
-    } else {
-#pragma unroll
-      for (int e = 0; e < E; ++e) Elem<T>::store(out + e, v[e]);
-    }
+  auto load = [&](int column) {
+    if (p.splits == 0) return Elem<T>::load(static_cast<const T*>(p.input) + row * p.row_stride + column);
+    const float sum = sum_slices(static_cast<const float*>(p.input) + row * p.row_stride + column,
+                                 static_cast<int64_t>(p.rows) * p.row_stride, p.splits);
+    return p.bias != nullptr ? sum + Elem<T>::load(static_cast<const T*>(p.bias) + column) : sum;
   };
   T* out = static_cast<T*>(p.q_out) + row * p.heads * p.size;
   if (is_k) {
@@ -94,11 +57,9 @@ __global__ void __launch_bounds__(256) attention_prep_kernel(const AttentionPrep
     const int64_t at = (slot * p.capacity + position) * p.kv_heads * p.size;
     out = static_cast<T*>(p.keys) + at;
     T* v_out = static_cast<T*>(p.values) + at;
-    for (int item = threadIdx.x * E; item < p.kv_heads * p.size; item += blockDim.x * E) {
+    for (int item = threadIdx.x; item < p.kv_heads * p.size; item += blockDim.x) {
       const int head = item / p.size, c = item - head * p.size;
-      float v[E] = {};
-      if (c < p.vdim) load(p.v_column + head * p.vdim + c, v);
-      store(v_out + item, v);
+      Elem<T>::store(v_out + item, c < p.vdim ? load(p.v_column + head * p.vdim + c) : 0.0f);
     }
   }
   for (int i = threadIdx.x; i < half; i += blockDim.x) {
@@ -107,14 +68,10 @@ __global__ void __launch_bounds__(256) attention_prep_kernel(const AttentionPrep
   }
   const int column = is_k ? p.k_column : p.q_column;
   float sum = 0.0f;
-  for (int item = threadIdx.x * E; item < count; item += blockDim.x * E) {
-    float v[E];
-    load(column + item, v);
-#pragma unroll
-    for (int e = 0; e < E; ++e) {
-      values[item + e] = v[e];
-      sum += v[e] * v[e];
-    }
+  for (int item = threadIdx.x; item < count; item += blockDim.x) {
+    const float v = load(column + item);
+    values[item] = v;
+    sum += v * v;
   }
   sum = warp_sum(sum);
   if ((threadIdx.x & 31) == 0) scratch[threadIdx.x >> 5] = sum;
@@ -123,23 +80,165 @@ __global__ void __launch_bounds__(256) attention_prep_kernel(const AttentionPrep
   for (int w = 0; w < static_cast<int>(blockDim.x >> 5); ++w) sum += scratch[w];
   const float factor = 1.0f / sqrtf(sum / count + p.eps);
   const T* weight = static_cast<const T*>(is_k ? p.k_weight : p.q_weight);
-  for (int item = threadIdx.x * E; item < heads * p.size; item += blockDim.x * E) {
+  for (int item = threadIdx.x; item < heads * p.size; item += blockDim.x) {
     const int head = item / p.size, c = item - head * p.size;
-    float v[E] = {};
+    float v = 0.0f;
     if (c < p.dim) {
       const int at = head * p.dim + c;
-#pragma unroll
-      for (int e = 0; e < E; ++e) {
-        v[e] = values[at + e] * factor * Elem<T>::load(weight + at + e);
-        if (c + e < p.rot_dims) {
-          const bool first = c + e < half;
-          const int i = first ? c + e : c + e - half, other = at + e + (first ? half : -half);
-          const float partner = values[other] * factor * Elem<T>::load(weight + other);
-          v[e] = v[e] * cosine[i] + (first ? -partner : partner) * sine[i];
-        }
+      v = values[at] * factor * Elem<T>::load(weight + at);
+      if (c < p.rot_dims) {
+        const bool first = c < half;
+        const int i = first ? c : c - half, other = at + (first ? half : -half);
+        const float partner = values[other] * factor * Elem<T>::load(weight + other);
+        v = v * cosine[i] + (first ? -partner : partner) * sine[i];
       }
     }
-    store(out + item, v);
+    Elem<T>::store(out + item, v);
+  }
+}
+
+// The same for sizes in whole quads: a CTA per row holds the projection in registers, Q quads a thread (the
+// queries' first, then the keys', then the values'), every load in flight at once.
+template <typename T>
+__device__ __forceinline__ float4 read_quad(const T* p) {
+  if constexpr (sizeof(T) == 4) {
+    return *reinterpret_cast<const float4*>(p);
+  } else {
+    const uint2 t = *reinterpret_cast<const uint2*>(p);
+    return make_float4(bf16_lo(t.x), bf16_hi(t.x), bf16_lo(t.y), bf16_hi(t.y));
+  }
+}
+template <typename T>
+__device__ __forceinline__ void write_quad(T* p, float4 v) {
+  if constexpr (sizeof(T) == 4) *reinterpret_cast<float4*>(p) = v;
+  else *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
+}
+
+template <typename T, int Q>
+__global__ void __launch_bounds__(512) attention_prep_quads_kernel(const AttentionPrepParams p, int dim_shift) {
+  extern __shared__ __align__(16) float normed[];  // q and k [(heads + kv_heads) * dim], then cos, sin [rot_dims / 2] each
+  __shared__ float scratch[2][16];
+  const int dq = p.dim / 4, half = p.rot_dims / 2;
+  const bool kv = p.keys != nullptr;
+  const int nq = p.heads * dq, nk = kv ? p.kv_heads * dq : 0, nv = kv ? p.kv_heads * (p.vdim / 4) : 0;
+  float* cosine = normed + (nq + nk) * 4;
+  float* sine = cosine + half;
+  grid_launch_dependents();
+  grid_dependency_wait_cta();
+  const int64_t row = blockIdx.x;
+  auto column_of = [&](int i) {
+    return i < nq ? p.q_column + i * 4 : i < nq + nk ? p.k_column + (i - nq) * 4 : p.v_column + (i - nq - nk) * 4;
+  };
+  float4 v[Q];
+#pragma unroll
+  for (int j = 0; j < Q; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    v[j] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    if (i >= nq + nk + nv) continue;
+    const int column = column_of(i);
+    if (p.splits > 0) {
+      const float* in = static_cast<const float*>(p.input) + row * p.row_stride + column;
+      const int64_t slice = static_cast<int64_t>(p.rows) * p.row_stride;
+      if (p.bias != nullptr) v[j] = read_quad<T>(static_cast<const T*>(p.bias) + column);
+      for (int s = 0; s < p.splits; s += 4) {
+        float4 t[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          t[e] = s + e < p.splits ? __ldcg(reinterpret_cast<const float4*>(in + (s + e) * slice))
+                                  : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          v[j].x += t[e].x; v[j].y += t[e].y; v[j].z += t[e].z; v[j].w += t[e].w;
+        }
+      }
+    } else {
+      v[j] = read_quad<T>(static_cast<const T*>(p.input) + row * p.row_stride + column);
+    }
+  }
+  const int sequence = p.batch.token_sequence[row];
+  const int slot = p.batch.slots[sequence];
+  const int64_t position = p.batch.position(sequence, row);
+  const T* q_weight = static_cast<const T*>(p.q_weight);
+  const T* k_weight = static_cast<const T*>(p.k_weight);
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    const double turns = static_cast<double>(position) * p.turns[i];
+    sincospif(2.0f * static_cast<float>(turns - rint(turns)), &sine[i], &cosine[i]);
+  }
+  float q_sum = 0.0f, k_sum = 0.0f;
+#pragma unroll
+  for (int j = 0; j < Q; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    const float squares = v[j].x * v[j].x + v[j].y * v[j].y + v[j].z * v[j].z + v[j].w * v[j].w;
+    if (i < nq) q_sum += squares;
+    else if (i < nq + nk) k_sum += squares;
+  }
+  q_sum = warp_sum(q_sum);
+  k_sum = warp_sum(k_sum);
+  const int warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+  if ((threadIdx.x & 31) == 0) {
+    scratch[0][warp] = q_sum;
+    scratch[1][warp] = k_sum;
+  }
+  __syncthreads();
+  q_sum = k_sum = 0.0f;
+  for (int w = 0; w < warps; ++w) {
+    q_sum += scratch[0][w];
+    k_sum += scratch[1][w];
+  }
+  const float q_factor = 1.0f / sqrtf(q_sum / (p.heads * p.dim) + p.eps);
+  const float k_factor = 1.0f / sqrtf(k_sum / (p.kv_heads * p.dim) + p.eps);
+#pragma unroll
+  for (int j = 0; j < Q; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    if (i >= nq + nk) continue;
+    const float4 w = i < nq ? read_quad<T>(q_weight + i * 4) : read_quad<T>(k_weight + (i - nq) * 4);
+    const float f = i < nq ? q_factor : k_factor;
+    v[j] = make_float4(v[j].x * f * w.x, v[j].y * f * w.y, v[j].z * f * w.z, v[j].w * f * w.w);
+    *reinterpret_cast<float4*>(normed + i * 4) = v[j];
+  }
+  __syncthreads();
+  const bool inside = slot >= 0 && position >= 0 && position < p.capacity;
+  if (kv && slot >= 0 && !inside && threadIdx.x == 0) atomicOr(p.status, B200_STATUS_KV_OVERFLOW);
+  const int64_t cache = (slot * p.capacity + position) * p.kv_heads * p.size;
+  T* q_out = static_cast<T*>(p.q_out) + row * p.heads * p.size;
+  T* k_out = static_cast<T*>(p.keys) + cache;
+  T* v_out = static_cast<T*>(p.values) + cache;
+#pragma unroll
+  for (int j = 0; j < Q; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    if (i >= nq + nk + nv || (i >= nq && !inside)) continue;
+    if (i >= nq + nk) {
+      const int quad = i - nq - nk, head = quad / (p.vdim / 4);
+      write_quad<T>(v_out + head * p.size + (quad - head * (p.vdim / 4)) * 4, v[j]);
+      continue;
+    }
+    const int quad = i < nq ? i : i - nq;
+    const int head = dim_shift >= 0 ? quad >> dim_shift : quad / dq, c = (quad - head * dq) * 4;
+    float4 out = v[j];
+    if (c < p.rot_dims) {
+      const bool first = c < half;
+      const int at = first ? c : c - half;
+      const float4 other = *reinterpret_cast<const float4*>(normed + i * 4 + (first ? half : -half));
+      const float4 cs = *reinterpret_cast<const float4*>(cosine + at);
+      float4 sn = *reinterpret_cast<const float4*>(sine + at);
+      if (first) sn = make_float4(-sn.x, -sn.y, -sn.z, -sn.w);
+      out = make_float4(out.x * cs.x + other.x * sn.x, out.y * cs.y + other.y * sn.y, out.z * cs.z + other.z * sn.z,
+                        out.w * cs.w + other.w * sn.w);
+    }
+    write_quad<T>((i < nq ? q_out : k_out) + head * p.size + c, out);
+  }
+  // zeros behind every head's dim / vdim
+  if (p.size > p.dim) {
+    const int pad = (p.size - p.dim) / 4;
+    for (int i = threadIdx.x; i < p.heads * pad; i += blockDim.x)
+      write_quad<T>(q_out + i / pad * p.size + p.dim + i % pad * 4, make_float4(0.0f, 0.0f, 0.0f, 0.0f));
+    for (int i = threadIdx.x; kv && inside && i < p.kv_heads * pad; i += blockDim.x)
+      write_quad<T>(k_out + i / pad * p.size + p.dim + i % pad * 4, make_float4(0.0f, 0.0f, 0.0f, 0.0f));
+  }
+  if (kv && inside && p.size > p.vdim) {
+    const int pad = (p.size - p.vdim) / 4;
+    for (int i = threadIdx.x; i < p.kv_heads * pad; i += blockDim.x)
+      write_quad<T>(v_out + i / pad * p.size + p.vdim + i % pad * 4, make_float4(0.0f, 0.0f, 0.0f, 0.0f));
   }
 }
 
@@ -240,19 +339,41 @@ extern "C" int b200_attention_prep(const b200_attention_prep_inputs* in, int dty
                         static_cast<int>(in->vdim), static_cast<int>(in->row_size), static_cast<int>(in->rot_dims),
                         static_cast<int>(in->q_column), static_cast<int>(in->k_column), static_cast<int>(in->v_column),
                         static_cast<int>(in->splits), in->row_stride, in->capacity, static_cast<float>(in->epsilon), status};
-  const bool quads = in->dim % 4 == 0 && (!kv || in->vdim % 4 == 0) && in->row_size % 4 == 0 && in->q_column % 4 == 0 &&
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const bool whole = in->dim % 4 == 0 && (!kv || in->vdim % 4 == 0) && in->row_size % 4 == 0 && in->q_column % 4 == 0 &&
                      in->k_column % 4 == 0 && in->v_column % 4 == 0 && in->row_stride % 4 == 0 && aligned16(in->input) &&
-                     aligned16(in->q_out) && aligned16(in->keys) && aligned16(in->values);
+                     aligned16(in->bias) && aligned16(in->q_weight) && aligned16(in->k_weight) && aligned16(in->q_out) &&
+                     aligned16(in->keys) && aligned16(in->values);
+  const int64_t quads = (in->heads * in->dim + (kv ? in->kv_heads * (in->dim + in->vdim) : 0)) / 4;
+  const int64_t quads_smem = (in->heads * in->dim + (kv ? in->kv_heads * in->dim : 0) + in->rot_dims) * static_cast<int64_t>(sizeof(float));
+  if (whole && in->rot_dims % 8 == 0 && quads <= 4096 && quads_smem <= 200 * 1024) {
+    int shift = 0;
+    while ((int64_t{4} << shift) < in->dim) ++shift;
+    if ((int64_t{4} << shift) != in->dim) shift = -1;
+    // few rows: a thread per quad or two; many: CTAs of a few warps, four quads a thread
+    const int64_t q = quads > 2048 ? 8 : in->rows <= 2 * kNumSMs && quads <= 1024 ? 2 : 4;
+    const int64_t threads = ceil_div(ceil_div(quads, q), 32) * 32;
+    auto go = [&](auto kernel) {
+      if (quads_smem > 48 * 1024 &&
+          cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(quads_smem)) != cudaSuccess)
+        return B200_ERR_LAUNCH;
+      return launch_chained(kernel, dim3(static_cast<unsigned>(in->rows)), dim3(static_cast<unsigned>(threads)),
+                            static_cast<size_t>(quads_smem), s, p, shift) == cudaSuccess ? launch_status() : B200_ERR_LAUNCH;
+    };
+    if (dtype == B200_F32) return q == 2 ? go(attention_prep_quads_kernel<float, 2>) : q == 4 ? go(attention_prep_quads_kernel<float, 4>)
+                                                                                           : go(attention_prep_quads_kernel<float, 8>);
+    return q == 2 ? go(attention_prep_quads_kernel<__nv_bfloat16, 2>) : q == 4 ? go(attention_prep_quads_kernel<__nv_bfloat16, 4>)
+                                                                              : go(attention_prep_quads_kernel<__nv_bfloat16, 8>);
+  }
   const dim3 grid(static_cast<unsigned>(in->rows), kv ? 2u : 1u);
   auto go = [&](auto kernel) {
     if (smem > 48 * 1024 &&
         cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)) != cudaSuccess)
       return B200_ERR_LAUNCH;
-    return launch_chained(kernel, grid, dim3(256), static_cast<size_t>(smem), static_cast<cudaStream_t>(stream), p) == cudaSuccess
-               ? launch_status() : B200_ERR_LAUNCH;
+    return launch_chained(kernel, grid, dim3(256), static_cast<size_t>(smem), s, p) == cudaSuccess ? launch_status()
+                                                                                                    : B200_ERR_LAUNCH;
   };
-  if (dtype == B200_F32) return quads ? go(attention_prep_kernel<float, 4>) : go(attention_prep_kernel<float, 1>);
-  return quads ? go(attention_prep_kernel<__nv_bfloat16, 4>) : go(attention_prep_kernel<__nv_bfloat16, 1>);
+  return dtype == B200_F32 ? go(attention_prep_kernel<float>) : go(attention_prep_kernel<__nv_bfloat16>);
 }
 
 extern "C" int b200_slot_attention(const void* q, const void* keys, const void* values, void* out,

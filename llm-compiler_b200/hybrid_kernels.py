@@ -546,76 +546,96 @@ def slot_attention(q: torch.Tensor, keys: torch.Tensor, values: torch.Tensor, ba
 
 
 @dataclass
-class SortedRows:
-    """Rows of a step sorted by the experts they go to: `rows` [sorted rows, columns], the choices' scores,
-    the table of tiles (expert, rows held) and, for every choice of every row, its place."""
+class ExpertOrder:
+    """The rows of a step in the order of the experts they go to: for every sorted row its row (`index`) and
+    score, the table of tiles (expert, rows held) and, for every row, its sorted rows (`places`)."""
 
-    rows: torch.Tensor
+    index: torch.Tensor
     scores: torch.Tensor
     tiles: torch.Tensor
     places: torch.Tensor
     tile: int
+    chosen: torch.Tensor  # [rows, top]
+    chosen_scores: torch.Tensor
 
 
-def expert_route(logits: torch.Tensor, counts: torch.Tensor, *, top: int):
-    """The `top` experts of every row and their sigmoid scores (both [rows, top]), and each choice's number
-    among its expert's. logits: fp32 [rows, >= experts] or split-K partials of them; counts: int32
-    [experts], zero before."""
-
-    device = _require_cuda(logits, counts)
-    if logits.dtype != torch.float32 or not logits.is_contiguous() or counts.dtype != torch.int32:
-        raise ValueError("the router's logits are contiguous fp32, the counts int32")
-    splits = logits.shape[0] if logits.ndim == 3 else 1
-    rows = logits.shape[-2]
-    chosen = torch.empty((rows, top), dtype=torch.int32, device=device)
-    scores = torch.empty((rows, top), dtype=torch.float32, device=device)
-    numbers = torch.empty_like(chosen)
-    rt = runtime(device)
-    code = _lib.load().b200_expert_route(logits.data_ptr(), chosen.data_ptr(), scores.data_ptr(), numbers.data_ptr(),
-                                         counts.data_ptr(), rows, counts.shape[0], top, splits, logits.shape[-1], _stream())
-    _check(code, "b200_expert_route")
-    _count(rt)
-    return chosen, scores, numbers
-
-
-def expert_place(h: torch.Tensor, chosen: torch.Tensor, scores: torch.Tensor, numbers: torch.Tensor,
-                 counts: torch.Tensor, *, tile: int) -> SortedRows:
-    """The rows of h sorted by expert, every expert starting at a multiple of `tile` rows."""
-
-    device = _require_cuda(h, chosen, scores, numbers, counts)
-    _require_rows(h, "the rows")
-    rows, top = chosen.shape
-    experts, columns = counts.shape[0], h.shape[1]
-    max_tiles = rows * top // tile + min(experts, rows * top)
-    placed = SortedRows(torch.empty((max_tiles * tile, columns), dtype=h.dtype, device=device),
+def _expert_order(rows: int, counters: torch.Tensor, top: int, always: int, tile: int):
+    experts, device = counters.shape[0] - 1, counters.device
+    if counters.dtype != torch.int32 or not 0 < top <= experts:
+        raise ValueError("a row takes some of the experts; counters are int32 [experts + 1]")
+    max_tiles = always * -(-rows // tile) + rows * top // tile + min(experts, rows * top)
+    int32 = dict(dtype=torch.int32, device=device)
+    order = ExpertOrder(torch.empty(max_tiles * tile, **int32),
                         torch.empty(max_tiles * tile, dtype=torch.float32, device=device),
-                        torch.empty((max_tiles, 2), dtype=torch.int32, device=device), torch.empty_like(chosen), tile)
+                        torch.empty((max_tiles, 2), **int32), torch.empty((rows, always + top), **int32), tile,
+                        torch.empty((rows, top), **int32), torch.empty((rows, top), dtype=torch.float32, device=device))
+    numbers = torch.empty((rows, top), **int32)
+    block = _lib.ExpertOrder(order.chosen.data_ptr(), order.chosen_scores.data_ptr(), numbers.data_ptr(),
+                             counters.data_ptr(), order.places.data_ptr(), order.index.data_ptr(),
+                             order.scores.data_ptr(), order.tiles.data_ptr(), experts, top, always, tile, max_tiles)
+    block.tensors = (order, numbers, counters)
+    return order, block
+
+
+def expert_select(h: torch.Tensor, router: torch.Tensor, counters: torch.Tensor, *, top: int, always: int,
+                  tile: int) -> ExpertOrder:
+    """The `top` experts of a few rows h by the router [>= experts, columns of h], in one launch. `always`
+    more experts, numbered behind the others, take every row with score 1. counters: int32 [experts + 1],
+    zero, and zero again behind the call."""
+
+    device = _require_cuda(h, router, counters)
+    _require_rows(h, "the rows")
+    if router.shape[1] != h.shape[1] or router.shape[0] < counters.shape[0] - 1 or router.dtype != h.dtype or \
+            not router.is_contiguous():
+        raise ValueError("the router needs a contiguous row of h's columns for every expert")
+    order, block = _expert_order(h.shape[0], counters, top, always, tile)
     rt = runtime(device)
-    code = _lib.load().b200_expert_place(
-        h.data_ptr(), chosen.data_ptr(), scores.data_ptr(), numbers.data_ptr(), counts.data_ptr(),
-        placed.places.data_ptr(), placed.rows.data_ptr(), placed.scores.data_ptr(), placed.tiles.data_ptr(), rows,
-        experts, top, tile, max_tiles, columns, h.stride(0), _code(h.dtype), _stream())
-    _check(code, "b200_expert_place")
+    _check(_lib.load().b200_expert_select(h.data_ptr(), router.data_ptr(), byref(block), h.shape[0], h.shape[1],
+                                          h.stride(0), _code(h.dtype), _stream()), "b200_expert_select")
     _count(rt)
-    return placed
+    return order
 
 
-def grouped_linear(x: torch.Tensor, weight: torch.Tensor, placed: SortedRows, *, swiglu: bool = False,
-                   clear: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """out[r] = weight[expert of r] x[r] over sorted rows; weight [experts, n, k]. swiglu: the rows of a
-    weight alternate gate and up, and the result is silu(s gate) * (s up) with the row's score s. `clear`: an
-    int32 vector set to zero on the way."""
+def expert_route(logits: torch.Tensor, h: torch.Tensor, counters: torch.Tensor, *, top: int, always: int,
+                 tile: int) -> Tuple[ExpertOrder, torch.Tensor]:
+    """The same for many rows from finished logits: fp32 [rows, >= experts] or split-K partials of them. Also
+    returns the rows of h in their order."""
 
-    device = _require_cuda(x, weight, placed.tiles, clear)
+    device = _require_cuda(logits, h, counters)
+    _require_rows(h, "the rows")
+    rows = logits.shape[-2]
+    if logits.dtype != torch.float32 or not logits.is_contiguous() or h.shape[0] != rows:
+        raise ValueError("the router's logits are contiguous fp32, a row for every row of h")
+    order, block = _expert_order(rows, counters, top, always, tile)
+    ordered = torch.empty((order.index.shape[0], h.shape[1]), dtype=h.dtype, device=device)
+    rt = runtime(device)
+    library = _lib.load()
+    _check(library.b200_expert_route(logits.data_ptr(), byref(block), rows, logits.shape[0] if logits.ndim == 3 else 1,
+                                     logits.shape[-1], _stream()), "b200_expert_route")
+    _check(library.b200_expert_place(byref(block), h.data_ptr(), ordered.data_ptr(), rows, h.shape[1], h.stride(0),
+                                     _code(h.dtype), _stream()), "b200_expert_place")
+    _count(rt, 2)
+    return order, ordered
+
+
+def grouped_linear(x: torch.Tensor, weight: torch.Tensor, order: ExpertOrder, *, gather: bool = False,
+                   swiglu: bool = False) -> torch.Tensor:
+    """out[r] = weight[expert of r] x[r] over sorted rows; weight [experts, n, k]. gather: x holds the step's
+    rows themselves, not sorted (at most `order.tile` of them). swiglu: the rows of a weight alternate gate and up, and the result is
+    silu(s gate) * (s up) with the row's score s."""
+
+    device = _require_cuda(x, weight, order.tiles)
     experts, n, k = weight.shape
-    if not (x.is_contiguous() and weight.is_contiguous()) or x.shape != (placed.rows.shape[0], k) or x.dtype != weight.dtype:
-        raise ValueError("grouped_linear needs contiguous sorted rows and weights [experts, n, k] of one dtype")
-    output = torch.empty((x.shape[0], n // 2 if swiglu else n), dtype=x.dtype, device=device)
+    sorted_rows = order.index.shape[0]
+    if not (x.is_contiguous() and weight.is_contiguous()) or x.ndim != 2 or x.shape[1] != k or x.dtype != weight.dtype or \
+            x.shape[0] != (order.places.shape[0] if gather else sorted_rows):
+        raise ValueError("grouped_linear needs contiguous rows and weights [experts, n, k] of one dtype")
+    output = torch.empty((sorted_rows, n // 2 if swiglu else n), dtype=x.dtype, device=device)
     rt = runtime(device)
     code = _lib.load().b200_grouped_linear(
-        x.data_ptr(), weight.data_ptr(), placed.tiles.data_ptr(), placed.scores.data_ptr() if swiglu else None,
-        output.data_ptr(), _ptr(clear), 0 if clear is None else clear.numel(), experts, placed.tile,
-        placed.tiles.shape[0], k, n, _lib.EPILOGUE_SWIGLU if swiglu else _lib.EPILOGUE_NONE, _code(x.dtype),
+        x.data_ptr(), weight.data_ptr(), order.tiles.data_ptr(), order.index.data_ptr() if gather else None,
+        order.scores.data_ptr() if swiglu else None, output.data_ptr(), experts, order.tile, order.tiles.shape[0],
+        x.shape[0], k, n, _lib.EPILOGUE_SWIGLU if swiglu else _lib.EPILOGUE_NONE, _code(x.dtype),
         rt.status.data_ptr(), _stream())
     _check(code, "b200_grouped_linear")
     _count(rt)

@@ -13,7 +13,7 @@ from typing import Dict, Iterator, List, Optional, Tuple
 import torch
 
 from .hybrid_config import ConfigError
-from .mixers import Attention, ExpertMlp, GatedMlp, HeadDelta, HybridLayer, Mixer
+from .mixers import Attention, ExpertMlp, HeadDelta, HybridLayer, Mixer
 
 ARCHITECTURE = "Lozanex"
 
@@ -181,7 +181,7 @@ def build_layers(config: LozanexConfig, weights: Dict[str, torch.Tensor]) -> Lis
         layer = HybridLayer(mixer, None, weights[p + "norm1"])
         if spec.mlp is not None:
             part = lambda prefix: {name: weights[f"{p}mlp.{prefix}.{name}"] for name in ("gate", "up", "down")}
-            shared = None if spec.mlp.get("shared") is None else GatedMlp(part("shared"), width=width)
+            shared = None if spec.mlp.get("shared") is None else part("shared")
             layer.mlp = ExpertMlp(weights[p + "mlp.router"], [part(f"e{e}") for e in range(spec.mlp["router"]["experts"])],
                                   width=width, top=spec.mlp["router"]["top"], shared=shared)
             layer.mlp_norm_out = weights[p + "norm2"]

@@ -374,38 +374,58 @@ class GatedMlp:
 
 class ExpertMlp:
     """Mixture of experts: sigmoid scores of a router, the `top` best experts per token, every expert a gated
-    MLP on the token scaled by its score; a shared gated MLP (None: none) runs for every token."""
+    MLP on the token scaled by its score; a shared gated MLP (None: none) runs for every token.
+
+    A gated MLP is the sum of its slices along the feed-forward width, so at decode sizes the shared one
+    runs as a few more experts of the others' size that take every token with score 1 (its weights stand
+    behind theirs); for prompts it is a dense product."""
 
     def __init__(self, router: torch.Tensor, experts: Sequence[Dict[str, torch.Tensor]], *, width: int, top: int,
-                 shared: Optional["GatedMlp"] = None) -> None:
-        self.top, self.shared, self.experts = top, shared, len(experts)
+                 shared: Optional[Dict[str, torch.Tensor]] = None) -> None:
+        self.top, self.experts = top, len(experts)
         self.w_router = pad_matrix(router, pad8(len(experts)), pad8(width))
         ff = pad8(experts[0]["gate"].shape[0])
+        shared_ff = 0 if shared is None else pad8(shared["gate"].shape[0])
+        self.slices = -(-shared_ff // ff)
         like = dict(dtype=router.dtype, device=router.device)
-        self.w_in = torch.empty((len(experts), 2 * ff, pad8(width)), **like)
-        self.w_out = torch.empty((len(experts), pad8(width), ff), **like)
+        self.w_in = torch.zeros((len(experts) + self.slices, 2 * ff, pad8(width)), **like)
+        self.w_out = torch.zeros((len(experts) + self.slices, pad8(width), ff), **like)
         for i, expert in enumerate(experts):
-            self.w_in[i].copy_(kernels.interleave_gate_up(pad_matrix(expert["gate"], ff, pad8(width)),
-                                                          pad_matrix(expert["up"], ff, pad8(width))))
-            self.w_out[i].copy_(pad_matrix(expert["down"], pad8(width), ff))
-        self.counts = torch.zeros(len(experts), dtype=torch.int32, device=router.device)  # zero between calls
+            mlp = GatedMlp(expert, width=width)
+            self.w_in[i].copy_(mlp.w_in)
+            self.w_out[i].copy_(mlp.w_out)
+        self.shared = None
+        if shared is not None:
+            self.shared = GatedMlp(shared, width=width)
+            flat = self.w_in[len(experts):].view(-1, pad8(width))[:2 * shared_ff]
+            flat.copy_(self.shared.w_in)
+            self.shared.w_in = flat  # (one copy serves both forms)
+            for i in range(self.slices):
+                part = self.shared.w_out[:, i * ff:(i + 1) * ff]
+                self.w_out[len(experts) + i, :, :part.shape[1]].copy_(part)
+        self.counters = torch.zeros(len(experts) + 1, dtype=torch.int32, device=router.device)  # zero between calls
 
     def tile_of(self, rows: int) -> int:
-        """Rows of a tile: near the average number of rows an expert gets."""
+        """Rows of a tile: at decode sizes every row (only those that it holds cost anything), else near the
+        average number of rows an expert gets."""
 
-        average = rows * self.top / self.experts
-        return next((tile for tile, most in ((16, 12), (32, 24), (64, 56), (128, 160)) if average <= most), 256)
+        if rows <= PARTIAL_ROWS:
+            return 64 if rows <= 64 else 128
+        return 128 if rows * self.top <= 160 * self.experts else 256
 
     def __call__(self, h: torch.Tensor) -> Summands:
-        if h.dtype == torch.bfloat16:  # (fp32 results either way)
-            logits = kernels.b200_linear_partial(h, self.w_router)
+        rows = h.shape[0]
+        tile, few = self.tile_of(rows), rows <= PARTIAL_ROWS
+        ordered = h
+        if few:
+            order = hk.expert_select(h, self.w_router, self.counters, top=self.top, always=self.slices, tile=tile)
         else:
-            logits = kernels.b200_linear(h, self.w_router)
-        placed = hk.expert_place(h, *hk.expert_route(logits, self.counts, top=self.top), self.counts,
-                                 tile=self.tile_of(h.shape[0]))
-        inner = hk.grouped_linear(placed.rows, self.w_in, placed, swiglu=True, clear=self.counts)
-        return Summands(None if self.shared is None else self.shared(h), None,
-                        hk.grouped_linear(inner, self.w_out, placed), placed.places)
+            logits = kernels.b200_linear_partial(h, self.w_router) if h.dtype == torch.bfloat16 \
+                else kernels.b200_linear(h, self.w_router)  # (fp32 results either way)
+            order, ordered = hk.expert_route(logits, h, self.counters, top=self.top, always=0, tile=tile)
+        inner = hk.grouped_linear(ordered, self.w_in, order, gather=few, swiglu=True)
+        return Summands(None if few or self.shared is None else self.shared(h), None,
+                        hk.grouped_linear(inner, self.w_out, order), order.places)
 
 
 @dataclass

@@ -80,7 +80,16 @@ def test_weights_are_checked_and_packed():
     mixed = oracle.silu(inner[:, 0::2]) * inner[:, 1::2]
     want = oracle.dense_mlp({name: weights["l0.mlp.e2." + name] for name in ("gate", "up", "down")}, h)
     assert torch.allclose((mixed @ experts.w_out[2].T)[:, :20], want, atol=1e-4)
-    assert [experts.tile_of(rows) for rows in (1, 30, 60, 200, 5000)] == [16, 32, 64, 128, 256]
+    assert [experts.tile_of(rows) for rows in (1, 64, 65, 128, 129, 5000)] == [64, 64, 128, 128, 128, 256]
+    # the shared expert in slices of the others' size: their sum is the whole
+    assert experts.slices == 2 and experts.w_in.shape[0] == 6
+    parts = [((oracle.silu(inner[:, 0::2]) * inner[:, 1::2]) @ experts.w_out[e].T)[:, :20]
+             for e in (4, 5) for inner in (rows @ experts.w_in[e].T,)]
+    shared = {name: weights["l0.mlp.shared." + name] for name in ("gate", "up", "down")}
+    assert torch.allclose(sum(parts), oracle.dense_mlp(shared, h), atol=1e-4)
+    inner = rows @ experts.shared.w_in.T
+    dense = (oracle.silu(inner[:, 0::2]) * inner[:, 1::2]) @ experts.shared.w_out.T
+    assert torch.allclose(dense[:, :20], oracle.dense_mlp(shared, h), atol=1e-4)
 
 
 # ------------------------------------------------------- the plain implementation itself ----

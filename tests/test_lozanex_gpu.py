@@ -16,7 +16,7 @@ from llm_compiler_b200 import hybrid_kernels as hk
 from llm_compiler_b200 import kernels, lozanex
 from llm_compiler_b200.cli import main
 from llm_compiler_b200.hybrid_engine import HybridEngine
-from llm_compiler_b200.mixers import Attention, ExpertMlp, GatedMlp, HeadDelta
+from llm_compiler_b200.mixers import Attention, ExpertMlp, HeadDelta
 from llm_compiler_b200.registry import load_model
 from llm_compiler_b200.safetensors_io import save_safetensors
 from llm_compiler_b200.scheduler import RequestScheduler
@@ -341,7 +341,7 @@ EXPERT_WIDTHS = [40, 264, 36, 72, 50]
 def expert_mlp(spec, weights, width):
     w = cuda(weights)
     part = lambda prefix: {name: w[f"{prefix}.{name}"] for name in ("gate", "up", "down")}
-    shared = None if spec["shared"] is None else GatedMlp(part("shared"), width=width)
+    shared = None if spec["shared"] is None else part("shared")
     return ExpertMlp(w["router"], [part(f"e{e}") for e in range(spec["router"]["experts"])], width=width,
                      top=spec["router"]["top"], shared=shared)
 
@@ -360,19 +360,20 @@ def padded(h, width):
 @BOTH
 @pytest.mark.parametrize("index", range(len(EXPERTS)))
 def test_mixture_of_experts(dtype, index):
-    """Row counts that take every tile size, called one after the other: the counters are zero again."""
+    """Decode sizes (one launch for the choice, the shared expert as slices) and prompts, called one after the
+    other: the counters are zero again."""
     spec, width = EXPERTS[index], EXPERT_WIDTHS[index]
     weights = expert_weights(index, dtype)
     mlp = expert_mlp(spec, weights, width)
     tiles = set()
-    for rows in (1, 20, 50, 130, 700):
+    for rows in (1, 20, 64, 65, 128, 129, 700):
         h = random_rows(rows, width, dtype, rows)
         got = summed(mlp(padded(h, width)))[:, :width]
         tiles.add(mlp.tile_of(rows))
         close(got, oracle.expert_mlp(double(weights), spec, h.double()), dtype)
-        assert torch.all(mlp.counts == 0)
+        assert torch.all(mlp.counters == 0)
     kernels.runtime().check_status()
-    assert index != 2 or len(tiles) == 5
+    assert len(tiles) >= 2
 
 
 @BOTH
@@ -395,43 +396,96 @@ def test_every_token_to_one_expert_and_a_score_that_matters(dtype):
 @pytest.mark.parametrize("tile", [16, 32, 64, 128, 256])
 @pytest.mark.parametrize("n,k", [(400, 136), (48, 24), (256, 512)])
 def test_grouped_linear_tiles(tile, n, k):
-    """Every tile size against plain products: experts without rows, with one, with a tile exactly, with more."""
+    """Every tile size against plain products: experts without rows, with one, with a tile
+    exactly, with more, and two that take every row."""
     g = torch.Generator().manual_seed(tile + n)
     held = [0, 1, tile, tile + 1, 0, 3 * tile - 1, 5]
     chosen = torch.cat([torch.full((c,), e, dtype=torch.int32) for e, c in enumerate(held)])
-    chosen = chosen[torch.randperm(len(chosen), generator=g)][:, None].contiguous()
-    counts = torch.zeros(len(held), dtype=torch.int32, device="cuda")
-    logits = torch.full((len(chosen), 8), -9.0)
-    logits[torch.arange(len(chosen)), chosen[:, 0].long()] = torch.randn(len(chosen), generator=g)
-    picked, scores, numbers = hk.expert_route(logits.cuda()[:, :7].contiguous(), counts, top=1)
-    assert torch.equal(picked.cpu(), chosen) and counts.tolist() == held
-    assert torch.allclose(scores.cpu()[:, 0], torch.sigmoid(logits.amax(1)), atol=1e-6)
-    x = torch.randn(len(chosen), k, generator=g).to(torch.bfloat16)
-    w = (torch.randn(7, n, k, generator=g) * k ** -0.5).to(torch.bfloat16)
-    placed = hk.expert_place(x.cuda(), picked, scores, numbers, counts, tile=tile)
-    places = placed.places.long()[:, 0]
-    assert len(set(places.tolist())) == len(chosen) and torch.equal(placed.rows[places].cpu(), x)
-    products = torch.einsum("rnk,rk->rn", w.double()[chosen[:, 0].long()], x.double())
-    close(hk.grouped_linear(placed.rows, w.cuda(), placed, clear=counts)[places], products, torch.bfloat16)
-    assert torch.all(counts == 0)
-    s = scores.double().cpu()
-    want = oracle.silu(s * products[:, 0::2]) * (s * products[:, 1::2])
-    close(hk.grouped_linear(placed.rows, w.cuda(), placed, swiglu=True)[places], want, torch.bfloat16)
+    chosen = chosen[torch.randperm(len(chosen), generator=g)].long()
+    rows = len(chosen)
+    logits = torch.full((rows, 8), -9.0)
+    logits[torch.arange(rows), chosen] = torch.randn(rows, generator=g)
+    logits[:, 7] = 50.0  # (no expert: a column of padding)
+    counters = torch.zeros(8, dtype=torch.int32, device="cuda")
+    x = torch.randn(rows, k, generator=g).to(torch.bfloat16).cuda()
+    order, ordered = hk.expert_route(logits.cuda(), x, counters, top=1, always=2, tile=tile)
+    assert torch.all(counters == 0) and torch.equal(order.chosen.cpu()[:, 0].long(), chosen)
+    assert torch.allclose(order.chosen_scores.cpu()[:, 0], torch.sigmoid(logits[torch.arange(rows), chosen]), atol=1e-6)
+    places = order.places.long()
+    assert places.shape == (rows, 3) and len(set(places.flatten().tolist())) == 3 * rows
+    assert torch.equal(order.index[places], torch.arange(rows, device="cuda", dtype=torch.int32)[:, None].expand(-1, 3))
+    table = order.tiles.tolist()
+    used = [t for t in table if t[0] >= 0]
+    assert table[len(used):] == [[-1, 0]] * (len(table) - len(used))
+    assert [sum(count for e, count in used if e == expert) for expert in range(9)] == held + [rows, rows]
+    w = (torch.randn(9, n, k, generator=g) * k ** -0.5).to(torch.bfloat16).cuda()
+    assert torch.equal(ordered[places], x[:, None].expand(-1, 3, -1))
+    unheld = torch.ones(ordered.shape[0], dtype=torch.bool, device="cuda")
+    unheld[places.flatten()] = False
+    ordered[unheld] = float("nan")  # rows that no tile holds hold anything
+    experts = torch.stack([torch.full_like(chosen, 7), torch.full_like(chosen, 8), chosen], 1)
+    products = torch.einsum("rjnk,rk->rjn", w.double().cpu()[experts], x.double().cpu())
+    scores = order.scores[places].double().cpu()[:, :, None]
+    assert torch.all(scores[:, :2] == 1)
+    gated = oracle.silu(scores * products[..., 0::2]) * (scores * products[..., 1::2])
+    for swiglu, want in ((False, products), (True, gated)):
+        got = hk.grouped_linear(ordered, w, order, swiglu=swiglu)[places]
+        close(got.flatten(0, 1), want.flatten(0, 1), torch.bfloat16)
     kernels.runtime().check_status()
 
 
-def test_routing_over_partial_sums_picks_the_largest():
+@BOTH
+@pytest.mark.parametrize("rows,experts,top,width", [(1, 5, 1, 40), (70, 99, 5, 136), (128, 3, 3, 264), (17, 300, 12, 1032)])
+def test_choice_in_one_launch(dtype, rows, experts, top, width):
+    """The router's products, the choice and the order against sorted logits of double precision."""
+    g = torch.Generator().manual_seed(rows)
+    h = torch.randn(rows, width, generator=g).to(dtype)
+    router = (torch.randn(experts, width, generator=g) * width ** -0.5).to(dtype)
+    counters = torch.zeros(experts + 1, dtype=torch.int32, device="cuda")
+    logits = h.double() @ router.double().T
+    want = torch.topk(logits, top, dim=-1)
+    for always in (0, 2):
+        order = hk.expert_select(h.cuda(), router.cuda(), counters, top=top, always=always, tile=16)
+        assert torch.equal(order.chosen.cpu().long(), want.indices) and torch.all(counters == 0)
+        assert torch.allclose(order.chosen_scores.cpu().double(), torch.sigmoid(want.values), atol=1e-6)
+        places = order.places.long()
+        assert len(set(places.flatten().tolist())) == rows * (top + always)
+        assert torch.equal(order.index[places[:, -1]].cpu(), torch.arange(rows, dtype=torch.int32))
+        own = order.tiles[places // 16].cpu()
+        assert torch.equal(own[:, always:, 0].long(), want.indices)
+        assert own[:, :always, 0].tolist() == [list(range(experts, experts + always))] * rows
+        assert torch.all(places.cpu() % 16 < own[..., 1])
+        assert torch.equal(order.scores[places[:, always:]], order.chosen_scores)
+
+
+@BOTH
+@pytest.mark.parametrize("rows,tile", [(1, 16), (16, 16), (33, 64), (64, 64), (100, 128), (128, 128), (200, 256)])
+def test_products_of_unsorted_rows(dtype, rows, tile):
+    """Decode sizes: every item multiplies all rows, a tile keeps those that it holds."""
+    g = torch.Generator().manual_seed(rows)
+    h = torch.randn(rows, 136, generator=g).to(dtype).cuda()
+    router = (torch.randn(11, 136, generator=g) * 0.1).to(dtype).cuda()
+    counters = torch.zeros(12, dtype=torch.int32, device="cuda")
+    order = hk.expert_select(h, router, counters, top=3, always=2, tile=tile)
+    w = (torch.randn(13, 272, 136, generator=g) * 0.1).to(dtype).cuda()
+    experts = torch.cat([torch.tensor([[11, 12]]).expand(rows, -1), order.chosen.cpu().long()], 1)
+    products = torch.einsum("rjnk,rk->rjn", w.double().cpu()[experts], h.double().cpu())
+    scores = order.scores[order.places.long()].double().cpu()[:, :, None]
+    gated = oracle.silu(scores * products[..., 0::2]) * (scores * products[..., 1::2])
+    for swiglu, want in ((False, products), (True, gated)):
+        got = hk.grouped_linear(h, w, order, gather=True, swiglu=swiglu)[order.places.long()]
+        close(got.flatten(0, 1), want.flatten(0, 1), dtype)
+    kernels.runtime().check_status()
+
+
+def test_choice_over_partial_sums():
     g = torch.Generator().manual_seed(0)
     parts = torch.randn(3, 70, 104, generator=g)
-    counts = torch.zeros(99, dtype=torch.int32, device="cuda")
-    chosen, scores, numbers = hk.expert_route(parts.cuda(), counts, top=5)
-    total = parts.sum(0)[:, :99]
-    want = torch.topk(total, 5, dim=-1)
-    assert torch.equal(chosen.cpu().long(), want.indices)
-    assert torch.allclose(scores.cpu(), torch.sigmoid(want.values), atol=1e-6)
-    assert torch.equal(counts.cpu(), torch.bincount(want.indices.flatten(), minlength=99).int())
-    taken = {(e, n) for e, n in zip(chosen.flatten().tolist(), numbers.flatten().tolist())}
-    assert len(taken) == 350 and all(n < counts[e] for e, n in taken)
+    counters = torch.zeros(100, dtype=torch.int32, device="cuda")
+    order, _ = hk.expert_route(parts.cuda(), torch.zeros(70, 8, device="cuda"), counters, top=5, always=0, tile=32)
+    want = torch.topk(parts.sum(0)[:, :99], 5, dim=-1)
+    assert torch.equal(order.chosen.cpu().long(), want.indices) and torch.all(counters == 0)
+    assert torch.allclose(order.chosen_scores.cpu(), torch.sigmoid(want.values), atol=1e-6)
 
 
 # ------------------------------------------------------------------------ whole model ----

@@ -128,16 +128,16 @@ def test_grouped_linear_wait_timeout_then_recovery(tile):
     g = torch.Generator().manual_seed(tile)
     x = torch.randn(40, 136, generator=g).bfloat16()
     w = (0.1 * torch.randn(3, 400, 136, generator=g)).bfloat16()
-    chosen = torch.arange(40, dtype=torch.int32).remainder(3)[:, None]
-    numbers = (torch.arange(40, dtype=torch.int32) // 3)[:, None].contiguous()
-    counts = torch.bincount(chosen[:, 0], minlength=3).to(torch.int32)
-    placed = hk.expert_place(x.cuda(), chosen.cuda(), torch.ones(40, 1).cuda(), numbers.cuda(), counts.cuda(), tile=tile)
+    chosen = torch.arange(40) % 3
+    logits = torch.nn.functional.one_hot(chosen, 4).float()
+    order, ordered = hk.expert_route(logits.cuda(), x.cuda(), torch.zeros(4, dtype=torch.int32, device="cuda"), top=1,
+                                     always=0, tile=tile)
     for _ in range(3):
         with waits_that_run_out():
-            hk.grouped_linear(placed.rows, w.cuda(), placed)
+            hk.grouped_linear(ordered, w.cuda(), order)
         expect_timeout()
-    out = hk.grouped_linear(placed.rows, w.cuda(), placed)[placed.places[:, 0].long()]
-    close(out, torch.einsum("rnk,rk->rn", w.float()[chosen[:, 0].long()], x.float()))
+    out = hk.grouped_linear(ordered, w.cuda(), order)[order.places[:, 0].long()]
+    close(out, torch.einsum("rnk,rk->rn", w.float()[chosen], x.float()))
     kernels.runtime().check_status()
 
 
