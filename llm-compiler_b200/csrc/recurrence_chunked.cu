@@ -115,7 +115,7 @@ __device__ __forceinline__ void solve_chunk(const ChunkParams& p, const __nv_bfl
                                             DecayedKey decayed_key) {
   using Layout = ChunkLayout<D>;
   const int v_row = (p.vdim + 31) / 32 * 32;
-  for (int tile = warp; tile < (D + v_row) / 16; tile += kIntraThreads / 32) {
+  for (int tile = warp; tile < (D + v_row) / 16; tile += blockDim.x / 32) {
     const int c0 = tile * 16 + (lane >> 2);  // fragment rows c0 and c0 + 8 are columns of [W | U]
     float rhs[kSubs][2][4];
 #pragma unroll
@@ -183,14 +183,14 @@ __device__ __forceinline__ void solve_chunk(const ChunkParams& p, const __nv_bfl
     }
   }
   __syncthreads();
-  for (int item = threadIdx.x; item < 2 * kChunk * D / 8; item += kIntraThreads)
+  for (int item = threadIdx.x; item < 2 * kChunk * D / 8; item += blockDim.x)
     reinterpret_cast<uint4*>(out + Layout::kW)[item] = reinterpret_cast<const uint4*>(staging)[item];
 }
 
 // (I + N)^-1 of the 16 x 16 diagonal blocks, one column a thread of the CTA's last 64
 __device__ __forceinline__ void invert_diagonal_blocks(const float* lower, int pitch, __nv_bfloat16* inverse) {
-  if (threadIdx.x < kIntraThreads - kChunk) return;
-  const int column = threadIdx.x - (kIntraThreads - kChunk), block = column / kSub * kSub, own = column % kSub;
+  if (threadIdx.x < blockDim.x - kChunk) return;
+  const int column = threadIdx.x - (blockDim.x - kChunk), block = column / kSub * kSub, own = column % kSub;
   float x[kSub];
 #pragma unroll
   for (int i = 0; i < kSub; ++i) {
@@ -282,8 +282,9 @@ template <int D>
 constexpr int intra_head_delta_smem_bytes() {
   return 4 * kChunk * (D + 8) * 2 + kChunk * (kChunk + 4) * 4 + 2 * kChunk * kTriangle * 2 + 2 * kChunk * kInverse * 2;
 }
+constexpr int kHeadDeltaThreads = 256;  // two CTAs per SM: one's loads and solve under the other's products
 template <int D>
-__global__ void __launch_bounds__(kIntraThreads) chunk_intra_head_delta_kernel(const ChunkParams p) {
+__global__ void __launch_bounds__(kHeadDeltaThreads, 2) chunk_intra_head_delta_kernel(const ChunkParams p) {
   constexpr int PM = kChunk + 4, PB = (D + 8) * 2;
   using Layout = ChunkLayout<D>;
   extern __shared__ __align__(128) unsigned char smem[];
@@ -300,15 +301,17 @@ __global__ void __launch_bounds__(kIntraThreads) chunk_intra_head_delta_kernel(c
   const int kv_head = head / (p.heads / p.kv_heads);
   unsigned char* out = p.workspace + (static_cast<int64_t>(chunk) * p.heads + head) * Layout::bytes(true, p.vdim);
   const bool whole = p.dim == D;
-  constexpr int kRounds = kChunk * D / 4 / kIntraThreads;
-  float4 q[kRounds], k[kRounds];
+  constexpr int kRounds = kChunk * D / 4 / kHeadDeltaThreads;
+  // (the queries' loads are in flight while the decays are summed up, the keys' while the queries are split)
+  auto load_rows = [&](const float* from, float4* rows) {
 #pragma unroll
-  for (int i = 0; i < kRounds; ++i) {
-    const int item = threadIdx.x + i * kIntraThreads, t = item / (D / 4), c = item % (D / 4) * 4;
-    const int64_t source = ((row0 + t) * p.kv_heads + kv_head) * p.dim;
-    q[i] = load4(p.q + source, c, p.dim, t < count, whole);
-    k[i] = load4(p.k + source, c, p.dim, t < count, whole);
-  }
+    for (int i = 0; i < kRounds; ++i) {
+      const int item = threadIdx.x + i * kHeadDeltaThreads, t = item / (D / 4), c = item % (D / 4) * 4;
+      rows[i] = load4(from + ((row0 + t) * p.kv_heads + kv_head) * p.dim, c, p.dim, t < count, whole);
+    }
+  };
+  float4 q[kRounds], k[kRounds];
+  load_rows(p.q, q);
   if (warp == 0) {  // two tokens a lane
     double x[2];
 #pragma unroll
@@ -334,76 +337,86 @@ __global__ void __launch_bounds__(kIntraThreads) chunk_intra_head_delta_kernel(c
   }
   __syncthreads();
   const double end = sums[kChunk - 1];
+  load_rows(p.k, k);
+  auto split_rows = [&](const float4* rows, unsigned char* planes, unsigned char* decayed, auto factor) {
 #pragma unroll
-  for (int i = 0; i < kRounds; ++i) {
-    const int item = threadIdx.x + i * kIntraThreads, t = item / (D / 4), c = item % (D / 4) * 4;
-    const float in = into[t], rest = exp2f(static_cast<float>(end - sums[t]));
-    uint2 high, low;
-    split4(q[i], high, low);
-    *reinterpret_cast<uint2*>(q_planes + t * PB + c * 2) = high;
-    *reinterpret_cast<uint2*>(q_planes + (kChunk + t) * PB + c * 2) = low;
-    split4(k[i], high, low);
-    *reinterpret_cast<uint2*>(k_planes + t * PB + c * 2) = high;
-    *reinterpret_cast<uint2*>(k_planes + (kChunk + t) * PB + c * 2) = low;
-    split4(mul4(q[i], make_float4(in, in, in, in)), high, low);
-    reinterpret_cast<uint2*>(out + Layout::kQ)[item] = high;
-    reinterpret_cast<uint2*>(out + Layout::kQ + Layout::kPlane)[item] = low;
-    split4(mul4(k[i], make_float4(rest, rest, rest, rest)), high, low);
-    reinterpret_cast<uint2*>(out + Layout::kK)[item] = high;
-    reinterpret_cast<uint2*>(out + Layout::kK + Layout::kPlane)[item] = low;
-  }
+    for (int i = 0; i < kRounds; ++i) {
+      const int item = threadIdx.x + i * kHeadDeltaThreads, t = item / (D / 4), c = item % (D / 4) * 4;
+      const float f = factor(t);
+      uint2 high, low;
+      split4(rows[i], high, low);
+      *reinterpret_cast<uint2*>(planes + t * PB + c * 2) = high;
+      *reinterpret_cast<uint2*>(planes + (kChunk + t) * PB + c * 2) = low;
+      split4(mul4(rows[i], make_float4(f, f, f, f)), high, low);
+      reinterpret_cast<uint2*>(decayed)[item] = high;
+      reinterpret_cast<uint2*>(decayed + Layout::kPlane)[item] = low;
+    }
+  };
+  split_rows(q, q_planes, out + Layout::kQ, [&](int t) { return into[t]; });
+  split_rows(k, k_planes, out + Layout::kK, [&](int t) { return exp2f(static_cast<float>(end - sums[t])); });
   if (threadIdx.x < D) reinterpret_cast<float*>(out + Layout::kEnd)[threadIdx.x] = into[kChunk - 1];
   __syncthreads();
-  // 16 warps: 16 rows x 16 columns of K K^T and of Q K^T each
-  const int m0 = (warp >> 2) * 16, n0 = (warp & 3) * 16;
-  float kk[2][4] = {}, qk[2][4] = {};
-  if (n0 <= m0) {
-    const uint32_t row_lane = (m0 + (lane & 15)) * PB + (lane >> 4) * 16;
-    const uint32_t ka_base = smem_u32(k_planes) + row_lane, qa_base = smem_u32(q_planes) + row_lane;
-    const uint32_t b_base = smem_u32(k_planes) + (n0 + ((lane >> 4) << 3) + (lane & 7)) * PB + ((lane >> 3) & 1) * 16;
+  // 16 x 16 tiles of K K^T and of Q K^T: the ten on and below the diagonal, then zeros above it
+  constexpr int kWarps = kHeadDeltaThreads / 32;
+  for (int tile = warp; tile < 16; tile += kWarps) {
+    int m = 0, n = tile;  // row by row below the diagonal; the last six above it
+    if (tile < 10) {
+      while (n > m) n -= ++m;
+    } else {
+      n = tile - 10;
+      while (n >= 3 - m) n -= 3 - m++;
+      n += m + 1;
+    }
+    const int m0 = m * 16, n0 = n * 16;
+    float kk[2][4] = {}, qk[2][4] = {};
+    if (n0 <= m0) {
+      const uint32_t row_lane = (m0 + (lane & 15)) * PB + (lane >> 4) * 16;
+      const uint32_t ka_base = smem_u32(k_planes) + row_lane, qa_base = smem_u32(q_planes) + row_lane;
+      const uint32_t b_base = smem_u32(k_planes) + (n0 + ((lane >> 4) << 3) + (lane & 7)) * PB + ((lane >> 3) & 1) * 16;
 #pragma unroll
-    for (int step = 0; step < D / 16; ++step) {
-      uint32_t kh[4], kl[4], qh[4], ql[4], bh[4], bl[4];
-      ldmatrix_x4(kh, ka_base + step * 32);
-      ldmatrix_x4(kl, ka_base + kChunk * PB + step * 32);
-      ldmatrix_x4(qh, qa_base + step * 32);
-      ldmatrix_x4(ql, qa_base + kChunk * PB + step * 32);
-      ldmatrix_x4(bh, b_base + step * 32);
-      ldmatrix_x4(bl, b_base + kChunk * PB + step * 32);
+      for (int step = 0; step < D / 16; ++step) {
+        uint32_t kh[4], kl[4], qh[4], ql[4], bh[4], bl[4];
+        ldmatrix_x4(kh, ka_base + step * 32);
+        ldmatrix_x4(kl, ka_base + kChunk * PB + step * 32);
+        ldmatrix_x4(qh, qa_base + step * 32);
+        ldmatrix_x4(ql, qa_base + kChunk * PB + step * 32);
+        ldmatrix_x4(bh, b_base + step * 32);
+        ldmatrix_x4(bl, b_base + kChunk * PB + step * 32);
 #pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        mma_bf16_16816(kk[h], kh, bh[h * 2], bh[h * 2 + 1]);
-        mma_bf16_16816(qk[h], qh, bh[h * 2], bh[h * 2 + 1]);
-        mma_bf16_16816(kk[h], kh, bl[h * 2], bl[h * 2 + 1]);
-        mma_bf16_16816(qk[h], qh, bl[h * 2], bl[h * 2 + 1]);
-        mma_bf16_16816(kk[h], kl, bh[h * 2], bh[h * 2 + 1]);
-        mma_bf16_16816(qk[h], ql, bh[h * 2], bh[h * 2 + 1]);
+        for (int h = 0; h < 2; ++h) {
+          mma_bf16_16816(kk[h], kh, bh[h * 2], bh[h * 2 + 1]);
+          mma_bf16_16816(qk[h], qh, bh[h * 2], bh[h * 2 + 1]);
+          mma_bf16_16816(kk[h], kh, bl[h * 2], bl[h * 2 + 1]);
+          mma_bf16_16816(qk[h], qh, bl[h * 2], bl[h * 2 + 1]);
+          mma_bf16_16816(kk[h], kl, bh[h * 2], bh[h * 2 + 1]);
+          mma_bf16_16816(qk[h], ql, bh[h * 2], bh[h * 2 + 1]);
+        }
       }
     }
+#pragma unroll
+    for (int h = 0; h < 2; ++h)
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int i = m0 + (lane >> 2) + half * 8, j = n0 + h * 8 + (lane & 3) * 2;
+        float a[2], l[2];
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const float f = i >= j + e ? exp2f(static_cast<float>(sums[i] - sums[j + e])) : 0.0f;
+          a[e] = qk[h][half * 2 + e] * f;
+          l[e] = i > j + e ? kk[h][half * 2 + e] * f * betas[i] : 0.0f;
+        }
+        uint32_t high, low;
+        split_bf16x2(a[0], a[1], high, low);
+        reinterpret_cast<uint32_t*>(out + Layout::kA)[(i * kChunk + j) / 2] = high;
+        reinterpret_cast<uint32_t*>(out + Layout::kA + Layout::kSquare)[(i * kChunk + j) / 2] = low;
+        if (n0 == m0) *reinterpret_cast<float2*>(lower + i * PM + j) = make_float2(l[0], l[1]);
+        if (n0 < m0) {
+          split_bf16x2(-l[0], -l[1], high, low);
+          *reinterpret_cast<uint32_t*>(triangle + i * kTriangle + j) = high;
+          *reinterpret_cast<uint32_t*>(triangle + (kChunk + i) * kTriangle + j) = low;
+        }
+      }
   }
-#pragma unroll
-  for (int h = 0; h < 2; ++h)
-#pragma unroll
-    for (int half = 0; half < 2; ++half) {
-      const int i = m0 + (lane >> 2) + half * 8, j = n0 + h * 8 + (lane & 3) * 2;
-      float a[2], l[2];
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const float f = i >= j + e ? exp2f(static_cast<float>(sums[i] - sums[j + e])) : 0.0f;
-        a[e] = qk[h][half * 2 + e] * f;
-        l[e] = i > j + e ? kk[h][half * 2 + e] * f * betas[i] : 0.0f;
-      }
-      uint32_t high, low;
-      split_bf16x2(a[0], a[1], high, low);
-      reinterpret_cast<uint32_t*>(out + Layout::kA)[(i * kChunk + j) / 2] = high;
-      reinterpret_cast<uint32_t*>(out + Layout::kA + Layout::kSquare)[(i * kChunk + j) / 2] = low;
-      if (n0 == m0) *reinterpret_cast<float2*>(lower + i * PM + j) = make_float2(l[0], l[1]);
-      if (n0 < m0) {
-        split_bf16x2(-l[0], -l[1], high, low);
-        *reinterpret_cast<uint32_t*>(triangle + i * kTriangle + j) = high;
-        *reinterpret_cast<uint32_t*>(triangle + (kChunk + i) * kTriangle + j) = low;
-      }
-    }
   __syncthreads();
   invert_diagonal_blocks(lower, PM, inverse);
   __syncthreads();
@@ -645,11 +658,13 @@ constexpr int inter_smem_bytes() {
   return (DELTA ? 6 : 4) * kChunk * (D + 8) * 2 + 2 * kChunk * (kChunk + 8) * 2 + 2 * D * (VB + 8) * 2 + 2 * kChunk * (VB + 8) * 2;
 }
 
-// Warps: H = VB / 16 share the columns of a 16-row tile. First product: 4 H warps on W S, 4 H on Q S;
+// Warps: H share the columns of a 16-row tile, 16 C each. First product: 4 H warps on W S, 4 H on Q S;
 // second: D / 16 x H warps on K^T U (their tile of S stays in registers), the last 4 H on A U.
+template <int VB>
+constexpr int kInterThreads = VB <= 32 ? VB * 16 : VB * 8;
 template <int D, int VB, bool DELTA>
-__global__ void __launch_bounds__(VB * 16, 1) chunk_inter_kernel(const ChunkParams p) {
-  constexpr int kThreads = VB * 16, H = VB / 16;
+__global__ void __launch_bounds__(kInterThreads<VB>, 1) chunk_inter_kernel(const ChunkParams p) {
+  constexpr int kThreads = kInterThreads<VB>, C = VB * 16 / kThreads, H = VB / (16 * C), T = 2 * C;  // T: n8 tiles of a warp
   constexpr int PB = (D + 8) * 2, PA = (kChunk + 8) * 2, PV = (VB + 8) * 2;  // byte pitches
   constexpr int kStateTiles = D / 16;
   using Layout = ChunkLayout<D>;
@@ -690,17 +705,17 @@ __global__ void __launch_bounds__(VB * 16, 1) chunk_inter_kernel(const ChunkPara
   load_first(0);
   load_second(0);
 
-  const int half = warp % H;                    // which 16 columns of this CTA's VB
-  const int column = half * 16 + (lane & 3) * 2;  // this lane's first column of n8 tile 0
+  const int half = warp % H;                          // which 16 C columns of this CTA's VB
+  const int column = half * 16 * C + (lane & 3) * 2;  // this lane's first column of n8 tile 0
   const bool reads_out = warp >= 4 * H;         // Q S and A U; else W S and U
   const int tile = warp / H % 4, t_row = tile * 16 + (lane >> 2);
   const bool owns_state = warp / H < kStateTiles;
   const int s_row = warp / H * 16 + (lane >> 2);
   float* state = p.state + (static_cast<int64_t>(slot) * p.heads + head) * p.dim * p.state_row;
   const bool fresh = p.batch.bases[sequence] == 0;
-  auto store_planes = [&](unsigned char* planes_at, int rows, int row, const float (&v)[2][4]) {
+  auto store_planes = [&](unsigned char* planes_at, int rows, int row, const float (*v)[4]) {
 #pragma unroll
-    for (int t = 0; t < 2; ++t)
+    for (int t = 0; t < T; ++t)
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         uint32_t high, low;
@@ -709,10 +724,10 @@ __global__ void __launch_bounds__(VB * 16, 1) chunk_inter_kernel(const ChunkPara
         *reinterpret_cast<uint32_t*>(planes_at + (rows + row + e * 8) * PV + (column + t * 8) * 2) = low;
       }
   };
-  float s[2][4] = {};
+  float s[T][4] = {};
   if (owns_state) {
 #pragma unroll
-    for (int t = 0; t < 2; ++t)
+    for (int t = 0; t < T; ++t)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int r = s_row + (e >> 1) * 8, c = v0 + column + t * 8 + (e & 1);
@@ -721,12 +736,12 @@ __global__ void __launch_bounds__(VB * 16, 1) chunk_inter_kernel(const ChunkPara
     store_planes(s_planes, D, s_row, s);
   }
   const int v_row = (p.vdim + 31) / 32 * 32;
-  float u0[2][4] = {}, end0 = 0.0f, end1 = 0.0f;  // fetched a chunk ahead
+  float u0[T][4] = {}, end0 = 0.0f, end1 = 0.0f;  // fetched a chunk ahead
   auto fetch = [&](int chunk) {
     const int64_t row0 = first + static_cast<int64_t>(chunk) * kChunk;
     if (!reads_out) {
 #pragma unroll
-      for (int t = 0; t < 2; ++t)
+      for (int t = 0; t < T; ++t)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int r = t_row + (e >> 1) * 8, c = v0 + column + t * 8 + (e & 1);
@@ -746,13 +761,13 @@ __global__ void __launch_bounds__(VB * 16, 1) chunk_inter_kernel(const ChunkPara
 
   // acc += A B: A given by its lanes' addresses (planes `a_low` bytes apart, `a_step` bytes a k16 step;
   // transposed when it lies [k][m]), B [k][VB] planes
-  const uint32_t b_lane = (lane & 15) * PV + (lane >> 4) * 16 + half * 32;
-  auto product = [&](float (&acc)[2][4], auto transposed, uint32_t a, int a_low, int a_step, uint32_t b, int b_low,
+  const uint32_t b_lane = (lane & 15) * PV + (lane >> 4) * 16 + half * 32 * C;
+  auto product = [&](float (*acc)[4], auto transposed, uint32_t a, int a_low, int a_step, uint32_t b, int b_low,
                      auto steps) {
-    float cross[2][4] = {};
+    float cross[T][4] = {};
 #pragma unroll
     for (int step = 0; step < decltype(steps)::value; ++step) {
-      uint32_t ah[4], al[4], bh[4], bl[4];
+      uint32_t ah[4], al[4];
       if (decltype(transposed)::value != 0) {
         ldmatrix_x4_trans(ah, a + step * a_step);
         ldmatrix_x4_trans(al, a + a_low + step * a_step);
@@ -760,17 +775,21 @@ __global__ void __launch_bounds__(VB * 16, 1) chunk_inter_kernel(const ChunkPara
         ldmatrix_x4(ah, a + step * a_step);
         ldmatrix_x4(al, a + a_low + step * a_step);
       }
-      ldmatrix_x4_trans(bh, b + step * 16 * PV);
-      ldmatrix_x4_trans(bl, b + b_low + step * 16 * PV);
 #pragma unroll
-      for (int t = 0; t < 2; ++t) {
-        mma_bf16_16816(acc[t], ah, bh[t * 2], bh[t * 2 + 1]);
-        mma_bf16_16816(cross[t], ah, bl[t * 2], bl[t * 2 + 1]);
-        mma_bf16_16816(cross[t], al, bh[t * 2], bh[t * 2 + 1]);
+      for (int c = 0; c < C; ++c) {
+        uint32_t bh[4], bl[4];
+        ldmatrix_x4_trans(bh, b + step * 16 * PV + c * 32);
+        ldmatrix_x4_trans(bl, b + b_low + step * 16 * PV + c * 32);
+#pragma unroll
+        for (int t = 0; t < 2; ++t) {
+          mma_bf16_16816(acc[c * 2 + t], ah, bh[t * 2], bh[t * 2 + 1]);
+          mma_bf16_16816(cross[c * 2 + t], ah, bl[t * 2], bl[t * 2 + 1]);
+          mma_bf16_16816(cross[c * 2 + t], al, bh[t * 2], bh[t * 2 + 1]);
+        }
       }
     }
 #pragma unroll
-    for (int t = 0; t < 2; ++t)
+    for (int t = 0; t < T; ++t)
 #pragma unroll
       for (int e = 0; e < 4; ++e) acc[t][e] += cross[t][e];
   };
@@ -778,14 +797,14 @@ __global__ void __launch_bounds__(VB * 16, 1) chunk_inter_kernel(const ChunkPara
   const uint32_t s_base = smem_u32(s_planes) + b_lane, u_base = smem_u32(u_planes) + b_lane;
   for (int chunk = 0; chunk < chunks; ++chunk) {
     const int64_t row0 = first + static_cast<int64_t>(chunk) * kChunk;
-    float acc[2][4] = {};
+    float acc[T][4] = {};
     if (reads_out) {
       product(acc, IntConstant<0>{}, smem_u32(q_planes) + row_lane, kChunk * PB, 32, s_base, D * PV, IntConstant<D / 16>{});
     } else {
       if (DELTA)
         product(acc, IntConstant<0>{}, smem_u32(w_planes) + row_lane, kChunk * PB, 32, s_base, D * PV, IntConstant<D / 16>{});
 #pragma unroll
-      for (int t = 0; t < 2; ++t)
+      for (int t = 0; t < T; ++t)
 #pragma unroll
         for (int e = 0; e < 4; ++e) acc[t][e] = u0[t][e] - acc[t][e];
       store_planes(u_planes, kChunk, t_row, acc);
@@ -799,7 +818,7 @@ __global__ void __launch_bounds__(VB * 16, 1) chunk_inter_kernel(const ChunkPara
     }
     if (owns_state) {
 #pragma unroll
-      for (int t = 0; t < 2; ++t) {
+      for (int t = 0; t < T; ++t) {
         s[t][0] *= e0; s[t][1] *= e0;
         s[t][2] *= e1; s[t][3] *= e1;
       }
@@ -812,7 +831,7 @@ __global__ void __launch_bounds__(VB * 16, 1) chunk_inter_kernel(const ChunkPara
       product(acc, IntConstant<0>{}, smem_u32(a_planes) + (tile * 16 + (lane & 15)) * PA + (lane >> 4) * 16, kChunk * PA, 32,
               u_base, kChunk * PV, IntConstant<kChunk / 16>{});
 #pragma unroll
-      for (int t = 0; t < 2; ++t)
+      for (int t = 0; t < T; ++t)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int64_t row = row0 + t_row + (e >> 1) * 8;
@@ -826,7 +845,7 @@ __global__ void __launch_bounds__(VB * 16, 1) chunk_inter_kernel(const ChunkPara
   }
   if (owns_state) {
 #pragma unroll
-    for (int t = 0; t < 2; ++t)
+    for (int t = 0; t < T; ++t)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int r = s_row + (e >> 1) * 8, c = v0 + column + t * 8 + (e & 1);
@@ -844,16 +863,22 @@ int launch_chunked(const ChunkParams& p, int64_t chunks, bool head_decay, cudaSt
                                                                         : intra_smem_bytes<D>();
   if (cudaFuncSetAttribute(intra, cudaFuncAttributeMaxDynamicSharedMemorySize, intra_smem) != cudaSuccess)
     return B200_ERR_LAUNCH;
-  intra<<<dim3(static_cast<unsigned>(chunks), static_cast<unsigned>(p.heads)), kIntraThreads, intra_smem, stream>>>(p);
+  intra<<<dim3(static_cast<unsigned>(chunks), static_cast<unsigned>(p.heads)),
+          DELTA && head_decay ? kHeadDeltaThreads : kIntraThreads, intra_smem, stream>>>(p);
   auto inter = [&](auto kernel, int vb, int smem) {
     if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess)
       return B200_ERR_LAUNCH;
     kernel<<<dim3(static_cast<unsigned>(ceil_div(p.vdim, vb)), static_cast<unsigned>(p.heads),
-                  static_cast<unsigned>(p.sequences)), vb * 16, smem, stream>>>(p);
+                  static_cast<unsigned>(p.sequences)), vb <= 32 ? vb * 16 : vb * 8, smem, stream>>>(p);
     return launch_status();
   };
-  // narrow column slices while the wide ones would leave half the SMs without a CTA
-  if (ceil_div(p.vdim, 32) * p.heads * p.sequences * 2 > kNumSMs)
+  // One CTA per SM: narrow column slices while the wide ones would leave half the SMs without a CTA, wide ones
+  // (1.5 times the work's time) where they save as much in waves.
+  const int64_t units = static_cast<int64_t>(p.heads) * p.sequences;
+  const int64_t waves32 = ceil_div(ceil_div(p.vdim, 32) * units, kNumSMs), waves64 = ceil_div(ceil_div(p.vdim, 64) * units, kNumSMs);
+  if (p.vdim > 32 && waves64 * 3 < waves32 * 2 + 1 && waves32 > 1)
+    return inter(chunk_inter_kernel<D, 64, DELTA>, 64, inter_smem_bytes<D, 64, DELTA>());
+  if (ceil_div(p.vdim, 32) * units * 2 > kNumSMs)
     return inter(chunk_inter_kernel<D, 32, DELTA>, 32, inter_smem_bytes<D, 32, DELTA>());
   return inter(chunk_inter_kernel<D, 16, DELTA>, 16, inter_smem_bytes<D, 16, DELTA>());
 }
