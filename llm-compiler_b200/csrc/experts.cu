@@ -128,10 +128,11 @@ __device__ __forceinline__ bool write_choice(const OrderParams& p, int64_t row, 
   return inside;
 }
 
-// The CTA that arrives last at the ticket (every thread gets the answer)
+// The CTA that arrives last at the ticket (every thread gets the answer). Thread 0 publishes what it has
+// written itself.
 __device__ __forceinline__ bool arrive_last(int32_t* ticket) {
   __shared__ int last;
-  __threadfence();
+  if (threadIdx.x == 0) __threadfence();
   __syncthreads();
   if (threadIdx.x == 0) last = atomicAdd(ticket, 1) == static_cast<int>(gridDim.x) - 1;
   __syncthreads();
@@ -144,10 +145,8 @@ template <typename T>
 __global__ void __launch_bounds__(512) expert_select_kernel(const OrderParams p, const T* h, const T* router, int width,
                                                             int64_t h_stride, int32_t* chosen, float* scores,
                                                             int early_weights) {
-  extern __shared__ float shared[];  // h [width], logits [experts], first rows [experts + 1], counts [experts]
+  extern __shared__ float logits[];  // [experts], then first rows [experts + 1], counts [experts]
   constexpr int V = Elem<T>::kPerVec;
-  float* row = shared;
-  float* logits = shared + width;
   int* first = reinterpret_cast<int*>(logits + p.experts);
   int* counts = first + p.experts + 1;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
@@ -158,25 +157,20 @@ __global__ void __launch_bounds__(512) expert_select_kernel(const OrderParams p,
       asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const char*>(router) + i * 128));
   }
   grid_dependency_wait_cta();
-  for (int c = threadIdx.x * V; c < width; c += blockDim.x * V) {
-    Vec16<T> t;
-    t.load(h + blockIdx.x * h_stride + c);
-#pragma unroll
-    for (int i = 0; i < V; ++i) row[c + i] = t.v[i];
-  }
-  __syncthreads();
+  const T* row = h + blockIdx.x * h_stride;
   for (int e0 = warp * 2; e0 < p.experts; e0 += warps * 2) {  // two experts a warp: twice the loads in flight
     const int e1 = e0 + 1 < p.experts ? e0 + 1 : e0;
     float a = 0.0f, b = 0.0f;
 #pragma unroll 4
     for (int c = lane * V; c < width; c += 32 * V) {
-      Vec16<T> ta, tb;
+      Vec16<T> x, ta, tb;
+      x.load(row + c);
       ta.load(router + static_cast<int64_t>(e0) * width + c);
       tb.load(router + static_cast<int64_t>(e1) * width + c);
 #pragma unroll
       for (int i = 0; i < V; ++i) {
-        a = fmaf(ta.v[i], row[c + i], a);
-        b = fmaf(tb.v[i], row[c + i], b);
+        a = fmaf(ta.v[i], x.v[i], a);
+        b = fmaf(tb.v[i], x.v[i], b);
       }
     }
     a = warp_sum(a);
@@ -383,7 +377,7 @@ extern "C" int b200_expert_select(const void* h, const void* router, const b200_
   if (dtype != B200_F32 && dtype != B200_BF16) return B200_ERR_UNSUPPORTED;
   if (width % 8 != 0 || h_row_stride % 8 != 0 || !aligned16(h) || !aligned16(router)) return B200_ERR_ALIGNMENT;
   if (rows == 0) return B200_OK;
-  const size_t smem = (width + 3 * p.experts + 1) * sizeof(float);
+  const size_t smem = (3 * p.experts + 1) * sizeof(float);
   if (rows > 65535 || smem > 200 * 1024) return B200_ERR_TOO_LARGE;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   auto go = [&](auto tag) {
