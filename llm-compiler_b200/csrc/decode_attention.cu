@@ -520,7 +520,7 @@ decode_attention_kernel(const DecodeParams p, const __grid_constant__ CUtensorMa
     trace.mark(0);
   }
   int64_t len = 0, slot_row = -1;  // slot_row: the buffer row of the first key this row sees
-  if (p.slots != nullptr) {
+  if (!FUSED && p.slots != nullptr) {
     const int slot = p.slots[b], position = p.bases[b];
     if (slot >= 0) {
       const int first = p.chunk > 0 ? position / p.chunk * p.chunk : 0;
@@ -679,7 +679,7 @@ decode_attention_kernel(const DecodeParams p, const __grid_constant__ CUtensorMa
       o_all += new_v[col] * wgt;
     }
     const int hq = kvh * p.groups + g0 + row;
-    if (p.slots != nullptr && n_tokens == 0) l_all = 1.0f;  // an idle row: zeros
+    if (!FUSED && p.slots != nullptr && n_tokens == 0) l_all = 1.0f;  // an idle row: zeros
     if (p.num_splits == 1) {
       p.out[(static_cast<int64_t>(b) * p.q_heads + hq) * D + col] =
           __float2bfloat16_rn(o_all / l_all);  // 0/0 = NaN for an empty sequence, as the oracle
@@ -720,7 +720,7 @@ decode_attention_kernel(const DecodeParams p, const __grid_constant__ CUtensorMa
           l_all += load_cluster_f32(staging + (16 * D + row * 2 + 1) * 4, s) * wgt;
           o_all += load_cluster_f32(staging + idx * 4, s) * wgt;
         }
-        if (p.slots != nullptr && n_tokens == 0) l_all = 1.0f;
+        if (!FUSED && p.slots != nullptr && n_tokens == 0) l_all = 1.0f;
         const int hq = kvh * p.groups + g0 + row;
         p.out[(static_cast<int64_t>(b) * p.q_heads + hq) * D + col] =
             __float2bfloat16_rn(o_all / l_all);
@@ -775,7 +775,7 @@ decode_attention_kernel(const DecodeParams p, const __grid_constant__ CUtensorMa
       l_all += __ldcg(p.ws_ml + (base + s) * 2 + 1) * wgt;
       o_all += __ldcg(p.ws_o + (base + s) * D + col) * wgt;
     }
-    if (p.slots != nullptr && n_tokens == 0) l_all = 1.0f;
+    if (!FUSED && p.slots != nullptr && n_tokens == 0) l_all = 1.0f;
     p.out[(static_cast<int64_t>(b) * p.q_heads + hq) * D + col] = __float2bfloat16_rn(o_all / l_all);
   }
 }

@@ -319,10 +319,13 @@ __global__ void __launch_bounds__(256) grouped_linear_generic_kernel(const Group
       ws[i / kDepth][i % kDepth] = n < p.n && c < p.k ? weight[static_cast<int64_t>(n) * p.k + c] : 0.0f;
     }
     __syncthreads();
+    float block[4] = {};
 #pragma unroll
     for (int c = 0; c < kDepth; ++c)
 #pragma unroll
-      for (int i = 0; i < 4; ++i) acc[i] = fmaf(xs[row + i][c], ws[column][c], acc[i]);
+      for (int i = 0; i < 4; ++i) block[i] = fmaf(xs[row + i][c], ws[column][c], block[i]);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) acc[i] += block[i];
     __syncthreads();
   }
   float* out = static_cast<float*>(p.out);

@@ -227,11 +227,7 @@ __global__ void __launch_bounds__(256) linear_generic_kernel(const LinearParamsG
   __shared__ float Bs[BKF][BN + 1];
   const int tx = threadIdx.x % 16, ty = threadIdx.x / 16;
   const int m_base = blockIdx.y * BM, n_base = blockIdx.x * BN;
-  float acc[4][4];
-#pragma unroll
-  for (int i = 0; i < 4; ++i)
-#pragma unroll
-    for (int j = 0; j < 4; ++j) acc[i][j] = 0.0f;
+  float acc[4][4] = {};  // a sum of the blocks' sums: rounding errors grow with K / 16 + 16, not with K
   for (int k0 = 0; k0 < p.k; k0 += BKF) {
     for (int id = threadIdx.x; id < BM * BKF; id += 256) {
       const int r = id / BKF, c = id % BKF;
@@ -241,6 +237,7 @@ __global__ void __launch_bounds__(256) linear_generic_kernel(const LinearParamsG
       Bs[c][r] = (n < p.n && kk < p.k) ? Elem<T>::load(p.w + static_cast<int64_t>(n) * p.k + kk) : 0.0f;
     }
     __syncthreads();
+    float block[4][4] = {};
 #pragma unroll
     for (int kk = 0; kk < BKF; ++kk) {
       float a[4], b[4];
@@ -251,8 +248,12 @@ __global__ void __launch_bounds__(256) linear_generic_kernel(const LinearParamsG
 #pragma unroll
       for (int i = 0; i < 4; ++i)
 #pragma unroll
-        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
+        for (int j = 0; j < 4; ++j) block[i][j] = fmaf(a[i], b[j], block[i][j]);
     }
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) acc[i][j] += block[i][j];
     __syncthreads();
   }
 #pragma unroll
