@@ -100,13 +100,14 @@ __global__ void __launch_bounds__(256) attention_prep_kernel(const AttentionPrep
 // The same for sizes in whole quads: a CTA per row holds the projection in registers, Q quads a thread (the
 // queries' first, then the keys', then the values'), every load in flight at once.
 template <typename T>
+struct RawQuad { using type = float4; };
+template <>
+struct RawQuad<__nv_bfloat16> { using type = uint2; };
+__device__ __forceinline__ float4 widen(float4 v) { return v; }
+__device__ __forceinline__ float4 widen(uint2 t) { return make_float4(bf16_lo(t.x), bf16_hi(t.x), bf16_lo(t.y), bf16_hi(t.y)); }
+template <typename T>
 __device__ __forceinline__ float4 read_quad(const T* p) {
-  if constexpr (sizeof(T) == 4) {
-    return *reinterpret_cast<const float4*>(p);
-  } else {
-    const uint2 t = *reinterpret_cast<const uint2*>(p);
-    return make_float4(bf16_lo(t.x), bf16_hi(t.x), bf16_lo(t.y), bf16_hi(t.y));
-  }
+  return widen(*reinterpret_cast<const typename RawQuad<T>::type*>(p));
 }
 template <typename T>
 __device__ __forceinline__ void write_quad(T* p, float4 v) {
@@ -114,10 +115,11 @@ __device__ __forceinline__ void write_quad(T* p, float4 v) {
   else *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
 }
 
-template <typename T, int Q>
-__global__ void __launch_bounds__(512) attention_prep_quads_kernel(const AttentionPrepParams p, int dim_shift) {
+// PLAIN: dim, vdim and the row size are one power of two.
+template <typename T, int Q, bool PLAIN>
+__global__ void __launch_bounds__(512) attention_prep_quads_kernel(const AttentionPrepParams p) {
   extern __shared__ __align__(16) float normed[];  // q and k [(heads + kv_heads) * dim], then cos, sin [rot_dims / 2] each
-  __shared__ float scratch[2][16];
+  __shared__ float scratch[2][16], factors[2];
   const int dq = p.dim / 4, half = p.rot_dims / 2;
   const bool kv = p.keys != nullptr;
   const int nq = p.heads * dq, nk = kv ? p.kv_heads * dq : 0, nv = kv ? p.kv_heads * (p.vdim / 4) : 0;
@@ -126,6 +128,7 @@ __global__ void __launch_bounds__(512) attention_prep_quads_kernel(const Attenti
   grid_launch_dependents();
   grid_dependency_wait_cta();
   const int64_t row = blockIdx.x;
+  const int sequence = p.batch.token_sequence[row];
   auto column_of = [&](int i) {
     return i < nq ? p.q_column + i * 4 : i < nq + nk ? p.k_column + (i - nq) * 4 : p.v_column + (i - nq - nk) * 4;
   };
@@ -155,11 +158,17 @@ __global__ void __launch_bounds__(512) attention_prep_quads_kernel(const Attenti
       v[j] = read_quad<T>(static_cast<const T*>(p.input) + row * p.row_stride + column);
     }
   }
-  const int sequence = p.batch.token_sequence[row];
+  using Raw = typename RawQuad<T>::type;
+  const Raw* q_weight = static_cast<const Raw*>(p.q_weight);
+  const Raw* k_weight = static_cast<const Raw*>(p.k_weight);
+  Raw weight[Q];
+#pragma unroll
+  for (int j = 0; j < Q; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    if (i < nq + nk) weight[j] = i < nq ? q_weight[i] : k_weight[i - nq];
+  }
   const int slot = p.batch.slots[sequence];
   const int64_t position = p.batch.position(sequence, row);
-  const T* q_weight = static_cast<const T*>(p.q_weight);
-  const T* k_weight = static_cast<const T*>(p.k_weight);
   for (int i = threadIdx.x; i < half; i += blockDim.x) {
     const double turns = static_cast<double>(position) * p.turns[i];
     sincospif(2.0f * static_cast<float>(turns - rint(turns)), &sine[i], &cosine[i]);
@@ -180,19 +189,20 @@ __global__ void __launch_bounds__(512) attention_prep_quads_kernel(const Attenti
     scratch[1][warp] = k_sum;
   }
   __syncthreads();
-  q_sum = k_sum = 0.0f;
-  for (int w = 0; w < warps; ++w) {
-    q_sum += scratch[0][w];
-    k_sum += scratch[1][w];
+  if (warp == 0) {  // half a warp for each of the two
+    const int lane = threadIdx.x & 31, which = lane >> 4;
+    float sum = (lane & 15) < warps ? scratch[which][lane & 15] : 0.0f;
+#pragma unroll
+    for (int o = 8; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+    if ((lane & 15) == 0) factors[which] = 1.0f / sqrtf(sum / ((which == 0 ? p.heads : p.kv_heads) * p.dim) + p.eps);
   }
-  const float q_factor = 1.0f / sqrtf(q_sum / (p.heads * p.dim) + p.eps);
-  const float k_factor = 1.0f / sqrtf(k_sum / (p.kv_heads * p.dim) + p.eps);
+  __syncthreads();
 #pragma unroll
   for (int j = 0; j < Q; ++j) {
     const int i = threadIdx.x + j * blockDim.x;
     if (i >= nq + nk) continue;
-    const float4 w = i < nq ? read_quad<T>(q_weight + i * 4) : read_quad<T>(k_weight + (i - nq) * 4);
-    const float f = i < nq ? q_factor : k_factor;
+    const float4 w = widen(weight[j]);
+    const float f = factors[i < nq ? 0 : 1];
     v[j] = make_float4(v[j].x * f * w.x, v[j].y * f * w.y, v[j].z * f * w.z, v[j].w * f * w.w);
     *reinterpret_cast<float4*>(normed + i * 4) = v[j];
   }
@@ -208,12 +218,13 @@ __global__ void __launch_bounds__(512) attention_prep_quads_kernel(const Attenti
     const int i = threadIdx.x + j * blockDim.x;
     if (i >= nq + nk + nv || (i >= nq && !inside)) continue;
     if (i >= nq + nk) {
-      const int quad = i - nq - nk, head = quad / (p.vdim / 4);
+      const int quad = i - nq - nk, head = PLAIN ? 0 : quad / (p.vdim / 4);
       write_quad<T>(v_out + head * p.size + (quad - head * (p.vdim / 4)) * 4, v[j]);
       continue;
     }
     const int quad = i < nq ? i : i - nq;
-    const int head = dim_shift >= 0 ? quad >> dim_shift : quad / dq, c = (quad - head * dq) * 4;
+    const int head = PLAIN ? 0 : quad / dq, within = quad - head * dq;  // (PLAIN: heads lie side by side)
+    const int c = (PLAIN ? quad & (dq - 1) : within) * 4;
     float4 out = v[j];
     if (c < p.rot_dims) {
       const bool first = c < half;
@@ -225,8 +236,9 @@ __global__ void __launch_bounds__(512) attention_prep_quads_kernel(const Attenti
       out = make_float4(out.x * cs.x + other.x * sn.x, out.y * cs.y + other.y * sn.y, out.z * cs.z + other.z * sn.z,
                         out.w * cs.w + other.w * sn.w);
     }
-    write_quad<T>((i < nq ? q_out : k_out) + head * p.size + c, out);
+    write_quad<T>((i < nq ? q_out : k_out) + head * p.size + within * 4, out);
   }
+  if (PLAIN) return;
   // zeros behind every head's dim / vdim
   if (p.size > p.dim) {
     const int pad = (p.size - p.dim) / 4;
@@ -347,9 +359,7 @@ extern "C" int b200_attention_prep(const b200_attention_prep_inputs* in, int dty
   const int64_t quads = (in->heads * in->dim + (kv ? in->kv_heads * (in->dim + in->vdim) : 0)) / 4;
   const int64_t quads_smem = (in->heads * in->dim + (kv ? in->kv_heads * in->dim : 0) + in->rot_dims) * static_cast<int64_t>(sizeof(float));
   if (whole && in->rot_dims % 8 == 0 && quads <= 4096 && quads_smem <= 200 * 1024) {
-    int shift = 0;
-    while ((int64_t{4} << shift) < in->dim) ++shift;
-    if ((int64_t{4} << shift) != in->dim) shift = -1;
+    const bool plain = (in->dim & (in->dim - 1)) == 0 && in->row_size == in->dim && (!kv || in->vdim == in->dim);
     // few rows: a thread per quad or two; many: CTAs of a few warps, four quads a thread
     const int64_t q = quads > 2048 ? 8 : in->rows <= 2 * kNumSMs && quads <= 1024 ? 2 : 4;
     const int64_t threads = ceil_div(ceil_div(quads, q), 32) * 32;
@@ -358,12 +368,16 @@ extern "C" int b200_attention_prep(const b200_attention_prep_inputs* in, int dty
           cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(quads_smem)) != cudaSuccess)
         return B200_ERR_LAUNCH;
       return launch_chained(kernel, dim3(static_cast<unsigned>(in->rows)), dim3(static_cast<unsigned>(threads)),
-                            static_cast<size_t>(quads_smem), s, p, shift) == cudaSuccess ? launch_status() : B200_ERR_LAUNCH;
+                            static_cast<size_t>(quads_smem), s, p) == cudaSuccess ? launch_status() : B200_ERR_LAUNCH;
     };
-    if (dtype == B200_F32) return q == 2 ? go(attention_prep_quads_kernel<float, 2>) : q == 4 ? go(attention_prep_quads_kernel<float, 4>)
-                                                                                           : go(attention_prep_quads_kernel<float, 8>);
-    return q == 2 ? go(attention_prep_quads_kernel<__nv_bfloat16, 2>) : q == 4 ? go(attention_prep_quads_kernel<__nv_bfloat16, 4>)
-                                                                              : go(attention_prep_quads_kernel<__nv_bfloat16, 8>);
+    auto pick = [&](auto tag) {
+      using T = typename decltype(tag)::type;
+      if (plain) return q == 2 ? go(attention_prep_quads_kernel<T, 2, true>) : q == 4 ? go(attention_prep_quads_kernel<T, 4, true>)
+                                                                                      : go(attention_prep_quads_kernel<T, 8, true>);
+      return q == 2 ? go(attention_prep_quads_kernel<T, 2, false>) : q == 4 ? go(attention_prep_quads_kernel<T, 4, false>)
+                                                                            : go(attention_prep_quads_kernel<T, 8, false>);
+    };
+    return dtype == B200_F32 ? pick(TypeTag<float>{}) : pick(TypeTag<__nv_bfloat16>{});
   }
   const dim3 grid(static_cast<unsigned>(in->rows), kv ? 2u : 1u);
   auto go = [&](auto kernel) {
